@@ -5,8 +5,9 @@ logic, usable without a GPU); this module wraps it and, on a device, owns the
 page memory itself.
 
 * A **cache group** is a set of layer caches with the same needs: all keys
-  (``window=None``) or the last ``window`` keys.  Every group has its own page
-  pool and its own block table per request.
+  (``window=None``), the last ``window`` keys, or those and a request's first
+  ``keep_first``.  Every group has its own page pool and its own block table
+  per request.
 * A **page** holds ``block_size`` tokens for every layer cache of its group.
 * A **state slot** is an index per live request into arrays of per-request
   state of fixed size (mixers with a recurrent state, sampling state); it is
@@ -38,7 +39,7 @@ def _native():
         I, P, L = ctypes.c_int, ctypes.c_void_p, ctypes.c_int64
         IP = ctypes.POINTER(ctypes.c_int)
         sigs = {
-            "cm_create": (P, [I, IP, IP, IP, I, I]),
+            "cm_create": (P, [I, IP, IP, IP, IP, I, I]),
             "cm_destroy": (None, [P]),
             "cm_admit": (I, [P, L]),
             "cm_find": (I, [P, L]),
@@ -69,11 +70,13 @@ def _native():
 
 @dataclass(frozen=True)
 class GroupSpec:
-    """What one cache group needs: ``window`` None keeps every key."""
+    """What one cache group needs: ``window`` None keeps every key; with a
+    window, a request's first ``keep_first`` tokens are kept beside it."""
 
     block_size: int
     num_pages: int
     window: Optional[int] = None
+    keep_first: int = 0
 
 
 _ERRORS = {-1: ("capacity", "the cache has no page or slot left"), -2: ("invalid_argument", "bad slot, group or length"), -3: ("state", "request is unknown, already live or already freed")}
@@ -101,6 +104,7 @@ class CacheManager:
             arr([g.block_size for g in groups]),
             arr([g.num_pages for g in groups]),
             arr([g.window or 0 for g in groups]),
+            arr([g.keep_first for g in groups]),
             max_requests,
             self.max_blocks,
         )

@@ -3,7 +3,8 @@
 For every run entry that owns a cache the model says what it needs
 (:class:`~alofa_b200.parts.base.PagedKV` or
 :class:`~alofa_b200.parts.base.SlotState`).  Paged caches are sorted into
-groups by their window (all keys, or the last ``window``); a group's page ids
+groups by their window (all keys, or the last ``window``, with or without a
+request's first tokens kept beside it); a group's page ids
 are valid in every layer cache of the group.  A layer cache is two tensors
 ``k, v: [num_pages * block_size, kv_heads, head_dim]``; cache slot
 ``page * block_size + offset`` holds one token (the reference keeps
@@ -48,19 +49,24 @@ def flat_specs(plan: dict) -> list:
     return out
 
 
+def group_key(spec) -> tuple:
+    """(window, first tokens kept beside it): paged caches of one key share a group."""
+    return spec.window, getattr(spec, "keep_first", 0) if spec.window is not None else 0
+
+
 def group_windows(plan: dict) -> list:
-    """The distinct windows of a cache plan, all-keys (None) first; empty when
-    no layer wants pages (the model then has state slots only, and neither the
-    cache manager nor the scheduler books a page for it)."""
-    windows = {spec.window for spec in flat_specs(plan) if isinstance(spec, (PagedKV, PagedRows))}
-    return ([None] if None in windows else []) + sorted(w for w in windows if w is not None)
+    """The distinct (window, first tokens kept) of a cache plan, all-keys (None)
+    first; empty when no layer wants pages (the model then has state slots only,
+    and neither the cache manager nor the scheduler books a page for it)."""
+    keys = {group_key(spec) for spec in flat_specs(plan) if isinstance(spec, (PagedKV, PagedRows))}
+    return sorted(keys, key=lambda k: (k[0] is not None, k[0] or 0, k[1]))
 
 
 class CacheStorage:
     def __init__(self, plan: dict, groups: list, max_requests: int, dtype: torch.dtype, device):
         """``plan``: run index -> cache spec (owners only); ``groups``: the
         :class:`GroupSpec` list in the order of :func:`group_windows`."""
-        windows = [g.window for g in groups]
+        windows = [(g.window, g.keep_first) for g in groups]
         self.groups = groups
         self.caches = {}
         self.bytes = 0
@@ -76,9 +82,9 @@ class CacheStorage:
     def _make(self, idx, spec):
         windows, groups, dtype, device = self._windows, self.groups, self.dtype, self.device
         if isinstance(spec, (PagedKV, PagedRows)):
-            if spec.window not in windows:
-                raise AlofaError("invalid_argument", "no cache group for this window", f"window={spec.window} groups={windows}")
-            gi = windows.index(spec.window)
+            if group_key(spec) not in windows:
+                raise AlofaError("invalid_argument", "no cache group for this window", f"window={group_key(spec)} groups={windows}")
+            gi = windows.index(group_key(spec))
             g = groups[gi]
             if isinstance(spec, PagedKV):
                 slots = g.num_pages * g.block_size
@@ -105,12 +111,12 @@ class CacheStorage:
 
     @staticmethod
     def bytes_per_token(plan: dict, dtype: torch.dtype) -> dict:
-        """window -> bytes of paged cache one token takes in that group."""
+        """(window, first tokens kept) -> bytes of paged cache one token takes in that group."""
         width = torch.empty((), dtype=dtype).element_size()
         out = {}
         for spec in flat_specs(plan):
             if isinstance(spec, PagedKV):
-                out[spec.window] = out.get(spec.window, 0) + (spec.num_kv_heads * spec.head_dim + (spec.v_heads or spec.num_kv_heads) * (spec.v_head_dim or spec.head_dim)) * width
+                out[group_key(spec)] = out.get(group_key(spec), 0) + (spec.num_kv_heads * spec.head_dim + (spec.v_heads or spec.num_kv_heads) * (spec.v_head_dim or spec.head_dim)) * width
             elif isinstance(spec, PagedRows):
-                out[spec.window] = out.get(spec.window, 0) + spec.width * width
+                out[group_key(spec)] = out.get(group_key(spec), 0) + spec.width * width
         return out

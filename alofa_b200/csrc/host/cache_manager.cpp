@@ -2,8 +2,8 @@
 // request and cache group, and fixed-size state slots.
 //
 // A cache group is a set of layer caches with the same needs: all keys of a
-// request (window == 0) or only the last `window` of them.  Every group has
-// pages of its own.  A page id names a slot in every layer cache of its
+// request (window == 0), only the last `window` of them, or those and the first
+// `keep` of the request.  Every group has pages of its own.  A page id names a slot in every layer cache of its
 // group, so a request has one block table per group, not per layer.
 //
 // Semantics follow the reference's physical pool (runtime/kv/pool.mojo:28-114:
@@ -29,6 +29,7 @@ struct Group {
   int page_size = 0;
   int num_pages = 0;
   int window = 0;  // 0: every key is kept
+  int keep = 0;    // with a window: so many first tokens of a request stay visible for good, and their pages with them
   std::vector<int32_t> refcount;
   std::vector<int32_t> free_stack;  // back() is handed out next
   int64_t allocs = 0, frees = 0;
@@ -71,8 +72,12 @@ int release_page(Group& g, int p) {
   return 0;
 }
 
+// Blocks that hold kept first tokens: no window ever gives them back.
+inline int blocks_kept(const Group& g) { return g.window > 0 ? ceil_div(g.keep, g.page_size) : 0; }
+
 // Blocks of a request that are wholly below the oldest key the next query
-// (at position `len`) can see in a window of `window` keys.
+// (at position `len`) can see in a window of `window` keys (those that hold
+// kept first tokens among them).
 inline int blocks_passed(const Group& g, int len) {
   if (g.window <= 0) return 0;
   int oldest_needed = len - g.window + 1;
@@ -84,20 +89,21 @@ inline int blocks_passed(const Group& g, int len) {
 
 extern "C" {
 
-void* cm_create(int n_groups, const int* page_size, const int* num_pages, const int* window,
+void* cm_create(int n_groups, const int* page_size, const int* num_pages, const int* window, const int* keep,
                 int max_requests, int max_blocks_per_request) {
   if (n_groups < 0 || max_requests <= 0 || max_blocks_per_request <= 0) return nullptr;  // no group: state slots only
   auto* m = new Manager();
   m->groups.resize(n_groups);
   for (int i = 0; i < n_groups; ++i) {
     Group& g = m->groups[i];
-    if (page_size[i] <= 0 || num_pages[i] <= 0 || window[i] < 0) {
+    if (page_size[i] <= 0 || num_pages[i] <= 0 || window[i] < 0 || keep[i] < 0 || (keep[i] > 0 && window[i] == 0)) {
       delete m;
       return nullptr;
     }
     g.page_size = page_size[i];
     g.num_pages = num_pages[i];
     g.window = window[i];
+    g.keep = keep[i];
     g.refcount.assign(g.num_pages, 0);
     g.free_stack.resize(g.num_pages);
     for (int p = 0; p < g.num_pages; ++p) g.free_stack[p] = g.num_pages - 1 - p;
@@ -192,7 +198,7 @@ int cm_advance(void* h, int s, int new_len) {
     Group& grp = m->groups[g];
     int passed = blocks_passed(grp, new_len);
     if (passed > (int)r.table[g].size()) passed = (int)r.table[g].size();
-    for (int b = r.first_block[g]; b < passed; ++b) {
+    for (int b = std::max(r.first_block[g], blocks_kept(grp)); b < passed; ++b) {
       if (r.table[g][b] >= 0) {
         if (release_page(grp, r.table[g][b]) < 0) return ERR_STATE;
         r.table[g][b] = -1;
@@ -450,7 +456,7 @@ int cm_defects(void* h) {
       for (size_t b = 0; b < r.table[g].size(); ++b) {
         int32_t p = r.table[g][b];
         if (p < 0) {
-          if ((int)b >= r.first_block[g]) defects++;
+          if ((int)b >= r.first_block[g] || (int)b < blocks_kept(grp)) defects++;
           continue;
         }
         if (p >= grp.num_pages) {

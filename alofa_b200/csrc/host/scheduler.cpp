@@ -17,6 +17,7 @@
 //     scheduler.mojo:539-557);
 //   * an arrival that does not fit now is deferred, not refused, and "newest"
 //     means latest admitted, not highest slot.
+#include <algorithm>
 #include <cstdint>
 #include <cstring>
 #include <vector>
@@ -38,7 +39,7 @@ struct Slot {
 
 struct Sched {
   int token_budget, max_chunk, max_batch, max_tokens, watermark_permille, max_wait_ticks, admission;
-  std::vector<int> page_size, window, capacity;
+  std::vector<int> page_size, window, capacity, keep;  // keep: first tokens of a request that stay beside the window
   std::vector<Slot> slots;
   std::vector<int> free_local, order;
   int64_t tick_seq = 0, preempt_total = 0, next_seq = 1;
@@ -53,7 +54,7 @@ int held(const Sched& s, int g, int len) {
   int blocks = ceil_div(len, s.page_size[g]);
   if (s.window[g] > 0) {
     int oldest = len - s.window[g] + 1;
-    if (oldest > 0) blocks -= oldest / s.page_size[g];
+    if (oldest > 0) blocks -= std::max(0, oldest / s.page_size[g] - ceil_div(s.keep[g], s.page_size[g]));
   }
   return blocks;
 }
@@ -64,7 +65,7 @@ int worst(const Sched& s, int g, int total) {
   if (s.window[g] <= 0) return ceil_div(total, s.page_size[g]);
   int span = s.window[g] + s.max_chunk;
   if (span > total) span = total;
-  return ceil_div(span, s.page_size[g]) + 1;
+  return std::min(ceil_div(total, s.page_size[g]), ceil_div(span, s.page_size[g]) + 1 + ceil_div(s.keep[g], s.page_size[g]));
 }
 
 int threshold(const Sched& s, int g) { return (int)((int64_t)s.capacity[g] * s.watermark_permille / 1000); }
@@ -192,7 +193,7 @@ extern "C" {
 
 // cfg: token_budget, max_chunk, max_batch, max_tokens, watermark_permille,
 //      max_wait_ticks, admission, n_groups, then per group page_size, window,
-//      capacity.  n_groups may be 0 (a model whose layers keep fixed-size state
+//      capacity, first tokens kept beside the window.  n_groups may be 0 (a model whose layers keep fixed-size state
 //      only): no page is ever booked, nothing is ever preempted, and admission is
 //      bounded by the request slots alone.
 void* sched_create(const int* cfg, int n) {
@@ -208,12 +209,13 @@ void* sched_create(const int* cfg, int n) {
   int G = cfg[7];
   bool ok = s->token_budget >= 0 && s->max_chunk > 0 && s->max_batch > 0 && s->max_tokens > 0 &&
             s->watermark_permille >= 0 && s->watermark_permille <= 1000 && s->max_wait_ticks >= 0 &&
-            (s->admission == ADMIT_COMMITTED || s->admission == ADMIT_OPTIMISTIC) && G >= 0 && n == 8 + 3 * G;
+            (s->admission == ADMIT_COMMITTED || s->admission == ADMIT_OPTIMISTIC) && G >= 0 && n == 8 + 4 * G;
   for (int g = 0; ok && g < G; ++g) {
-    s->page_size.push_back(cfg[8 + 3 * g]);
-    s->window.push_back(cfg[9 + 3 * g]);
-    s->capacity.push_back(cfg[10 + 3 * g]);
-    ok = s->page_size[g] > 0 && s->window[g] >= 0 && s->capacity[g] > 0;
+    s->page_size.push_back(cfg[8 + 4 * g]);
+    s->window.push_back(cfg[9 + 4 * g]);
+    s->capacity.push_back(cfg[10 + 4 * g]);
+    s->keep.push_back(cfg[11 + 4 * g]);
+    ok = s->page_size[g] > 0 && s->window[g] >= 0 && s->capacity[g] > 0 && s->keep[g] >= 0;
   }
   if (!ok) {
     delete s;

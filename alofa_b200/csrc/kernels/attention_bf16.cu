@@ -11,18 +11,22 @@
 // mma.sync m16n8k16 (bf16 operands); softmax is the streaming form in fp32:
 // running maximum, exp2 with the scale folded in, rescaled sums.
 // Visibility: key j is seen by the row at position P when j <= P and, with a
-// window, j > P - window.
+// window, j > P - window or j < keep (a request's first keys, kept beside the
+// window).  Key blocks that a tile cannot see are never touched (their pages
+// may have been given back): the blocks walked are the kept ones, then those
+// from the window's start on (see SeenBlocks).
 //
 // Decode-only launches may split the keys of a request over several CTAs
 // (split s owns keys [s * split_keys, (s + 1) * split_keys), a function of the
-// key index alone); the partial (output, maximum, sum) triples are merged by
+// key index alone; with kept keys the same of the blocks walked, counted
+// through); the partial (output, maximum, sum) triples are merged by
 // attention_combine_kernel in split order.
 //
 // Prompt portions go to the tcgen05 kernel of attention_prefill_tc.cuh instead
 // when the head size is 64 or 128 and a page holds whole 64-key blocks; decode
 // tokens of small head groups to attention_decode_kernel below.
 //
-// HEAD_DIM is a compile-time constant (a multiple of 16 up to 128): the
+// HEAD_DIM and V_DIM are compile-time constants (multiples of 16 up to 128): the
 // library is built per head size.  Formulas: src/alofa/kernels/cpu/scalar.mojo:392-470,
 // paged addressing src/alofa/kernels/cpu/paged.mojo:249-336.
 #include "common.cuh"
@@ -30,14 +34,14 @@
 #include "attention_core.cuh"
 
 struct AttnParams {
-  bf16* out;             // [T, nh, HD]
+  bf16* out;             // [T, nh, VD]
   const bf16* q;         // [T, nh, HD]
   const bf16* k_cache;   // [slots, nkv, HD]
-  const bf16* v_cache;
+  const bf16* v_cache;   // [slots, nkv, VD]
   const int* q_start;    // [R + 1] first row of each request in this step
   const int* kv_len;     // [R] keys of each request after this step
   const int* block_table;  // [R, max_blocks]
-  float* partial_o;      // split mode: [splits, T * nh, HD]
+  float* partial_o;      // split mode: [splits, T * nh, VD]
   float* partial_ml;     // split mode: [splits, T * nh, 2]
   int max_blocks, page_size, nh, nkv, window, split_keys, n_splits, n_rows_total, table_entries;
   float scale_log2;      // scale * log2(e)
@@ -46,6 +50,13 @@ struct AttnParams {
 #endif
   int* status;           // set to 2 when a wait on a bulk copy gave up (may be null)
   const float* sink;     // [nh] or null: one more term exp(sink[h]) of the softmax's denominator, with no key and no value
+  int keep;              // with a window: keys j < keep are seen beside it
+  const float* gate;     // [T, gate_ld] or null: the finished output of head h is multiplied by sigmoid(gate[t, h])
+  int gate_ld;
+#ifdef DISTANCE_BIAS
+  const float* slopes;   // [nh]: slopes[h] * (P - j) is taken off the score of key j
+  float slope_mul;       // 1 / scale: the bias in units of the raw dot products
+#endif
 };
 
 // The sink's share of a row's sum whose terms are scaled by 2^-m_log2 (m_log2: the row's maximum in log2 units).
@@ -54,37 +65,80 @@ __device__ __forceinline__ float sink_term(const float* sink, int head, float m_
   return sink ? exp2f(fmaf(sink[head], 1.4426950408889634f, -m_log2)) : 0.f;
 }
 
+// A head's gate on its finished output.
+__device__ __forceinline__ float gate_of_head(const float* gate, int ld, int token, int head) {
+  return gate ? 1.0f / (1.0f + expf(-gate[(size_t)token * ld + head])) : 1.0f;
+}
+
 // How far back the query at position pos sees, itself included (0: every key).  A negative `window` is a mask in chunks of
 // that many positions counted from the sequence's start: the query sees the keys of its own chunk, which is a window of
 // pos % chunk + 1 keys.  A window's start never moves back as the position grows, whichever kind it is.
 __device__ __forceinline__ int window_at(int window, int pos) { return window >= 0 ? window : pos % (-window) + 1; }
 
+constexpr bool TMA_SIZES = HD % 64 == 0 && VD % 64 == 0;  // head sizes the kernels fed by bulk tensor copies take
+
+// The blocks of N keys that queries see whose last key is k_hi and whose window starts at k_lo (0: no window, or not left
+// yet), walked as numbers lo .. hi: first the `kept` blocks that hold a request's kept first keys, then those from the
+// window's first on.  Without kept keys a number is the block's own.
+template <int N>
+struct SeenBlocks {
+  int lo, hi, kept, gap;
+  __device__ __forceinline__ SeenBlocks(int keep, int k_lo, int k_hi) {
+    const int first = k_lo / N;
+    kept = keep > 0 ? min((keep + N - 1) / N, first) : 0;
+    gap = keep > 0 ? first - kept : 0;
+    lo = keep > 0 ? 0 : first;
+    hi = k_hi / N - gap;
+  }
+  __device__ __forceinline__ int block(int i) const { return i < kept ? i : i + gap; }
+};
+
+// A CTA's copy of the block-table entries it may use: those of the kept keys, then those from the window's start on.
+struct TableCopy {
+  int kept, shift, entries;
+  __device__ __forceinline__ TableCopy(int keep, int k_lo, int k_hi, int page_size) {
+    const int last = k_hi / page_size;
+    kept = keep > 0 ? min((keep + page_size - 1) / page_size, last + 1) : 0;
+    const int first = max(kept, k_lo / page_size);
+    shift = first - kept;
+    entries = kept + max(0, last - first + 1);
+  }
+  __device__ __forceinline__ int source(int i) const { return i < kept ? i : i + shift; }  // the i-th copied entry
+  __device__ __forceinline__ int index(int e) const { return e < kept ? e : e - shift; }   // where entry e lies in the copy
+};
+
 #include "attention_prefill_tc.cuh"
 
 // Copy keys [j0, j0 + 64) of one KV head, keys and values, into shared tiles
-// [64][ROW]; rows past j_end (exclusive) or before j_begin are zero-filled.
-// `table` is the shared copy of the request's block-table entries from entry
-// `first_entry` on (a lookup in global memory here would stall every copy
+// [64][ROW] and [64][VROW]; rows past k_hi, and rows before k_lo that are not
+// kept, are zero-filled.  `table` is the shared copy of the request's
+// block-table entries (a lookup in global memory here would stall every copy
 // behind it).  When a page holds whole key blocks (page_size % 64 == 0) the
 // block lies in one page and a row's address is the block's base plus a fixed
 // stride; else every row looks its page up.
 __device__ __forceinline__ void load_kv_tiles(bf16* k_tile, bf16* v_tile, const bf16* k_cache, const bf16* v_cache, const int* table,
-                                              int first_entry, int page_size, bool block_in_page, int nkv, int kvh, int j0, int j_begin,
-                                              int j_end) {
-  if constexpr (128 % CHUNKS != 0) {
-    // head sizes whose rows do not divide a round of 128 threads: one chunk at a time
+                                              const TableCopy& copy, int page_size, bool block_in_page, int nkv, int kvh, int j0, int k_lo,
+                                              int k_hi, int keep) {
+  auto seen = [&](int j) { return j <= k_hi && (j >= k_lo || j < keep); };
+  auto slot_of = [&](int j) -> size_t {
+    const int e = j / page_size;
+    return (size_t)(table[copy.index(e)] * page_size + (j - e * page_size)) * nkv + kvh;
+  };
+  if constexpr (VD != HD || 128 % CHUNKS != 0) {
+    // keys and values of different sizes, or head sizes whose rows do not divide a round of 128 threads: one chunk at a time
     for (int idx = threadIdx.x; idx < BLOCK_N * CHUNKS; idx += 128) {
       const int r = idx / CHUNKS, c = idx % CHUNKS;
-      const int j = j0 + r;
-      const bool ok = j >= j_begin && j < j_end;
-      size_t offset = 0;
-      if (ok) {
-        const int e = j / page_size;
-        const int slot = table[e - first_entry] * page_size + (j - e * page_size);
-        offset = ((size_t)slot * nkv + kvh) * HD + c * 8;
+      const bool ok = seen(j0 + r);
+      const size_t row = ok ? slot_of(j0 + r) : 0;
+      cp_async16((uint32_t)__cvta_generic_to_shared(k_tile + r * ROW + c * 8), k_cache + (ok ? row * HD + c * 8 : 0), ok);
+      if constexpr (VD == HD) cp_async16((uint32_t)__cvta_generic_to_shared(v_tile + r * VROW + c * 8), v_cache + (ok ? row * VD + c * 8 : 0), ok);
+    }
+    if constexpr (VD != HD) {
+      for (int idx = threadIdx.x; idx < BLOCK_N * VCHUNKS; idx += 128) {
+        const int r = idx / VCHUNKS, c = idx % VCHUNKS;
+        const bool ok = seen(j0 + r);
+        cp_async16((uint32_t)__cvta_generic_to_shared(v_tile + r * VROW + c * 8), v_cache + (ok ? slot_of(j0 + r) * VD + c * 8 : 0), ok);
       }
-      cp_async16((uint32_t)__cvta_generic_to_shared(k_tile + r * ROW + c * 8), k_cache + offset, ok);
-      cp_async16((uint32_t)__cvta_generic_to_shared(v_tile + r * ROW + c * 8), v_cache + offset, ok);
     }
     return;
   }
@@ -94,13 +148,12 @@ __device__ __forceinline__ void load_kv_tiles(bf16* k_tile, bf16* v_tile, const 
   constexpr int ROWS_PER_ROUND = (128 % CHUNKS == 0) ? 128 / CHUNKS : 1;
   if (block_in_page) {
     const int e = j0 / page_size;
-    const size_t first_slot = (size_t)table[e - first_entry] * page_size + (j0 - e * page_size);
+    const size_t first_slot = (size_t)table[copy.index(e)] * page_size + (j0 - e * page_size);
     const size_t base = ((first_slot + r0) * nkv + kvh) * HD + c * 8;
     const size_t step = (size_t)ROWS_PER_ROUND * nkv * HD;
 #pragma unroll
     for (int it = 0; it < BLOCK_N / ROWS_PER_ROUND; ++it) {
-      const int j = j0 + r0 + it * ROWS_PER_ROUND;
-      const bool ok = j >= j_begin && j < j_end;
+      const bool ok = seen(j0 + r0 + it * ROWS_PER_ROUND);
       const size_t offset = ok ? base + it * step : 0;
       cp_async16(k_dst + it * ROWS_PER_ROUND * ROW * 2, k_cache + offset, ok);
       cp_async16(v_dst + it * ROWS_PER_ROUND * ROW * 2, v_cache + offset, ok);
@@ -110,13 +163,8 @@ __device__ __forceinline__ void load_kv_tiles(bf16* k_tile, bf16* v_tile, const 
 #pragma unroll
   for (int it = 0; it < BLOCK_N / ROWS_PER_ROUND; ++it) {
     const int j = j0 + r0 + it * ROWS_PER_ROUND;
-    const bool ok = j >= j_begin && j < j_end;
-    size_t offset = 0;
-    if (ok) {
-      const int e = j / page_size;
-      const int slot = table[e - first_entry] * page_size + (j - e * page_size);
-      offset = ((size_t)slot * nkv + kvh) * HD + c * 8;
-    }
+    const bool ok = seen(j);
+    const size_t offset = ok ? slot_of(j) * HD + c * 8 : 0;
     cp_async16(k_dst + it * ROWS_PER_ROUND * ROW * 2, k_cache + offset, ok);
     cp_async16(v_dst + it * ROWS_PER_ROUND * ROW * 2, v_cache + offset, ok);
   }
@@ -129,7 +177,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* q_tile = reinterpret_cast<bf16*>(smem_raw);          // [64][ROW]
   bf16* k_tiles = q_tile + BLOCK_M * ROW;                    // [STAGES][64][ROW]
-  bf16* v_tiles = k_tiles + STAGES * BLOCK_N * ROW;          // [STAGES][64][ROW]
+  bf16* v_tiles = k_tiles + STAGES * BLOCK_N * ROW;          // [STAGES][64][VROW]
   pdl_begin();
 
   const int seq = blockIdx.z, kvh = blockIdx.y;
@@ -149,20 +197,25 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
   int k_hi = pos0 + t_last;  // last visible key of the tile (inclusive)
   int k_lo = 0;
   if (p.window != 0) k_lo = max(0, pos0 + t_first - window_at(p.window, pos0 + t_first) + 1);
+  const SeenBlocks<BLOCK_N> walk(p.keep, k_lo, k_hi);
+  int nb_lo = walk.lo, nb_hi = walk.hi;  // the numbers of the blocks this CTA walks
   if (SPLIT) {
-    k_lo = max(k_lo, split * p.split_keys);
-    k_hi = min(k_hi, (split + 1) * p.split_keys - 1);
-    if (k_lo > k_hi) return;
+    nb_lo = max(nb_lo, split * (p.split_keys / BLOCK_N));
+    nb_hi = min(nb_hi, (split + 1) * (p.split_keys / BLOCK_N) - 1);
+    if (nb_lo > nb_hi) return;
+    if (p.keep == 0) {  // only this split's entries of the block table
+      k_lo = max(k_lo, split * p.split_keys);
+      k_hi = min(k_hi, (split + 1) * p.split_keys - 1);
+    }
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // the block-table entries this CTA will use, copied to shared memory once
-  int* table = reinterpret_cast<int*>(v_tiles + STAGES * BLOCK_N * ROW);
-  const int first_entry = k_lo / p.page_size;
+  int* table = reinterpret_cast<int*>(v_tiles + STAGES * BLOCK_N * VROW);
+  const TableCopy copy(p.keep, k_lo, k_hi, p.page_size);
   const bool block_in_page = p.page_size % BLOCK_N == 0;
   {
-    const int* src = p.block_table + (size_t)seq * p.max_blocks + first_entry;
-    const int n_entries = k_hi / p.page_size - first_entry + 1;
-    for (int e = threadIdx.x; e < n_entries; e += 128) table[e] = src[e];
+    const int* src = p.block_table + (size_t)seq * p.max_blocks;
+    for (int e = threadIdx.x; e < copy.entries; e += 128) table[e] = src[copy.source(e)];
     __syncthreads();
   }
 
@@ -175,12 +228,11 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
     if (ok) src = p.q + ((size_t)(row_begin + row / g) * p.nh + kvh * g + row % g) * HD + c * 8;
     cp_async16((uint32_t)__cvta_generic_to_shared(q_tile + r * ROW + c * 8), src, ok);
   }
-  const int nb_lo = k_lo / BLOCK_N, nb_hi = k_hi / BLOCK_N;
 #pragma unroll
   for (int st = 0; st < STAGES; ++st) {  // one commit group per stage, empty past the last block
     if (nb_lo + st <= nb_hi) {
-      load_kv_tiles(k_tiles + st * BLOCK_N * ROW, v_tiles + st * BLOCK_N * ROW, p.k_cache, p.v_cache, table, first_entry, p.page_size,
-                    block_in_page, p.nkv, kvh, (nb_lo + st) * BLOCK_N, k_lo, k_hi + 1);
+      load_kv_tiles(k_tiles + st * BLOCK_N * ROW, v_tiles + st * BLOCK_N * VROW, p.k_cache, p.v_cache, table, copy, p.page_size,
+                    block_in_page, p.nkv, kvh, walk.block(nb_lo + st) * BLOCK_N, k_lo, k_hi, p.keep);
     }
     cp_async_commit();
   }
@@ -190,6 +242,9 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
   const int pos_lo = pos0 + min(r_lo, n_rows - 1) / g, pos_hi = pos0 + min(r_hi, n_rows - 1) / g;
   const int warp_pos_min = pos0 + min(row0 + warp * 16, n_rows - 1) / g;
   const int warp_pos_max = pos0 + min(row0 + warp * 16 + 15, n_rows - 1) / g;
+#ifdef DISTANCE_BIAS
+  const float slope_lo = p.slopes[kvh * g + min(r_lo, n_rows - 1) % g] * p.slope_mul, slope_hi = p.slopes[kvh * g + min(r_hi, n_rows - 1) % g] * p.slope_mul;
+#endif
 
   uint32_t qf[KSTEPS][4];
   float o[DTILES][4];
@@ -209,7 +264,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
       }
     }
     const bf16* kt = k_tiles + buf * BLOCK_N * ROW;
-    const bf16* vt = v_tiles + buf * BLOCK_N * ROW;
+    const bf16* vt = v_tiles + buf * BLOCK_N * VROW;
 
     // ---- S = Q K^T : 16 rows x 64 keys per warp ---------------------------------
     float s[BLOCK_N / 8][4];
@@ -234,9 +289,16 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
       for (int e = 0; e < 4; ++e) s[n][e] = cap_score(s[n][e], p.cap_in, p.cap_out);
 #endif
     // ---- visibility -------------------------------------------------------------
-    const int j0 = nb * BLOCK_N;
-    const bool all_visible = (j0 + BLOCK_N - 1 <= min(warp_pos_min, k_hi)) && (j0 >= k_lo) &&
-                             (p.window == 0 || j0 > warp_pos_max - window_at(p.window, warp_pos_max));
+    const int j0 = walk.block(nb) * BLOCK_N;
+#ifdef DISTANCE_BIAS
+#pragma unroll
+    for (int n = 0; n < BLOCK_N / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        s[n][e] = fmaf(e < 2 ? slope_lo : slope_hi, (float)(j0 + n * 8 + (lane & 3) * 2 + (e & 1) - (e < 2 ? pos_lo : pos_hi)), s[n][e]);
+#endif
+    const bool all_visible = j0 + BLOCK_N - 1 <= warp_pos_min &&
+                             (p.window == 0 || j0 > warp_pos_max - window_at(p.window, warp_pos_max) || j0 + BLOCK_N <= p.keep);
     if (!all_visible) {
 #pragma unroll
       for (int n = 0; n < BLOCK_N / 8; ++n) {
@@ -244,9 +306,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + n * 8 + (lane & 3) * 2 + (e & 1);
           const int pos = (e < 2) ? pos_lo : pos_hi;
-          bool vis = j <= pos && j >= k_lo && j <= k_hi;
-          if (p.window != 0) vis = vis && j > pos - window_at(p.window, pos);
-          if (!vis) s[n][e] = -INFINITY;
+          if (!key_seen(j, pos, window_at(p.window, pos), p.keep)) s[n][e] = -INFINITY;
         }
       }
     }
@@ -293,10 +353,10 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
 #pragma unroll
     for (int kk = 0; kk < BLOCK_N / 16; ++kk) {
 #pragma unroll
-      for (int d2 = 0; d2 < HD / 16; ++d2) {
+      for (int d2 = 0; d2 < VD / 16; ++d2) {
         // keys kk*16 .. +15 (k), dims d2*16 .. +15 (n): transposed 8x8 loads
         uint32_t vf[4];
-        const bf16* src = vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ROW + d2 * 16 + (lane >> 4) * 8;
+        const bf16* src = vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VROW + d2 * 16 + (lane >> 4) * 8;
         ldmatrix_x4_trans(vf, (uint32_t)__cvta_generic_to_shared(src));
         mma_16816(o[2 * d2], pf[kk], vf[0], vf[1]);
         mma_16816(o[2 * d2 + 1], pf[kk], vf[2], vf[3]);
@@ -304,8 +364,8 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
     }
     __syncthreads();  // everyone is done with this buffer before it is refilled
     if (nb + STAGES <= nb_hi) {
-      load_kv_tiles(k_tiles + buf * BLOCK_N * ROW, v_tiles + buf * BLOCK_N * ROW, p.k_cache, p.v_cache, table, first_entry, p.page_size,
-                    block_in_page, p.nkv, kvh, (nb + STAGES) * BLOCK_N, k_lo, k_hi + 1);
+      load_kv_tiles(k_tiles + buf * BLOCK_N * ROW, v_tiles + buf * BLOCK_N * VROW, p.k_cache, p.v_cache, table, copy, p.page_size,
+                    block_in_page, p.nkv, kvh, walk.block(nb + STAGES) * BLOCK_N, k_lo, k_hi, p.keep);
     }
     cp_async_commit();
   }
@@ -321,7 +381,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
     const float l = half ? l_hi : l_lo, m = half ? m_hi : m_lo;
     const size_t out_row = (size_t)(row_begin + row / g) * p.nh + kvh * g + row % g;
     if (SPLIT) {
-      float* po = p.partial_o + ((size_t)split * p.n_rows_total + out_row) * HD;
+      float* po = p.partial_o + ((size_t)split * p.n_rows_total + out_row) * VD;
 #pragma unroll
       for (int d = 0; d < DTILES; ++d)
         *reinterpret_cast<float2*>(po + d * 8 + (lane & 3) * 2) = make_float2(o[d][half * 2], o[d][half * 2 + 1]);
@@ -331,8 +391,9 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
         ml[1] = l;
       }
     } else {
-      const float inv = 1.0f / (l + sink_term(p.sink, kvh * g + row % g, m * p.scale_log2));
-      bf16* po = p.out + out_row * HD;
+      const int head = kvh * g + row % g;
+      const float inv = gate_of_head(p.gate, p.gate_ld, row_begin + row / g, head) / (l + sink_term(p.sink, head, m * p.scale_log2));
+      bf16* po = p.out + out_row * VD;
 #pragma unroll
       for (int d = 0; d < DTILES; ++d)
         *reinterpret_cast<uint32_t*>(po + d * 8 + (lane & 3) * 2) = pack_bf16(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
@@ -359,7 +420,7 @@ __global__ void __launch_bounds__(128) attention_bf16_kernel(const AttnParams p)
 // arrives by bulk tensor copies - keys and values, 128-byte swizzled, each on
 // its own mbarrier of the warp - issued by one lane; else by 16-byte cp.async
 // copies into padded tiles, one block after the other.
-constexpr int TILE_BYTES_TMA = BLOCK_N * HD * 2;  // one dense tile
+constexpr int K_TILE_TMA = BLOCK_N * HD * 2, V_TILE_TMA = BLOCK_N * VD * 2;  // bytes of a dense tile
 
 // LONG: splits of more than one block per warp; without it a warp's keys and values come on one
 // barrier and nothing is refilled.
@@ -367,12 +428,12 @@ template <int WARPS, bool TMA, bool LONG>
 __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const AttnParams p, const __grid_constant__ CUtensorMap map_k,
                                                                       const __grid_constant__ CUtensorMap map_v) {
   constexpr int THREADS = WARPS * 32;
-  constexpr int TILE_ELEMS = TMA ? BLOCK_N * HD : BLOCK_N * ROW;
+  constexpr int K_ELEMS = TMA ? BLOCK_N * HD : BLOCK_N * ROW, V_ELEMS = TMA ? BLOCK_N * VD : BLOCK_N * VROW;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* aligned = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   bf16* k_tiles = reinterpret_cast<bf16*>(aligned);       // [WARPS] tiles of 64 keys
-  bf16* v_tiles = k_tiles + WARPS * TILE_ELEMS;           // [WARPS] tiles of 64 keys
-  bf16* q_tile = v_tiles + WARPS * TILE_ELEMS;            // [16][ROW]
+  bf16* v_tiles = k_tiles + WARPS * K_ELEMS;              // [WARPS] tiles of 64 values
+  bf16* q_tile = v_tiles + WARPS * V_ELEMS;               // [16][ROW]
   // the merge buffers reuse the key tiles once every warp is done with them
   float* merge_o = reinterpret_cast<float*>(k_tiles);     // [WARPS][16][MERGE_ROW]
   float* merge_ml = merge_o + WARPS * 16 * MERGE_ROW;     // [WARPS][16][2]
@@ -392,49 +453,58 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
   int k_lo = 0;
   const int window = window_at(p.window, pos);  // of this one position
   if (window > 0) k_lo = max(0, pos - window + 1);
-  k_lo = max(k_lo, split * p.split_keys);
-  const int k_hi = min(pos, (split + 1) * p.split_keys - 1);
-  if (k_lo > k_hi) return;
+  const SeenBlocks<BLOCK_N> walk(p.keep, k_lo, pos);
+  const int b_lo = max(walk.lo, split * (p.split_keys / BLOCK_N)), b_hi = min(walk.hi, (split + 1) * (p.split_keys / BLOCK_N) - 1);
+  if (b_lo > b_hi) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  // this warp's blocks of keys: first, first + WARPS, ... up to last (block numbers within the request)
-  const int b_lo = k_lo / BLOCK_N, b_hi = k_hi / BLOCK_N;
+  // this warp's blocks of keys: first, first + WARPS, ... up to last (numbers of the walk over the request's blocks)
   const int mine = split * (p.split_keys / BLOCK_N) + warp;
   const int first = mine >= b_lo ? mine : mine + (b_lo - mine + WARPS - 1) / WARPS * WARPS;
   const bool has_keys = first <= b_hi;
   const int last = !has_keys ? first - WARPS : LONG ? first + (b_hi - first) / WARPS * WARPS : first;
-  bf16* kt = k_tiles + warp * TILE_ELEMS;
-  bf16* vt = v_tiles + warp * TILE_ELEMS;
+  bf16* kt = k_tiles + warp * K_ELEMS;
+  bf16* vt = v_tiles + warp * V_ELEMS;
+#ifdef DISTANCE_BIAS
+  const float slope_lo = (lane >> 2) < g ? p.slopes[kvh * g + (lane >> 2)] * p.slope_mul : 0.f;
+  const float slope_hi = (lane >> 2) + 8 < g ? p.slopes[kvh * g + (lane >> 2) + 8] * p.slope_mul : 0.f;
+#endif
   // a block lies inside one page, its 64 rows are consecutive cache slots
   auto block_row = [&](int block) {
-    const int j = block * BLOCK_N, e = j / p.page_size;
+    const int j = walk.block(block) * BLOCK_N, e = j / p.page_size;
     return p.block_table[(size_t)seq * p.max_blocks + e] * p.page_size + (j - e * p.page_size);
   };
   auto fetch_keys = [&](int row) {  // one lane
-    mbar_expect_tx(&k_bar[warp], TILE_BYTES_TMA);
+    mbar_expect_tx(&k_bar[warp], K_TILE_TMA);
 #pragma unroll
     for (int sub = 0; sub < HD / 64; ++sub)
       tma_load_2d(reinterpret_cast<uint8_t*>(kt) + sub * BLOCK_N * 128, &map_k, &k_bar[warp], kvh * HD + sub * 64, row);
   };
   auto fetch_values = [&](int row) {  // one lane
-    mbar_expect_tx(&v_bar[warp], TILE_BYTES_TMA);
+    mbar_expect_tx(&v_bar[warp], V_TILE_TMA);
 #pragma unroll
-    for (int sub = 0; sub < HD / 64; ++sub)
-      tma_load_2d(reinterpret_cast<uint8_t*>(vt) + sub * BLOCK_N * 128, &map_v, &v_bar[warp], kvh * HD + sub * 64, row);
+    for (int sub = 0; sub < VD / 64; ++sub)
+      tma_load_2d(reinterpret_cast<uint8_t*>(vt) + sub * BLOCK_N * 128, &map_v, &v_bar[warp], kvh * VD + sub * 64, row);
   };
   auto fetch_padded = [&](int block) {  // the whole warp
     const int* table = p.block_table + (size_t)seq * p.max_blocks;
+    const int j0 = walk.block(block) * BLOCK_N;
+    auto row_of = [&](int j) -> size_t {
+      const int e = j / p.page_size;
+      return (size_t)(table[e] * p.page_size + (j - e * p.page_size)) * p.nkv + kvh;
+    };
     for (int idx = lane; idx < BLOCK_N * CHUNKS; idx += 32) {
       const int r = idx / CHUNKS, c = idx % CHUNKS;
-      const int j = block * BLOCK_N + r;
-      const bool ok = j >= k_lo && j <= k_hi;
-      size_t offset = 0;
-      if (ok) {
-        const int e = j / p.page_size;
-        const int slot = table[e] * p.page_size + (j - e * p.page_size);
-        offset = ((size_t)slot * p.nkv + kvh) * HD + c * 8;
+      const bool ok = key_seen(j0 + r, pos, window, p.keep);
+      const size_t row = ok ? row_of(j0 + r) : 0;
+      cp_async16((uint32_t)__cvta_generic_to_shared(kt + r * ROW + c * 8), p.k_cache + (ok ? row * HD + c * 8 : 0), ok);
+      if constexpr (VD == HD) cp_async16((uint32_t)__cvta_generic_to_shared(vt + r * VROW + c * 8), p.v_cache + (ok ? row * VD + c * 8 : 0), ok);
+    }
+    if constexpr (VD != HD) {
+      for (int idx = lane; idx < BLOCK_N * VCHUNKS; idx += 32) {
+        const int r = idx / VCHUNKS, c = idx % VCHUNKS;
+        const bool ok = key_seen(j0 + r, pos, window, p.keep);
+        cp_async16((uint32_t)__cvta_generic_to_shared(vt + r * VROW + c * 8), p.v_cache + (ok ? row_of(j0 + r) * VD + c * 8 : 0), ok);
       }
-      cp_async16((uint32_t)__cvta_generic_to_shared(kt + r * ROW + c * 8), p.k_cache + offset, ok);
-      cp_async16((uint32_t)__cvta_generic_to_shared(vt + r * ROW + c * 8), p.v_cache + offset, ok);
     }
   };
   auto fetch_first = [&](int row) {  // one lane
@@ -442,11 +512,11 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
       fetch_keys(row);
       fetch_values(row);
     } else {
-      mbar_expect_tx(&k_bar[warp], 2 * TILE_BYTES_TMA);
+      mbar_expect_tx(&k_bar[warp], K_TILE_TMA + V_TILE_TMA);
 #pragma unroll
-      for (int sub = 0; sub < HD / 64; ++sub) {
-        tma_load_2d(reinterpret_cast<uint8_t*>(kt) + sub * BLOCK_N * 128, &map_k, &k_bar[warp], kvh * HD + sub * 64, row);
-        tma_load_2d(reinterpret_cast<uint8_t*>(vt) + sub * BLOCK_N * 128, &map_v, &k_bar[warp], kvh * HD + sub * 64, row);
+      for (int sub = 0; sub < (HD > VD ? HD : VD) / 64; ++sub) {
+        if (sub < HD / 64) tma_load_2d(reinterpret_cast<uint8_t*>(kt) + sub * BLOCK_N * 128, &map_k, &k_bar[warp], kvh * HD + sub * 64, row);
+        if (sub < VD / 64) tma_load_2d(reinterpret_cast<uint8_t*>(vt) + sub * BLOCK_N * 128, &map_v, &k_bar[warp], kvh * VD + sub * 64, row);
       }
     }
   };
@@ -458,7 +528,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
   const int token = p.q_start[seq];
   // A block that ends before the query's own position holds only keys of earlier steps: its copy
   // need not wait for the kernel that writes this step's key and may start at once.
-  const bool early = TMA && has_keys && first * BLOCK_N + BLOCK_N - 1 < pos;
+  const bool early = TMA && has_keys && walk.block(first) * BLOCK_N + BLOCK_N - 1 < pos;
   if (early && lane == 0) fetch_first(row_first);
   pdl_wait();
 
@@ -502,7 +572,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
         if (LONG && lane == 0 && block + 2 * WARPS <= last) row_after = block_row(block + 2 * WARPS);
         bool values_here = true;
         attend_block<true>(
-            st, qf, kt_s, vt_s, block * BLOCK_N, lane, pos, k_lo, k_hi, window, p.scale_log2 CAP_ARGS(p),
+            st, qf, kt_s, vt_s, walk.block(block) * BLOCK_N, lane, pos, window, p.keep, p.scale_log2 CAP_ARGS(p) BIAS_PASS,
             [&] {
               if (more) {
                 __syncwarp();  // every lane has taken its scores from the key tile
@@ -519,7 +589,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
         }
         row_next = row_after;
       } else {
-        attend_block<false>(st, qf, kt_s, vt_s, block * BLOCK_N, lane, pos, k_lo, k_hi, window, p.scale_log2 CAP_ARGS(p));
+        attend_block<false>(st, qf, kt_s, vt_s, walk.block(block) * BLOCK_N, lane, pos, window, p.keep, p.scale_log2 CAP_ARGS(p) BIAS_PASS);
         if (more) {
           __syncwarp();
           fetch_padded(block + WARPS);
@@ -555,8 +625,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
   }
   __syncthreads();
   const bool single = gridDim.x == 1;
-  for (int idx = threadIdx.x; idx < g * HD; idx += THREADS) {
-    const int r = idx / HD, d = idx % HD;
+  for (int idx = threadIdx.x; idx < g * VD; idx += THREADS) {
+    const int r = idx / VD, d = idx % VD;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) m = fmaxf(m, merge_ml[w * 32 + r * 2]);
@@ -570,9 +640,9 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
     }
     const size_t out_row = (size_t)token * p.nh + kvh * g + r;
     if (single) {
-      p.out[out_row * HD + d] = __float2bfloat16_rn(acc / (l + sink_term(p.sink, kvh * g + r, m)));
+      p.out[out_row * VD + d] = __float2bfloat16_rn(acc * gate_of_head(p.gate, p.gate_ld, token, kvh * g + r) / (l + sink_term(p.sink, kvh * g + r, m)));
     } else {
-      p.partial_o[((size_t)split * p.n_rows_total + out_row) * HD + d] = acc;
+      p.partial_o[((size_t)split * p.n_rows_total + out_row) * VD + d] = acc;
       if (d == 0) {
         float* ml = p.partial_ml + ((size_t)split * p.n_rows_total + out_row) * 2;
         ml[0] = m;
@@ -583,8 +653,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_decode_kernel(const Attn
 }
 
 static size_t decode_smem_bytes(int warps, bool tma) {
-  const size_t tile = tma ? (size_t)BLOCK_N * HD * sizeof(bf16) : (size_t)BLOCK_N * ROW * sizeof(bf16);
-  const size_t tiles = 2 * warps * tile;
+  const size_t tiles = (size_t)warps * BLOCK_N * (tma ? HD + VD : ROW + VROW) * sizeof(bf16);
   const size_t merge = (size_t)warps * 16 * MERGE_ROW * sizeof(float) + (size_t)warps * 32 * sizeof(float);
   return 1024 + (tiles > merge ? tiles : merge) + (size_t)16 * ROW * sizeof(bf16);
 }
@@ -612,17 +681,18 @@ static int launch_decode(const AttnParams& p, const CUtensorMap& map_k, const CU
   return launch_decode_as<WARPS, TMA, false>(p, map_k, map_v, n_splits, nkv, n_seqs, stream);
 }
 
-// Merge the splits of every (token, head) row in split order.  One block of HD
-// threads per row; a row's splits are those its visible keys fall into.
+// Merge the splits of every (token, head) row in split order.  One block of VD
+// threads per row; a row's splits are those its visible keys fall into (keep > 0: those the walk over its blocks fell into).
 __global__ void attention_combine_kernel(bf16* __restrict__ out, const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                                          const int* __restrict__ positions, int nh, int window, int split_keys, int n_rows_total,
-                                         const float* __restrict__ sink) {
+                                         const float* __restrict__ sink, int keep, const float* __restrict__ gate, int gate_ld) {
   const int row = blockIdx.x;       // token * nh + head
   pdl_begin();
   const int P = positions[row / nh];
   int k_lo = 0;
   if (window != 0) k_lo = max(0, P - window_at(window, P) + 1);
-  const int s_lo = k_lo / split_keys, s_hi = P / split_keys;
+  const SeenBlocks<BLOCK_N> walk(keep, k_lo, P);
+  const int s_lo = walk.lo / (split_keys / BLOCK_N), s_hi = walk.hi / (split_keys / BLOCK_N);
   float m = -INFINITY;
   for (int s = s_lo; s <= s_hi; ++s) m = fmaxf(m, partial_ml[((size_t)s * n_rows_total + row) * 2]);
   float l = 0.f, acc = 0.f;
@@ -631,14 +701,14 @@ __global__ void attention_combine_kernel(bf16* __restrict__ out, const float* __
     const float* ml = partial_ml + ((size_t)s * n_rows_total + row) * 2;
     const float w = (ml[0] == -INFINITY) ? 0.f : fast_exp2(ml[0] - m);
     l += ml[1] * w;
-    acc += partial_o[((size_t)s * n_rows_total + row) * HD + d] * w;
+    acc += partial_o[((size_t)s * n_rows_total + row) * VD + d] * w;
   }
-  out[(size_t)row * HD + d] = __float2bfloat16_rn(acc / (l + sink_term(sink, row % nh, m)));
+  out[(size_t)row * VD + d] = __float2bfloat16_rn(acc * gate_of_head(gate, gate_ld, row / nh, row % nh) / (l + sink_term(sink, row % nh, m)));
 }
 
 constexpr int PREFILL_STAGES = 2, SPLIT_STAGES = 4;
 static size_t attention_smem_bytes(int stages, int table_entries) {
-  return (size_t)(BLOCK_M + 2 * stages * BLOCK_N) * ROW * sizeof(bf16) + (size_t)table_entries * sizeof(int);
+  return ((size_t)(BLOCK_M + stages * BLOCK_N) * ROW + (size_t)stages * BLOCK_N * VROW) * sizeof(bf16) + (size_t)table_entries * sizeof(int);
 }
 
 ALOFA_API int alofa_attention_head_dim() { return HD; }
@@ -646,14 +716,14 @@ ALOFA_API int alofa_attention_head_dim() { return HD; }
 // The decode kernel's wide form: one CTA per SM with as many warps as its shared memory holds
 // key and value tiles for (16 KB a warp at head size 64, 32 KB at 128), on pages of whole key
 // blocks.  Taken when a launch's splits are a multiple of WIDE_WARPS * 64 keys.
-constexpr int WIDE_WARPS = HD == 64 ? 8 : HD == 128 ? 6 : 0;
+constexpr int WIDE_WARPS = !TMA_SIZES ? 0 : HD + VD <= 128 ? 8 : 6;
 ALOFA_API int alofa_attention_decode_wide_warps() { return WIDE_WARPS; }
 
 // How many CTAs of the decode kernel with `warps` warps (4, or the wide form's) the device holds
 // at a time: what a caller sizes the key splits by, so that a step's CTAs are resident together.
 // 0 when that kernel does not exist here or the device cannot be asked.
 ALOFA_API int alofa_attention_decode_slots(int page_size, int warps) {
-  const bool tma = (HD == 64 || HD == 128) && page_size % BLOCK_N == 0;
+  const bool tma = TMA_SIZES && page_size % BLOCK_N == 0;
   int device = 0, sms = 0, per_sm = 0;
   if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess) return 0;
   cudaError_t rc;
@@ -681,12 +751,13 @@ ALOFA_API int alofa_attention_decode_slots(int page_size, int warps) {
   return sms * per_sm;
 }
 
-// Merge the splits a launch with do_combine = 0 left behind: out [T, nh, HD] bf16.
+// Merge the splits a launch with do_combine = 0 left behind: out [T, nh, VD] bf16.
 ALOFA_API int alofa_attention_combine(void* out, const float* partial_o, const float* partial_ml, const int* positions, int n_tokens, int nh,
                                       int window, int split_keys, const float* sink, cudaStream_t stream) {
   if (n_tokens <= 0) return ALOFA_OK;
-  if (!partial_o || !partial_ml || !positions || split_keys <= 0) return ALOFA_ERR_ARGUMENT;
-  launch_dep(attention_combine_kernel, n_tokens * nh, HD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, n_tokens * nh, sink);
+  if (!partial_o || !partial_ml || !positions || split_keys <= 0 || split_keys % BLOCK_N) return ALOFA_ERR_ARGUMENT;
+  launch_dep(attention_combine_kernel, n_tokens * nh, VD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, n_tokens * nh, sink, 0,
+             (const float*)nullptr, 0);
   return launch_status();
 }
 
@@ -702,20 +773,34 @@ ALOFA_API int alofa_attention_bf16(void* out, const void* q, const void* k_cache
                                    const int* block_table, int max_blocks, int page_size, int n_seqs, int n_tokens, int tiles, int nh, int nkv,
                                    int window, float scale, int n_splits, int split_keys, float* partial_o, float* partial_ml,
                                    int max_kv_len, long long cache_slots, int* status, int do_combine, float softcap, const float* sink,
-                                   cudaStream_t stream) {
+                                   int keep, const float* slopes, const float* gate, int gate_ld, cudaStream_t stream) {
   if (n_seqs <= 0 || n_tokens <= 0) return ALOFA_OK;
 #ifdef SOFTCAP
   if (!(softcap > 0.f) || !(scale > 0.f)) return ALOFA_ERR_ARGUMENT;
 #else
   if (softcap != 0.f) return ALOFA_ERR_ARGUMENT;  // only a library built with SOFTCAP caps its scores
 #endif
+#ifdef DISTANCE_BIAS
+  if (!slopes || !(scale > 0.f)) return ALOFA_ERR_ARGUMENT;
+#else
+  if (slopes) return ALOFA_ERR_ARGUMENT;  // only a library built with DISTANCE_BIAS biases its scores
+#endif
+  if (keep < 0 || (keep > 0 && window <= 0) || (gate && gate_ld < nh)) return ALOFA_ERR_ARGUMENT;
   if (nkv <= 0 || nh % nkv != 0 || page_size <= 0 || tiles <= 0) return ALOFA_ERR_ARGUMENT;
   if (n_splits > 0 && (split_keys <= 0 || split_keys % BLOCK_N != 0 || !partial_o || !partial_ml || !positions)) return ALOFA_ERR_ARGUMENT;
   const bool decode_only = n_seqs == n_tokens;
   if (n_splits > 0 && decode_only && nh / nkv > BLOCK_M) return ALOFA_ERR_ARGUMENT;
-  if (sink && n_splits > 1 && !do_combine) return ALOFA_ERR_ARGUMENT;  // the sink is added where the splits are merged: here
+  if ((sink || gate || keep > 0) && n_splits > 1 && !do_combine) return ALOFA_ERR_ARGUMENT;  // what completes a row is done where the splits are merged: here
+  if (keep > 0 && n_splits > 0 && !decode_only) return ALOFA_ERR_ARGUMENT;  // the tiles of a prompt walk their own blocks: a row's splits could not be told
   AttnParams p;
   p.sink = sink;
+  p.keep = keep;
+  p.gate = gate;
+  p.gate_ld = gate_ld;
+#ifdef DISTANCE_BIAS
+  p.slopes = slopes;
+  p.slope_mul = 1.0f / scale;
+#endif
   p.out = (bf16*)out;
   p.q = (const bf16*)q;
   p.status = status;
@@ -740,7 +825,7 @@ ALOFA_API int alofa_attention_bf16(void* out, const void* q, const void* k_cache
   p.cap_out = softcap / scale;
 #endif
   // entries of a block table one CTA may touch: a split's keys, or up to the longest request
-  const int reach = n_splits > 0 ? split_keys : max_kv_len;
+  const int reach = n_splits > 0 && keep == 0 ? split_keys : max_kv_len;
   p.table_entries = reach / page_size + 2;
   const size_t smem = attention_smem_bytes((n_splits > 0 && decode_only) ? SPLIT_STAGES : PREFILL_STAGES, p.table_entries);
   if (smem > 200 * 1024) return ALOFA_ERR_ARGUMENT;
@@ -762,12 +847,12 @@ ALOFA_API int alofa_attention_bf16(void* out, const void* q, const void* k_cache
   if (n_splits > 0 && decode_only && nh / nkv <= 16 &&
       (split_keys % (4 * BLOCK_N) == 0 || split_keys == 2 * BLOCK_N || (WIDE_WARPS > 0 && split_keys % ((WIDE_WARPS > 0 ? WIDE_WARPS : 4) * BLOCK_N) == 0))) {
     // decode tokens of small head groups: the key blocks of a split side by side on the warps
-    // pages that hold whole key blocks and rows of 128 or 256 bytes: bulk tensor copies
+    // pages that hold whole key blocks, rows of 128 or 256 bytes: bulk tensor copies
     CUtensorMap map_k, map_v;
-    bool tma = (HD == 64 || HD == 128) && page_size % BLOCK_N == 0 && cache_slots > 0 && ((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0;
+    bool tma = TMA_SIZES && page_size % BLOCK_N == 0 && cache_slots > 0 && ((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0;
     if (tma)
       tma = make_tensor_map_bf16(&map_k, k_cache, (uint64_t)cache_slots, (uint64_t)nkv * HD, BLOCK_N, 64) &&
-            make_tensor_map_bf16(&map_v, v_cache, (uint64_t)cache_slots, (uint64_t)nkv * HD, BLOCK_N, 64);
+            make_tensor_map_bf16(&map_v, v_cache, (uint64_t)cache_slots, (uint64_t)nkv * VD, BLOCK_N, 64);
     if (!tma) {
       memset(&map_k, 0, sizeof(map_k));
       memset(&map_v, 0, sizeof(map_v));
@@ -782,17 +867,20 @@ ALOFA_API int alofa_attention_bf16(void* out, const void* q, const void* k_cache
       rc = tma ? launch_decode<2, true>(p, map_k, map_v, n_splits, nkv, n_seqs, stream) : launch_decode<2, false>(p, map_k, map_v, n_splits, nkv, n_seqs, stream);
     if (rc != ALOFA_OK) return rc;
     if (n_splits > 1 && do_combine)
-      launch_dep(attention_combine_kernel, n_tokens * nh, HD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink);
+      launch_dep(attention_combine_kernel, n_tokens * nh, VD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink, keep,
+                 gate, gate_ld);
   } else if (n_splits > 0 && !decode_only) {
     // prompt portions: every query tile's keys split over n_splits CTAs, so that the tiles
     // at the end of a long prompt do not set the pace
     launch_dep(attention_bf16_kernel<true, PREFILL_STAGES>, dim3(tiles * n_splits, nkv, n_seqs), 128, smem, stream, p);
     if (cudaGetLastError() != cudaSuccess) return ALOFA_ERR_LAUNCH;
-    launch_dep(attention_combine_kernel, n_tokens * nh, HD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink);
+    launch_dep(attention_combine_kernel, n_tokens * nh, VD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink, keep,
+                 gate, gate_ld);
   } else if (n_splits > 0) {
     launch_dep(attention_bf16_kernel<true, SPLIT_STAGES>, dim3(n_splits, nkv, n_seqs), 128, smem, stream, p);
     if (cudaGetLastError() != cudaSuccess) return ALOFA_ERR_LAUNCH;
-    launch_dep(attention_combine_kernel, n_tokens * nh, HD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink);
+    launch_dep(attention_combine_kernel, n_tokens * nh, VD, 0, stream, (bf16*)out, partial_o, partial_ml, positions, nh, window, split_keys, p.n_rows_total, p.sink, keep,
+                 gate, gate_ld);
   } else {
     // prompt portions: the tcgen05 kernel where the head size and the pages are its own
     // (ALOFA_ATTENTION_TC=0 keeps the mma.sync kernel), else mma.sync

@@ -2,8 +2,8 @@
 // size, the asynchronous-copy / ldmatrix / mma.sync wrappers, and attend_block,
 // which runs 16 query rows against one 64-key block held in shared memory with
 // the streaming softmax in fp32 (running maximum, exp2 with the scale folded
-// in, rescaled sums).  HEAD_DIM is a compile-time constant (a multiple of 16 up
-// to 128).  Formulas: src/alofa/kernels/cpu/scalar.mojo:392-470.
+// in, rescaled sums).  HEAD_DIM (keys) and V_DIM (values; the same unless given)
+// are compile-time constants, multiples of 16 up to 128.  Formulas: src/alofa/kernels/cpu/scalar.mojo:392-470.
 #pragma once
 #include "common.cuh"
 
@@ -11,14 +11,22 @@
 #define HEAD_DIM 64
 #endif
 
-constexpr int HD = HEAD_DIM;
+#ifndef V_DIM
+#define V_DIM HEAD_DIM
+#endif
+
+constexpr int HD = HEAD_DIM;  // channels of a query or key head
+constexpr int VD = V_DIM;     // channels of a value head
 constexpr int BLOCK_M = 64;   // query rows per CTA (4 warps x 16)
 constexpr int BLOCK_N = 64;   // keys per block
 constexpr int ROW = HD + 8;   // shared-memory row in elements: 16 bytes of padding keep ldmatrix conflict-free
+constexpr int VROW = VD + 8;
 constexpr int KSTEPS = HD / 16;
-constexpr int DTILES = HD / 8;
+constexpr int DTILES = VD / 8;
 constexpr int CHUNKS = HD / 8;  // 16-byte chunks per row
+constexpr int VCHUNKS = VD / 8;
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 128, "head_dim must be a multiple of 16 between 16 and 128");
+static_assert(VD % 16 == 0 && VD >= 16 && VD <= 128, "the values' head size must be a multiple of 16 between 16 and 128");
 
 __device__ __forceinline__ void cp_async16(uint32_t smem, const void* gptr, bool pred) {
   const int bytes = pred ? 16 : 0;
@@ -57,16 +65,16 @@ struct RowState {
 };
 
 // Shared-memory address of the 16-byte chunk at (row, col) of a 64-key tile.
-// Padded layout: rows of ROW elements (the cp.async path).  Swizzled layout (what a
+// Padded layout: rows of `pitch` elements (the cp.async path).  Swizzled layout (what a
 // TMA load with 128-byte swizzle leaves): sub-tiles of 64 dims, rows of 128 bytes,
 // the chunk index XOR-ed with the low bits of the row.
 template <bool SWIZZLED>
-__device__ __forceinline__ uint32_t tile_addr(uint32_t base, int row, int col) {
+__device__ __forceinline__ uint32_t tile_addr(uint32_t base, int row, int col, int pitch) {
   if (SWIZZLED) {
     const int sub = col >> 6, chunk = (col & 63) >> 3;
     return base + sub * (BLOCK_N * 128) + row * 128 + ((chunk ^ (row & 7)) << 4);
   }
-  return base + (row * ROW + col) * 2;
+  return base + (row * pitch + col) * 2;
 }
 
 // A library built with SOFTCAP bounds the scaled scores by softcap * tanh(score / softcap) before the
@@ -89,12 +97,25 @@ __device__ __forceinline__ float cap_score(float dot, float cap_in, float cap_ou
 #define CAP_ARGS(p)
 #endif
 
+// A library built with DISTANCE_BIAS takes slope_h * (query position - key position) off the scaled (and capped) score.  The
+// scores are raw dot products until the scale is folded into the exponent, so the slopes come divided by the scale.
+#ifdef DISTANCE_BIAS
+#define BIAS_PARAMS , float slope_lo, float slope_hi
+#define BIAS_PASS , slope_lo, slope_hi
+#else
+#define BIAS_PARAMS
+#define BIAS_PASS
+#endif
+
+// Whether the query at `pos` sees key j: the last `window` keys (0: every key), and beside a window the first `keep`.
+__device__ __forceinline__ bool key_seen(int j, int pos, int window, int keep) { return j <= pos && (window <= 0 || j > pos - window || j < keep); }
+
 // One warp: 16 query rows against the 64 keys of one block held in shared tiles.
 // keys_done() runs when the key tile has been read for the last time (it may be
 // refilled), values_wanted() just before the value tile is read for the first time.
 template <bool SWIZZLED, class KeysDone, class ValuesWanted>
 __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[KSTEPS][4], uint32_t kt, uint32_t vt, int j0, int lane,
-                                             int pos, int k_lo, int k_hi, int window, float scale_log2 CAP_PARAMS, KeysDone keys_done,
+                                             int pos, int window, int keep, float scale_log2 CAP_PARAMS BIAS_PARAMS, KeysDone keys_done,
                                              ValuesWanted values_wanted) {
   float s[BLOCK_N / 8][4];
 #pragma unroll
@@ -104,7 +125,7 @@ __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[
 #pragma unroll
     for (int n2 = 0; n2 < BLOCK_N / 16; ++n2) {
       uint32_t kf[4];
-      ldmatrix_x4(kf, tile_addr<SWIZZLED>(kt, n2 * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 16 + ((lane >> 3) & 1) * 8));
+      ldmatrix_x4(kf, tile_addr<SWIZZLED>(kt, n2 * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 16 + ((lane >> 3) & 1) * 8, ROW));
       mma_16816(s[2 * n2], qf[ks], kf[0], kf[1]);
       mma_16816(s[2 * n2 + 1], qf[ks], kf[2], kf[3]);
     }
@@ -116,16 +137,20 @@ __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[n][e] = cap_score(s[n][e], cap_in, cap_out);
 #endif
-  const bool all_visible = j0 >= k_lo && j0 + BLOCK_N - 1 <= k_hi && (window <= 0 || j0 > pos - window);
+#ifdef DISTANCE_BIAS
+#pragma unroll
+  for (int n = 0; n < BLOCK_N / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[n][e] = fmaf(e < 2 ? slope_lo : slope_hi, (float)(j0 + n * 8 + (lane & 3) * 2 + (e & 1) - pos), s[n][e]);
+#endif
+  const bool all_visible = j0 + BLOCK_N - 1 <= pos && (window <= 0 || j0 > pos - window || j0 + BLOCK_N <= keep);
   if (!all_visible) {
 #pragma unroll
     for (int n = 0; n < BLOCK_N / 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int j = j0 + n * 8 + (lane & 3) * 2 + (e & 1);
-        bool vis = j <= pos && j >= k_lo && j <= k_hi;
-        if (window > 0) vis = vis && j > pos - window;
-        if (!vis) s[n][e] = -INFINITY;
+        if (!key_seen(j, pos, window, keep)) s[n][e] = -INFINITY;
       }
   }
   float bm_lo = -INFINITY, bm_hi = -INFINITY;
@@ -169,9 +194,9 @@ __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[
 #pragma unroll
   for (int kk = 0; kk < BLOCK_N / 16; ++kk) {
 #pragma unroll
-    for (int d2 = 0; d2 < HD / 16; ++d2) {
+    for (int d2 = 0; d2 < VD / 16; ++d2) {
       uint32_t vf[4];
-      ldmatrix_x4_trans(vf, tile_addr<SWIZZLED>(vt, kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, d2 * 16 + (lane >> 4) * 8));
+      ldmatrix_x4_trans(vf, tile_addr<SWIZZLED>(vt, kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, d2 * 16 + (lane >> 4) * 8, VROW));
       mma_16816(st.o[2 * d2], pf[kk], vf[0], vf[1]);
       mma_16816(st.o[2 * d2 + 1], pf[kk], vf[2], vf[3]);
     }
@@ -180,9 +205,9 @@ __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[
 
 template <bool SWIZZLED>
 __device__ __forceinline__ void attend_block(RowState& st, const uint32_t (&qf)[KSTEPS][4], uint32_t kt, uint32_t vt, int j0, int lane,
-                                             int pos, int k_lo, int k_hi, int window, float scale_log2 CAP_PARAMS) {
-  attend_block<SWIZZLED>(st, qf, kt, vt, j0, lane, pos, k_lo, k_hi, window, scale_log2 CAP_PASS, [] {}, [] {});
+                                             int pos, int window, int keep, float scale_log2 CAP_PARAMS BIAS_PARAMS) {
+  attend_block<SWIZZLED>(st, qf, kt, vt, j0, lane, pos, window, keep, scale_log2 CAP_PASS BIAS_PASS, [] {}, [] {});
 }
 
-constexpr int MERGE_ROW = HD + 4;  // floats per merged row in shared memory
+constexpr int MERGE_ROW = VD + 4;  // floats per merged row in shared memory
 

@@ -1,5 +1,5 @@
 // Causal grouped-query attention of prompt portions on the fifth-generation
-// tensor cores (tcgen05), for head sizes 64 and 128 and pages that hold whole
+// tensor cores (tcgen05), for head sizes 64 and 128 (keys and values may differ) and pages that hold whole
 // 64-key blocks.  Included by attention_bf16.cu, which owns AttnParams.
 //
 // One CTA owns 128 query rows of one (request, KV head): a row is a (token,
@@ -30,11 +30,12 @@
 
 constexpr int TC_BM = 128;                       // query rows per CTA
 constexpr int TC_BN = 128;                       // keys per block
-constexpr int TC_PANELS = HD / 64;               // 64-wide panels of a head
+constexpr int TC_PANELS = HD / 64;               // 64-wide panels of a query or key head
+constexpr int TC_V_PANELS = VD / 64;             // and of a value head
 constexpr int TC_PANEL_BYTES = 128 * 128;        // 128 rows of 128 bytes
-constexpr int TC_KV_BYTES = TC_PANELS * TC_PANEL_BYTES;  // one key (or value) block
+constexpr int TC_K_BYTES = TC_PANELS * TC_PANEL_BYTES, TC_STAGE_BYTES = (TC_PANELS + TC_V_PANELS) * TC_PANEL_BYTES;  // a key block; a key and a value block
 constexpr int TC_Q_BYTES = TC_PANELS * TC_PANEL_BYTES;
-constexpr int TC_STAGES = HD <= 64 ? 4 : 2;
+constexpr int TC_STAGES = HD + VD <= 128 ? 4 : HD + VD <= 192 ? 3 : 2;
 constexpr int TC_THREADS = 320;  // a warp of copies, a warp of MMAs, eight of softmax
 constexpr float TC_RESCALE_ABOVE = 8.0f;         // log2 units a row's maximum may outgrow the one in use
 
@@ -61,7 +62,7 @@ __device__ __forceinline__ uint64_t smem_desc_mn_sw128(uint32_t addr, uint32_t p
 }
 
 static size_t prefill_tc_smem_bytes(int table_entries) {
-  return 1024 + (size_t)TC_Q_BYTES + (size_t)TC_STAGES * 2 * TC_KV_BYTES + (size_t)table_entries * sizeof(int);
+  return 1024 + (size_t)TC_Q_BYTES + (size_t)TC_STAGES * TC_STAGE_BYTES + (size_t)table_entries * sizeof(int);
 }
 
 __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(const AttnParams p, const __grid_constant__ CUtensorMap map_k,
@@ -70,7 +71,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* q_tile = smem;                                   // [panel][128 rows][128 B], K-major
   uint8_t* kv_ring = q_tile + TC_Q_BYTES;                   // [stage][K | V][panel][128 keys][128 B]
-  int* table = reinterpret_cast<int*>(kv_ring + TC_STAGES * 2 * TC_KV_BYTES);  // the request's block-table entries from the first block on
+  int* table = reinterpret_cast<int*>(kv_ring + TC_STAGES * TC_STAGE_BYTES);  // the request's block-table entries that this tile may see
   __shared__ uint64_t kv_full[TC_STAGES], kv_free[TC_STAGES], s_full[2], q_ready, p_full, pv_done, pair_bar[4];
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
@@ -91,7 +92,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
   const int t_first = row0 / g, t_last = last_row / g;
   const int k_hi = pos0 + t_last;  // last visible key of the tile
   const int k_lo = p.window != 0 ? max(0, pos0 + t_first - window_at(p.window, pos0 + t_first) + 1) : 0;
-  const int jb0 = k_lo / TC_BN, nblk = k_hi / TC_BN - jb0 + 1;
+  const SeenBlocks<TC_BN> walk(p.keep, k_lo, k_hi);
+  const int jb0 = walk.lo, nblk = walk.hi - walk.lo + 1;
 
   if (threadIdx.x == 0) {
     abort_flag = 0;
@@ -118,27 +120,30 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
 
   if (warp == 0) {
     // ---- the key and value blocks ------------------------------------------------------
-    const int first_entry = (jb0 * TC_BN) / p.page_size;
-    const int n_entries = k_hi / p.page_size - first_entry + 1;
-    for (int e = lane; e < n_entries; e += 32) table[e] = p.block_table[(size_t)seq * p.max_blocks + first_entry + e];
+    const TableCopy copy(p.keep, k_lo / TC_BN * TC_BN, k_hi, p.page_size);
+    for (int e = lane; e < copy.entries; e += 32) table[e] = p.block_table[(size_t)seq * p.max_blocks + copy.source(e)];
     __syncwarp();
     if (lane == 0) {
       for (int i = 0; i < nblk; ++i) {
         const int s = i % TC_STAGES;
         if (i >= TC_STAGES && !mbar_wait(&kv_free[s], ((i / TC_STAGES) - 1) & 1, &abort_flag)) break;
-        uint8_t* k_stage = kv_ring + (size_t)s * 2 * TC_KV_BYTES;
-        uint8_t* v_stage = k_stage + TC_KV_BYTES;
-        mbar_expect_tx(&kv_full[s], 2 * TC_KV_BYTES);
+        uint8_t* k_stage = kv_ring + (size_t)s * TC_STAGE_BYTES;
+        uint8_t* v_stage = k_stage + TC_K_BYTES;
+        mbar_expect_tx(&kv_full[s], TC_STAGE_BYTES);
+        const int j_block = walk.block(jb0 + i) * TC_BN;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          int j = (jb0 + i) * TC_BN + half * 64;
-          if (j > k_hi) j -= 64;  // nothing there: the first half again, every key of it masked
+          int j = j_block + half * 64;
+          // nothing of this half can be seen (it lies past the tile's last key, or between the kept keys and the window, where its
+          // page may be gone): the other half again, every key of it masked
+          const bool unseen = j > k_hi || (p.keep > 0 && j >= p.keep && j + 63 < k_lo);
+          if (unseen) j = j_block + (half ^ 1) * 64;
           const int e = j / p.page_size;
-          const int slot0 = table[e - first_entry] * p.page_size + (j - e * p.page_size);
+          const int slot0 = table[copy.index(e)] * p.page_size + (j - e * p.page_size);
 #pragma unroll
-          for (int pn = 0; pn < TC_PANELS; ++pn) {
-            tma_load_2d(k_stage + pn * TC_PANEL_BYTES + half * 8192, &map_k, &kv_full[s], kvh * HD + pn * 64, slot0);
-            tma_load_2d(v_stage + pn * TC_PANEL_BYTES + half * 8192, &map_v, &kv_full[s], kvh * HD + pn * 64, slot0);
+          for (int pn = 0; pn < (TC_PANELS > TC_V_PANELS ? TC_PANELS : TC_V_PANELS); ++pn) {
+            if (pn < TC_PANELS) tma_load_2d(k_stage + pn * TC_PANEL_BYTES + half * 8192, &map_k, &kv_full[s], kvh * HD + pn * 64, slot0);
+            if (pn < TC_V_PANELS) tma_load_2d(v_stage + pn * TC_PANEL_BYTES + half * 8192, &map_v, &kv_full[s], kvh * VD + pn * 64, slot0);
           }
         }
       }
@@ -147,13 +152,13 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
     // ---- the MMAs ------------------------------------------------------------------------
     if (lane == 0) {
       constexpr uint32_t IDESC_QK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TC_BN >> 3) << 17) | ((uint32_t)(TC_BM >> 4) << 24);
-      constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(HD >> 3) << 17) | ((uint32_t)(TC_BM >> 4) << 24);
+      constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(VD >> 3) << 17) | ((uint32_t)(TC_BM >> 4) << 24);
       const uint32_t q_addr = smem_u32(q_tile);
       auto issue_qk = [&](int i) -> bool {  // S[i & 1] = Q K_i^T
         const int s = i % TC_STAGES;
         if (!mbar_wait(&kv_full[s], (i / TC_STAGES) & 1, &abort_flag)) return false;
         tc_fence_after();
-        const uint32_t k_addr = smem_u32(kv_ring + (size_t)s * 2 * TC_KV_BYTES);
+        const uint32_t k_addr = smem_u32(kv_ring + (size_t)s * TC_STAGE_BYTES);
 #pragma unroll
         for (int k = 0; k < HD / UMMA_K; ++k) {
           const uint32_t off = (k >> 2) * TC_PANEL_BYTES + (k & 3) * 32;
@@ -171,7 +176,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
         if (i + 1 < nblk) ok = issue_qk(i + 1);
         if (!ok || !mbar_wait(&p_full, i & 1, &abort_flag)) break;
         tc_fence_after();
-        const uint32_t v_addr = smem_u32(kv_ring + (size_t)(i % TC_STAGES) * 2 * TC_KV_BYTES + TC_KV_BYTES);
+        const uint32_t v_addr = smem_u32(kv_ring + (size_t)(i % TC_STAGES) * TC_STAGE_BYTES + TC_K_BYTES);
 #pragma unroll
         for (int k = 0; k < TC_BN / UMMA_K; ++k) {  // O += P V_i, sixteen keys (eight packed columns of P) at a time
           const uint64_t desc_v = smem_desc_mn_sw128(v_addr + k * 2048, TC_PANEL_BYTES);
@@ -192,6 +197,9 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
     const bool row_ok = R < n_rows;
     const int my_pos = pos0 + (row_ok ? R / g : 0);
     const int my_lo = p.window != 0 ? max(0, my_pos - window_at(p.window, my_pos) + 1) : 0;
+#ifdef DISTANCE_BIAS
+    const float slope = row_ok ? p.slopes[kvh * g + R % g] * p.slope_mul : 0.f;
+#endif
     uint32_t pair_phase = 0;
     auto pair_sync = [&]() -> bool {  // the two warps of a quadrant meet (bounded, like every wait here)
       mbar_arrive(&pair_bar[q4]);
@@ -213,7 +221,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
       mbar_arrive(&q_ready);
     }
     constexpr int COLS = TC_BN / 2;  // key columns per thread
-    constexpr int OCOLS = HD / 2;    // output columns per thread
+    constexpr int OCOLS = VD / 2;    // output columns per thread
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     float m_used = -INFINITY;  // the maximum (log2 units) that P, O and the sums are scaled by
     float l = 0.f;             // this thread's share of the row's sum
@@ -236,13 +244,18 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
 #pragma unroll
       for (int j = 0; j < COLS; ++j) s[j] = cap_score(s[j], p.cap_in, p.cap_out);
 #endif
-      const int j0 = (jb0 + i) * TC_BN + half * COLS;
-      const bool all_visible = row_ok && j0 + COLS - 1 <= my_pos && j0 >= my_lo;
+      const int j0 = walk.block(jb0 + i) * TC_BN + half * COLS;
+#ifdef DISTANCE_BIAS
+      const float bias0 = slope * (float)(j0 - my_pos);
+#pragma unroll
+      for (int j = 0; j < COLS; ++j) s[j] += fmaf(slope, (float)j, bias0);
+#endif
+      const bool all_visible = row_ok && j0 + COLS - 1 <= my_pos && (j0 >= my_lo || j0 + COLS <= p.keep);
       if (!all_visible) {
 #pragma unroll
         for (int j = 0; j < COLS; ++j) {
           const int kj = j0 + j;
-          if (!row_ok || kj > my_pos || kj < my_lo) s[j] = -INFINITY;
+          if (!row_ok || kj > my_pos || (kj < my_lo && kj >= p.keep)) s[j] = -INFINITY;
         }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};  // four chains, not one of 64
@@ -328,8 +341,9 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
     l += row_max[0][half ^ 1][r];
     if (ok) {
       tc_fence_after();
-      const float inv = 1.0f / (l + sink_term(p.sink, kvh * g + (row_ok ? R % g : 0), m_used));
-      bf16* dst = p.out + ((size_t)(row_begin + (row_ok ? R / g : 0)) * p.nh + kvh * g + (row_ok ? R % g : 0)) * HD + half * OCOLS;
+      const int token = row_begin + (row_ok ? R / g : 0), head = kvh * g + (row_ok ? R % g : 0);
+      const float inv = gate_of_head(p.gate, p.gate_ld, token, head) / (l + sink_term(p.sink, head, m_used));
+      bf16* dst = p.out + ((size_t)token * p.nh + head) * VD + half * OCOLS;
 #pragma unroll
       for (int c0 = 0; c0 < OCOLS; c0 += 16) {
         uint32_t v[16];
@@ -354,14 +368,14 @@ __global__ void __launch_bounds__(TC_THREADS, 1) attention_prefill_tc_kernel(con
 // Launch for a step with prompt portions; false when the shapes are not the kernel's.
 static bool launch_prefill_tc(const AttnParams& p, const void* k_cache, const void* v_cache, long long cache_slots, int tiles64, int nkv, int n_seqs,
                               int max_kv_len, cudaStream_t stream, int* rc) {
-  if (!(HD == 64 || HD == 128) || p.page_size % 64 != 0 || cache_slots <= 0) return false;
+  if (!TMA_SIZES || p.page_size % 64 != 0 || cache_slots <= 0) return false;
   if (((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) || ((uintptr_t)p.q & 15) || ((uintptr_t)p.out & 15)) return false;
-  const int entries = max_kv_len / p.page_size + 2;
+  const int entries = max_kv_len / p.page_size + 2;  // enough for the kept keys' entries too: they are among the request's
   const size_t smem = prefill_tc_smem_bytes(entries);
   if (smem > 220 * 1024) return false;
   CUtensorMap map_k, map_v;
   if (!make_tensor_map_bf16(&map_k, k_cache, (uint64_t)cache_slots, (uint64_t)nkv * HD, 64, 64) ||
-      !make_tensor_map_bf16(&map_v, v_cache, (uint64_t)cache_slots, (uint64_t)nkv * HD, 64, 64))
+      !make_tensor_map_bf16(&map_v, v_cache, (uint64_t)cache_slots, (uint64_t)nkv * VD, 64, 64))
     return false;
   static bool configured = false;
   if (!configured) {

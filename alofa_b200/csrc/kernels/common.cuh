@@ -50,6 +50,27 @@ __device__ __forceinline__ float silu_times(float g, float u) {
   return g * r * u;
 }
 
+// What a gated product makes of its two sums.  alpha == 0: silu(g) * u.  alpha > 0: the clamped form, g and u held to
+// `limit` (g from above only) and then g * sigmoid(alpha g) * (u + 1).  gate_times uses the library functions (the 32-bit
+// path), fast_gate_times the hardware approximations of silu_times (the bfloat16 kernels).
+__device__ __forceinline__ float gate_times(float g, float u, float alpha, float limit) {
+  if (alpha == 0.f) return g / (1.0f + expf(-g)) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+__device__ __forceinline__ float clamped_gate_times(float g, float u, float alpha, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * alpha * g));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return g * r * (u + 1.0f);
+}
+__device__ __forceinline__ float fast_gate_times(float g, float u, float alpha, float limit) {
+  return alpha == 0.f ? silu_times(g, u) : clamped_gate_times(g, u, alpha, limit);
+}
+
 // Activations that an epilogue may apply to its fp32 sums (after the bias): the precise library
 // functions, the same in every kernel that takes an activation code.
 enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_RELU = 4, ACT_RELU_SQUARED = 5 };

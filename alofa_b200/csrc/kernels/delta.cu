@@ -6,7 +6,7 @@
 //   c = x + 1/2 where x >= 0 and sigmoid(x) where x < 0; the output is S_t * silu(gate).
 //
 // The gated delta rule over a matrix state per head (N key channels x P value channels), with one
-// decay per head and key channel:
+// decay per head and key channel, or one per head (g_t then is a number):
 //   S <- diag(g_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 // so the read-out sees the token's own write.  A value channel's column of S never meets another
 // column: o_t[p] = (g S[:, p]) . q + u[p] (k . q), and u[p] needs (g S[:, p]) . k.  Both dot
@@ -113,14 +113,14 @@ ALOFA_API int alofa_min_gru(void* out, const float* u, int ld, int z_off, int x_
 // u [T, ldu] the gate logit of each head at column b_off.
 //   qn = q / sqrt(sum(q^2) + unit_eps) * q_scale,  kn = k / sqrt(sum(k^2) + unit_eps)   per group
 //   kq[t, g] = kn . qn
-//   g[t, h, n] = exp(-exp(A_log[h]) * softplus(dz[t, h, n] + dt_bias[h, n]))
+//   g[t, h, n] = exp(-exp(A_log[h]) * softplus(dz[t, h, n] + dt_bias[h, n]))      (ND = N decays a head, or ND = 1: g[t, h])
 //   beta[t, h] = sigmoid(u[t, b_off + h])
 // One block per token, a warp per group in turn.
 // ---------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) delta_prepare_kernel(float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ kq, float* __restrict__ g,
                                                             float* __restrict__ beta, const float* __restrict__ conv, int ldc, const float* __restrict__ dz, int ldz,
                                                             const float* __restrict__ u, int ldu, int b_off, const float* __restrict__ dt_bias,
-                                                            const float* __restrict__ A_log, int H, int G, int N, float unit_eps, float q_scale) {
+                                                            const float* __restrict__ A_log, int H, int G, int N, int ND, float unit_eps, float q_scale) {
   pdl_begin();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
   const float* row = conv + (size_t)t * ldc;
@@ -145,19 +145,19 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(float* __restrict__ 
     dot = warp_sum(dot);
     if (lane == 0) kq[(size_t)t * G + grp] = dot;
   }
-  for (int e = threadIdx.x; e < H * N; e += blockDim.x) {
-    const int h = e / N;
-    g[(size_t)t * H * N + e] = expf(-expf(A_log[h]) * softplus_f(dz[(size_t)t * ldz + e] + dt_bias[e]));
+  for (int e = threadIdx.x; e < H * ND; e += blockDim.x) {
+    const int h = e / ND;
+    g[(size_t)t * H * ND + e] = expf(-expf(A_log[h]) * softplus_f(dz[(size_t)t * ldz + e] + dt_bias[e]));
   }
   for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(size_t)t * H + h] = sigmoid_f(u[(size_t)t * ldu + b_off + h]);
 }
 
 ALOFA_API int alofa_delta_prepare(float* qn, float* kn, float* kq, float* g, float* beta, const float* conv, int ldc, const float* dz, int ldz, const float* u, int ldu,
-                                  int b_off, const float* dt_bias, const float* A_log, int n_tokens, int H, int G, int N, float unit_eps, float q_scale,
+                                  int b_off, const float* dt_bias, const float* A_log, int n_tokens, int H, int G, int N, int ND, float unit_eps, float q_scale,
                                   cudaStream_t stream) {
   if (n_tokens <= 0) return ALOFA_OK;
-  if (H <= 0 || G <= 0 || H % G || N <= 0) return ALOFA_ERR_ARGUMENT;
-  launch_dep(delta_prepare_kernel, n_tokens, 256, 0, stream, qn, kn, kq, g, beta, conv, ldc, dz, ldz, u, ldu, b_off, dt_bias, A_log, H, G, N, unit_eps, q_scale);
+  if (H <= 0 || G <= 0 || H % G || N <= 0 || (ND != N && ND != 1)) return ALOFA_ERR_ARGUMENT;
+  launch_dep(delta_prepare_kernel, n_tokens, 256, 0, stream, qn, kn, kq, g, beta, conv, ldc, dz, ldz, u, ldu, b_off, dt_bias, A_log, H, G, N, ND, unit_eps, q_scale);
   return launch_status();
 }
 
@@ -169,14 +169,14 @@ ALOFA_API int alofa_delta_prepare(float* qn, float* kn, float* kq, float* g, flo
 // 16 bytes each, and the NS threads' loads lie side by side in shared memory).  The state lies
 // in memory as [head][value channel][key channel].  Keys, queries, decays, values, beta and k . q
 // of TC tokens at a time come into shared memory by asynchronous copies, the next ones while
-// these are worked on.
+// these are worked on.  ONE: one decay per head: it travels beside beta and k . q and multiplies the column.
 // ---------------------------------------------------------------------------
 struct DeltaArgs {
   float* y;                              // [T, H * P]
   const float* v; int ldv, v_off;        // values: v[t * ldv + v_off + h * P + p]
   const float* kn; const float* qn;      // [T, G, N]
   const float* kq;                       // [T, G]
-  const float* g;                        // [T, H, N]
+  const float* g;                        // [T, H, N], ONE: [T, H]
   const float* beta;                     // [T, H]
   float* state; long long slot_stride;
   const int* q_start; const int* state_slots;
@@ -194,12 +194,12 @@ __device__ __forceinline__ void delta_cp_done() {
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
-template <int R>
+template <int R, bool ONE>
 __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
   extern __shared__ __align__(16) float delta_smem[];
   const int N = a.N, P = a.P, NS = a.NS, PC = a.PC, TC = a.TC;
   const int NW = NS * R;                       // key channels a stage holds per token (zeros past N)
-  const int per_stage = TC * (3 * NW + PC + 4);  // k, q, g, v, then beta and k.q (two words, padded to four)
+  const int per_stage = TC * ((ONE ? 2 : 3) * NW + PC + 4);  // k, q, g (unless ONE), v, then beta, k.q and (ONE) the decay (padded to four words)
   const int h = blockIdx.x, s = blockIdx.y, p0 = blockIdx.z * PC;
   const int tid = threadIdx.x, nthreads = blockDim.x;
   const int pl = tid / NS, ns = tid - pl * NS;
@@ -222,7 +222,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
     float* ks = delta_smem + which * per_stage;
     float* qs = ks + TC * NW;
     float* gs = qs + TC * NW;
-    float* vs = gs + TC * NW;
+    float* vs = ONE ? gs : gs + TC * NW;
     float* bs = vs + TC * PC;
     const int live = min(TC, t1 - c0);
     if (a.vec) {
@@ -232,7 +232,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
         const size_t t = c0 + tt;
         delta_cp16(ks + tt * NW + c, a.kn + (t * a.G + grp) * N + c);
         delta_cp16(qs + tt * NW + c, a.qn + (t * a.G + grp) * N + c);
-        delta_cp16(gs + tt * NW + c, a.g + (t * a.H + h) * N + c);
+        if (!ONE) delta_cp16(gs + tt * NW + c, a.g + (t * a.H + h) * N + c);
       }
       const int p4 = PC >> 2;
       for (int e = tid; e < live * p4; e += nthreads) {
@@ -245,7 +245,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
         const size_t t = c0 + tt;
         delta_cp4(ks + tt * NW + c, a.kn + (t * a.G + grp) * N + c);
         delta_cp4(qs + tt * NW + c, a.qn + (t * a.G + grp) * N + c);
-        delta_cp4(gs + tt * NW + c, a.g + (t * a.H + h) * N + c);
+        if (!ONE) delta_cp4(gs + tt * NW + c, a.g + (t * a.H + h) * N + c);
       }
       for (int e = tid; e < live * PC; e += nthreads) {
         const int tt = e / PC, c = e - tt * PC;
@@ -255,6 +255,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
     for (int tt = tid; tt < live; tt += nthreads) {
       delta_cp4(bs + 4 * tt, a.beta + (size_t)(c0 + tt) * a.H + h);
       delta_cp4(bs + 4 * tt + 1, a.kq + (size_t)(c0 + tt) * a.G + grp);
+      if (ONE) delta_cp4(bs + 4 * tt + 2, a.g + (size_t)(c0 + tt) * a.H + h);
     }
   };
 
@@ -268,17 +269,18 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
     const float* ks = delta_smem + which * per_stage;
     const float* qs = ks + TC * NW;
     const float* gs = qs + TC * NW;
-    const float* vs = gs + TC * NW;
+    const float* vs = ONE ? gs : gs + TC * NW;
     const float* bs = vs + TC * PC;
     for (int tt = 0; tt < live; ++tt) {
       const float4* kr = reinterpret_cast<const float4*>(ks + tt * NW) + ns;
       const float4* qr = reinterpret_cast<const float4*>(qs + tt * NW) + ns;
       const float4* gr = reinterpret_cast<const float4*>(gs + tt * NW) + ns;
+      const float decay = ONE ? bs[4 * tt + 2] : 0.f;
       float kk[R];
       float r0 = 0.f, r1 = 0.f, w0 = 0.f, w1 = 0.f;
 #pragma unroll
       for (int j4 = 0; j4 < R / 4; ++j4) {
-        const float4 k4 = kr[j4 * NS], q4 = qr[j4 * NS], g4 = gr[j4 * NS];
+        const float4 k4 = kr[j4 * NS], q4 = qr[j4 * NS], g4 = ONE ? make_float4(decay, decay, decay, decay) : gr[j4 * NS];
         const int j = 4 * j4;
         kk[j] = k4.x, kk[j + 1] = k4.y, kk[j + 2] = k4.z, kk[j + 3] = k4.w;
         st[j] *= g4.x, st[j + 1] *= g4.y, st[j + 2] *= g4.z, st[j + 3] *= g4.w;
@@ -312,21 +314,21 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
   }
 }
 
-template <int R>
+template <int R, bool ONE>
 static int delta_scan_launch(const DeltaArgs& a, int n_seqs, int threads, size_t smem, cudaStream_t stream) {
   static size_t set = 48 * 1024;
   if (smem > set) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
+    if (cudaFuncSetAttribute(delta_scan_kernel<R, ONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
     set = smem;
   }
-  launch_dep(delta_scan_kernel<R>, dim3(a.H, n_seqs, (a.P + a.PC - 1) / a.PC), threads, smem, stream, a);
+  launch_dep(delta_scan_kernel<R, ONE>, dim3(a.H, n_seqs, (a.P + a.PC - 1) / a.PC), threads, smem, stream, a);
   return launch_status();
 }
 
-// spread: how many blocks the scan should have at least, if the value channels allow it.
+// one_decay: g is [T, H], one decay per head.  spread: how many blocks the scan should have at least, if the value channels allow it.
 ALOFA_API int alofa_delta_scan(float* y, const float* v, int ldv, int v_off, const float* kn, const float* qn, const float* kq, const float* g, const float* beta,
                                float* state, long long slot_stride, const int* q_start, const int* state_slots, int n_tokens, int n_seqs, int H, int G, int N, int P,
-                               int spread, cudaStream_t stream) {
+                               int one_decay, int spread, cudaStream_t stream) {
   if (n_seqs <= 0 || n_tokens <= 0) return ALOFA_OK;
   if (H <= 0 || G <= 0 || H % G || N <= 0 || N > 1024 || P <= 0) return ALOFA_ERR_ARGUMENT;
   int R = N <= 64 ? 8 : (N <= 256 ? 16 : 32);
@@ -345,13 +347,19 @@ ALOFA_API int alofa_delta_scan(float* y, const float* v, int ldv, int v_off, con
   if (PC < 4) PC = 4;
   const int threads = (PC * NS + 31) / 32 * 32;
   const bool vec = N % 4 == 0 && P % 4 == 0 && PC % 4 == 0 && ldv % 4 == 0 && v_off % 4 == 0 && ((uintptr_t)v % 16 == 0) && ((uintptr_t)kn % 16 == 0) &&
-                   ((uintptr_t)qn % 16 == 0) && ((uintptr_t)g % 16 == 0);
+                   ((uintptr_t)qn % 16 == 0) && (one_decay || (uintptr_t)g % 16 == 0);
   int TC = 16;
-  while (TC > 2 && (size_t)2 * TC * (3 * NS * R + PC + 4) * sizeof(float) > 160 * 1024) TC /= 2;
-  const size_t smem = (size_t)2 * TC * (3 * NS * R + PC + 4) * sizeof(float);
+  const int wide = one_decay ? 2 : 3;  // rows of N numbers a token brings
+  while (TC > 2 && (size_t)2 * TC * (wide * NS * R + PC + 4) * sizeof(float) > 160 * 1024) TC /= 2;
+  const size_t smem = (size_t)2 * TC * (wide * NS * R + PC + 4) * sizeof(float);
   if (smem > 200 * 1024) return ALOFA_ERR_ARGUMENT;
   DeltaArgs a = {y, v, ldv, v_off, kn, qn, kq, g, beta, state, slot_stride, q_start, state_slots, H, G, N, P, NS, PC, TC, vec ? 1 : 0};
-  if (R == 8) return delta_scan_launch<8>(a, n_seqs, threads, smem, stream);
-  if (R == 16) return delta_scan_launch<16>(a, n_seqs, threads, smem, stream);
-  return delta_scan_launch<32>(a, n_seqs, threads, smem, stream);
+  if (one_decay) {
+    if (R == 8) return delta_scan_launch<8, true>(a, n_seqs, threads, smem, stream);
+    if (R == 16) return delta_scan_launch<16, true>(a, n_seqs, threads, smem, stream);
+    return delta_scan_launch<32, true>(a, n_seqs, threads, smem, stream);
+  }
+  if (R == 8) return delta_scan_launch<8, false>(a, n_seqs, threads, smem, stream);
+  if (R == 16) return delta_scan_launch<16, false>(a, n_seqs, threads, smem, stream);
+  return delta_scan_launch<32, false>(a, n_seqs, threads, smem, stream);
 }

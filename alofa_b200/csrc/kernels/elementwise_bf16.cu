@@ -5,7 +5,8 @@
 //
 //   alofa_norm_fused        h += bias + sum_z partial[z]  (optional), then
 //                           x = h / sqrt(mean(h^2) + eps) * w      (RMSNorm,
-//                           src/alofa/kernels/cpu/scalar.mojo:93-129)
+//                           src/alofa/kernels/cpu/scalar.mojo:93-129), or with a shift
+//                           x = (h - mean) / sqrt(variance + eps) * w + shift  (layer norm)
 //   alofa_stream_settle     h = base + accumulator: the residual stream of a small decode
 //                           step brought back to one fp32 tensor (see STREAM_SCALE)
 //   alofa_rope_store_fused  qkv = bias + sum_z partial[z] (or a bf16 tensor),
@@ -70,7 +71,7 @@ __global__ void __launch_bounds__(256) norm_fused_kernel(TO* __restrict__ out, f
                                                          const float* __restrict__ partial, const float* __restrict__ bias,
                                                          const int* __restrict__ rows, int n_tokens, int hidden, int splits, float eps,
                                                          const float* __restrict__ base, long long* __restrict__ acc,
-                                                         long long* __restrict__ other) {
+                                                         long long* __restrict__ other, const float* __restrict__ shift) {
   extern __shared__ float row_buf[];  // hidden floats
   __shared__ float scratch[32];
   const int n4 = hidden >> 2;
@@ -83,7 +84,7 @@ __global__ void __launch_bounds__(256) norm_fused_kernel(TO* __restrict__ out, f
   float4* hr = reinterpret_cast<float4*>(h + (size_t)src * hidden);
   const float4* br = base ? reinterpret_cast<const float4*>(base + (size_t)src * hidden) : hr;
   const size_t plane4 = ((size_t)n_tokens * hidden) >> 2;
-  float ss = 0.f;
+  float ss = 0.f, sum = 0.f;
   for (int c = threadIdx.x; c < n4; c += blockDim.x) {
     float4 v = br[c];
     if (acc) {
@@ -123,14 +124,32 @@ __global__ void __launch_bounds__(256) norm_fused_kernel(TO* __restrict__ out, f
     ss = fmaf(v.y, v.y, ss);
     ss = fmaf(v.z, v.z, ss);
     ss = fmaf(v.w, v.w, ss);
+    sum += (v.x + v.y) + (v.z + v.w);
   }
   pdl_launch();
+  float mean = 0.f;
+  if (shift) {  // the squared deviations from the mean, in a second pass over what this thread left in shared memory
+    mean = block_sum(sum, scratch) / (float)hidden;
+    ss = 0.f;
+    for (int c = threadIdx.x; c < n4; c += blockDim.x) {
+      const float4 v = reinterpret_cast<float4*>(row_buf)[c];
+      const float a = v.x - mean, b = v.y - mean, d = v.z - mean, e = v.w - mean;
+      ss = fmaf(a, a, ss);
+      ss = fmaf(b, b, ss);
+      ss = fmaf(d, d, ss);
+      ss = fmaf(e, e, ss);
+    }
+  }
   ss = block_sum(ss, scratch);
   const float scale = 1.0f / sqrtf(ss / (float)hidden + eps);
   for (int c = threadIdx.x; c < n4; c += blockDim.x) {
     const float4 v = reinterpret_cast<float4*>(row_buf)[c];
     const float4 g = c == (int)threadIdx.x ? g_first : reinterpret_cast<const float4*>(w)[c];
-    const float y0 = v.x * scale * g.x, y1 = v.y * scale * g.y, y2 = v.z * scale * g.z, y3 = v.w * scale * g.w;
+    float y0 = (v.x - mean) * scale * g.x, y1 = (v.y - mean) * scale * g.y, y2 = (v.z - mean) * scale * g.z, y3 = (v.w - mean) * scale * g.w;
+    if (shift) {
+      const float4 b = reinterpret_cast<const float4*>(shift)[c];
+      y0 += b.x, y1 += b.y, y2 += b.z, y3 += b.w;
+    }
     if (sizeof(TO) == 2) {
       __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
       uint2 packed = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
@@ -149,7 +168,7 @@ template <typename TO, int CHUNKS>
 __global__ void __launch_bounds__(256) norm_rows_kernel(TO* __restrict__ out, float* __restrict__ h, const float* __restrict__ w,
                                                         const float* __restrict__ partial, const float* __restrict__ bias,
                                                         const int* __restrict__ rows, int n_rows, int n_tokens, int hidden, int splits,
-                                                        float eps) {
+                                                        float eps, const float* __restrict__ shift) {
   pdl_begin();
   const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= n_rows) return;
@@ -187,6 +206,16 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(TO* __restrict__ out, fl
       }
     }
   }
+  float mean = 0.f;
+  if (shift) {  // layer norm: deviations from the row's mean (groups past the row's end stay zero)
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    mean = warp_sum(sum) / (float)hidden;
+#pragma unroll
+    for (int i = 0; i < CHUNKS; ++i)
+      if (lane + i * 32 < n4) v[i].x -= mean, v[i].y -= mean, v[i].z -= mean, v[i].w -= mean;
+  }
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < CHUNKS; ++i) {
@@ -202,7 +231,11 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(TO* __restrict__ out, fl
     const int c = lane + i * 32;
     if (c >= n4) break;
     const float4 g = reinterpret_cast<const float4*>(w)[c];
-    const float y0 = v[i].x * scale * g.x, y1 = v[i].y * scale * g.y, y2 = v[i].z * scale * g.z, y3 = v[i].w * scale * g.w;
+    float y0 = v[i].x * scale * g.x, y1 = v[i].y * scale * g.y, y2 = v[i].z * scale * g.z, y3 = v[i].w * scale * g.w;
+    if (shift) {
+      const float4 b = reinterpret_cast<const float4*>(shift)[c];
+      y0 += b.x, y1 += b.y, y2 += b.z, y3 += b.w;
+    }
     if (sizeof(TO) == 2) {
       __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
       reinterpret_cast<uint2*>(out + (size_t)r * hidden)[c] = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
@@ -214,45 +247,45 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(TO* __restrict__ out, fl
 
 template <typename TO, int CHUNKS>
 static void launch_norm_rows(TO* out, float* h, const float* w, const float* partial, const float* bias, const int* rows, int n_rows,
-                             int n_tokens, int hidden, int splits, float eps, cudaStream_t stream) {
+                             int n_tokens, int hidden, int splits, float eps, const float* shift, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
     prefer_max_shared(norm_rows_kernel<TO, CHUNKS>);
     configured = true;
   }
-  launch_dep(norm_rows_kernel<TO, CHUNKS>, (unsigned)((n_rows + 7) / 8), 256, 0, stream, out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps);
+  launch_dep(norm_rows_kernel<TO, CHUNKS>, (unsigned)((n_rows + 7) / 8), 256, 0, stream, out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift);
 }
 template <typename TO>
 static void dispatch_norm_rows(TO* out, float* h, const float* w, const float* partial, const float* bias, const int* rows, int n_rows,
-                               int n_tokens, int hidden, int splits, float eps, cudaStream_t stream) {
-  if (hidden <= 1024) launch_norm_rows<TO, 8>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, stream);
-  else if (hidden <= 2048) launch_norm_rows<TO, 16>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, stream);
-  else launch_norm_rows<TO, 32>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, stream);
+                               int n_tokens, int hidden, int splits, float eps, const float* shift, cudaStream_t stream) {
+  if (hidden <= 1024) launch_norm_rows<TO, 8>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift, stream);
+  else if (hidden <= 2048) launch_norm_rows<TO, 16>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift, stream);
+  else launch_norm_rows<TO, 32>(out, h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift, stream);
 }
 
 // base (optional): the rows are read from `base` instead of h (h is written, complete).  acc
 // (optional, with rows == nullptr only): a fixed-point accumulator [n_tokens, hidden] added on
-// top and left zero, as is `other`.
+// top and left zero, as is `other`.  shift (optional): layer norm, else RMSNorm.
 ALOFA_API int alofa_norm_fused(void* out, void* h, const float* w, const float* partial, const float* bias, const int* rows, int n_rows,
                                int n_tokens, int hidden, int splits, float eps, int out_bf16, const float* base, long long* acc,
-                               long long* other, cudaStream_t stream) {
+                               long long* other, const float* shift, cudaStream_t stream) {
   if (n_rows <= 0) return ALOFA_OK;
   if (hidden % 4 != 0 || hidden > 12288) return ALOFA_ERR_ARGUMENT;
   if ((acc || base) && (rows || n_rows != n_tokens)) return ALOFA_ERR_ARGUMENT;
   if (n_rows >= 256 && hidden <= 4096 && !acc && !base) {  // many rows: a warp each, the row in registers
     if (out_bf16)
-      dispatch_norm_rows<bf16>((bf16*)out, (float*)h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, stream);
+      dispatch_norm_rows<bf16>((bf16*)out, (float*)h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift, stream);
     else
-      dispatch_norm_rows<float>((float*)out, (float*)h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, stream);
+      dispatch_norm_rows<float>((float*)out, (float*)h, w, partial, bias, rows, n_rows, n_tokens, hidden, splits, eps, shift, stream);
     return launch_status();
   }
   const size_t smem = (size_t)hidden * sizeof(float);
   ALOFA_PREFER_MAX_SHARED(norm_fused_kernel<bf16>);
   ALOFA_PREFER_MAX_SHARED(norm_fused_kernel<float>);
   if (out_bf16)
-    launch_dep(norm_fused_kernel<bf16>, n_rows, 256, smem, stream, (bf16*)out, (float*)h, w, partial, bias, rows, n_tokens, hidden, splits, eps, base, acc, other);
+    launch_dep(norm_fused_kernel<bf16>, n_rows, 256, smem, stream, (bf16*)out, (float*)h, w, partial, bias, rows, n_tokens, hidden, splits, eps, base, acc, other, shift);
   else
-    launch_dep(norm_fused_kernel<float>, n_rows, 256, smem, stream, (float*)out, (float*)h, w, partial, bias, rows, n_tokens, hidden, splits, eps, base, acc, other);
+    launch_dep(norm_fused_kernel<float>, n_rows, 256, smem, stream, (float*)out, (float*)h, w, partial, bias, rows, n_tokens, hidden, splits, eps, base, acc, other, shift);
   return launch_status();
 }
 

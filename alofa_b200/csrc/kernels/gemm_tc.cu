@@ -12,7 +12,7 @@
 // accumulator with tcgen05.ld (lane = feature) and write it out:
 //   EPI_STORE    out[t, f] = acc + bias[f]                (bf16 or fp32)
 //   EPI_RESIDUAL out[t, f] += acc + bias[f]               (fp32 residual stream)
-//   EPI_GATED    W = [gate; up]: out[t, f] = silu(g) * u  (two accumulators)
+//   EPI_GATED    W = [gate; up]: out[t, f] = silu(g) * u  (two accumulators), or the clamped form (fast_gate_times)
 //   EPI_PARTIAL  ws[z, t, f] = acc                        (split-K; see reduce)
 //   EPI_ROPE     W = [q; k; v]: bias, NeoX rotation of q and k, q to its buffer,
 //                k and v to their cache slots
@@ -79,6 +79,7 @@ struct GemmArgs {
   int k_slices_per_split;
   int out_bf16;
   int act;            // EPI_STORE: an activation on the sums plus bias (codes of common.cuh), 0 for none
+  float gate_alpha, gate_limit;  // EPI_GATED: the form of the gate (fast_gate_times)
   // Tokens on M, EPI_STORE, by tile: the weight is [batches * N, K] and the token tile i (128 rows)
   // multiplies by the rows of batch tile_batch[i], negative: the tile is empty (the experts of a routed
   // feed-forward, rows sorted by expert and padded to whole tiles; the array is written on the device)
@@ -491,7 +492,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           if (N_ACC == 2) p[plane] = __uint_as_float(r1[j]);
         } else if (EPI == EPI_GATED) {
           const float g = a0 + bias0, u = __uint_as_float(r1[j]) + bias1;
-          const float y = silu_times(g, u);
+          const float y = fast_gate_times(g, u, args.gate_alpha, args.gate_limit);
           if (args.out_bf16) ((bf16*)args.out)[(size_t)t * args.N + f] = __float2bfloat16_rn(y);
           else ((float*)args.out)[(size_t)t * args.N + f] = y;
         } else {
@@ -704,16 +705,25 @@ __device__ __forceinline__ void tokens_epilogue_staged(const GemmArgs& args, uin
       if (GATED) tmem_ld16(taddr + FEATS, r1);
       tmem_ld_wait();
       float v[16];
+      if (GATED && args.gate_alpha != 0.f) {  // the clamped form of the gate, outside the loop of the usual one
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        float a = __uint_as_float(r0[j]);
-        if (!split && args.bias && f + j < N) a += args.bias[f + j];
-        if (GATED) {
-          float u = __uint_as_float(r1[j]);
-          if (args.bias && f + j < N) u += args.bias[N + f + j];
-          a = silu_times(a, u);
+        for (int j = 0; j < 16; ++j) {
+          float a = __uint_as_float(r0[j]), u = __uint_as_float(r1[j]);
+          if (args.bias && f + j < N) a += args.bias[f + j], u += args.bias[N + f + j];
+          v[j] = clamped_gate_times(a, u, args.gate_alpha, args.gate_limit);
         }
-        v[j] = a;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          float a = __uint_as_float(r0[j]);
+          if (!split && args.bias && f + j < N) a += args.bias[f + j];
+          if (GATED) {
+            float u = __uint_as_float(r1[j]);
+            if (args.bias && f + j < N) u += args.bias[N + f + j];
+            a = silu_times(a, u);
+          }
+          v[j] = a;
+        }
       }
       if (EPI == EPI_STORE && !split && args.act) {
 #pragma unroll
@@ -945,7 +955,7 @@ gemm_tc_tokens_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
         }
         if (GATED) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = silu_times(v[j], u[j]);
+          for (int j = 0; j < 16; ++j) v[j] = fast_gate_times(v[j], u[j], args.gate_alpha, args.gate_limit);
         }
         if (EPI == EPI_STORE && args.act) {
 #pragma unroll
@@ -1307,7 +1317,7 @@ gemm_tc_tokens_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
 // ---------------------------------------------------------------------------
 template <int EPI>
 __global__ void splitk_reduce_kernel(void* __restrict__ out, const float* __restrict__ partial, const float* __restrict__ bias, int T, int N,
-                                     int splits, int out_bf16, int act) {
+                                     int splits, int out_bf16, int act, float gate_alpha, float gate_limit) {
   constexpr int N_ACC = (EPI == EPI_GATED) ? 2 : 1;
   const size_t plane = (size_t)T * N;
   pdl_begin();
@@ -1335,7 +1345,7 @@ __global__ void splitk_reduce_kernel(void* __restrict__ out, const float* __rest
   }
   float y = a0;
   if (EPI == EPI_STORE && act) y = activate_out_of_line(a0, act);
-  if (EPI == EPI_GATED) y = silu_times(a0, a1);
+  if (EPI == EPI_GATED) y = fast_gate_times(a0, a1, gate_alpha, gate_limit);
   if (EPI == EPI_RESIDUAL) {
     ((float*)out)[idx] += y;
   } else if (out_bf16) {
@@ -1624,7 +1634,7 @@ ALOFA_API int alofa_gemm_tc(void* out, const void* x, const void* w, const float
                             int bn, int splits, int do_reduce, int* status, int b_kind, const float* b_src, const float* b_ml,
                             const int* b_positions, int b_heads, int b_head_dim, int b_window, int b_split_keys, long long* acc,
                             const long long* n_acc, const float* n_gamma, float n_eps, float* n_out, long long* n_zero, const int* tile_batch,
-                            int batches, cudaStream_t stream) {
+                            int batches, float gate_alpha, float gate_limit, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return ALOFA_OK;
   const int act = epi >> 4;  // EPI_STORE | (code << 4): an activation on the sums plus bias
   epi &= 15;
@@ -1675,6 +1685,8 @@ ALOFA_API int alofa_gemm_tc(void* out, const void* x, const void* w, const float
   splits = (total_slices + args.k_slices_per_split - 1) / args.k_slices_per_split;  // no empty split
   args.out_bf16 = out_bf16;
   args.act = act;
+  args.gate_alpha = gate_alpha;
+  args.gate_limit = gate_limit;
   args.tile_batch = tile_batch;
   args.pair = pair ? 1 : 0;
   args.few = few;
@@ -1709,16 +1721,16 @@ ALOFA_API int alofa_gemm_tc(void* out, const void* x, const void* w, const float
   const size_t plane = (size_t)T * N;
   const int threads = 256;
   const unsigned blocks = (unsigned)((plane + threads - 1) / threads);
-  if (epi == EPI_STORE) launch_dep(splitk_reduce_kernel<EPI_STORE>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
-  else if (epi == EPI_RESIDUAL) launch_dep(splitk_reduce_kernel<EPI_RESIDUAL>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
-  else launch_dep(splitk_reduce_kernel<EPI_GATED>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
+  if (epi == EPI_STORE) launch_dep(splitk_reduce_kernel<EPI_STORE>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
+  else if (epi == EPI_RESIDUAL) launch_dep(splitk_reduce_kernel<EPI_RESIDUAL>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
+  else launch_dep(splitk_reduce_kernel<EPI_GATED>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
   return launch_status();
 }
 
 // The second stage alone: out (op)= bias + sum_z partial[z], for partial sums a
 // deferred product left behind.
 ALOFA_API int alofa_splitk_reduce(void* out, const float* partial, const float* bias, int T, int N, int splits, int epi, int out_bf16,
-                                  cudaStream_t stream) {
+                                  float gate_alpha, float gate_limit, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return ALOFA_OK;
   const int act = epi >> 4;
   epi &= 15;
@@ -1726,9 +1738,9 @@ ALOFA_API int alofa_splitk_reduce(void* out, const float* partial, const float* 
   const size_t plane = (size_t)T * N;
   const int threads = 256;
   const unsigned blocks = (unsigned)((plane + threads - 1) / threads);
-  if (epi == EPI_STORE) launch_dep(splitk_reduce_kernel<EPI_STORE>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
-  else if (epi == EPI_RESIDUAL) launch_dep(splitk_reduce_kernel<EPI_RESIDUAL>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
-  else if (epi == EPI_GATED) launch_dep(splitk_reduce_kernel<EPI_GATED>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act);
+  if (epi == EPI_STORE) launch_dep(splitk_reduce_kernel<EPI_STORE>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
+  else if (epi == EPI_RESIDUAL) launch_dep(splitk_reduce_kernel<EPI_RESIDUAL>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
+  else if (epi == EPI_GATED) launch_dep(splitk_reduce_kernel<EPI_GATED>, blocks, threads, 0, stream, out, partial, bias, T, N, splits, out_bf16, act, gate_alpha, gate_limit);
   else return ALOFA_ERR_ARGUMENT;
   return launch_status();
 }

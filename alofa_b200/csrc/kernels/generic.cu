@@ -46,31 +46,39 @@ ALOFA_API int alofa_embed_gather(void* out, const void* table, const int* ids, c
 
 // ---------------------------------------------------------------------------
 // RMSNorm: y = x * (1/sqrt(mean(x^2) + eps)) * w, one block per output row.
-// `rows` (optional) picks the input row of each output row.
+// `rows` (optional) picks the input row of each output row.  With `shift`
+// (optional) the layer norm instead: y = (x - mean) / sqrt(variance + eps) * w +
+// shift, the variance being the mean of the squared deviations.
 // ---------------------------------------------------------------------------
 template <typename TO>
 __global__ void rmsnorm_kernel(TO* __restrict__ out, const float* __restrict__ x, const float* __restrict__ w,
-                               const int* __restrict__ rows, int hidden, float eps) {
+                               const float* __restrict__ shift, const int* __restrict__ rows, int hidden, float eps) {
   __shared__ float scratch[32];
   const int r = blockIdx.x;
   const float* xr = x + (size_t)(rows ? rows[r] : r) * hidden;
+  float mean = 0.f;
+  if (shift) {
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) mean += xr[c];
+    mean = block_sum(mean, scratch) / (float)hidden;
+  }
   float ss = 0.f;
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-    const float v = xr[c];
+    const float v = xr[c] - mean;
     ss = fmaf(v, v, ss);
   }
   ss = block_sum(ss, scratch);
   const float scale = 1.0f / sqrtf(ss / (float)hidden + eps);
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) out[(size_t)r * hidden + c] = from_f<TO>(xr[c] * scale * w[c]);
+  if (shift) for (int c = threadIdx.x; c < hidden; c += blockDim.x) out[(size_t)r * hidden + c] = from_f<TO>((xr[c] - mean) * scale * w[c] + shift[c]);
+  else for (int c = threadIdx.x; c < hidden; c += blockDim.x) out[(size_t)r * hidden + c] = from_f<TO>(xr[c] * scale * w[c]);
 }
 
-ALOFA_API int alofa_rmsnorm(void* out, const void* x, const void* w, const int* rows, int n_rows, int hidden, float eps,
+ALOFA_API int alofa_rmsnorm(void* out, const void* x, const void* w, const float* shift, const int* rows, int n_rows, int hidden, float eps,
                             int out_bf16, cudaStream_t stream) {
   if (n_rows <= 0) return ALOFA_OK;
   if (out_bf16)
-    rmsnorm_kernel<bf16><<<n_rows, 256, 0, stream>>>((bf16*)out, (const float*)x, (const float*)w, rows, hidden, eps);
+    rmsnorm_kernel<bf16><<<n_rows, 256, 0, stream>>>((bf16*)out, (const float*)x, (const float*)w, shift, rows, hidden, eps);
   else
-    rmsnorm_kernel<float><<<n_rows, 256, 0, stream>>>((float*)out, (const float*)x, (const float*)w, rows, hidden, eps);
+    rmsnorm_kernel<float><<<n_rows, 256, 0, stream>>>((float*)out, (const float*)x, (const float*)w, shift, rows, hidden, eps);
   return launch_status();
 }
 
@@ -78,7 +86,7 @@ ALOFA_API int alofa_rmsnorm(void* out, const void* x, const void* w, const int* 
 // Matrix product y = x W^T (+ bias), W row-major [N, K].
 //   EPI_STORE    out[m, n] = acc
 //   EPI_RESIDUAL out[m, n] += acc        (out is the fp32 residual stream)
-//   EPI_GATED    W holds [gate; up] (2N rows): out[m, n] = silu(gate) * up
+//   EPI_GATED    W holds [gate; up] (2N rows): out[m, n] = silu(gate) * up, or the clamped form of gate_times
 // EPI_STORE | (code << 4): out[m, n] = act(acc + bias), the activation codes of common.cuh.
 // 64x64 tile, 16-deep slices, 256 threads with 4x4 outputs each; every output
 // is summed by one thread over k ascending.
@@ -88,7 +96,7 @@ enum { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GATED = 2 };
 template <typename TA, typename TW, typename TO, int EPI>
 __global__ void __launch_bounds__(256) gemm_generic_kernel(TO* __restrict__ out, const TA* __restrict__ x,
                                                            const TW* __restrict__ w, const float* __restrict__ bias, int M,
-                                                           int N, int K, int act) {
+                                                           int N, int K, int act, float gate_alpha, float gate_limit) {
   constexpr int BM = 64, BN = 64, BK = 16;
   constexpr int NW = (EPI == EPI_GATED) ? 2 : 1;
   __shared__ float xs[BK][BM + 1];
@@ -150,7 +158,7 @@ __global__ void __launch_bounds__(256) gemm_generic_kernel(TO* __restrict__ out,
           g += bias[gn];
           u += bias[N + gn];
         }
-        out[o] = from_f<TO>(g / (1.0f + expf(-g)) * u);
+        out[o] = from_f<TO>(gate_times(g, u, gate_alpha, gate_limit));
       } else {
         float v = acc[0][i][j];
         if (bias) v += bias[gn];
@@ -165,17 +173,17 @@ __global__ void __launch_bounds__(256) gemm_generic_kernel(TO* __restrict__ out,
 
 template <typename TA, typename TW, typename TO>
 static int gemm_generic_launch(void* out, const void* x, const void* w, const float* bias, int M, int N, int K, int epi,
-                               cudaStream_t stream) {
+                               float gate_alpha, float gate_limit, cudaStream_t stream) {
   const int act = epi >> 4;  // EPI_STORE only: an activation on the sums (codes of common.cuh)
   epi &= 15;
   if (act && epi != EPI_STORE) return ALOFA_ERR_ARGUMENT;
   dim3 grid((N + 63) / 64, (M + 63) / 64);
   if (epi == EPI_STORE)
-    gemm_generic_kernel<TA, TW, TO, EPI_STORE><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act);
+    gemm_generic_kernel<TA, TW, TO, EPI_STORE><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act, gate_alpha, gate_limit);
   else if (epi == EPI_RESIDUAL)
-    gemm_generic_kernel<TA, TW, TO, EPI_RESIDUAL><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act);
+    gemm_generic_kernel<TA, TW, TO, EPI_RESIDUAL><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act, gate_alpha, gate_limit);
   else if (epi == EPI_GATED)
-    gemm_generic_kernel<TA, TW, TO, EPI_GATED><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act);
+    gemm_generic_kernel<TA, TW, TO, EPI_GATED><<<grid, 256, 0, stream>>>((TO*)out, (const TA*)x, (const TW*)w, bias, M, N, K, act, gate_alpha, gate_limit);
   else
     return ALOFA_ERR_ARGUMENT;
   return launch_status();
@@ -184,21 +192,21 @@ static int gemm_generic_launch(void* out, const void* x, const void* w, const fl
 // dtype flags: 0 = fp32, 1 = bf16.  N is the number of output columns (for
 // EPI_GATED the weight has 2N rows).  EPI_RESIDUAL requires an fp32 output.
 ALOFA_API int alofa_gemm_generic(void* out, const void* x, const void* w, const void* bias, int M, int N, int K, int epi,
-                                 int x_bf16, int w_bf16, int out_bf16, cudaStream_t stream) {
+                                 int x_bf16, int w_bf16, int out_bf16, float gate_alpha, float gate_limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return ALOFA_OK;
   if (K <= 0) return ALOFA_ERR_ARGUMENT;
   if ((epi & 15) == EPI_RESIDUAL && out_bf16) return ALOFA_ERR_ARGUMENT;
   const float* b = (const float*)bias;
   const int key = (x_bf16 ? 4 : 0) | (w_bf16 ? 2 : 0) | (out_bf16 ? 1 : 0);
   switch (key) {
-    case 0: return gemm_generic_launch<float, float, float>(out, x, w, b, M, N, K, epi, stream);
-    case 1: return gemm_generic_launch<float, float, bf16>(out, x, w, b, M, N, K, epi, stream);
-    case 2: return gemm_generic_launch<float, bf16, float>(out, x, w, b, M, N, K, epi, stream);
-    case 3: return gemm_generic_launch<float, bf16, bf16>(out, x, w, b, M, N, K, epi, stream);
-    case 4: return gemm_generic_launch<bf16, float, float>(out, x, w, b, M, N, K, epi, stream);
-    case 5: return gemm_generic_launch<bf16, float, bf16>(out, x, w, b, M, N, K, epi, stream);
-    case 6: return gemm_generic_launch<bf16, bf16, float>(out, x, w, b, M, N, K, epi, stream);
-    default: return gemm_generic_launch<bf16, bf16, bf16>(out, x, w, b, M, N, K, epi, stream);
+    case 0: return gemm_generic_launch<float, float, float>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 1: return gemm_generic_launch<float, float, bf16>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 2: return gemm_generic_launch<float, bf16, float>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 3: return gemm_generic_launch<float, bf16, bf16>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 4: return gemm_generic_launch<bf16, float, float>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 5: return gemm_generic_launch<bf16, float, bf16>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    case 6: return gemm_generic_launch<bf16, bf16, float>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
+    default: return gemm_generic_launch<bf16, bf16, bf16>(out, x, w, b, M, N, K, epi, gate_alpha, gate_limit, stream);
   }
 }
 
@@ -279,14 +287,15 @@ ALOFA_API int alofa_rope_store(void* q_out, void* k_cache, void* v_cache, const 
 // rescaled as in streaming softmax.  score = dot * scale, then (softcap > 0)
 // softcap * tanh(score / softcap), all in fp32.  Keys have hd numbers per head,
 // values vd (the two caches have their own row widths); v_share neighbouring key heads read one value
-// head; chunk > 0: a query sees only the keys of its own chunk of that many positions.
+// head; chunk > 0: a query sees only the keys of its own chunk of that many positions.  keep > 0: keys j < keep are
+// seen beside the window.  slopes: slopes[h] * (P - j) is taken off the score (after scale and cap).
 // ---------------------------------------------------------------------------
 template <typename T, typename TO>
 __global__ void __launch_bounds__(128) paged_attention_generic_kernel(
     TO* __restrict__ out, const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
     const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
     int max_blocks, int page_size, int nh, int nkv, int hd, int vd, int window, float scale, float softcap, const float* __restrict__ sink,
-    int chunk, int v_share) {
+    int chunk, int v_share, int keep, const float* __restrict__ slopes) {
   extern __shared__ float smem[];
   float* qs = smem;          // hd
   float* ps = smem + hd;     // 128
@@ -304,10 +313,13 @@ __global__ void __launch_bounds__(128) paged_attention_generic_kernel(
   // a sink is one more term of the softmax's denominator, exp(sink[h]), that belongs to no key and has no value
   float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;
   float acc0 = 0.f, acc1 = 0.f;  // dims tid and tid + 128
+  const int kept = min(keep, first);  // keys [0, kept) and [first, P] are seen
+  const float slope = slopes ? slopes[h] : 0.f;
   __syncthreads();
-  for (int c0 = (first / 128) * 128; c0 <= P; c0 += 128) {
+  for (int c0 = kept > 0 ? 0 : (first / 128) * 128; c0 <= P; c0 += 128) {
+    if (c0 >= kept) c0 = max(c0, (first / 128) * 128);  // nothing between the kept keys and the window
     const int j = c0 + tid;
-    const bool visible = j >= first && j <= P;
+    const bool visible = (j >= first || j < kept) && j <= P;
     float s = -INFINITY;
     int slot = -1;
     if (visible) {
@@ -318,6 +330,7 @@ __global__ void __launch_bounds__(128) paged_attention_generic_kernel(
       for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], to_f(kr[d]), dot);
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      s -= slope * (float)(P - j);
     }
     pages[tid] = slot;
     const float cmax = block_max(s, scratch);
@@ -350,22 +363,22 @@ ALOFA_API int alofa_paged_attention_generic(void* out, const void* q, const void
                                             const int* positions, const int* seq_of_token, const int* block_table,
                                             int max_blocks, int page_size, int n_tokens, int nh, int nkv, int hd,
                                             int vd, int window, float scale, float softcap, const float* sink, int is_bf16, int chunk, int v_share,
-                                            int out_f32, cudaStream_t stream) {
+                                            int out_f32, int keep, const float* slopes, cudaStream_t stream) {
   if (n_tokens <= 0) return ALOFA_OK;
-  if (hd <= 0 || vd <= 0 || vd > 256 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || chunk < 0 || v_share <= 0 || nkv % v_share != 0) return ALOFA_ERR_ARGUMENT;
+  if (hd <= 0 || vd <= 0 || vd > 256 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || chunk < 0 || v_share <= 0 || nkv % v_share != 0 || keep < 0) return ALOFA_ERR_ARGUMENT;
   dim3 grid(n_tokens, nh);
   const size_t smem = (size_t)(hd + 128) * sizeof(float);
   if (is_bf16 && out_f32)
     paged_attention_generic_kernel<bf16, float><<<grid, 128, smem, stream>>>(
         (float*)out, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, positions, seq_of_token, block_table,
-        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share);
+        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share, keep, slopes);
   else if (is_bf16)
     paged_attention_generic_kernel<bf16, bf16><<<grid, 128, smem, stream>>>(
         (bf16*)out, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, positions, seq_of_token, block_table,
-        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share);
+        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share, keep, slopes);
   else
     paged_attention_generic_kernel<float, float><<<grid, 128, smem, stream>>>(
         (float*)out, (const float*)q, (const float*)k_cache, (const float*)v_cache, positions, seq_of_token, block_table,
-        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share);
+        max_blocks, page_size, nh, nkv, hd, vd, window, scale, softcap, sink, chunk, v_share, keep, slopes);
   return launch_status();
 }

@@ -672,7 +672,7 @@ template <typename T, int TT>
 __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate,
                                                          const T* __restrict__ x, const float* __restrict__ wr, int T_, int E, int top, int hidden,
                                                          int gated, int softmax, int renormalize, const float* __restrict__ correction,
-                                                         float renorm_eps, int groups, int keep, float route_scale) {
+                                                         float renorm_eps, int groups, int keep, float route_scale, int group_best) {
   extern __shared__ __align__(16) uint8_t router_smem[];
   const int cols = E + (gated ? 1 : 0);
   float* z = reinterpret_cast<float*>(router_smem);      // [TT][cols]
@@ -746,7 +746,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
     __syncwarp();
     if (groups > 1) {
       // experts form `groups` equal groups of neighbours; a group's score is the sum of its two largest choice
-      // scores (score + correction); only experts of the `keep` best groups can be chosen (ties: the lower group)
+      // scores (score + correction), or (group_best) the largest alone; only experts of the `keep` best groups can be chosen (ties: the lower group)
       const int per = E / groups;
       float* gs = gsc + r * groups;
       for (int g = lane; g < groups; g += 32) {
@@ -756,7 +756,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
           if (v > a) b = a, a = v;
           else if (v > b) b = v;
         }
-        gs[g] = per > 1 ? a + b : a;
+        gs[g] = per > 1 && !group_best ? a + b : a;
       }
       __syncwarp();
       for (int g = lane; g < groups; g += 32) {
@@ -802,7 +802,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
 
 template <typename T, int TT>
 static int moe_router_launch(int* choice, float* weight, float* gate, const void* x, const float* wr, int T_, int E, int top, int hidden, int softmax,
-                             int renormalize, const float* correction, float renorm_eps, int groups, int keep, float route_scale, cudaStream_t stream) {
+                             int renormalize, const float* correction, float renorm_eps, int groups, int keep, float route_scale, int group_best, cudaStream_t stream) {
   const int cols = E + (gate ? 1 : 0);
   const size_t smem = ((size_t)TT * (cols + groups) + 4) * sizeof(float) + (size_t)TT * hidden * sizeof(T);
   static size_t set = 0;
@@ -811,7 +811,7 @@ static int moe_router_launch(int* choice, float* weight, float* gate, const void
     set = smem;
   }
   launch_dep(moe_router_kernel<T, TT>, (T_ + TT - 1) / TT, 256, smem, stream, choice, weight, gate, (const T*)x, wr, T_, E, top, hidden, gate ? 1 : 0, softmax,
-             renormalize, correction, renorm_eps, groups, keep, route_scale);
+             renormalize, correction, renorm_eps, groups, keep, route_scale, group_best);
   return launch_status();
 }
 
@@ -820,7 +820,7 @@ static int moe_router_launch(int* choice, float* weight, float* gate, const void
 // choice scores) can be chosen.  route_scale: a factor on the weights.
 ALOFA_API int alofa_moe_router(int* choice, float* weight, float* gate, const void* x, const float* wr, int T, int E, int top, int hidden, int softmax,
                                int renormalize, int x_bf16, const float* correction, float renorm_eps, int groups, int keep, float route_scale,
-                               cudaStream_t stream) {
+                               int group_best, cudaStream_t stream) {
   if (T <= 0) return ALOFA_OK;
   if (E <= 0 || top <= 0 || top > E || top > 32) return ALOFA_ERR_ARGUMENT;
   if (groups < 1) groups = 1;
@@ -829,11 +829,11 @@ ALOFA_API int alofa_moe_router(int* choice, float* weight, float* gate, const vo
   const size_t room = 200 * 1024;
   // few tokens: two to a block, so that a decode step's tokens are spread over more than a handful of SMs
   if (8 * row <= room && T > 512)
-    return x_bf16 ? moe_router_launch<bf16, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, stream)
-                  : moe_router_launch<float, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, stream);
+    return x_bf16 ? moe_router_launch<bf16, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
+                  : moe_router_launch<float, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream);
   if (2 * row <= room)
-    return x_bf16 ? moe_router_launch<bf16, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, stream)
-                  : moe_router_launch<float, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, stream);
+    return x_bf16 ? moe_router_launch<bf16, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
+                  : moe_router_launch<float, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream);
   return ALOFA_ERR_ARGUMENT;
 }
 
@@ -1005,22 +1005,22 @@ ALOFA_API int alofa_moe_combine(float* y, const float* ys, const int* dest, cons
   return launch_status();
 }
 
-// mid[r, c] = silu(gu[r, c]) * gu[r, ff + c]: the gated activation of rows that hold [gate | up] side by side (fp32 sums in, compute dtype out).
+// mid[r, c] = silu(gu[r, c]) * gu[r, ff + c] (or the clamped form, see gate_times): the gated activation of rows that hold [gate | up] side by side (fp32 sums in, compute dtype out).
 template <typename T>
-__global__ void gate_up_kernel(T* __restrict__ mid, const float* __restrict__ gu, long long count, int ff) {
+__global__ void gate_up_kernel(T* __restrict__ mid, const float* __restrict__ gu, long long count, int ff, float alpha, float limit) {
   pdl_begin();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= count) return;
   const long long r = i / ff;
   const int c = (int)(i - r * ff);
   const float g = gu[r * 2 * ff + c], u = gu[r * 2 * ff + ff + c];
-  mid[i] = from_f<T>(g / (1.0f + expf(-g)) * u);
+  mid[i] = from_f<T>(gate_times(g, u, alpha, limit));
 }
 
-ALOFA_API int alofa_gate_up(void* mid, const float* gu, long long rows, int ff, int out_bf16, cudaStream_t stream) {
+ALOFA_API int alofa_gate_up(void* mid, const float* gu, long long rows, int ff, int out_bf16, float alpha, float limit, cudaStream_t stream) {
   const long long count = rows * ff;
   if (count <= 0) return ALOFA_OK;
-  if (out_bf16) launch_dep(gate_up_kernel<bf16>, (unsigned)((count + 255) / 256), 256, 0, stream, (bf16*)mid, gu, count, ff);
-  else launch_dep(gate_up_kernel<float>, (unsigned)((count + 255) / 256), 256, 0, stream, (float*)mid, gu, count, ff);
+  if (out_bf16) launch_dep(gate_up_kernel<bf16>, (unsigned)((count + 255) / 256), 256, 0, stream, (bf16*)mid, gu, count, ff, alpha, limit);
+  else launch_dep(gate_up_kernel<float>, (unsigned)((count + 255) / 256), 256, 0, stream, (float*)mid, gu, count, ff, alpha, limit);
   return launch_status();
 }

@@ -586,6 +586,155 @@ ALOFA_API int alofa_qkv_prepare(void* q_out, void* k_cache, void* v_cache, const
 }
 
 // ---------------------------------------------------------------------------
+// The same preparation where q and k are each normed over ALL their heads at once: a row of ld fp32 sums [q: H * d |
+// k: G * d | v: G * dv | more].  q / sqrt(mean(q^2) + eps) * q_w (q_w [H * d]) to its buffer, k likewise (k_w [G * d]) and v to
+// the token's cache slot.  v_first (optional, fp32 [T, G * dv]): the values of the first of several layers that mix
+// theirs.  mix null: this is that layer, its values are left there; else v <- (1 - mix) v + mix v_first before it is
+// stored.  One block per token: the row's q and k wait in shared memory for their sums.
+// ---------------------------------------------------------------------------
+template <typename T, int V>
+struct PackedStore;
+template <>
+struct PackedStore<float, 4> {
+  static __device__ __forceinline__ void put(float* to, const float (&x)[4]) { *reinterpret_cast<float4*>(to) = make_float4(x[0], x[1], x[2], x[3]); }
+};
+template <>
+struct PackedStore<bf16, 4> {
+  static __device__ __forceinline__ void put(bf16* to, const float (&x)[4]) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+    *reinterpret_cast<uint2*>(to) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+  }
+};
+template <typename T>
+struct PackedStore<T, 1> {
+  static __device__ __forceinline__ void put(T* to, const float (&x)[1]) { *to = from_f<T>(x[0]); }
+};
+
+// V columns of a row from `col` on: finished sums, or planes of them added in split order with the bias on top
+template <int V>
+__device__ __forceinline__ void row_columns(float (&x)[V], const float* row, int col, int splits, long long plane, const float* bias) {
+  const int planes = splits > 0 ? splits : 1;
+#pragma unroll
+  for (int i = 0; i < V; ++i) x[i] = 0.f;
+  for (int z = 0; z < planes; ++z) {
+    const float* p = row + (size_t)z * plane + col;
+    if constexpr (V == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(p);
+      x[0] += a.x, x[1] += a.y, x[2] += a.z, x[3] += a.w;
+    } else {
+      x[0] += p[0];
+    }
+  }
+  if (bias) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[i] += bias[col + i];
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) qkv_prepare_rows_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ qkv, int ld,
+                                                                const int* __restrict__ slot_map, int nq, int nk, int nv, const float* __restrict__ q_w,
+                                                                const float* __restrict__ k_w, float eps, float* __restrict__ v_first, const float* __restrict__ mix,
+                                                                int splits, long long plane, const float* __restrict__ bias, float* __restrict__ extra_out, int extra_at,
+                                                                int extra_n) {
+  extern __shared__ __align__(16) float row_smem[];  // nq + nk numbers
+  __shared__ float scratch[32];
+  pdl_begin();
+  const int t = blockIdx.x;
+  const float* row = qkv + (size_t)t * ld;
+  const int slot = slot_map[t];
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+    float x[V];
+    row_columns<V>(x, row, c, splits, plane, bias);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      row_smem[c + i] = x[i];
+      ss = fmaf(x[i], x[i], ss);
+    }
+    if (c < nq) sq += ss;
+    else sk += ss;
+  }
+  const float lambda = mix ? *mix : 0.f;
+  for (int c = threadIdx.x * V; c < nv; c += blockDim.x * V) {
+    float x[V];
+    row_columns<V>(x, row, nq + nk + c, splits, plane, bias);
+    if (v_first) {
+      float* f = v_first + (size_t)t * nv + c;
+      if (mix) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[i] = (1.0f - lambda) * x[i] + lambda * f[i];
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[i] = x[i];
+      }
+    }
+    PackedStore<T, V>::put(v_cache + (size_t)slot * nv + c, x);
+  }
+  if (extra_out)
+    for (int c = threadIdx.x; c < extra_n; c += blockDim.x) {
+      float x[1];
+      row_columns<1>(x, row, extra_at + c, splits, plane, bias);
+      extra_out[(size_t)t * extra_n + c] = x[0];
+    }
+  sq = block_sum(sq, scratch);
+  sk = block_sum(sk, scratch);
+  const float rq = 1.0f / sqrtf(sq / (float)nq + eps), rk = 1.0f / sqrtf(sk / (float)nk + eps);
+  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+    const bool is_q = c < nq;
+    const float* w = is_q ? q_w + c : k_w + (c - nq);
+    const float r = is_q ? rq : rk;
+    float x[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[i] = row_smem[c + i] * r * w[i];
+    PackedStore<T, V>::put(is_q ? q_out + (size_t)t * nq + c : k_cache + (size_t)slot * nk + (c - nq), x);
+  }
+}
+
+template <typename T, int V>
+static int qkv_prepare_rows_launch(void* q_out, void* k_cache, void* v_cache, const float* qkv, int ld, const int* slot_map, int n_tokens, int nq, int nk, int nv,
+                                   const float* q_w, const float* k_w, float eps, float* v_first, const float* mix, int splits, long long plane, const float* bias,
+                                   float* extra_out, int extra_at, int extra_n, cudaStream_t stream) {
+  const size_t smem = (size_t)(nq + nk) * sizeof(float);
+  if (smem > 200 * 1024) return ALOFA_ERR_ARGUMENT;
+  static size_t set = 48 * 1024;
+  if (smem > set) {
+    if (cudaFuncSetAttribute(qkv_prepare_rows_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
+    set = smem;
+  }
+  const int groups = (nq + nk + V - 1) / V;  // what the threads of a block share: with few tokens a wide block, whose loads are all in flight at once
+  int threads = groups >= 1024 ? 1024 : (groups + 31) / 32 * 32;
+  if (n_tokens > 148 && threads > 256) threads = 256;
+  launch_dep(qkv_prepare_rows_kernel<T, V>, n_tokens, threads, smem, stream, (T*)q_out, (T*)k_cache, (T*)v_cache, qkv, ld, slot_map, nq, nk, nv, q_w, k_w, eps, v_first,
+             mix, splits, plane, bias, extra_out, extra_at, extra_n);
+  return launch_status();
+}
+
+// nq, nk, nv: columns of q (all heads), k and v.  splits, plane, bias and the extra columns as in alofa_qkv_prepare.
+ALOFA_API int alofa_qkv_prepare_rows(void* q_out, void* k_cache, void* v_cache, const float* qkv, int ld, const int* slot_map, int n_tokens, int nq, int nk, int nv,
+                                     const float* q_w, const float* k_w, float eps, float* v_first, const float* mix, int is_bf16, int splits, long long plane,
+                                     const float* bias, float* extra_out, int extra_at, int extra_n, cudaStream_t stream) {
+  if (n_tokens <= 0) return ALOFA_OK;
+  if (nq <= 0 || nk <= 0 || nv <= 0 || !q_w || !k_w || (mix && !v_first) || ld < nq + nk + nv || splits < 0 || (splits > 0 && plane < (long long)n_tokens * ld) ||
+      (extra_out && (extra_n <= 0 || extra_at < 0 || extra_at + extra_n > ld)))
+    return ALOFA_ERR_ARGUMENT;
+  if (splits == 0) bias = nullptr;
+  const bool four = nq % 4 == 0 && nk % 4 == 0 && nv % 4 == 0 && ld % 4 == 0 && plane % 4 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)q_out % 16 == 0 &&
+                    (uintptr_t)k_cache % 16 == 0 && (uintptr_t)v_cache % 16 == 0;
+#define ROWS_CASE(TT, VV) \
+  return qkv_prepare_rows_launch<TT, VV>(q_out, k_cache, v_cache, qkv, ld, slot_map, n_tokens, nq, nk, nv, q_w, k_w, eps, v_first, mix, splits, plane, bias, extra_out, \
+                                         extra_at, extra_n, stream)
+  if (is_bf16) {
+    if (four) ROWS_CASE(bf16, 4);
+    ROWS_CASE(bf16, 1);
+  }
+  if (four) ROWS_CASE(float, 4);
+  ROWS_CASE(float, 1);
+#undef ROWS_CASE
+}
+
+// ---------------------------------------------------------------------------
 // heads_finish: what some attentions do to a head's output before the output projection, one warp per
 // (token, head), fp32.  a [T, H * maps, dv] fp32 holds the attention outputs in the order qkv_prepare
 // gave the queries ([key head][map][head of the group]); the tensor-core attention kernels leave them in bfloat16.

@@ -38,10 +38,10 @@ def _generic():
         lib = load_library("alofa_generic", ["kernels/generic.cu"])
         sigs = {
             "alofa_embed_gather": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
-            "alofa_rmsnorm": [_P, _P, _P, _P, _I, _I, _F, _I, _P],
-            "alofa_gemm_generic": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+            "alofa_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _P],
+            "alofa_gemm_generic": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
             "alofa_rope_store": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
-            "alofa_paged_attention_generic": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _P],
+            "alofa_paged_attention_generic": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _I, _I, _I, _P, _P],
         }
         for name, args in sigs.items():
             fn = getattr(lib, name)
@@ -72,9 +72,9 @@ def _gemm_tc():
     if lib is None:
         lib = load_library("alofa_gemm_tc", ["kernels/gemm_tc.cu"])
         lib.alofa_gemm_tc.restype = _I
-        lib.alofa_gemm_tc.argtypes = [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _I, _P]
+        lib.alofa_gemm_tc.argtypes = [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _I, _F, _F, _P]
         lib.alofa_splitk_reduce.restype = _I
-        lib.alofa_splitk_reduce.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _P]
+        lib.alofa_splitk_reduce.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P]
         lib.alofa_gemm_tc_reduces_in_cluster.restype = _I
         lib.alofa_gemm_tc_reduces_in_cluster.argtypes = [_I, _I, _I]
         lib.alofa_gemm_tc_rope.restype = _I
@@ -87,17 +87,23 @@ def _gemm_tc():
     return lib
 
 
-def _attention(head_dim: int, capped: bool = False):
-    """The attention library of one head size; ``capped``: the build whose scores are bounded by softcap * tanh(. / softcap)."""
-    key = f"attention_hd{head_dim}" + ("_cap" if capped else "")
+def _attention(head_dim: int, capped: bool = False, v_dim=None, distance: bool = False):
+    """The attention library of one size of key heads and (``v_dim``, when it differs) value heads; ``capped``: the build
+    whose scores are bounded by softcap * tanh(. / softcap); ``distance``: the one that takes a distance bias off them."""
+    v_dim = v_dim or head_dim
+    key = f"attention_hd{head_dim}" + (f"_v{v_dim}" if v_dim != head_dim else "") + ("_cap" if capped else "") + ("_dist" if distance else "")
     lib = _libs.get(key)
     if lib is None:
         defines = {"HEAD_DIM": head_dim}
         if capped:
             defines["SOFTCAP"] = 1
+        if v_dim != head_dim:
+            defines["V_DIM"] = v_dim
+        if distance:
+            defines["DISTANCE_BIAS"] = 1
         lib = load_library(f"alofa_{key}", ["kernels/attention_bf16.cu"], defines=defines)
         lib.alofa_attention_bf16.restype = _I
-        lib.alofa_attention_bf16.argtypes = [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _I, ctypes.c_longlong, _P, _I, _F, _P, _P]
+        lib.alofa_attention_bf16.argtypes = [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _I, ctypes.c_longlong, _P, _I, _F, _P, _I, _P, _P, _I, _P]
         lib.alofa_attention_combine.restype = _I
         lib.alofa_attention_combine.argtypes = [_P, _P, _P, _P, _I, _I, _I, _I, _P, _P]
         lib.alofa_attention_decode_wide_warps.restype = _I
@@ -111,25 +117,25 @@ def _attention(head_dim: int, capped: bool = False):
 _decode_slots = {}
 
 
-def attention_decode_wide_warps(head_dim: int, capped: bool = False) -> int:
+def attention_decode_wide_warps(head_dim: int, capped: bool = False, v_dim=None, distance: bool = False) -> int:
     """Warps of the decode attention kernel's wide form at this head size (one
     CTA per SM; its splits are multiples of 64 keys a warp), 0 when it has none."""
-    return _attention(head_dim, capped).alofa_attention_decode_wide_warps()
+    return _attention(head_dim, capped, v_dim, distance).alofa_attention_decode_wide_warps()
 
 
-def attention_decode_slots(head_dim: int, page_size: int, warps: int = 4, capped: bool = False) -> int:
+def attention_decode_slots(head_dim: int, page_size: int, warps: int = 4, capped: bool = False, v_dim=None, distance: bool = False) -> int:
     """How many CTAs of the decode attention kernel with ``warps`` warps (4, or
     the wide form's) the device holds at a time, 0 when that kernel is not
     built for this head size and kind of page (asked once each)."""
-    key = (head_dim, page_size % 64 == 0, warps, capped)
+    key = (head_dim, page_size % 64 == 0, warps, capped, v_dim or head_dim, distance)
     if key not in _decode_slots:
-        _decode_slots[key] = max(0, _attention(head_dim, capped).alofa_attention_decode_slots(page_size, warps))
+        _decode_slots[key] = max(0, _attention(head_dim, capped, v_dim, distance).alofa_attention_decode_slots(page_size, warps))
     return _decode_slots[key]
 
 
-def attention_bf16_supported(head_dim: int) -> bool:
-    """Head sizes the bfloat16 attention kernel is built for."""
-    return head_dim % 16 == 0 and 16 <= head_dim <= 128
+def attention_bf16_supported(head_dim: int, v_dim=None) -> bool:
+    """Sizes of key and value heads (the same unless given) the bfloat16 attention kernel is built for."""
+    return all(d % 16 == 0 and 16 <= d <= 128 for d in (head_dim, v_dim or head_dim))
 
 
 def _elementwise():
@@ -137,7 +143,7 @@ def _elementwise():
     if lib is None:
         lib = load_library("alofa_elementwise_bf16", ["kernels/elementwise_bf16.cu"])
         lib.alofa_norm_fused.restype = _I
-        lib.alofa_norm_fused.argtypes = [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P]
+        lib.alofa_norm_fused.argtypes = [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P, _P]
         lib.alofa_stream_settle.restype = _I
         lib.alofa_stream_settle.argtypes = [_P, _P, _P, _P, _I, _P]
         lib.alofa_rope_store_fused.restype = _I
@@ -214,23 +220,32 @@ def embed_gather(out, table, ids, status=None, src=None, fed=None) -> None:
     )
 
 
-def rmsnorm(out, x, weight, eps: float, rows=None) -> None:
-    """out[r] = rmsnorm(x[rows[r] or r]) * weight; x fp32, weight fp32."""
+def rmsnorm(out, x, weight, eps: float, rows=None, shift=None) -> None:
+    """out[r] = rmsnorm(x[rows[r] or r]) * weight; x fp32, weight fp32.  With
+    ``shift`` (fp32) the layer norm: (x - mean) / sqrt(variance + eps) * weight
+    + shift."""
     n, hidden = out.shape
-    if x.shape[-1] != hidden or weight.shape[0] != hidden:
+    if x.shape[-1] != hidden or weight.shape[0] != hidden or (shift is not None and shift.shape[0] != hidden):
         raise AlofaError("invalid_argument", "rmsnorm sizes disagree", f"out={tuple(out.shape)} x={tuple(x.shape)} w={tuple(weight.shape)}")
     _done(
         _generic().alofa_rmsnorm(
             _dev(out, "out"), _dev(x, "x", torch.float32), _dev(weight, "weight", torch.float32),
+            _dev(shift, "shift", torch.float32) if shift is not None else None,
             _dev(rows, "rows", torch.int32) if rows is not None else None, n, hidden, float(eps), _is_bf16(out, "out"), _stream(),
         ),
         "rmsnorm",
     )
 
 
-def gemm_generic(out, x, w, bias, epi: int, act: int = 0) -> None:
+SILU_GATE = (0.0, 0.0)  # what a gated product makes of its sums: silu(g) * u
+
+
+def gemm_generic(out, x, w, bias, epi: int, act: int = 0, gate=SILU_GATE) -> None:
     """out = x @ w.T (+bias) with the epilogue ``epi``; any sizes.  ``act``
-    (EPI_STORE only): a code of ``ACTIVATIONS`` applied to the fp32 sums."""
+    (EPI_STORE only): a code of ``ACTIVATIONS`` applied to the fp32 sums.
+    ``gate`` = (alpha, limit) (EPI_GATED only): with alpha > 0 the clamped form
+    ``g = min(g, limit), u = clamp(u, -limit, limit): g * sigmoid(alpha g) * (u
+    + 1)`` instead of ``silu(g) * u``."""
     m, k = x.shape
     n = out.shape[1]
     rows_w = 2 * n if epi == EPI_GATED else n
@@ -239,7 +254,7 @@ def gemm_generic(out, x, w, bias, epi: int, act: int = 0) -> None:
     _done(
         _generic().alofa_gemm_generic(
             _dev(out, "out"), _dev(x, "x"), _dev(w, "w"), _dev(bias, "bias", torch.float32) if bias is not None else None,
-            m, n, k, epi | (act << 4), _is_bf16(x, "x"), _is_bf16(w, "w"), _is_bf16(out, "out"), _stream(),
+            m, n, k, epi | (act << 4), _is_bf16(x, "x"), _is_bf16(w, "w"), _is_bf16(out, "out"), float(gate[0]), float(gate[1]), _stream(),
         ),
         "gemm_generic", f"M={m} N={n} K={k} epi={epi}",
     )
@@ -266,7 +281,7 @@ def rope_store(q_out, k_cache, v_cache, qkv, cos_sin, positions, slot_map, nh, n
 
 
 def paged_attention_generic(out, q, k_cache, v_cache, positions, seq_of_token, block_table, page_size, nh, nkv, hd, window, scale, softcap: float = 0.0, vd=None, sink=None,
-                            chunk: int = 0, v_share: int = 1) -> None:
+                            chunk: int = 0, v_share: int = 1, keep: int = 0, slopes=None) -> None:
     """Causal grouped-query attention over the paged cache for every size and
     both dtypes; fp32 scores and softmax.  ``softcap`` > 0 bounds the scaled
     scores by ``softcap * tanh(score / softcap)``; ``vd`` is the values' head
@@ -275,8 +290,10 @@ def paged_attention_generic(out, q, k_cache, v_cache, positions, seq_of_token, b
     belongs to no key and has no value.  ``chunk`` > 0: a query at position p
     sees only the keys from ``p - p % chunk`` on.  ``v_share``: so many
     neighbouring key heads read one value head (the value cache has ``nkv /
-    v_share`` heads).  ``out`` may be fp32 while q and the caches are
-    bfloat16."""
+    v_share`` heads).  ``keep`` > 0: keys j < keep are seen beside the window.
+    ``slopes`` (fp32, one per head): ``slopes[h] * (p - j)`` is taken off the
+    score of key j after scale and cap.  ``out`` may be fp32 while q and the
+    caches are bfloat16."""
     n = q.shape[0]
     vd = hd if vd is None else vd
     dt = q.dtype
@@ -288,7 +305,8 @@ def paged_attention_generic(out, q, k_cache, v_cache, positions, seq_of_token, b
             _dev(out, "out"), _dev(q, "q"), _dev(k_cache, "k_cache", dt), _dev(v_cache, "v_cache", dt),
             _dev(positions, "positions", torch.int32), _dev(seq_of_token, "seq_of_token", torch.int32), _dev(block_table, "block_table", torch.int32),
             block_table.shape[1], page_size, n, nh, nkv, hd, vd, int(window or 0), float(scale), float(softcap or 0.0),
-            _dev(sink, "sink", torch.float32) if sink is not None else None, _is_bf16(q, "q"), int(chunk or 0), int(v_share), 1 if out.dtype == torch.float32 else 0, _stream(),
+            _dev(sink, "sink", torch.float32) if sink is not None else None, _is_bf16(q, "q"), int(chunk or 0), int(v_share), 1 if out.dtype == torch.float32 else 0,
+            int(keep or 0), _dev(slopes, "slopes", torch.float32) if slopes is not None else None, _stream(),
         ),
         "paged_attention_generic", f"heads={nh} kv_heads={nkv} head_dim={hd} v_head_dim={vd}",
     )
@@ -362,7 +380,7 @@ B_ROWS, B_MERGED_SPLITS, B_NORMED = 0, 1, 2
 
 
 def gemm_tc(out, x, w, bias, epi: int, bn: int, splits: int = 1, partial=None, status=None, reduce: bool = True, computed=None, acc=None, act: int = 0,
-            tile_batch=None, batches: int = 1) -> bool:
+            tile_batch=None, batches: int = 1, gate=SILU_GATE) -> bool:
     """Tensor-core product ``out = x @ w.T`` (bf16 operands, fp32 sums) with
     the epilogue fused.  Returns False, having launched nothing, when the
     kernel does not take these sizes (depth not a multiple of 8, unaligned).
@@ -385,7 +403,8 @@ def gemm_tc(out, x, w, bias, epi: int, bn: int, splits: int = 1, partial=None, s
     ``tile_batch`` (int32 on the device; tokens on M, EPI_STORE or EPI_GATED,
     no bias): ``w`` is [batches * N, K] (gated: [batches * 2N, K], a batch's
     gate rows before its up rows) and the i-th tile of 128 token rows multiplies
-    by the rows of batch ``tile_batch[i]``; a negative entry skips the tile."""
+    by the rows of batch ``tile_batch[i]``; a negative entry skips the tile.
+    ``gate`` (EPI_GATED): as in :func:`gemm_generic`."""
     n = out.shape[1]
     rows_w = (2 * n if epi == EPI_GATED else n) * (batches if tile_batch is not None else 1)
     k = w.shape[1]
@@ -416,7 +435,7 @@ def gemm_tc(out, x, w, bias, epi: int, bn: int, splits: int = 1, partial=None, s
         _dev(status, "status", torch.int32) if status is not None else None,
         b_kind, b_src, b_ml, b_pos, heads, hd, window, split_keys,
         _dev(acc, "acc", i64) if acc is not None else None, n_acc, n_gamma, float(n_eps), n_out, n_zero,
-        _dev(tile_batch, "tile_batch", torch.int32) if tile_batch is not None else None, batches, _stream(),
+        _dev(tile_batch, "tile_batch", torch.int32) if tile_batch is not None else None, batches, float(gate[0]), float(gate[1]), _stream(),
     )
     if rc == 1:
         return False
@@ -461,7 +480,8 @@ def gemm_tc_rope(x, w, bias, q_out, k_cache, v_cache, slot_map, positions, cos_s
 
 
 def attention_bf16(out, q, k_cache, v_cache, q_start, kv_len, positions, block_table, page_size, n_seqs, max_q_len, nh, nkv, hd, window, scale,
-                   n_splits: int = 0, split_keys: int = 0, partial_o=None, partial_ml=None, max_kv_len: int = 0, status=None, combine: bool = True, softcap: float = 0.0, sink=None) -> None:
+                   n_splits: int = 0, split_keys: int = 0, partial_o=None, partial_ml=None, max_kv_len: int = 0, status=None, combine: bool = True, softcap: float = 0.0, sink=None,
+                   keep: int = 0, slopes=None, gate=None, gate_at: int = 0) -> None:
     """Causal GQA over the paged bf16 cache for a step's requests; with
     ``n_splits`` > 0 the keys of each request (decode tokens) or of each query
     tile (prompt portions) are split over several CTAs and merged - unless
@@ -469,12 +489,23 @@ def attention_bf16(out, q, k_cache, v_cache, q_start, kv_len, positions, block_t
     keep the splits for :func:`attention_combine` or a product that merges them.
     ``softcap`` > 0 (the library built for it): scaled scores are bounded by
     ``softcap * tanh(score / softcap)``.  ``sink`` [nh] fp32: one more term
-    ``exp(sink[h])`` of every row's denominator (merged splits only)."""
+    ``exp(sink[h])`` of every row's denominator (merged splits only).
+    ``keep`` > 0: the keys j < keep are seen beside the window; the splits then
+    go by the blocks of 64 keys a request can see, the kept ones first.
+    ``slopes`` [nh] fp32 (the library built for it): ``slopes[h]`` times the
+    distance of query and key is taken off every score.  ``gate`` (fp32 [T, ld],
+    sums of a projection): head h's finished output is multiplied by
+    ``sigmoid(gate[t, gate_at + h])``.  The values' head size is the value cache's own."""
     n = q.shape[0]
     bf = torch.bfloat16
+    vd = v_cache.shape[2]
+    if tuple(out.shape) != (n, nh * vd) or tuple(q.shape) != (n, nh * hd) or tuple(k_cache.shape[1:]) != (nkv, hd) or v_cache.shape[1] != nkv:
+        raise AlofaError("invalid_argument", "attention sizes disagree", f"q={tuple(q.shape)} out={tuple(out.shape)} k={tuple(k_cache.shape)} v={tuple(v_cache.shape)}")
+    if (sink is not None and sink.shape[0] != nh) or (slopes is not None and slopes.shape[0] != nh) or (gate is not None and (gate.shape[0] != n or gate_at + nh > gate.shape[1])):
+        raise AlofaError("invalid_argument", "attention: a number per head disagrees with the heads", f"heads={nh}")
     g = nh // nkv
     tiles = -(-(max_q_len * g) // 64)
-    rc = _attention(hd, softcap > 0).alofa_attention_bf16(
+    rc = _attention(hd, softcap > 0, vd, slopes is not None).alofa_attention_bf16(
         _dev(out, "out", bf), _dev(q, "q", bf), _dev(k_cache, "k_cache", bf), _dev(v_cache, "v_cache", bf),
         _dev(q_start, "q_start", torch.int32), _dev(kv_len, "kv_len", torch.int32), _dev(positions, "positions", torch.int32),
         _dev(block_table, "block_table", torch.int32),
@@ -483,18 +514,20 @@ def attention_bf16(out, q, k_cache, v_cache, q_start, kv_len, positions, block_t
         _dev(partial_ml, "partial_ml", torch.float32) if partial_ml is not None else None,
         int(max_kv_len) if max_kv_len else block_table.shape[1] * page_size, k_cache.shape[0],
         _dev(status, "status", torch.int32) if status is not None else None, 1 if combine else 0, float(softcap or 0.0),
-        _dev(sink, "sink", torch.float32) if sink is not None else None, _stream(),
+        _dev(sink, "sink", torch.float32) if sink is not None else None, int(keep or 0), _dev(slopes, "slopes", torch.float32) if slopes is not None else None,
+        _dev(gate, "gate", torch.float32) + 4 * gate_at if gate is not None else None, gate.shape[1] if gate is not None else 0, _stream(),
     )
     _done(rc, "attention_bf16", f"hd={hd} nh={nh} nkv={nkv} splits={n_splits}")
     if n_splits > 1 and combine:
         count_launches(1)
 
 
-def attention_combine(out, partial_o, partial_ml, positions, nh: int, hd: int, window, split_keys: int, sink=None, capped: bool = False) -> None:
-    """Merge the key splits of decode tokens: out [T, nh * hd] bf16.  ``capped``:
-    take the kernel from the library built for capped scores (the one the
-    splits came from), so that no second library is built for it."""
-    rc = _attention(hd, capped).alofa_attention_combine(
+def attention_combine(out, partial_o, partial_ml, positions, nh: int, hd: int, window, split_keys: int, sink=None, capped: bool = False, key_dim=None, distance: bool = False) -> None:
+    """Merge the key splits of decode tokens: out [T, nh * hd] bf16.  ``capped``,
+    ``key_dim`` (the keys' head size where it is not the values' ``hd``) and
+    ``distance`` name the library the splits came from, so that no second
+    library is built for it."""
+    rc = _attention(key_dim or hd, capped, hd, distance).alofa_attention_combine(
         _dev(out, "out", torch.bfloat16), _dev(partial_o, "partial_o", torch.float32), _dev(partial_ml, "partial_ml", torch.float32),
         _dev(positions, "positions", torch.int32), out.shape[0], nh, int(window or 0), split_keys,
         _dev(sink, "sink", torch.float32) if sink is not None else None, _stream(),
@@ -502,13 +535,14 @@ def attention_combine(out, partial_o, partial_ml, positions, nh: int, hd: int, w
     _done(rc, "attention_combine")
 
 
-def norm_fused(out, h, weight, eps: float, rows=None, partial=None, splits: int = 0, bias=None, base=None, acc=None, other=None) -> bool:
+def norm_fused(out, h, weight, eps: float, rows=None, partial=None, splits: int = 0, bias=None, base=None, acc=None, other=None, shift=None) -> bool:
     """RMSNorm of rows of the fp32 stream ``h`` (vectorised; hidden % 4 == 0).
     With ``partial`` [splits, T, hidden] the pending partial sums (and bias)
     are first added into ``h``.  With ``base`` the stream's values are read
     from there (``h`` is written, complete), with ``acc`` (int64, units of
     2^-32; every row, ``rows`` None) that accumulator is added on top and left
-    zero, as is ``other``.  Returns False when the size is not taken."""
+    zero, as is ``other``.  With ``shift`` (fp32) the layer norm instead.
+    Returns False when the size is not taken."""
     n, hidden = out.shape
     if hidden % 4:
         return False
@@ -518,7 +552,7 @@ def norm_fused(out, h, weight, eps: float, rows=None, partial=None, splits: int 
         _dev(bias, "bias", f32) if bias is not None else None, _dev(rows, "rows", torch.int32) if rows is not None else None,
         n, h.shape[0], hidden, splits, float(eps), _is_bf16(out, "out"),
         _dev(base, "base", f32) if base is not None else None, _dev(acc, "acc", i64) if acc is not None else None,
-        _dev(other, "other", i64) if other is not None else None, _stream(),
+        _dev(other, "other", i64) if other is not None else None, _dev(shift, "shift", f32) if shift is not None else None, _stream(),
     )
     if rc == 1:
         return False
@@ -560,7 +594,7 @@ def splitk_reduce(out, partial, bias, splits: int, epi: int) -> None:
     _done(
         _gemm_tc().alofa_splitk_reduce(
             _dev(out, "out"), _dev(partial, "partial", torch.float32), _dev(bias, "bias", torch.float32) if bias is not None else None,
-            t, n, splits, epi, _is_bf16(out, "out"), _stream(),
+            t, n, splits, epi, _is_bf16(out, "out"), 0.0, 0.0, _stream(),
         ),
         "splitk_reduce",
     )
@@ -586,12 +620,12 @@ def _latent():
             "alofa_sandwich_norm": [_P, _P, _P, _F, _P, _P, _F, _I, _I, _I, _I, _L, _P, _P],
             "alofa_concat_rows": [_P, _P, _P, _I, _I, _I, _P],
             "alofa_moe_route": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-            "alofa_moe_router": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _P],
+            "alofa_moe_router": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _I, _P],
             "alofa_cast_rows": [_P, _P, _L, _I, _P],
             "alofa_moe_sort": [_P, _P, _P, _I, _I, _I, _I, _P],
             "alofa_moe_scatter": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
             "alofa_moe_combine": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _I, _P],
-            "alofa_gate_up": [_P, _P, _L, _I, _I, _P],
+            "alofa_gate_up": [_P, _P, _L, _I, _I, _F, _F, _P],
         }
         for name, args in sigs.items():
             fn = getattr(lib, name)
@@ -782,8 +816,9 @@ def gemm_by_tile(out, x, w, tile_batch, tile_rows: int, act: str = "none") -> No
     gemm_batched(out, x, w, 1, rows, n, k, k, 0, k, n * k, n, 0, act=act, tile_batch=tile_batch, tile_rows=tile_rows)
 
 
-def gemm_by_tile_gated(out, x, w, tile_batch, tile_rows: int) -> bool:
-    """``out[rows of tile i] = silu(x_i @ Wg^T) * (x_i @ Wu^T)`` with ``w``
+def gemm_by_tile_gated(out, x, w, tile_batch, tile_rows: int, gate=SILU_GATE) -> bool:
+    """``out[rows of tile i] = silu(x_i @ Wg^T) * (x_i @ Wu^T)`` (or the clamped
+    form, ``gate`` as in :func:`gemm_generic`) with ``w``
     [batches, 2N, K] holding each batch's gate rows before its up rows: the
     tcgen05 product with the gated epilogue.  False, having launched nothing,
     for operands it does not take (the caller then multiplies and gates in
@@ -793,7 +828,7 @@ def gemm_by_tile_gated(out, x, w, tile_batch, tile_rows: int) -> bool:
     if (tile_rows != MOE_TILE_TC or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or k % 8 or rows % 128 or n2 % 2
             or os.environ.get("ALOFA_BY_TILE_TC", "1") == "0"):
         return False
-    return gemm_tc(out, x, w.view(batches * n2, k), None, EPI_GATED, -256, tile_batch=tile_batch, batches=batches)
+    return gemm_tc(out, x, w.view(batches * n2, k), None, EPI_GATED, -256, tile_batch=tile_batch, batches=batches, gate=gate)
 
 
 def moe_route(choice, weight, gate, z, experts: int, top: int, softmax: bool = False, renormalize: bool = False) -> None:
@@ -809,7 +844,7 @@ def moe_route(choice, weight, gate, z, experts: int, top: int, softmax: bool = F
 
 
 def moe_router(choice, weight, gate, x, wr, experts: int, top: int, softmax: bool = False, renormalize: bool = False, correction=None,
-               renorm_eps: float = 0.0, groups: int = 1, keep: int = 1, route_scale: float = 1.0) -> None:
+               renorm_eps: float = 0.0, groups: int = 1, keep: int = 1, route_scale: float = 1.0, group_best: bool = False) -> None:
     """:func:`moe_route` with the router's product in the same kernel: ``x``
     [T, hidden] in the compute dtype, ``wr`` fp32 [experts (+1 with ``gate``),
     hidden]; logits and scores are fp32.  ``correction`` (fp32 [experts]) is
@@ -817,7 +852,7 @@ def moe_router(choice, weight, gate, x, wr, experts: int, top: int, softmax: boo
     ``renorm_eps`` is added to the sum that ``renormalize`` divides by.
     ``groups`` > 1: the experts form that many equal groups of neighbours; a
     group's score is the sum of its two largest choice scores (score +
-    correction), and only experts of the ``keep`` best groups can be chosen.
+    correction; ``group_best``: the largest alone), and only experts of the ``keep`` best groups can be chosen.
     ``route_scale``: a factor on the weights."""
     i32, f32 = torch.int32, torch.float32
     if wr.shape != (experts + (1 if gate is not None else 0), x.shape[1]) or (correction is not None and correction.shape[0] != experts):
@@ -826,7 +861,7 @@ def moe_router(choice, weight, gate, x, wr, experts: int, top: int, softmax: boo
         _latent().alofa_moe_router(_dev(choice, "choice", i32), _dev(weight, "weight", f32), _dev(gate, "gate", f32) if gate is not None else None, _dev(x, "x"),
                                    _dev(wr, "wr", f32), x.shape[0], experts, top, x.shape[1], 1 if softmax else 0, 1 if renormalize else 0, _is_bf16(x, "x"),
                                    _dev(correction, "correction", f32) if correction is not None else None, float(renorm_eps), int(groups), int(keep), float(route_scale),
-                                   _stream()),
+                                   1 if group_best else 0, _stream()),
         "moe_router", f"experts={experts} top={top} groups={groups} keep={keep}",
     )
 
@@ -859,13 +894,14 @@ def moe_combine(y, ys, dest, weight, shared, gate, top: int, x=None, add: bool =
     )
 
 
-def gate_up(mid, gu) -> None:
-    """mid[r, c] = silu(gu[r, c]) * gu[r, ff + c] for rows of fp32 sums that
-    hold gate and up side by side; ``mid`` in its own dtype."""
+def gate_up(mid, gu, gate=SILU_GATE) -> None:
+    """mid[r, c] = silu(gu[r, c]) * gu[r, ff + c] (or the clamped form, ``gate``
+    as in :func:`gemm_generic`) for rows of fp32 sums that hold gate and up
+    side by side; ``mid`` in its own dtype."""
     rows, ff = mid.shape
     if tuple(gu.shape) != (rows, 2 * ff):
         raise AlofaError("invalid_argument", "gate_up sizes disagree", f"mid={tuple(mid.shape)} gu={tuple(gu.shape)}")
-    _done(_latent().alofa_gate_up(_dev(mid, "mid"), _dev(gu, "gu", torch.float32), rows, ff, _is_bf16(mid, "mid"), _stream()), "gate_up")
+    _done(_latent().alofa_gate_up(_dev(mid, "mid"), _dev(gu, "gu", torch.float32), rows, ff, _is_bf16(mid, "mid"), float(gate[0]), float(gate[1]), _stream()), "gate_up")
 
 
 def latent_attention_bf16_supported(kv_rank: int, rot: int) -> bool:
@@ -932,6 +968,7 @@ def _recurrent():
             "alofa_gated_group_norm": [_P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _F, _I, _I, _P],
             "alofa_branch_norm_add": [_P, _P, _P, _P, _P, _I, _I, _F, _F, _P],
             "alofa_qkv_prepare": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _F, _I, _P, _I, _F, _I, _I, _I, _I, _L, _P, _P, _I, _I, _P],
+            "alofa_qkv_prepare_rows": [_P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _I, _L, _P, _P, _I, _I, _P],
             "alofa_heads_finish": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _I, _I, _P],
         }
         for name, args in sigs.items():
@@ -1116,6 +1153,43 @@ def qkv_prepare(q_out, k_cache, v_cache, qkv, positions, slot_map, heads: int, k
     )
 
 
+def _owed_or_finished(qkv, what: str):
+    """(tensor, splits, plane, bias) of a product's output: finished sums [T, ld], or the partial sums it left owed."""
+    if isinstance(qkv, torch.Tensor):
+        return qkv, 0, 0, None
+    sums = qkv.sums
+    if sums.shape[0] != int(qkv.splits) or not sums.is_contiguous():
+        raise AlofaError("invalid_argument", f"{what}: owed sums disagree with their count", f"sums={tuple(sums.shape)} splits={qkv.splits}")
+    return sums[0], int(qkv.splits), sums.shape[1] * sums.shape[2], qkv.bias
+
+
+def qkv_prepare_rows(q_out, k_cache, v_cache, qkv, slot_map, q_weight, k_weight, eps: float, v_first=None, mix=None, extra_out=None, extra_at: int = 0) -> None:
+    """:func:`qkv_prepare` where q and k are each normed over all their heads at
+    once: from rows of fp32 sums [q | k | v | more], ``q / sqrt(mean(q^2) + eps)
+    * q_weight`` (fp32, one number per column) to ``q_out`` [T, nq], k likewise
+    and v to the tokens' cache slots.  ``v_first`` (fp32 [T, nv]): without
+    ``mix`` the values are also left there; with ``mix`` (one fp32 number on the
+    device) they become ``(1 - mix) v + mix v_first`` before they are stored.
+    ``qkv`` may be the partial sums a product left owed, ``extra_out`` /
+    ``extra_at`` are as in :func:`qkv_prepare`."""
+    f32 = torch.float32
+    qkv, splits, plane, bias = _owed_or_finished(qkv, "qkv_prepare_rows")
+    n, nq = q_out.shape
+    dt = q_out.dtype
+    nk, nv = k_cache.shape[1] * k_cache.shape[2], v_cache.shape[1] * v_cache.shape[2]
+    if (qkv.shape[0] != n or qkv.shape[1] < nq + nk + nv or q_weight.shape[0] != nq or k_weight.shape[0] != nk or (v_first is not None and tuple(v_first.shape) != (n, nv))
+            or (mix is not None and (v_first is None or mix.numel() != 1)) or (extra_out is not None and (extra_out.shape[0] != n or extra_at + extra_out.shape[1] > qkv.shape[1]))):
+        raise AlofaError("invalid_argument", "qkv_prepare_rows sizes disagree", f"qkv={tuple(qkv.shape)} q={tuple(q_out.shape)} k={tuple(k_cache.shape)} v={tuple(v_cache.shape)}")
+    opt = lambda t_, name: _dev(t_, name, f32) if t_ is not None else None
+    _done(
+        _recurrent().alofa_qkv_prepare_rows(_dev(q_out, "q_out"), _dev(k_cache, "k_cache", dt), _dev(v_cache, "v_cache", dt), _dev(qkv, "qkv", f32), qkv.shape[1],
+                                            _dev(slot_map, "slot_map", torch.int32), n, nq, nk, nv, _dev(q_weight, "q_weight", f32), _dev(k_weight, "k_weight", f32), float(eps),
+                                            opt(v_first, "v_first"), opt(mix, "mix"), _is_bf16(q_out, "q_out"), splits, plane, opt(bias, "bias"),
+                                            opt(extra_out, "extra_out"), int(extra_at), extra_out.shape[1] if extra_out is not None else 0, _stream()),
+        "qkv_prepare_rows", f"nq={nq} nk={nk} nv={nv}",
+    )
+
+
 def heads_finish(out, a, heads: int, kv_heads: int, dv: int, maps: int = 1, difference: float = 0.0, eps: float = 0.0, post: float = 1.0, gate=None, g_off: int = 0) -> None:
     """What stands between some attentions and their output projection, fp32:
     ``a`` [T, heads * maps * dv] (fp32, or bfloat16 like ``out``) holds the attention outputs in the order
@@ -1221,8 +1295,8 @@ def _delta():
         lib = load_library("alofa_delta", ["kernels/delta.cu"])
         sigs = {
             "alofa_min_gru": [_P, _P, _I, _I, _I, _I, _P, _L, _P, _P, _I, _I, _I, _I, _P],
-            "alofa_delta_prepare": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P],
-            "alofa_delta_scan": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+            "alofa_delta_prepare": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
+            "alofa_delta_scan": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         }
         for name, args in sigs.items():
             fn = getattr(lib, name)
@@ -1253,21 +1327,23 @@ def min_gru(out, u, z_off: int, x_off: int, g_off: int, state, q_start, state_sl
                                  _dev(q_start, "q_start", i32), _dev(state_slots, "state_slots", i32), n_seqs, n, width, _is_bf16(out, "out"), _stream()), "min_gru")
 
 
-def delta_prepare(qn, kn, kq, g, beta, conv, dz, u, b_off: int, dt_bias, a_log, heads: int, groups: int, n: int, unit_eps: float, q_scale: float) -> None:
+def delta_prepare(qn, kn, kq, g, beta, conv, dz, u, b_off: int, dt_bias, a_log, heads: int, groups: int, n: int, unit_eps: float, q_scale: float, dz_off: int = 0) -> None:
     """What :func:`delta_scan` reads, all fp32: from conv [T, ld] = [q: groups *
     n | k: groups * n | v ...] the unit vectors ``qn = q / sqrt(sum q^2 +
     unit_eps) * q_scale`` and ``kn`` (no scale) per group, ``kq = kn . qn``;
     from the first heads * n columns of dz [T, ld''] the decays ``g = exp(-exp(a_log[h]) * softplus(dz +
-    dt_bias))``; from u [T, ld'] ``beta = sigmoid(u[t, b_off + h])``."""
+    dt_bias))`` (``dt_bias`` of ``heads`` numbers: one decay per head, from ``heads`` columns starting at
+    ``dz_off``, g [T, heads]); from u [T, ld'] ``beta = sigmoid(u[t, b_off + h])``."""
     f32 = torch.float32
     rows = conv.shape[0]
-    if (tuple(qn.shape) != (rows, groups * n) or tuple(kn.shape) != (rows, groups * n) or tuple(kq.shape) != (rows, groups) or tuple(g.shape) != (rows, heads * n)
-            or tuple(beta.shape) != (rows, heads) or dz.shape[0] != rows or dz.shape[1] < heads * n or conv.shape[1] < 2 * groups * n or u.shape[0] != rows
-            or b_off + heads > u.shape[1] or dt_bias.shape[0] != heads * n or a_log.shape[0] != heads):
+    decays = dt_bias.shape[0] // heads  # a head's
+    if (tuple(qn.shape) != (rows, groups * n) or tuple(kn.shape) != (rows, groups * n) or tuple(kq.shape) != (rows, groups) or tuple(g.shape) != (rows, heads * decays)
+            or tuple(beta.shape) != (rows, heads) or dz.shape[0] != rows or dz.shape[1] < dz_off + heads * decays or conv.shape[1] < 2 * groups * n or u.shape[0] != rows
+            or b_off + heads > u.shape[1] or decays not in (1, n) or dt_bias.shape[0] != heads * decays or a_log.shape[0] != heads):
         raise AlofaError("invalid_argument", "delta_prepare sizes disagree", f"conv={tuple(conv.shape)} dz={tuple(dz.shape)} heads={heads} groups={groups} n={n}")
     _done(_delta().alofa_delta_prepare(_dev(qn, "qn", f32), _dev(kn, "kn", f32), _dev(kq, "kq", f32), _dev(g, "g", f32), _dev(beta, "beta", f32), _dev(conv, "conv", f32),
-                                       conv.shape[1], _dev(dz, "dz", f32), dz.shape[1], _dev(u, "u", f32), u.shape[1], b_off, _dev(dt_bias, "dt_bias", f32), _dev(a_log, "a_log", f32),
-                                       rows, heads, groups, n, float(unit_eps), float(q_scale), _stream()), "delta_prepare")
+                                       conv.shape[1], _dev(dz, "dz", f32) + 4 * dz_off, dz.shape[1], _dev(u, "u", f32), u.shape[1], b_off, _dev(dt_bias, "dt_bias", f32), _dev(a_log, "a_log", f32),
+                                       rows, heads, groups, n, decays, float(unit_eps), float(q_scale), _stream()), "delta_prepare")
 
 
 def delta_scan(y, v, v_off: int, kn, qn, kq, g, beta, state, q_start, state_slots, n_seqs: int, heads: int, groups: int, n: int, p: int, spread: int = 0) -> None:
@@ -1276,16 +1352,17 @@ def delta_scan(y, v, v_off: int, kn, qn, kq, g, beta, state, q_start, state_slot
     k_t u^T; y_t = S^T q_t``.  The state [slots, >= heads * p * n] (per head
     [p][n]) is read and left up to date; v fp32 [T, ld] at column offset
     ``v_off`` (heads * p columns); head h reads the keys and queries of group
-    ``h // (heads / groups)``."""
+    ``h // (heads / groups)``.  ``g`` [T, heads * n], or [T, heads]: one decay per head."""
     f32, i32 = torch.float32, torch.int32
     rows = y.shape[0]
+    one = n > 1 and tuple(g.shape) == (rows, heads)
     if (tuple(y.shape) != (rows, heads * p) or v.shape[0] != rows or v_off + heads * p > v.shape[1] or tuple(kn.shape) != (rows, groups * n)
-            or tuple(qn.shape) != (rows, groups * n) or tuple(kq.shape) != (rows, groups) or tuple(g.shape) != (rows, heads * n) or tuple(beta.shape) != (rows, heads)):
+            or tuple(qn.shape) != (rows, groups * n) or tuple(kq.shape) != (rows, groups) or (not one and tuple(g.shape) != (rows, heads * n)) or tuple(beta.shape) != (rows, heads)):
         raise AlofaError("invalid_argument", "delta_scan sizes disagree", f"y={tuple(y.shape)} v={tuple(v.shape)} heads={heads} groups={groups} n={n} p={p}")
     _slot_state(state, heads * p * n, "delta_scan")
     _done(_delta().alofa_delta_scan(_dev(y, "y", f32), _dev(v, "v", f32), v.shape[1], v_off, _dev(kn, "kn", f32), _dev(qn, "qn", f32), _dev(kq, "kq", f32), _dev(g, "g", f32),
                                     _dev(beta, "beta", f32), state.data_ptr(), state.stride(0), _dev(q_start, "q_start", i32), _dev(state_slots, "state_slots", i32),
-                                    rows, n_seqs, heads, groups, n, p, spread, _stream()), "delta_scan", f"heads={heads} groups={groups} n={n} p={p}")
+                                    rows, n_seqs, heads, groups, n, p, 1 if one else 0, spread, _stream()), "delta_scan", f"heads={heads} groups={groups} n={n} p={p}")
 
 
 # -- the real-gated linear recurrent unit ------------------------------------------------------------

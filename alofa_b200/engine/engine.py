@@ -89,7 +89,7 @@ class Engine:
         capacity = cfg.capacity_blocks or cfg.max_batch * blocks_per_request
         step_tokens = max(cfg.token_budget, cfg.max_batch, 1)
         self.runner = StepRunner(self.model, cfg.block_size, capacity, cfg.max_batch, self.max_tokens, step_tokens, cfg.cuda_graphs)
-        groups = [(g.block_size, g.window or 0, g.num_pages) for g in self.runner.group_specs]
+        groups = [(g.block_size, g.window or 0, g.num_pages, g.keep_first) for g in self.runner.group_specs]
         self.sched_config = SchedConfig(
             token_budget=cfg.token_budget, max_chunk=min(cfg.max_chunk, step_tokens), max_batch=cfg.max_batch, max_tokens=self.max_tokens,
             watermark_permille=cfg.watermark_permille, max_wait_ticks=cfg.max_wait_ticks, admission=admission, groups=groups,

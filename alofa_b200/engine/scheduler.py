@@ -42,7 +42,8 @@ def _native():
 @dataclass
 class SchedConfig:
     """``groups``: one ``(page_size, window, capacity_pages)`` per cache group
-    (window 0 = all keys).  ``admission``: "committed" admits a request only
+    (window 0 = all keys), or with a fourth number, the first tokens of a
+    request that are kept beside the window.  ``admission``: "committed" admits a request only
     if every live request could grow to its full length beside it (nothing is
     ever preempted); "optimistic" admits while the prompts fit and lets decode
     growth preempt the newest running request."""
@@ -60,8 +61,8 @@ class SchedConfig:
         if self.admission not in ADMISSION:
             raise AlofaError("invalid_argument", "admission must be committed or optimistic", f"admission={self.admission}")
         out = [self.token_budget, self.max_chunk, self.max_batch, self.max_tokens, self.watermark_permille, self.max_wait_ticks, ADMISSION[self.admission], len(self.groups)]
-        for ps, win, cap in self.groups:
-            out += [ps, win or 0, cap]
+        for ps, win, cap, *keep in self.groups:
+            out += [ps, win or 0, cap, keep[0] if keep else 0]
         return out
 
 
@@ -180,7 +181,7 @@ def _triples(values) -> str:
 def format_config(cfg: SchedConfig) -> str:
     return (
         f"CFG b={cfg.token_budget} c={cfg.max_chunk} n={cfg.max_batch} m={cfg.max_tokens} w={cfg.watermark_permille} "
-        f"t={cfg.max_wait_ticks} a={ADMISSION[cfg.admission]} G={_triples([(p, w or 0, c) for p, w, c in cfg.groups])}"
+        f"t={cfg.max_wait_ticks} a={ADMISSION[cfg.admission]} G={_triples([(p, w or 0, c, *(k for k in keep if k)) for p, w, c, *keep in cfg.groups])}"
     )
 
 

@@ -75,7 +75,7 @@ class StepRunner:
         windows = group_windows(plan)
         if isinstance(num_pages, int):
             num_pages = [num_pages] * len(windows)
-        self.group_specs = [GroupSpec(block_size, n, w) for n, w in zip(num_pages, windows)]
+        self.group_specs = [GroupSpec(block_size, n, w, keep) for n, (w, keep) in zip(num_pages, windows)]
         self.manager = CacheManager(self.group_specs, max_requests, self.max_tokens)
         self.storage = CacheStorage(plan, self.group_specs, max_requests, self.rt.dtype, self.rt.device)
         self.has_paged = any(isinstance(s, (PagedKV, PagedRows)) for s in flat_specs(plan))

@@ -30,13 +30,19 @@ class PagedAttend:
     split over CTAs.  The mixer gives ``nh``, ``nkv``, ``hd`` (keys and values
     alike), ``q_dim``, ``window``, ``scale``, ``softcap`` (0: none), ``sink``
     (None, or a score per head that the softmax's denominator holds beside the
-    keys': the kernel that completes a row's sum adds it) and ``chunk`` (0, or
+    keys': the kernel that completes a row's sum adds it), ``chunk`` (0, or
     the size of the chunks, counted from the sequence's start, that a query
-    does not see out of; the kernels take it as a negative window)."""
+    does not see out of; the kernels take it as a negative window),
+    ``keep_first`` (keys before it are seen beside the window), ``slopes``
+    (None, or a number per head: that times the distance of query and key is
+    taken off the score) and ``vd`` (the values' head size, None: the keys')."""
 
     softcap = 0.0
     sink = None
     chunk = 0
+    keep_first = 0
+    slopes = None
+    vd = None
 
     # Keys per CTA, at least, when a decode-only step splits each request's keys: four 64-key
     # blocks, one per warp.  Splits grow in steps of this (a warp then takes several blocks in
@@ -89,44 +95,54 @@ class PagedAttend:
             per_split = max(per_split, unit * -(-longest // (unit * cls.MERGE_IN_PRODUCT_SPLITS)))
         return per_split
 
-    def attend(self, ctx, q, cache, group):
+    def attend(self, ctx, q, cache, group, gate=None):
         """Attention of the step's rows over the cache: the tensor-core kernels
         for bfloat16 and head sizes they are built for, else the generic one.
         Returns the output rows, or a :class:`MergedSplits` for the product
-        that follows to merge."""
-        out = ctx.buf((q.shape[0], self.q_dim), q.dtype)
-        if q.dtype == torch.bfloat16 and ops.attention_bf16_supported(self.hd):
+        that follows to merge.  ``gate``: (fp32 sums of a projection, the heads'
+        first column) whose sigmoid multiplies every head's output (the
+        tensor-core kernels only)."""
+        vd = self.vd or self.hd
+        out = ctx.buf((q.shape[0], self.nh * vd), q.dtype)
+        if q.dtype == torch.bfloat16 and ops.attention_bf16_supported(self.hd, vd):
             splits, po, pml = 0, None, None
-            longest = ctx.max_context if ctx.capturing else ctx.max_kv_len
+            longest, longest_now = ctx.max_context if ctx.capturing else ctx.max_kv_len, ctx.max_kv_len
+            reach = longest  # the longest context
+            if self.keep_first and ctx.decode_only:
+                # key splits then go by the blocks a request can see: those of the kept keys, and those its window touches
+                seen = 64 * (-(-self.keep_first // 64) + (self.window + 62) // 64 + 1)
+                longest, longest_now = min(longest, seen), min(longest_now, seen)
+            distance = self.slopes is not None
             per_split = self.SPLIT_KEYS
             group_size = self.nh // self.nkv
             if ctx.decode_only and group_size <= 16:
                 capped = self.softcap > 0
-                wide_warps = ops.attention_decode_wide_warps(self.hd, capped)
-                per_split = self.decode_split_keys(ctx.n_tokens, ctx.n_seqs * self.nkv, longest, ctx.max_kv_len,
-                                                   ops.attention_decode_slots(self.hd, group.page_size, wide_warps, capped) if wide_warps else 0,
-                                                   ops.attention_decode_slots(self.hd, group.page_size, 4, capped), 64 * wide_warps)
+                wide_warps = ops.attention_decode_wide_warps(self.hd, capped, vd, distance)
+                per_split = self.decode_split_keys(ctx.n_tokens, ctx.n_seqs * self.nkv, longest, longest_now,
+                                                   ops.attention_decode_slots(self.hd, group.page_size, wide_warps, capped, vd, distance) if wide_warps else 0,
+                                                   ops.attention_decode_slots(self.hd, group.page_size, 4, capped, vd, distance), 64 * wide_warps)
             if not ctx.decode_only:
                 per_split = self.PROMPT_SPLIT_KEYS or (1 << 30)
             if ctx.decode_only and self.nh // self.nkv <= 64 and (longest > per_split or self.nh // self.nkv <= 16):
                 splits = max(1, -(-longest // per_split))
-            elif not ctx.decode_only and longest > per_split:
+            elif not ctx.decode_only and longest > per_split and not self.keep_first:
                 splits = -(-longest // per_split)
             if splits:
-                po = ctx.buf((splits, ctx.n_tokens * self.nh, self.hd), torch.float32)
+                po = ctx.buf((splits, ctx.n_tokens * self.nh, vd), torch.float32)
                 pml = ctx.buf((splits, ctx.n_tokens * self.nh, 2), torch.float32)
-            unmerged = ctx.decode_only and 1 < splits <= self.MERGE_IN_PRODUCT_SPLITS and self.nh // self.nkv <= 16 and ctx.n_tokens <= 16 and self.sink is None and not self.chunk
+            plain = self.sink is None and gate is None and not self.chunk and not self.keep_first  # nothing is done to a row once it is complete
+            unmerged = ctx.decode_only and 1 < splits <= self.MERGE_IN_PRODUCT_SPLITS and self.nh // self.nkv <= 16 and ctx.n_tokens <= 16 and plain
             ops.attention_bf16(
                 out, q, cache.k, cache.v, ctx.q_start, ctx.kv_len, ctx.positions, group.block_table, group.page_size, ctx.n_seqs, ctx.max_q_len,
-                self.nh, self.nkv, self.hd, -self.chunk if self.chunk else self.window, self.scale, splits, per_split, po, pml, longest, ctx.status, combine=not unmerged, softcap=self.softcap,
-                sink=self.sink,
+                self.nh, self.nkv, self.hd, -self.chunk if self.chunk else self.window, self.scale, splits, per_split, po, pml, reach, ctx.status, combine=not unmerged, softcap=self.softcap,
+                sink=self.sink, keep=self.keep_first, slopes=self.slopes, gate=gate[0] if gate else None, gate_at=gate[1] if gate else 0,
             )
             if unmerged:
-                return MergedSplits(po, pml, ctx.positions, ctx.n_tokens, self.nh, self.hd, self.window, per_split, ctx.buf, capped=self.softcap > 0)
+                return MergedSplits(po, pml, ctx.positions, ctx.n_tokens, self.nh, vd, self.window, per_split, ctx.buf, capped=self.softcap > 0, key_dim=self.hd, distance=distance)
             return out
         ops.paged_attention_generic(
             out, q, cache.k, cache.v, ctx.positions, ctx.seq_of_token, group.block_table, group.page_size,
-            self.nh, self.nkv, self.hd, self.window, self.scale, self.softcap, None, self.sink, self.chunk,
+            self.nh, self.nkv, self.hd, self.window, self.scale, self.softcap, vd, self.sink, self.chunk, 1, self.keep_first, self.slopes,
         )
         return out
 

@@ -18,7 +18,8 @@ norm_a(mixer(h)); h += norm_b(feed_forward(h))``; the sublayers read the
 stream itself (the feed-forward may be absent).
 
 ``prenorm_residual``: ``h += mixer(norm_a(h)); h += feed_forward(norm_b(h))``
-(src/alofa/model/arch/qwen.mojo:1367-1372, 1418-1510).  The residual stream
+(the feed-forward may be absent;
+src/alofa/model/arch/qwen.mojo:1367-1372, 1418-1510).  The residual stream
 ``h`` is fp32; the parts add into it."""
 from __future__ import annotations
 
@@ -36,12 +37,14 @@ class PrenormResidual(Part):
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
         self.mixer = build_part("mixer", self.param("mixer"), rt)
-        self.feed_forward = build_part("feed_forward", self.param("feed_forward"), rt)
         self.mixer_norm = build_part("norm", self.param("mixer_norm"), rt)
-        self.feed_forward_norm = build_part("norm", self.param("feed_forward_norm"), rt)
+        ff = self.params.get("feed_forward")
+        self.feed_forward = build_part("feed_forward", ff, rt) if ff is not None else None
+        self.feed_forward_norm = build_part("norm", self.param("feed_forward_norm"), rt) if ff is not None else None
+        self.shared_value_width = getattr(self.mixer, "shared_value_width", 0)  # the model keeps a step's first values for mixers that mix theirs with them
 
     def parts(self):
-        return (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None)
 
     def tensors(self):
         out = {}
@@ -77,6 +80,8 @@ class PrenormResidual(Part):
     def forward(self, ctx, h, cache, writes=True):
         x = self._norm(self.mixer_norm, ctx, h, self.mixer)
         self.mixer.forward(ctx, x, h, cache, writes)
+        if self.feed_forward is None:
+            return
         x = self._norm(self.feed_forward_norm, ctx, h, self.feed_forward)
         self.feed_forward.forward(ctx, x, h)
 

@@ -111,7 +111,7 @@ def plan(linear):
             partial = buf(shape, torch.float32) if buf is not None else torch.empty(shape, dtype=torch.float32, device=w.device)
         deferred = defer and splits > 1 and n_acc == 1 and acc is None and not linear.act  # whoever adds deferred sums up applies no activation
         dst = partial[0] if deferred else out  # a deferred product writes partial sums only
-        if not ops.gemm_tc(dst, x, w, linear.bias, linear.epi, bn, splits, partial, reduce=not deferred, computed=computed, acc=acc, act=linear.act):
+        if not ops.gemm_tc(dst, x, w, linear.bias, linear.epi, bn, splits, partial, reduce=not deferred, computed=computed, acc=acc, act=linear.act, gate=linear.gate):
             if normed:
                 lazy.undo()
                 return run(out, lazy.rows(), defer, buf)

@@ -50,13 +50,31 @@ class GatedMLP(Part):
         add_into_stream(ctx, self.down, h, act)
 
 
+def gate_form(params: dict, activation: str) -> tuple:
+    """(alpha, limit) of a gated feed-forward for :func:`ops.gemm_generic`: the
+    plain silu gate, or the clamped one with its ``gate_alpha`` and
+    ``gate_limit`` (absent: no limit)."""
+    if activation == "silu":
+        return ops.SILU_GATE
+    if activation != "clamped_silu":
+        raise AlofaError("unsupported", "a gated feed-forward takes the silu or clamped_silu activation", f"activation={activation}")
+    alpha, limit = float(params.get("gate_alpha") or 0.0), params.get("gate_limit")
+    limit = float("inf") if limit is None else float(limit)
+    if not alpha > 0 or not limit > 0:
+        raise AlofaError("invalid_argument", "a clamped gate needs a positive alpha and limit", f"alpha={alpha} limit={limit}")
+    return alpha, limit
+
+
 class DenseMLP(Part):
     """``Wdown act(Wup x (+ bup)) (+ bdown)`` with tensors ``<prefix>up``,
     ``<prefix>down`` (``.b`` for the biases); ``activation``: gelu_erf (the
     exact one), gelu_tanh, silu, relu.  The activation is taken on the fp32
     sums, before they are rounded to the compute dtype.  ``gated``: ``Wdown
     (silu(Wgate x) * (Wup x))`` with a third tensor ``<prefix>gate``, no
-    biases (gate and up are one product whose epilogue multiplies them)."""
+    biases (gate and up are one product whose epilogue multiplies them);
+    ``activation`` "clamped_silu" with ``gate_alpha`` and ``gate_limit``: ``g =
+    min(Wgate x, limit), u = clamp(Wup x, -limit, limit), Wdown (g sigmoid(alpha
+    g) (u + 1))``."""
 
     family = "feed_forward"
     graph_safe = True
@@ -70,11 +88,12 @@ class DenseMLP(Part):
         self.act = str(self.param("activation", "gelu_erf"))
         self.bias = bool(self.params.get("bias", False))
         self.gated = bool(self.params.get("gated", False))
-        if self.act not in ops.ACTIVATIONS:
+        self.gate = gate_form(self.params, self.act) if self.gated else ops.SILU_GATE
+        if not self.gated and self.act not in ops.ACTIVATIONS:
             raise AlofaError("unsupported", "unknown activation", f"activation={self.act} known={sorted(ops.ACTIVATIONS)}")
-        if self.gated and (self.act != "silu" or self.bias):
-            raise AlofaError("unsupported", "a gated feed-forward takes the silu activation and no biases", f"activation={self.act} bias={self.bias}")
-        self.up = self.down = None
+        if self.gated and self.bias:
+            raise AlofaError("unsupported", "a gated feed-forward takes no biases", f"activation={self.act}")
+        self.up = self.down = self.down_add = None
 
     def tensors(self):
         pre = self.prefix
@@ -89,7 +108,8 @@ class DenseMLP(Part):
     def load(self, state):
         pre = self.prefix
         if self.gated:  # gate rows first, then up rows
-            self.up = Linear(torch.cat([state[pre + "gate"], state[pre + "up"]], dim=0), None, GATED)
+            self.up = Linear(torch.cat([state[pre + "gate"], state[pre + "up"]], dim=0), None, GATED, gate=self.gate)
+            self.down_add = Linear(state[pre + "down"], None, RESIDUAL)
         else:
             self.up = Linear(state[pre + "up"], as_float32_vector(state[pre + "up.b"]) if self.bias else None, STORE, act=self.act)
         self.down = Linear(state[pre + "down"], as_float32_vector(state[pre + "down.b"]) if self.bias else None, STORE)
@@ -103,6 +123,8 @@ class DenseMLP(Part):
         self.up(mid, x, buf=ctx.buf)  # bias and activation on the fp32 sums, in the product's epilogue
         if store:
             return self.down(h, mid, defer=defer, buf=ctx.buf)  # None, or the split sums a caller that asked for them adds up itself
+        if self.gated:
+            add_into_stream(ctx, self.down_add, h, mid)
         else:
             y = ctx.buf((n, self.hidden), torch.float32)
             self.down(y, mid, buf=ctx.buf)

@@ -43,10 +43,10 @@ class MergedSplits:
 
     dtype = torch.bfloat16
 
-    def __init__(self, partial_o, partial_ml, positions, tokens: int, heads: int, head_dim: int, window, split_keys: int, buf, capped: bool = False):
+    def __init__(self, partial_o, partial_ml, positions, tokens: int, heads: int, head_dim: int, window, split_keys: int, buf, capped: bool = False, key_dim=None, distance: bool = False):
         self.partial_o, self.partial_ml, self.positions = partial_o, partial_ml, positions
         self.buf = buf  # the step's scratch allocator
-        self.capped = capped  # the splits came from the library built for capped scores
+        self.library = {"capped": capped, "key_dim": key_dim, "distance": distance}  # the attention library the splits came from
         self.heads, self.head_dim, self.window, self.split_keys = heads, head_dim, window, split_keys
         self.shape = (tokens, heads * head_dim)
 
@@ -58,7 +58,7 @@ class MergedSplits:
 
     def rows(self) -> torch.Tensor:
         out = self.buf(self.shape, torch.bfloat16)
-        ops.attention_combine(out, self.partial_o, self.partial_ml, self.positions, self.heads, self.head_dim, self.window, self.split_keys, capped=self.capped)
+        ops.attention_combine(out, self.partial_o, self.partial_ml, self.positions, self.heads, self.head_dim, self.window, self.split_keys, **self.library)
         return out
 
 
@@ -111,12 +111,14 @@ ACCUMULATED = object()  # what a residual product returns when it added its sums
 class Linear:
     """``epi`` STORE: out = act(x W^T + b), ``act`` a name of
     ``ops.ACTIVATIONS`` taken on the fp32 sums.  RESIDUAL: out (fp32) += x W^T
-    + b.  GATED: W = [gate; up]: out = silu(x Wg^T) * (x Wu^T)."""
+    + b.  GATED: W = [gate; up]: out = silu(x Wg^T) * (x Wu^T), or with ``gate``
+    = (alpha, limit) the clamped form of :func:`ops.gemm_generic`."""
 
-    def __init__(self, weight: torch.Tensor, bias, epi: int = STORE, act: str = "none"):
+    def __init__(self, weight: torch.Tensor, bias, epi: int = STORE, act: str = "none", gate=ops.SILU_GATE):
         self.weight = weight.contiguous()
         self.bias = bias
         self.epi = epi
+        self.gate = gate
         self.act = ops.ACTIVATIONS[act]
         if self.act and epi != STORE:
             raise AlofaError("invalid_argument", "only a stored product takes an activation", f"epi={epi} act={act}")
@@ -155,7 +157,7 @@ class Linear:
                 return done if isinstance(done, Partial) else None
         if not isinstance(x, torch.Tensor):
             x = x.rows()
-        ops.gemm_generic(out, x, self.weight, self.bias, self.epi, self.act)
+        ops.gemm_generic(out, x, self.weight, self.bias, self.epi, self.act, self.gate)
         return None
 
 

@@ -28,6 +28,11 @@ class Model:
         # a block may read the embedding output of the step's tokens later on (ctx.embedding_output)
         self.keeps_embedding = any(getattr(block, "needs_embedding_output", False) for block in self.layers)
         # blocks that keep several copies of the residual stream say how many (ctx.streams); every block of a model says the same
+        # mixers that mix their values with those of the first of them: the values of a step's tokens are kept for it (ctx.first_values)
+        widths = {int(getattr(block, "shared_value_width", 0)) for block in self.layers} - {0}
+        if len(widths) > 1:
+            raise AlofaError("unsupported", "layers that mix their values must have the same number of them", f"widths={sorted(widths)}")
+        self.shared_value_width = widths.pop() if widths else 0
         copies = {int(getattr(block, "stream_copies", 0)) for block in self.layers}
         if len(copies) > 1:
             raise AlofaError("unsupported", "blocks over several residual streams cannot be mixed with others", f"stream_copies={sorted(copies)}")
@@ -56,7 +61,7 @@ class Model:
         layer that needs most): what the step runner sizes its arena from."""
         hidden = self.spec.hidden_size
         per_layer = max([getattr(block, "scratch_row_bytes", lambda: 0)() for block in self.layers] + [8 * hidden])
-        return 4 * hidden + 4 * hidden + (4 * hidden if self.keeps_embedding else 0) + (4 * hidden * self.stream_copies if self.stream_copies > 1 else 0), per_layer
+        return 4 * hidden + 4 * hidden + (4 * hidden if self.keeps_embedding else 0) + 4 * self.shared_value_width + (4 * hidden * self.stream_copies if self.stream_copies > 1 else 0), per_layer
 
     def cache_plan(self) -> dict:
         """run index -> cache spec, for the entries that own a cache."""
@@ -72,6 +77,8 @@ class Model:
         if self.keeps_embedding:
             ctx.embedding_output = ctx.buf(tuple(h.shape), torch.float32)
             ctx.embedding_output.copy_(h)
+        if self.shared_value_width:
+            ctx.first_values = ctx.buf((ctx.n_tokens, self.shared_value_width), torch.float32)
         if self.stream_copies:
             ctx.open_streams(h, self.stream_copies)
         for i, (layer, cache) in enumerate(self.run):

@@ -1,6 +1,8 @@
 """RMSNorm: ``y = x / sqrt(mean(x^2) + eps) * w`` per row, fp32 sums; no bias,
 no mean subtraction, the weight is used as stored
-(src/alofa/kernels/cpu/scalar.mojo:93-129)."""
+(src/alofa/kernels/cpu/scalar.mojo:93-129).  Layer norm: ``y = (x - mean) /
+sqrt(variance + eps) * w + b``, the variance being the mean of the squared
+deviations, ``b`` the tensor of the weight's name with ``.b`` added."""
 from __future__ import annotations
 
 import torch
@@ -20,6 +22,7 @@ class RMSNorm(Part):
         self.eps = float(self.param("eps"))
         self.name = self.prefix + str(self.params.get("weight_name", "weight"))  # the tensor's name: prefix + "weight" unless the spec says otherwise
         self.weight = None
+        self.shift = None  # a layer norm's bias
 
     def tensors(self):
         return {self.name: TensorSpec((self.size,), "ones")}
@@ -49,7 +52,7 @@ class RMSNorm(Part):
         pend = ctx.take_pending(h)
         if pend is not None and pend.acc is not None:
             acc, other = ctx.accumulators(h, pend)
-            if rows is None and ops.norm_fused(out, h, self.weight, self.eps, None, base=pend.base if pend.base is not h else None, acc=acc, other=other):
+            if rows is None and ops.norm_fused(out, h, self.weight, self.eps, None, base=pend.base if pend.base is not h else None, acc=acc, other=other, shift=self.shift):
                 return out
             ops.stream_settle(h, pend.base, acc, other)  # picked rows, or a width the fused kernel refuses: the whole stream first
             pend = None
@@ -60,15 +63,30 @@ class RMSNorm(Part):
             owed = pend.partial
             base = pend.base if pend.base is not h else None
             if rows is None or base is None:
-                if ops.norm_fused(out, h, self.weight, self.eps, rows, owed.sums, owed.splits, owed.bias, base=base if rows is None else None):
+                if ops.norm_fused(out, h, self.weight, self.eps, rows, owed.sums, owed.splits, owed.bias, base=base if rows is None else None, shift=self.shift):
                     return out
             if base is not None:
                 h.copy_(base)
             ops.splitk_reduce(h, owed.sums, owed.bias, owed.splits, ops.EPI_RESIDUAL)
-        if self.rt.dtype == torch.bfloat16 and ops.norm_fused(out, h, self.weight, self.eps, rows):
+        if self.rt.dtype == torch.bfloat16 and ops.norm_fused(out, h, self.weight, self.eps, rows, shift=self.shift):
             return out
-        ops.rmsnorm(out, h, self.weight, self.eps, rows)
+        ops.rmsnorm(out, h, self.weight, self.eps, rows, self.shift)
         return out
 
 
+class LayerNorm(RMSNorm):
+    gives_normed_rows = False  # no product makes these rows itself
+
+    def tensors(self):
+        return {self.name: TensorSpec((self.size,), "ones"), self.name + ".b": TensorSpec((self.size,))}
+
+    def load(self, state):
+        super().load(state)
+        self.shift = as_float32_vector(state[self.name + ".b"])
+
+    def forward(self, ctx, h, rows=None, lazy=False):
+        return self.rows_now(ctx, h, rows)
+
+
 register_part("norm", "rmsnorm", RMSNorm)
+register_part("norm", "layernorm", LayerNorm)

@@ -4,7 +4,9 @@ options of designs that take positions in by other means:
 * ``qk_norm``: q and k are divided by their root mean square over the head's
   channels (eps inside the root); with ``norm_weight`` then multiplied by a
   plain weight of ``dim`` numbers, one for the queries and one for the keys
-  (``q.norm``, ``k.norm``), shared by all heads;
+  (``q.norm``, ``k.norm``), shared by all heads; ``norm_over`` "projection":
+  by the root mean square over all heads' channels at once, times a weight of
+  that size;
 * ``q_temp_coef`` / ``q_temp_every``: the query at position p is multiplied by
   ``1 + coef * ln(floor((p + 1) / every) + 1)``;
 * ``scale``: scores are ``(q . k) * scale``;
@@ -13,7 +15,16 @@ options of designs that take positions in by other means:
 * ``position``: a position part whose rotation (neighbouring pairs, angles in
   fp32 in the kernel) turns the first dimensions of every q and k head;
 * ``sink``: the softmax's denominator holds one more term ``exp(sink)`` that
-  belongs to no key and has no value (0.0: "one added to the denominator");
+  belongs to no key and has no value (0.0: "one added to the denominator";
+  "learned": a number per head, tensor ``sink``);
+* ``distance_bias``: ``slope_h * (i - j)`` is taken off the (scaled, capped) score
+  of query i and key j, ``slope_h = 2^(-8 (h + 1) / heads)``;
+* ``window`` with ``keep_first``: query i sees key j when ``i - j < window`` or
+  ``j < keep_first``;
+* ``value_mix``: "first": this layer's values, as projected, are left in
+  ``ctx.first_values``; "later": ``v <- (1 - m) v + m v_first`` with one number m
+  (tensor ``vmix``, which the first such layer has too but does not use) before
+  the values are cached;
 * ``values`` "keys": there is no value projection, the values are the keys
   as projected, before their norm;
 * ``gate``: head h's output is multiplied by ``sigmoid(W_g x)_h`` (``g``
@@ -67,7 +78,12 @@ class NormedAttention(PagedAttend, Part):
         self.every = int(self.params.get("q_temp_every") or 1)
         self.window = self.params.get("window")
         self.bias = bool(self.params.get("bias", False))
-        self.sink_score = self.params.get("sink")  # None: no sink
+        self.sink_score = self.params.get("sink")  # None: no sink; "learned": a tensor
+        self.norm_rows = str(self.params.get("norm_over", "head")) == "projection"
+        self.distance_bias = bool(self.params.get("distance_bias", False))
+        self.keep_first = int(self.params.get("keep_first") or 0) if self.window else 0  # every key is visible anyway without a window
+        self.value_mix = self.params.get("value_mix")  # None, "first" or "later"
+        self.mix = None
         self.sink = None
         self.norm_weight = bool(self.params.get("norm_weight", False))
         self.values_from_keys = str(self.params.get("values", "projected")) == "keys"
@@ -92,6 +108,12 @@ class NormedAttention(PagedAttend, Part):
             raise AlofaError("invalid_argument", "keys that are also the values have the values' size", f"dim={self.dim} vdim={self.vdim}")
         if self.chunk < 0 or (self.chunk and self.window):
             raise AlofaError("invalid_argument", "a chunked mask takes a positive size and no window beside it", f"chunk={self.chunk} window={self.window}")
+        if self.norm_rows and (not self.norm_weight or self.maps > 1 or self.values_from_keys or self.position is not None or self.coef):
+            raise AlofaError("unsupported", "norms over the whole projection have weights, one map a head, values of their own and no rotation or temperature", f"params={self.params}")
+        if self.value_mix not in (None, "first", "later") or (self.value_mix and not self.norm_rows):
+            raise AlofaError("unsupported", "values are mixed by the kernel that norms whole projections", f"params={self.params}")
+        if self.keep_first < 0 or (self.distance_bias and self.maps > 1):
+            raise AlofaError("invalid_argument", "keep_first must not be negative, and two maps a head take no distance bias", f"params={self.params}")
         if self.norm_weight and not self.qk_norm:
             raise AlofaError("invalid_argument", "a norm's weight needs the norm", f"params={self.params}")
         if self.every <= 0 or self.softcap < 0:
@@ -101,14 +123,16 @@ class NormedAttention(PagedAttend, Part):
         self.rows = self.q_dim + self.k_dim + self.v_dim + (self.heads if self.gate else 0)  # [q | k | v | gate]
         # the bfloat16 tensor-core kernels take keys and values of one size and as many value heads as key heads: with several maps a
         # head the values are then kept once per map (the every-size kernel reads one value head for all of a key head's maps)
-        self.tensor_cores = rt.dtype == torch.bfloat16 and self.dim == self.vdim and ops.attention_bf16_supported(self.dim)
+        self.tensor_cores = (rt.dtype == torch.bfloat16 and (self.dim == self.vdim or self.maps == 1) and ops.attention_bf16_supported(self.dim, self.vdim)
+                             and (self.scale > 0 or not self.distance_bias))  # there the bias is taken off in units of the scale
         self.v_copies = self.maps if self.tensor_cores else 1
-        self.nh, self.nkv, self.hd = self.heads * self.maps, self.kv_heads * self.maps, self.dim  # what the shared choice of kernels goes by (keys and values alike only)
+        self.nh, self.nkv, self.hd, self.vd = self.heads * self.maps, self.kv_heads * self.maps, self.dim, self.vdim  # what the shared choice of kernels goes by
+        self.shared_value_width = self.v_dim if self.value_mix else 0
 
     def cache_spec(self):
         # a chunk never reaches further back than its own size: the pages behind it are given back like a window's
         value_heads = self.kv_heads * self.v_copies
-        return PagedKV(self.kv_heads * self.maps, self.dim, self.chunk or self.window, self.vdim, None if value_heads == self.kv_heads * self.maps else value_heads)
+        return PagedKV(self.kv_heads * self.maps, self.dim, self.chunk or self.window, self.vdim, None if value_heads == self.kv_heads * self.maps else value_heads, self.keep_first)
 
     def scratch_row_bytes(self) -> int:
         return 4 * self.rows + 4 * self.q_dim + 4 * (self.maps + 1) * self.heads * self.vdim + 8 * self.hidden
@@ -121,7 +145,12 @@ class NormedAttention(PagedAttend, Part):
         if self.bias:
             t.update({pre + n + ".b": TensorSpec((t[pre + n].shape[0],)) for n in self._stacked()})
         if self.norm_weight:
-            t.update({pre + "q.norm": TensorSpec((self.dim,), "ones"), pre + "k.norm": TensorSpec((self.dim,), "ones")})
+            sizes = (self.q_dim, self.k_dim) if self.norm_rows else (self.dim, self.dim)
+            t.update({pre + "q.norm": TensorSpec((sizes[0],), "ones"), pre + "k.norm": TensorSpec((sizes[1],), "ones")})
+        if self.sink_score == "learned":
+            t[pre + "sink"] = TensorSpec((self.heads,))
+        if self.value_mix:
+            t[pre + "vmix"] = TensorSpec(())
         if self.gate:
             t[pre + "g"] = TensorSpec((self.heads, self.hidden))
         if self.out_bias:
@@ -144,7 +173,13 @@ class NormedAttention(PagedAttend, Part):
         if self.position is not None:
             self.position.load(state)
         dev = state[pre + "o"].device
-        if self.sink_score is not None:
+        if self.distance_bias:
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)], dtype=torch.float64).to(torch.float32).to(dev)
+        if self.value_mix == "later":
+            self.mix = as_float32_vector(state[pre + "vmix"].reshape(1))
+        if self.sink_score == "learned":
+            self.sink = as_float32_vector(state[pre + "sink"])
+        elif self.sink_score is not None:
             self.sink = torch.full((self.heads,), float(self.sink_score), dtype=torch.float32, device=dev)
         if self.norm_weight:
             self.q_weight, self.k_weight = as_float32_vector(state[pre + "q.norm"]), as_float32_vector(state[pre + "k.norm"])
@@ -170,25 +205,29 @@ class NormedAttention(PagedAttend, Part):
         gates, gates_at = (sums, g_off) if self.gate else (None, 0)
         if owed is not None and self.gate:
             gates, gates_at = ctx.buf((n, self.heads), torch.float32), 0  # the gates' logits, finished, for the kernel after the attention
-        ops.qkv_prepare(q, cache.k, cache.v, sums if owed is None else owed, ctx.positions, group.slot_map, self.heads, self.kv_heads, self.dim, self.vdim, self.qk_norm,
-                        self.eps, self.coef, self.every, self.position.frequencies() if rotated else None, self.rot_dims, self.maps, self.q_weight, self.k_weight,
-                        float(getattr(self.position, "magnitude", 1.0)) if rotated else 1.0, self.values_from_keys, self.v_copies,
-                        gates if owed is not None and self.gate else None, g_off)
-        if self.tensor_cores or (self.dim == self.vdim and self.maps == 1 and not self.chunk):
-            out = self.attend(ctx, q, cache, group)  # the tensor-core kernels in bfloat16 for the head sizes they are built for, else the every-size kernel
-            if (self.gate or self.maps > 1) and not isinstance(out, torch.Tensor):
-                out = out.rows()
+        if self.norm_rows:
+            ops.qkv_prepare_rows(q, cache.k, cache.v, sums if owed is None else owed, group.slot_map, self.q_weight, self.k_weight, self.eps,
+                                 ctx.first_values if self.value_mix else None, self.mix, gates if owed is not None and self.gate else None, g_off)
+        else:
+            ops.qkv_prepare(q, cache.k, cache.v, sums if owed is None else owed, ctx.positions, group.slot_map, self.heads, self.kv_heads, self.dim, self.vdim, self.qk_norm,
+                            self.eps, self.coef, self.every, self.position.frequencies() if rotated else None, self.rot_dims, self.maps, self.q_weight, self.k_weight,
+                            float(getattr(self.position, "magnitude", 1.0)) if rotated else 1.0, self.values_from_keys, self.v_copies,
+                            gates if owed is not None and self.gate else None, g_off)
+        if self.tensor_cores:
+            # the tensor-core kernels, which multiply a head's gate in where they complete its rows
+            out = self.attend(ctx, q, cache, group, (gates, gates_at) if self.gate and self.maps == 1 else None)
             if self.maps > 1:
+                if not isinstance(out, torch.Tensor):
+                    out = out.rows()
                 a, out = out, ctx.buf((n, self.heads * self.vdim), dt)
                 ops.heads_finish(out, a, self.heads, self.kv_heads, self.vdim, self.maps, self.difference, self.eps, 1.0 - self.diff, gates, gates_at)
-            elif self.gate:
-                ops.head_gate(out, gates, gates_at, self.heads, self.vdim)
         else:
             # the every-size kernel; what is still to be combined or gated stays fp32 until it has been
             plain = self.maps == 1 and not self.gate
             a = ctx.buf((n, self.heads * self.maps * self.vdim), dt if plain else torch.float32)
             ops.paged_attention_generic(a, q, cache.k, cache.v, ctx.positions, ctx.seq_of_token, group.block_table, group.page_size, self.heads * self.maps,
-                                        self.kv_heads * self.maps, self.dim, self.window, self.scale, self.softcap, self.vdim, self.sink, self.chunk, self.maps)
+                                        self.kv_heads * self.maps, self.dim, self.window, self.scale, self.softcap, self.vdim, self.sink, self.chunk, self.maps,
+                                            self.keep_first, self.slopes)
             out = a
             if not plain:
                 out = ctx.buf((n, self.heads * self.vdim), dt)

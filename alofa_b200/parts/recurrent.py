@@ -36,7 +36,10 @@ convolution per channel (no bias) and silu, q and k are made unit vectors per
 head (q also times ``dim^(-1/2)``), ``beta = sigmoid(W_b h)``, ``g =
 exp(-exp(A_log) * softplus(W_a2 (W_a1 h) + dt_bias))``; every head's output is
 RMS-normed over its value channels with one weight shared by the heads and
-multiplied by ``sigmoid(W_g2 (W_g1 h))``, then projected.
+multiplied by ``sigmoid(W_g2 (W_g1 h))``, then projected.  Options:
+``decay_per`` "head" (one decay per head, ``dt_bias`` of ``heads`` numbers),
+``low_rank`` False (the decays' and the gate's logits are ``W_a h`` and ``W_g
+h``, in one stacked projection with q, k, v and beta), ``gate`` "silu".
 
 ``gated_lru``: the recurrent block with a real-gated linear recurrent unit.
 Two branches of ``width`` channels: ``y = act(W_y h + b_y)`` and ``u =
@@ -258,9 +261,14 @@ class GatedDelta(Part):
         if self.dim > 1024:
             raise AlofaError("unsupported", "the recurrence kernel holds at most 1,024 key channels a head", f"dim={self.dim}")
         self.qk, self.v = self.kv_heads * self.dim, self.heads * self.vdim
-        self.decays = self.heads * self.dim
+        self.low_rank = bool(self.params.get("low_rank", True))
+        per, gate = str(self.params.get("decay_per", "channel")), str(self.params.get("gate", "sigmoid"))
+        if per not in ("channel", "head") or gate not in ("sigmoid", "silu"):
+            raise AlofaError("unsupported", "a delta rule has a decay per channel or per head and a sigmoid or silu gate", f"decay_per={per} gate={gate}")
+        self.gate_sigmoid = gate == "sigmoid"
+        self.decays = self.heads * (self.dim if per == "channel" else 1)
         self.channels = 2 * self.qk + self.v  # what passes the convolution: q, k, v
-        self.in_rows = self.channels + self.heads  # [q | k | v | beta]
+        self.in_rows = self.channels + self.heads + (0 if self.low_rank else self.decays + self.v)  # [q | k | v | beta] (and [decays | gate])
         self.scan_words = self.heads * self.vdim * self.dim
         self.conv_words = (self.taps - 1) * self.channels
         self.rank_a = self.rank_g = None  # the inner sizes of the decays' and the gate's projections, from the tensors
@@ -274,20 +282,35 @@ class GatedDelta(Part):
 
     def tensors(self):
         pre = self.prefix
-        ra, rg = -int(self.params.get("decay_rank") or 16), -int(self.params.get("gate_rank") or 16)  # the files' own; these for random weights
-        return {
+        t = {
             pre + "q": TensorSpec((self.qk, self.hidden)), pre + "q.conv": TensorSpec((self.qk, self.taps)),
             pre + "k": TensorSpec((self.qk, self.hidden)), pre + "k.conv": TensorSpec((self.qk, self.taps)),
             pre + "v": TensorSpec((self.v, self.hidden)), pre + "v.conv": TensorSpec((self.v, self.taps)),
             pre + "b": TensorSpec((self.heads, self.hidden)), pre + "A_log": TensorSpec((self.heads,)), pre + "norm": TensorSpec((self.vdim,), "ones"),
-            pre + "a1": TensorSpec((ra, self.hidden)), pre + "a2": TensorSpec((self.decays, ra)), pre + "dt_bias": TensorSpec((self.decays,)),
-            pre + "g1": TensorSpec((rg, self.hidden)), pre + "g2": TensorSpec((self.v, rg)), pre + "o": TensorSpec((self.hidden, self.v)),
+            pre + "dt_bias": TensorSpec((self.decays,)), pre + "o": TensorSpec((self.hidden, self.v)),
         }
+        if self.low_rank:
+            ra, rg = -int(self.params.get("decay_rank") or 16), -int(self.params.get("gate_rank") or 16)  # the files' own; these for random weights
+            t.update({pre + "a1": TensorSpec((ra, self.hidden)), pre + "a2": TensorSpec((self.decays, ra)), pre + "g1": TensorSpec((rg, self.hidden)),
+                      pre + "g2": TensorSpec((self.v, rg))})
+        else:
+            t.update({pre + "a": TensorSpec((self.decays, self.hidden)), pre + "g": TensorSpec((self.v, self.hidden))})
+        return t
 
     def load(self, state):
         pre = self.prefix
-        self.w_in = Linear(torch.cat([state[pre + n] for n in ("q", "k", "v", "b")], dim=0), None, STORE)
+        self.w_in = Linear(torch.cat([state[pre + n] for n in ("q", "k", "v", "b") + (() if self.low_rank else ("a", "g"))], dim=0), None, STORE)
         self.conv_w = torch.cat([state[pre + n + ".conv"] for n in ("q", "k", "v")], dim=0).to(torch.float32).contiguous()
+        if self.low_rank:
+            self._load_low_rank(state)
+        self.dt_bias = as_float32_vector(state[pre + "dt_bias"])
+        self.a_log = as_float32_vector(state[pre + "A_log"])
+        self.norm_w = as_float32_vector(state[pre + "norm"])
+        self.out_add = Linear(state[pre + "o"], None, RESIDUAL)
+        self.out_store = Linear(state[pre + "o"], None, STORE)
+
+    def _load_low_rank(self, state):
+        pre = self.prefix
         a1, a2, g1, g2 = (state[pre + n] for n in ("a1", "a2", "g1", "g2"))
         self.rank_a, self.rank_g = a1.shape[0], g1.shape[0]
         if a2.shape[1] != self.rank_a or g2.shape[1] != self.rank_g:
@@ -299,31 +322,28 @@ class GatedDelta(Part):
         second[: self.decays, : self.rank_a] = a2
         second[self.decays :, self.rank_a :] = g2
         self.high = Linear(second, None, STORE)
-        self.dt_bias = as_float32_vector(state[pre + "dt_bias"])
-        self.a_log = as_float32_vector(state[pre + "A_log"])
-        self.norm_w = as_float32_vector(state[pre + "norm"])
-        self.out_add = Linear(state[pre + "o"], None, RESIDUAL)
-        self.out_store = Linear(state[pre + "o"], None, STORE)
 
     def forward(self, ctx, x, h, cache, writes=True, store=False):
         n, f32 = x.shape[0], torch.float32
         H, G, N, P = self.heads, self.kv_heads, self.dim, self.vdim
-        u = ctx.buf((n, self.in_rows), f32)  # [q | k | v | beta], the projection's fp32 sums
+        u = ctx.buf((n, self.in_rows), f32)  # [q | k | v | beta] (and the logits below), the projection's fp32 sums
         self.w_in(u, x, buf=ctx.buf)
-        low = ctx.buf((n, self.rank_a + self.rank_g), self.rt.dtype)
-        self.low(low, x, buf=ctx.buf)
-        z = ctx.buf((n, self.decays + self.v), f32)  # the decays' logits, then the output gate's
-        self.high(z, low, buf=ctx.buf)
+        z, at = u, self.channels + H  # the decays' logits, then the output gate's
+        if self.low_rank:
+            low = ctx.buf((n, self.rank_a + self.rank_g), self.rt.dtype)
+            self.low(low, x, buf=ctx.buf)
+            z, at = ctx.buf((n, self.decays + self.v), f32), 0
+            self.high(z, low, buf=ctx.buf)
         st = cache.state
         xc = ctx.buf((n, self.channels), f32)
         ops.causal_conv(xc, u, 0, self.conv_w, None, st[:, self.scan_words:], ctx.q_start, ctx.state_slots, ctx.seq_of_token, ctx.n_seqs)
         qn, kn = ctx.buf((n, self.qk), f32), ctx.buf((n, self.qk), f32)
         kq, g, beta = ctx.buf((n, G), f32), ctx.buf((n, self.decays), f32), ctx.buf((n, H), f32)
-        ops.delta_prepare(qn, kn, kq, g, beta, xc, z, u, self.channels, self.dt_bias, self.a_log, H, G, N, self.UNIT_EPS, N ** -0.5)
+        ops.delta_prepare(qn, kn, kq, g, beta, xc, z, u, self.channels, self.dt_bias, self.a_log, H, G, N, self.UNIT_EPS, N ** -0.5, at)
         y = ctx.buf((n, self.v), f32)
         ops.delta_scan(y, xc, 2 * self.qk, kn, qn, kq, g, beta, st, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, G, N, P, spread=SCAN_SPREAD)
         normed = ctx.buf((n, self.v), self.rt.dtype)
-        ops.gated_group_norm(normed, y, z, self.decays, self.norm_w, H, self.eps, gate_first=False, sigmoid=True)
+        ops.gated_group_norm(normed, y, z, at + self.decays, self.norm_w, H, self.eps, gate_first=False, sigmoid=self.gate_sigmoid)
         _project_out(ctx, self.out_add, self.out_store, h, normed, store)
 
 

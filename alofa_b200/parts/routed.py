@@ -6,13 +6,16 @@ them are fp32 (``score``: "sigmoid" per expert, or "softmax" over the experts);
 the ``top`` largest scores choose the experts and are their weights
 (``renormalize``: divided by their sum).  The weight multiplies the expert's
 input (``weight_on_input``) or its output.  Options: ``gated`` experts
-``Wdown (act(Wgate .) * (Wup .))`` (tensors ``e<i>.gate``); ``correction``, a
+``Wdown (act(Wgate .) * (Wup .))`` (tensors ``e<i>.gate``), or with the
+activation "clamped_silu" the clamped form (``gate_alpha``, ``gate_limit``, see
+:class:`~alofa_b200.parts.feed_forward.DenseMLP`); ``correction``, a
 stored vector added to the scores for the choice only (the weights stay the
 scores); ``identity``: the last so many of the router's outputs are experts
 without tensors whose output is their input; ``renorm_eps`` added to the sum
 that ``renormalize`` divides by; ``groups`` / ``keep``: the experts form
 ``groups`` equal groups of neighbours, a group's score is the sum of its two
-largest choice scores (score + correction), and only experts of the ``keep``
+largest choice scores (score + correction; ``group_score`` "best": the largest
+alone), and only experts of the ``keep``
 best groups can be chosen; ``route_scale``: a factor on the weights.  A shared
 expert of the same form
 (``shared_ff`` > 0) runs for every token and is added, times ``sigmoid(x
@@ -31,7 +34,7 @@ import torch
 from ..csrc import ops
 from ..errors import AlofaError
 from .base import Part, TensorSpec, register_part
-from .feed_forward import DenseMLP
+from .feed_forward import DenseMLP, gate_form
 from .linear import STORE, Linear
 
 
@@ -64,11 +67,11 @@ class RoutedExperts(Part):
             raise AlofaError("invalid_argument", "groups must divide the experts, and the groups kept must hold at least top experts",
                              f"experts={self.experts} groups={self.groups} keep={self.keep} top={self.top}")
         self.routed = self.experts + self.identity  # outputs of the router
-        if self.gated and self.act != "silu":
-            raise AlofaError("unsupported", "gated experts take the silu activation only", f"activation={self.act}")
+        self.gate_form = gate_form(self.params, self.act) if self.gated else ops.SILU_GATE
+        self.group_best = str(self.params.get("group_score", "top_two")) == "best"
         if self.identity and self.weight_on_input:
             raise AlofaError("unsupported", "identity experts need the weight on the expert's output")
-        if self.act not in ops.ACTIVATIONS or self.score not in ("sigmoid", "softmax"):
+        if (not self.gated and self.act not in ops.ACTIVATIONS) or self.score not in ("sigmoid", "softmax"):
             raise AlofaError("unsupported", "unknown activation or score of a routed feed-forward", f"activation={self.act} score={self.score}")
         if not 0 < self.top <= min(self.experts + int(self.params.get("identity") or 0), 32) or self.experts <= 0:
             raise AlofaError("invalid_argument", "top must lie in [1, min(experts, 32)]", f"top={self.top} experts={self.experts}")
@@ -76,7 +79,8 @@ class RoutedExperts(Part):
         if self.shared_ff:
             from ..config.spec import PartSpec
 
-            self.shared = DenseMLP(PartSpec("mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_ff, "activation": self.act, "bias": False, "gated": self.gated},
+            self.shared = DenseMLP(PartSpec("mlp", {"hidden_size": self.hidden, "intermediate_size": self.shared_ff, "activation": self.act, "bias": False, "gated": self.gated,
+                                            "gate_alpha": self.params.get("gate_alpha"), "gate_limit": self.params.get("gate_limit")},
                                             prefix=self.prefix + "shared."), rt)
 
     def tensors(self):
@@ -119,7 +123,7 @@ class RoutedExperts(Part):
         choice, weight = ctx.buf((n, top), i32), ctx.buf((n, top), f32)
         gate = ctx.buf((n,), f32) if self.shared_gate else None
         ops.moe_router(choice, weight, gate, x, self.router, self.routed, top, self.score == "softmax", self.renormalize, self.correction, self.renorm_eps,
-                       self.groups, self.keep, self.route_scale)
+                       self.groups, self.keep, self.route_scale, self.group_best)
         pairs = n * top
         tiles = -(-pairs // tile) + self.experts  # every expert may end on a tile that is not full
         dest, tile_expert = ctx.buf((n, top), i32), ctx.buf((tiles,), i32)
@@ -130,10 +134,10 @@ class RoutedExperts(Part):
         mid = ctx.buf((rows, self.ff), dt)
         if self.gated:
             # gate and up in one product whose epilogue multiplies them (the tcgen05 kernel), else the sums of both and a kernel that gates
-            if not ops.gemm_by_tile_gated(mid, xs, self.up, tile_expert, tile):
+            if not ops.gemm_by_tile_gated(mid, xs, self.up, tile_expert, tile, self.gate_form):
                 both = ctx.buf((rows, 2 * self.ff), f32)
                 ops.gemm_by_tile(both, xs, self.up, tile_expert, tile)
-                ops.gate_up(mid, both)
+                ops.gate_up(mid, both, self.gate_form)
         else:
             ops.gemm_by_tile(mid, xs, self.up, tile_expert, tile, act=self.act)
         ys = ctx.buf((rows, self.hidden), f32)
