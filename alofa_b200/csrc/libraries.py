@@ -20,6 +20,9 @@ def all_libraries() -> list:
         {"name": "alofa_latent_attention_kv64_r32", "sources": ["kernels/latent_attention_bf16.cu"], "defines": {"KV_RANK": 64, "ROT": 32}},
         {"name": "alofa_latent_attention_kv96_r16", "sources": ["kernels/latent_attention_bf16.cu"], "defines": {"KV_RANK": 96, "ROT": 16}},
         *[{"name": f"alofa_attention_hd{hd}", "sources": ["kernels/attention_bf16.cu"], "defines": {"HEAD_DIM": hd}} for hd in (16, 32, 48, 64, 80, 96, 128)],
+        # the build that takes a distance bias off its scores, per sizes of key and value heads at first use; the tests' sizes ahead
+        *[{"name": f"alofa_attention_hd{hd}" + (f"_v{vd}" if vd != hd else "") + "_dist", "sources": ["kernels/attention_bf16.cu"],
+           "defines": {"HEAD_DIM": hd, "DISTANCE_BIAS": 1, **({"V_DIM": vd} if vd != hd else {})}} for hd, vd in ((64, 64), (128, 128), (64, 128), (128, 64), (32, 48))],
         # the build whose scores are capped (softcap * tanh(score / softcap)), likewise per head size at first use; two sizes ahead
         *[{"name": f"alofa_attention_hd{hd}_cap", "sources": ["kernels/attention_bf16.cu"], "defines": {"HEAD_DIM": hd, "SOFTCAP": 1}} for hd in (64, 128)],
     ]

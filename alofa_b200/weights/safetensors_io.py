@@ -130,4 +130,4 @@ def write_safetensors(path, tensors: dict, metadata: dict | None = None) -> None
         fh.write(struct.pack("<Q", len(text)))
         fh.write(text)
         for t in blobs:
-            fh.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            fh.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")

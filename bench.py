@@ -605,6 +605,50 @@ def kikerax_numbers(z: dict, b: dict) -> dict:
             "attn_flops_per_pair": n_pair * 4.0 * h * d, "head_flops": 2.0 * w * z["vocab"], "state_bytes_per_request": 2 * state_bytes + chunk_bytes}
 
 
+# --design pekerax: biased attention with a window, kept first tokens and a sink, and the delta rule with one decay per head, in
+# turn; dense and routed feed-forwards; beside the Dibulix design (pre-norm, the delta rule with a decay per channel, windowed
+# attention with a sink) and, for the routed feed-forward, the Kikerax design, at the same width, layers, heads, experts and
+# vocabulary.  The delta rule has Dibulix's sizes; attention heads of 128 over a window of 1,024 beside 64 kept tokens; Kikerax's
+# groups of experts.
+PEKERAX_SIZES = {
+    "1k": dict(kv_heads=2, att_dim=128, att_vdim=128, window=1024, keep_first=64, delta_heads=4, delta_kv_heads=2, delta_dim=128, delta_vdim=256, conv=4, groups=4, keep=2),
+    "2k": dict(kv_heads=4, att_dim=128, att_vdim=128, window=1024, keep_first=64, delta_heads=8, delta_kv_heads=4, delta_dim=128, delta_vdim=256, conv=4, groups=8, keep=4),
+}
+
+
+def pekerax_config(z: dict, b: dict):
+    """Attention with a dense feed-forward, the delta rule with routed experts, attention with routed experts and the delta rule with a dense feed-forward, in turn."""
+    from alofa_b200.models.pekerax import BiasedAttentionConfig, DeltaConfig, FeedForwardConfig, PekeraxConfig, PekeraxLayer
+
+    attention = BiasedAttentionConfig(z["heads"], b["kv_heads"], b["att_dim"], b["att_vdim"], b["att_dim"] ** -0.5, True, b["window"], b["keep_first"])
+    delta = DeltaConfig(b["delta_heads"], b["delta_kv_heads"], b["delta_dim"], b["delta_vdim"], b["conv"])
+    dense = FeedForwardConfig("dense", z["ff"], 7.0)
+    routed = FeedForwardConfig("moe", z["expert_ff"], 7.0, z["experts"], z["top"], {"count": b["groups"], "keep": b["keep"]})
+    kinds = (("attention", attention, dense), ("delta", delta, routed), ("attention", attention, routed), ("delta", delta, dense))
+    return PekeraxConfig(z["vocab"], z["width"], 1e-6, z["width"] ** 0.5, [PekeraxLayer(*kinds[i % 4]) for i in range(z["layers"])])
+
+
+def pekerax_numbers(z: dict, b: dict) -> dict:
+    """Bytes a decode step reads and flops a token costs for the Pekerax sizes (bf16 weights and caches, fp32 states).  The
+    bench's prompts are longer than the window, so a decode step reads the window's and the kept rows per request, whatever
+    the context: that is counted as state, and nothing grows with the context."""
+    w, h, g = z["width"], z["heads"], b["kv_heads"]
+    att = w * ((h + g) * b["att_dim"] + g * b["att_vdim"] + h) + h * b["att_vdim"] * w
+    qk, v = b["delta_kv_heads"] * b["delta_dim"], b["delta_heads"] * b["delta_vdim"]
+    delta = w * (2 * qk + v + 2 * b["delta_heads"] + v) + v * w
+    dense = 3 * w * z["ff"]
+    expert, router = 3 * w * z["expert_ff"], z["experts"] * w
+    kinds = [("att", "dense"), ("delta", "moe"), ("att", "moe"), ("delta", "dense")]
+    used = [kinds[i % 4] for i in range(z["layers"])]
+    n = {k: sum(k in pair for pair in used) for k in ("att", "delta", "dense", "moe")}
+    shared = n["att"] * att + n["delta"] * delta + n["dense"] * dense + n["moe"] * router
+    state_bytes = 4 * n["delta"] * (b["delta_heads"] * b["delta_dim"] * b["delta_vdim"] + (b["conv"] - 1) * (2 * qk + v))
+    window_bytes = 2 * (b["window"] + b["keep_first"]) * n["att"] * g * (b["att_dim"] + b["att_vdim"])
+    return {"weight_bytes": 2 * (shared + n["moe"] * z["experts"] * expert + z["vocab"] * w), "kv_bytes_per_token": 0,
+            "flops_per_token": 2.0 * (shared + n["moe"] * z["top"] * expert), "attn_flops_per_pair": n["att"] * 2.0 * h * (b["att_dim"] + b["att_vdim"]),
+            "head_flops": 2.0 * w * z["vocab"], "state_bytes_per_request": 2 * state_bytes + window_bytes}
+
+
 class KernelClock:
     """Times every kernel call of the package's ops module with its own pair of CUDA events during one
     step (run outright, no graph), and sets each beside the time its own operands allow: the larger of
@@ -658,7 +702,7 @@ class KernelClock:
             # y, v, ., kn, qn, kq, g, beta, state, q_start, slots, n_seqs, heads, groups, n, p: the rows once, the live requests' states read and written
             y, n_seqs, heads, groups, n, p = args[0], args[11], args[12], args[13], args[14], args[15]
             rows = y.shape[0]
-            byts = 4 * rows * (2 * heads * p + 2 * groups * n + heads * n + heads + groups) + 8 * n_seqs * heads * n * p
+            byts = 4 * rows * (2 * heads * p + 2 * groups * n + args[6].shape[1] + heads + groups) + 8 * n_seqs * heads * n * p
             # 32-bit by the design: the decay's multiply, the two dot products with key and query and the write's multiply-add per
             # state element and token on the fp32 pipe, against the nominal fp32 rate: 128 lanes x 2 x 1.965 GHz per SM
             import torch as _t
@@ -666,6 +710,11 @@ class KernelClock:
             fp32_rate = _t.cuda.get_device_properties(0).multi_processor_count * 128 * 2 * 1.965e9
             ideal = max(7.0 * rows * heads * n * p / fp32_rate, byts / (self.peaks["hbm_gbs"] * 1e9)) * 1e6
             return ideal, 7.0 * rows * heads * n * p, byts
+        elif name == "qkv_prepare_rows":
+            # q_out, k_cache, v_cache, qkv: a step's rows of the projection (or its split sums) read, q, keys and values written, the shared values once
+            q, k, v, qkv = args[:4]
+            sums = qkv if isinstance(qkv, torch.Tensor) else qkv.sums
+            byts = sums.numel() * 4 + q.numel() * q.element_size() + q.shape[0] * (k[0].numel() + v[0].numel()) * k.element_size() + 4 * q.shape[0] * v[0].numel()
         elif name == "min_gru":
             out, n_seqs = args[0], args[8]
             byts = out.numel() * (12 + out.element_size()) + 8 * n_seqs * out.shape[1]
@@ -818,7 +867,7 @@ class DesignBench(Bench):
                 runner.release(s_)
         finally:
             runner.cuda_graphs, runner.prompt_graphs = graphs
-        return {"prefill_2048": prefill[:8], f"decode_b{batch}": decode[:8]}
+        return {"prefill_2048": prefill[:12], f"decode_b{batch}": decode[:12]}
 
 
 def design_numbers(design: str, z: dict, routed_only: bool = False) -> dict:
@@ -863,17 +912,21 @@ def darolix_numbers(z: dict, d: dict) -> dict:
 
 def run_designs(args) -> dict:
     """Prefill and decode of a design beside its closest existing design at equal layer sizes (Kotutar
-    beside Qwen2, Darolix beside Kotutar, Dibulix beside Darolix), and the kernels of one step of each
-    against their own rooflines."""
-    from alofa_b200.models import darolix, dibulix, kikerax, kotutar, qwen2
+    beside Qwen2, Darolix beside Kotutar, Dibulix and Kikerax beside Darolix, Pekerax beside Dibulix and
+    Kikerax), and the kernels of one step of each against their own rooflines."""
+    from alofa_b200.models import darolix, dibulix, kikerax, kotutar, pekerax, qwen2
 
-    pair = {"kikerax": "Kikerax design beside Darolix", "dibulix": "Dibulix design beside Darolix", "darolix": "Darolix design beside Kotutar", "kotutar": "Kotutar design beside Qwen2"}[args.design]
+    pair = {"pekerax": "Pekerax design beside Dibulix and Kikerax", "kikerax": "Kikerax design beside Darolix", "dibulix": "Dibulix design beside Darolix", "darolix": "Darolix design beside Kotutar", "kotutar": "Kotutar design beside Qwen2"}[args.design]
     out = {"metric": f"prefill and decode of the {pair} at equal layer sizes", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
            "prompt_tokens": PROMPT_LEN, "context": CONTEXT, "steps": args.steps, "warmup": args.warmup, "sizes": {}}
     for size in ([args.size] if args.size else sorted(DESIGN_SIZES)):
         z = DESIGN_SIZES[size]
         row = {"sizes": z}
-        if args.design == "kikerax":
+        if args.design == "pekerax":
+            row["pekerax_sizes"], row["dibulix_sizes"], row["kikerax_sizes"] = PEKERAX_SIZES[size], DIBULIX_SIZES[size], KIKERAX_SIZES[size]
+            arms = (("pekerax", pekerax.NAME, pekerax_config(z, PEKERAX_SIZES[size])), ("dibulix", dibulix.NAME, dibulix_config(z, DIBULIX_SIZES[size])),
+                    ("kikerax", kikerax.NAME, kikerax_config(z, KIKERAX_SIZES[size])))
+        elif args.design == "kikerax":
             row["kikerax_sizes"], row["darolix_sizes"] = KIKERAX_SIZES[size], DAROLIX_SIZES[size]
             arms = (("kikerax", kikerax.NAME, kikerax_config(z, KIKERAX_SIZES[size])), ("darolix", darolix.NAME, darolix_config(z, DAROLIX_SIZES[size])))
         elif args.design == "dibulix":
@@ -885,7 +938,9 @@ def run_designs(args) -> dict:
         else:
             arms = (("kotutar", kotutar.NAME, kotutar_config(z)), ("qwen2", qwen2.NAME, qwen2_config_like(z)))
         for design, name, cfg in arms:
-            if design == "kikerax":
+            if design == "pekerax":
+                n = pekerax_numbers(z, PEKERAX_SIZES[size])
+            elif design == "kikerax":
                 n = kikerax_numbers(z, KIKERAX_SIZES[size])
             elif design == "dibulix":
                 n = dibulix_numbers(z, DIBULIX_SIZES[size])
@@ -893,7 +948,7 @@ def run_designs(args) -> dict:
                 n = darolix_numbers(z, DAROLIX_SIZES[size])
             else:
                 n = design_numbers(design, z, routed_only=args.design == "darolix")
-            window = DIBULIX_SIZES[size]["window"] if design == "dibulix" else 0
+            window = {"dibulix": DIBULIX_SIZES[size]["window"], "pekerax": PEKERAX_SIZES[size]["window"] + PEKERAX_SIZES[size]["keep_first"]}.get(design, 0)
             bench = DesignBench(name, cfg, f"{design} {size}", z["vocab"], n["weight_bytes"], n["kv_bytes_per_token"], n["flops_per_token"], n["attn_flops_per_pair"], 64,
                                 n.get("state_bytes_per_request", 0), window=window)
             res = {"prefill_2048": bench.prefill(args.warmup)}
@@ -925,7 +980,7 @@ def main() -> int:
     ap.add_argument("--phase", choices=["all", "decode", "prefill"], default="all", help="profiling aid: run only one part; the JSON line then lacks the others")
     ap.add_argument("--shape", choices=sorted(SHAPES), default="0.5b", help="whose layer sizes the headline run has")
     ap.add_argument("--no-extra", dest="extra", action="store_false", help="leave out the measurements beside the headline (long contexts, the 1.5B and 7B shapes)")
-    ap.add_argument("--design", choices=["kotutar", "darolix", "dibulix", "kikerax"], help="instead of the headline run: this design beside its closest existing one (Qwen2 for kotutar, Kotutar for darolix, Darolix for dibulix and kikerax) at equal layer sizes (prefill, decode, kernels against their rooflines)")
+    ap.add_argument("--design", choices=["kotutar", "darolix", "dibulix", "kikerax", "pekerax"], help="instead of the headline run: this design beside its closest existing one (Qwen2 for kotutar, Kotutar for darolix, Darolix for dibulix and kikerax, Dibulix and Kikerax for pekerax) at equal layer sizes (prefill, decode, kernels against their rooflines)")
     ap.add_argument("--size", choices=sorted(DESIGN_SIZES), help="with --design: one of the sizes only")
     args = ap.parse_args()
     if args.impl == "reference":

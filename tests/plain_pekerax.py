@@ -196,7 +196,7 @@ def routed(w, p, mlp, h):
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, g in zip(chosen[t], weights[t]):
-            out[t] += g * clamped_gated(w, f"{p}e{e}.", h[t : t + 1], mlp["expert"]["limit"])[0]
+            out[t] += g * clamped_gated(w, f"{p}e{e}.", h[t : t + 1], mlp["expert"].get("limit", np.inf))[0]
     return out
 
 
@@ -224,7 +224,7 @@ def forward(w, cfg, tokens, streams=False, margins=False):
         if mlp:
             h = layer_norm(x, w[p + "norm2"], w[p + "norm2.b"], eps)
             if mlp["kind"] == "dense":
-                x = x + clamped_gated(w, p + "mlp.", h, mlp["limit"])
+                x = x + clamped_gated(w, p + "mlp.", h, mlp.get("limit", np.inf))
             else:
                 worst = np.minimum(worst, route(w, p + "mlp.", mlp["router"], h)[2])
                 x = x + routed(w, p + "mlp.", mlp, h)

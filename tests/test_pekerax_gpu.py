@@ -1,0 +1,750 @@
+"""Pekerax on the GPU against the plain implementation (tests/plain_pekerax.py).
+
+Mechanisms alone (kernels against the plain function of the same mechanism):
+attention with a distance bias, a window beside kept first tokens, a sink per
+head, norms over the whole projection and a gate, on the every-size kernel and
+on the tensor-core kernels (keys and values of different sizes, one to twenty
+heads on a key head), over pages of which those that nothing may see are
+poisoned, in prompts, portions and decoding at lengths around page and window
+borders; one key made to stand out just inside and just outside the window and
+the kept tokens; a far key among hundreds; sinks; mixed values and split sums
+still owed; the delta rule with one decay per head over portions and reused
+slots, a far token read back; the clamped gate in every product that has one;
+the router; the layer norm.  Then whole models of five configurations, in 32-bit
+and bfloat16: whole prompts, prefill against token-by-token decoding, portions
+down to two tokens, batches of unequal requests in a pool so small that pages
+and slots are used again, long decoding from the first token, the stream after
+every layer, and greedy generation through the engine and the programs."""
+import json
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import plain_pekerax as plain
+import replay
+import tiny_pekerax as tiny
+from gpu_util import assert_close, dev, rounded
+
+pytestmark = pytest.mark.gpu
+
+F32, BF16 = torch.float32, torch.bfloat16
+# Largest |engine - plain| on logits, times max(1, max|plain|): fp32 sums against float64; bfloat16 rounds
+# activations and cache rows to 8 bits of mantissa.
+TOL = {"float32": 3e-5, "bfloat16": 9e-2}
+KERNEL_TOL = {F32: 2e-5, BF16: 3e-2}
+
+
+class Owed:
+    """What a product leaves when its reader is to add its split sums up: planes [splits, rows, columns] and a bias."""
+
+    def __init__(self, sums, bias=None):
+        self.sums, self.splits, self.bias = sums, sums.shape[0], bias
+
+
+# ---------------------------------------------------------------------------------------------------
+# attention: the kernels' pipeline (prepare, attend, gate) against the plain mixer with weights that pick
+# q, k, v and the gates' logits out of the input, so that a test can make them what it wants
+# ---------------------------------------------------------------------------------------------------
+def picking_weights(rng, m, prefix="a."):
+    """The input is [q | k | v | gate logits]; the projections pick their columns; the output projection is the identity."""
+    H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    nq, nk, nv = H * d, G * d, G * dv
+    eye = np.eye(nq + nk + nv + H)
+    w = {"q": eye[:nq], "k": eye[nq : nq + nk], "v": eye[nq + nk : nq + nk + nv], "g": eye[nq + nk + nv :], "o": np.eye(H * dv), "q.norm": rounded(1 + 0.3 * rng.standard_normal(nq), F32),
+         "k.norm": rounded(1 + 0.3 * rng.standard_normal(nk), F32), "sink": rounded(rng.standard_normal(H) + 0.5, F32), "vmix": np.array(0.0)}
+    return {prefix + n: v for n, v in w.items()}, eye.shape[0]
+
+
+class PagedCase:
+    """Requests of given lengths over one paged cache with block tables in random order."""
+
+    def __init__(self, rng, m, lengths, page, dtype):
+        self.page, self.lengths, self.m = page, lengths, m
+        blocks = [-(-n // page) for n in lengths]
+        order = rng.permutation(sum(blocks) + 3)
+        self.table = np.full((len(lengths), max(blocks) + 1), -1, dtype=np.int32)
+        at = 0
+        for r, b in enumerate(blocks):
+            self.table[r, :b] = order[at : at + b]
+            at += b
+        slots = (sum(blocks) + 3) * page
+        self.k = torch.empty((slots, m["kv_heads"], m["dim"]), dtype=dtype, device="cuda")
+        self.v = torch.empty((slots, m["kv_heads"], m["vdim"]), dtype=dtype, device="cuda")
+        self.table_dev = dev(self.table)
+        self.clear()
+
+    def clear(self):
+        self.k.fill_(60.0)  # what lies in slots that nothing may see must not matter
+        self.v.fill_(-900.0)
+
+    def slot_map(self, r, lo, hi):
+        return np.array([self.table[r, j // self.page] * self.page + j % self.page for j in range(lo, hi)], dtype=np.int32)
+
+    def poison_passed_pages(self, spans):
+        """What the cache manager may have given away by the next step: pages neither kept nor within reach of the window."""
+        mask = self.m.get("mask")
+        if not mask:
+            return
+        for r, _, hi in spans:
+            for b in range(-(-mask.get("keep_first", 0) // self.page), max(0, hi - mask["size"] + 1) // self.page):
+                s = self.table[r, b] * self.page
+                self.k[s : s + self.page] = 60.0
+                self.v[s : s + self.page] = -900.0
+
+
+def attend(case, w, rows, spans, dtype, eps, tensor_cores, prefix="a.", split_keys=256):
+    """The kernels' pipeline over the rows ``spans`` = [(request, lo, hi)] of ``rows[request]`` in one step."""
+    from alofa_b200.csrc import ops
+
+    m = case.m
+    H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    mask = m.get("mask") or {}
+    window, keep = mask.get("size"), mask.get("keep_first", 0)
+    sums = dev(np.concatenate([rows[r][lo:hi] for r, lo, hi in spans]), F32)
+    n = sums.shape[0]
+    positions = dev(np.concatenate([np.arange(lo, hi, dtype=np.int32) for _, lo, hi in spans]))
+    q = torch.empty((n, H * d), dtype=dtype, device="cuda")
+    ops.qkv_prepare_rows(q, case.k, case.v, sums, dev(np.concatenate([case.slot_map(r, lo, hi) for r, lo, hi in spans])), dev(w[prefix + "q.norm"], F32), dev(w[prefix + "k.norm"], F32), eps)
+    sink, slopes, g_at = dev(w[prefix + "sink"], F32), dev(plain.slopes(H), F32), sums.shape[1] - H
+    out = torch.empty((n, H * dv), dtype=dtype, device="cuda")
+    if tensor_cores:
+        counts = [hi - lo for _, lo, hi in spans]
+        q_start = dev(np.concatenate([[0], np.cumsum(counts)]).astype(np.int32))
+        kv_len = dev(np.array([hi for _, _, hi in spans], dtype=np.int32))
+        table = dev(case.table[[r for r, _, _ in spans]])
+        longest = max(hi for _, _, hi in spans)
+        splits, po, pml = 0, None, None
+        if max(counts) == 1:  # a decode step: every request's keys in splits
+            reach = longest if not (window and keep) else min(longest, 64 * (-(-keep // 64) + (window + 62) // 64 + 1))
+            splits = -(-reach // split_keys)
+            po = torch.full((splits, n * H, dv), 1e9, dtype=F32, device="cuda")
+            pml = torch.full((splits, n * H, 2), 1e9, dtype=F32, device="cuda")
+        status = torch.zeros(4, dtype=torch.int32, device="cuda")
+        ops.attention_bf16(out, q, case.k, case.v, q_start, kv_len, positions, table, case.page, len(spans), max(counts), H, G, d, window, m["scale"], splits, split_keys, po, pml,
+                           longest, status, sink=sink, keep=keep if window else 0, slopes=slopes, gate=sums, gate_at=g_at)
+        assert int(status.sum()) == 0
+    else:
+        seq = dev(np.concatenate([np.full(hi - lo, r, dtype=np.int32) for r, lo, hi in spans]))
+        a = torch.empty((n, H * dv), dtype=F32, device="cuda")
+        ops.paged_attention_generic(a, q, case.k, case.v, positions, seq, case.table_dev, case.page, H, G, d, window, m["scale"], 0.0, dv, sink, 0, 1, keep if window else 0, slopes)
+        ops.heads_finish(out, a, H, G, dv, gate=sums, g_off=g_at)
+    return out.float().cpu().numpy()
+
+
+def in_steps(case, w, rows, dtype, eps, cuts, tensor_cores):
+    """Every request whole in one step; then again from an empty cache in portions of ``cuts`` (1: decoding) with all requests in every step."""
+    whole = attend(case, w, rows, [(r, 0, n) for r, n in enumerate(case.lengths)], dtype, eps, tensor_cores)
+    split = np.cumsum([0] + list(case.lengths))
+    out = [[whole[split[r] : split[r + 1]] for r in range(len(rows))]]
+    case.clear()
+    got, at, step = [[] for _ in rows], [0] * len(rows), 0
+    while any(at[r] < n for r, n in enumerate(case.lengths)):
+        spans = []
+        for r, n in enumerate(case.lengths):
+            if at[r] < n:
+                c = min(cuts[(step + r) % len(cuts)], n - at[r])
+                spans.append((r, at[r], at[r] + c))
+        step += 1
+        res, k = attend(case, w, rows, spans, dtype, eps, tensor_cores, split_keys=128 if step % 2 else 256), 0
+        for r, lo, hi in spans:
+            got[r].append(res[k : k + hi - lo])
+            k += hi - lo
+            at[r] = hi
+        case.poison_passed_pages(spans)
+    out.append([np.concatenate(g) for g in got])
+    return out
+
+
+def case_mixer(H, G, d, dv, window, keep, scale=None):
+    m = {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "scale": scale or 1.5 / np.sqrt(d)}
+    if window is not None:
+        m["mask"] = {"size": window, "keep_first": keep}
+    return m
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("H,G,d,dv,window,keep", [(4, 2, 16, 24, 9, 5), (3, 3, 12, 8, 21, 0), (2, 1, 10, 30, None, 0), (1, 1, 8, 130, 2, 1), (6, 2, 40, 72, 32, 40), (2, 2, 136, 64, 150, 17)])
+def test_biased_attention_on_the_every_size_kernel(dtype, H, G, d, dv, window, keep):
+    """Whole prompts, portions that end inside windows and pages, and decoding, at lengths around page (16) and window
+    borders; pages that nothing may see are poisoned from step to step."""
+    rng = np.random.default_rng(3)
+    m = case_mixer(H, G, d, dv, window, keep)
+    w, width = picking_weights(rng, m)
+    near = [window - 1, window, window + 1, window + keep, window + keep + 1, 2 * window + 16] if window else [60]
+    lengths = sorted({n for n in [1, 2, 15, 16, 17, 33, 70, keep, keep + 1] + near if n > 0})
+    rows = [rounded(rng.standard_normal((n, width)), F32) for n in lengths]
+    want = [plain.attention(w, "a.", m, x, 1e-5)[0] for x in rows]
+    for cuts in ((1,), (5, 2, 16, 3, 2, 33)):
+        case = PagedCase(rng, m, lengths, 16, dtype)
+        for what, got in zip(("whole", f"portions of {cuts}"), in_steps(case, w, rows, dtype, 1e-5, cuts, False)):
+            for r, n in enumerate(lengths):
+                assert_close(got[r], want[r], KERNEL_TOL[dtype], f"{what}: request of {n} tokens")
+
+
+@pytest.mark.parametrize("H,G,d,dv,window,keep,page", [
+    (4, 2, 64, 64, 64, 70, 64), (4, 2, 64, 64, 100, 20, 64), (4, 2, 64, 64, None, 0, 64), (4, 1, 64, 64, 1, 64, 64), (2, 2, 64, 64, 130, 0, 64), (2, 1, 64, 64, 50, 7, 16),
+    (6, 2, 64, 128, 100, 33, 64), (3, 3, 64, 128, None, 0, 64), (2, 1, 128, 64, 90, 129, 64), (4, 1, 128, 64, 200, 1, 32), (2, 1, 128, 128, 256, 65, 64),
+    (20, 1, 32, 48, 40, 10, 16), (20, 1, 32, 48, 70, 100, 64), (34, 2, 32, 48, None, 0, 48), (4, 2, 32, 48, 65, 3, 64), (2, 2, 32, 48, 17, 16, 16)])
+def test_biased_attention_on_the_tensor_core_kernels(H, G, d, dv, window, keep, page):
+    """bfloat16: the tcgen05 / mma.sync prompt kernels and the decode kernels in key splits, keys and values of one size and
+    of two, key heads with one to twenty heads, pages of whole key blocks and smaller ones."""
+    rng = np.random.default_rng(13)
+    m = case_mixer(H, G, d, dv, window, keep)
+    w, width = picking_weights(rng, m)
+    c = window or 50
+    lengths = sorted({n for n in [1, 2, 63, 64, 65, c - 1, c, c + 1, c + keep, c + keep + 1, 257, 400] if n > 0})
+    rows = [rounded(rng.standard_normal((n, width)), F32) for n in lengths]
+    want = [plain.attention(w, "a.", m, x, 1e-5)[0] for x in rows]
+    for cuts in ((1,), (5, 2, 64, 3, 2, 130)):
+        case = PagedCase(rng, m, lengths, page, BF16)
+        for what, got in zip(("whole", f"portions of {cuts}"), in_steps(case, w, rows, BF16, 1e-5, cuts, True)):
+            for r, n in enumerate(lengths):
+                assert_close(got[r], want[r], KERNEL_TOL[BF16], f"{what}: request of {n} tokens")
+
+
+PATHS = [(F32, 16, 16, False), (BF16, 16, 24, False), (BF16, 64, 64, True), (BF16, 32, 48, True)]
+
+
+@pytest.mark.parametrize("dtype,d,dv,tensor_cores", PATHS)
+@pytest.mark.parametrize("window,keep", [(3, 2), (16, 5), (40, 17), (64, 1), (100, 64), (33, 0)])
+def test_a_key_just_inside_and_just_outside_the_window_and_the_kept_tokens(dtype, d, dv, tensor_cores, window, keep):
+    """The last key that a far query may not see and the first that it may, at the window's edge and at the kept tokens'
+    edge, all point the query's way and hold large values of alternating sign: the sum of the right ones and no other."""
+    rng = np.random.default_rng(4)
+    H, G = 2, 1
+    m = case_mixer(H, G, d, dv, window, keep, scale=1.0)
+    w, width = picking_weights(rng, m)
+    for n in ("q.norm", "k.norm"):
+        w["a." + n] = np.ones_like(w["a." + n])
+    n = window + max(keep, 8) + 70
+    x = rounded(0.2 * rng.standard_normal((n, width)), F32)
+    i = n - 3  # the query
+    way = rng.standard_normal(d)
+    kcol, vcol = H * d, H * d + G * d
+    x[i, : H * d] = np.tile(way, H)
+    for j, value in ((i - window, 30.0), (i - window + 1, -20.0), (keep, 30.0)) + (((keep - 1, 45.0),) if keep else ()):
+        x[j, kcol : kcol + d] = way
+        x[j, vcol : vcol + dv] = value
+    x[:, -H:] = 3.0
+    x = rounded(x, F32)
+    want = plain.attention(w, "a.", m, x, 1e-6)[0]
+    wrong = [plain.attention(w, "a.", dict(m, mask={"size": window + a, "keep_first": keep + b}), x, 1e-6)[0][i] for a, b in ((1, 0), (-1, 0), (0, 1)) + (((0, -1),) if keep else ())]
+    assert all(np.abs(want[i] - other)[-dv:].max() > 1.0 for other in wrong), "the test's keys do not stand out"
+    for cuts in ((1,), (7, 2, 64)):
+        case = PagedCase(rng, m, [n], 64 if tensor_cores and d == 64 else 16, dtype)
+        for got in in_steps(case, w, [x], dtype, 1e-6, cuts, tensor_cores):
+            assert_close(got[0], want, KERNEL_TOL[dtype], f"window {window}, kept {keep}, cuts {cuts}")
+
+
+@pytest.mark.parametrize("dtype,d,dv,tensor_cores", PATHS)
+def test_one_far_key_among_hundreds_and_the_bias_on_it(dtype, d, dv, tensor_cores):
+    """Key 3 of 700 and the last query point the same way: against the last head's slope its score stays far above the
+    others and the output is (nearly) its value; against the first head's slope it is gone."""
+    rng = np.random.default_rng(6)
+    H, G = 4, 1
+    m = case_mixer(H, G, d, dv, None, 0, scale=16.0 / d)
+    w, width = picking_weights(rng, m)
+    for n in ("q.norm", "k.norm"):
+        w["a." + n] = np.ones_like(w["a." + n])
+    w["a.sink"] = np.full(H, -2.0)
+    x = rounded(0.3 * rng.standard_normal((700, width)), F32)
+    way = rng.standard_normal(d)
+    x[3, H * d : H * d + d] = way
+    x[3, H * d + d : H * d + d + dv] = 9.0
+    x[699, : H * d] = np.tile(way, H)
+    x[:, -H:] = 30.0  # the gates wide open
+    x = rounded(x, F32)
+    want = plain.attention(w, "a.", m, x, 1e-6)[0]
+    assert want[699, -1] > 7.5 and abs(want[699, 0]) < 1.0, "the test's far key does not stand out"
+    case = PagedCase(rng, m, [700], 16, dtype)
+    attend(case, w, [x], [(0, 0, 699)], dtype, 1e-6, tensor_cores)
+    assert_close(attend(case, w, [x], [(0, 699, 700)], dtype, 1e-6, tensor_cores), want[699:], KERNEL_TOL[dtype], "last query")
+
+
+@pytest.mark.parametrize("dtype,d,dv,tensor_cores", PATHS)
+@pytest.mark.parametrize("sink", [-30.0, 0.0, 4.0, 30.0])
+def test_sinks_take_their_share_once(dtype, d, dv, tensor_cores, sink):
+    """Equal scores over a window: the output is the values' weighted mean times the part the sink leaves, however many
+    key splits and blocks the row was merged from."""
+    rng = np.random.default_rng(7)
+    m = case_mixer(2, 1, d, dv, 300, 20, scale=0.01)
+    w, width = picking_weights(rng, m)
+    w["a.sink"] = np.array([sink, sink - 1.0])
+    x = rounded(rng.standard_normal((420, width)), F32)
+    x[:, 3 * d : 3 * d + dv] += 3.0
+    want = plain.attention(w, "a.", m, x, 1e-6)[0]
+    for cuts in ((1,), (130, 2)):
+        case = PagedCase(rng, m, [420], 16, dtype)
+        for got in in_steps(case, w, [x], dtype, 1e-6, cuts, tensor_cores):
+            assert_close(got[0], want, KERNEL_TOL[dtype], f"sink {sink}, cuts {cuts}")
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("H,G,d,dv,n", [(4, 2, 24, 40, 37), (3, 1, 7, 5, 9), (16, 4, 128, 128, 3), (5, 5, 10, 30, 200)])
+def test_norms_over_the_whole_projection_mixed_values_and_owed_sums(dtype, H, G, d, dv, n):
+    """q, keys, values (left for the later layers, and mixed with the first layer's) and gate logits from finished sums
+    and from planes of split sums with a bias on top."""
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(15)
+    nq, nk, nv = H * d, G * d, G * dv
+    ld = nq + nk + nv + H
+    planes, bias = rounded(rng.standard_normal((3, n, ld)), F32), rounded(rng.standard_normal(ld), F32)
+    whole = rounded(planes.sum(axis=0) + bias, F32)
+    wq, wk = rounded(1 + 0.2 * rng.standard_normal(nq), F32), rounded(1 + 0.2 * rng.standard_normal(nk), F32)
+    first, lam = rounded(rng.standard_normal((n, nv)), F32), 0.3
+    slots = rng.permutation(4 * n)[:n].astype(np.int32)
+    for sums in (dev(whole, F32), Owed(dev(planes, F32), dev(bias, F32))):
+        for mix in (None, lam):
+            q = torch.zeros((n, nq), dtype=dtype, device="cuda")
+            k, v = torch.zeros((4 * n, G, d), dtype=dtype, device="cuda"), torch.zeros((4 * n, G, dv), dtype=dtype, device="cuda")
+            gates = torch.zeros((n, H), dtype=F32, device="cuda")
+            vf = dev(first, F32) if mix is not None else torch.zeros((n, nv), dtype=F32, device="cuda")
+            ops.qkv_prepare_rows(q, k, v, sums, dev(slots), dev(wq, F32), dev(wk, F32), 1e-5, vf, dev(np.array([lam]), F32) if mix is not None else None, gates, ld - H)
+            tol = 4e-6 if dtype == F32 else 1e-2
+            assert_close(q.float().cpu(), plain.rms_norm(whole[:, :nq], wq, 1e-5), tol, "q")
+            assert_close(k.float().cpu().numpy()[slots].reshape(n, nk), plain.rms_norm(whole[:, nq : nq + nk], wk, 1e-5), tol, "keys")
+            own = whole[:, nq + nk : nq + nk + nv]
+            assert_close(v.float().cpu().numpy()[slots].reshape(n, nv), plain.mixed_values(own, first if mix is not None else None, lam), tol, "values")
+            assert_close(vf.cpu(), own if mix is None else first, 2e-6, "the first layer's values")
+            assert_close(gates.cpu(), whole[:, ld - H :], 2e-6, "gate logits")
+            unused = np.setdiff1d(np.arange(4 * n), slots)
+            assert float(k[unused].abs().max()) == 0.0 and float(v[unused].abs().max()) == 0.0
+
+
+# ---------------------------------------------------------------------------------------------------
+# the delta rule
+# ---------------------------------------------------------------------------------------------------
+def delta_weights(rng, m, slow=False, prefix="d."):
+    """The input is [q | k | v | beta | decay | gate logits]; the projections pick their columns; the output projection is the identity."""
+    H, G, n, P, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+    sizes = {"q": G * n, "k": G * n, "v": H * P, "b": H, "a": H, "g": H * P}
+    eye, at, w = np.eye(sum(sizes.values())), 0, {}
+    for name, size in sizes.items():
+        w[name] = eye[at : at + size]
+        at += size
+    for name in ("q", "k", "v"):
+        w[name + ".conv"] = rounded(rng.standard_normal((sizes[name], K)) / np.sqrt(K) + (np.arange(K) == K - 1), F32)
+    w.update({"A_log": rounded(rng.uniform(-9.0, -8.0, H) if slow else rng.uniform(-4.0, 0.5, H), F32), "dt_bias": rounded(rng.standard_normal(H), F32),
+              "norm": rounded(1 + 0.3 * rng.standard_normal(P), F32), "o": np.eye(H * P)})
+    return {prefix + k: v for k, v in w.items()}, eye.shape[0]
+
+
+class Delta:
+    """The kernels of the mixer with a state per slot, as the part runs them."""
+
+    def __init__(self, w, m, slots, dtype, eps, prefix="d."):
+        self.m, self.dtype, self.eps = m, dtype, eps
+        H, G, n, P = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        self.channels, self.words = 2 * G * n + H * P, H * n * P
+        self.state = torch.zeros((slots, self.words + (m["conv"] - 1) * self.channels), dtype=F32, device="cuda")
+        self.conv = dev(np.concatenate([w[prefix + s + ".conv"] for s in ("q", "k", "v")]), F32)
+        self.a_log, self.dt_bias, self.norm = (dev(w[prefix + s], F32) for s in ("A_log", "dt_bias", "norm"))
+
+    def step(self, x, counts, slots):
+        from alofa_b200.csrc import ops
+
+        H, G, n, P = self.m["heads"], self.m["kv_heads"], self.m["dim"], self.m["vdim"]
+        q_start = dev(np.concatenate([[0], np.cumsum(counts)]).astype(np.int32))
+        seq = dev(np.concatenate([np.full(c, s, dtype=np.int32) for s, c in enumerate(counts)]))
+        slots = dev(np.asarray(slots, dtype=np.int32))
+        T, u = x.shape[0], dev(x, F32)
+        new = lambda *shape: torch.empty(shape, dtype=F32, device="cuda")
+        xc = new(T, self.channels)
+        ops.causal_conv(xc, u, 0, self.conv, None, self.state[:, self.words :], q_start, slots, seq, len(counts))
+        qn, kn, kq, g, beta, y = new(T, G * n), new(T, G * n), new(T, G), new(T, H), new(T, H), new(T, H * P)
+        ops.delta_prepare(qn, kn, kq, g, beta, xc, u, u, self.channels, self.dt_bias, self.a_log, H, G, n, 1e-6, n ** -0.5, self.channels + H)
+        ops.delta_scan(y, xc, 2 * G * n, kn, qn, kq, g, beta, self.state, q_start, slots, len(counts), H, G, n, P, spread=128)
+        out = torch.empty((T, H * P), dtype=self.dtype, device="cuda")
+        ops.gated_group_norm(out, y, u, self.channels + 2 * H, self.norm, H, self.eps, gate_first=False)
+        return out.float().cpu().numpy()
+
+
+def walk(lengths, cuts, slots_of, xs, mixer):
+    """Requests of ``lengths`` tokens through steps: request r brings ``cuts[(step + r) % len(cuts)]`` tokens and sits out
+    every third step; every request's rows in order."""
+    got, at, step = [[] for _ in lengths], [0] * len(lengths), 0
+    while any(at[r] < lengths[r] for r in range(len(lengths))):
+        live = [r for r in range(len(lengths)) if at[r] < lengths[r] and (step + r) % 3 != 2]
+        step += 1
+        if not live:
+            continue
+        counts = [min(cuts[(step + r) % len(cuts)], lengths[r] - at[r]) for r in live]
+        rows, k = mixer.step(np.concatenate([xs[r][at[r] : at[r] + c] for r, c in zip(live, counts)]), counts, [slots_of[r] for r in live]), 0
+        for r, c in zip(live, counts):
+            got[r].append(rows[k : k + c])
+            k += c
+            at[r] += c
+    return [np.concatenate(g) for g in got]
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("H,G,n,P,K", [(6, 3, 12, 20, 4), (2, 2, 16, 8, 1), (5, 1, 7, 9, 3), (4, 2, 64, 32, 2), (1, 1, 128, 256, 4), (2, 1, 130, 6, 2), (3, 3, 1, 4, 2), (2, 1, 300, 12, 3)])
+def test_delta_rule_with_one_decay_a_head_over_portions_in_slots_used_out_of_order(dtype, H, G, n, P, K):
+    """Convolutions and recurrence carried from step to step: portions of 1, 2 and many tokens, requests that sit steps
+    out, slots in another order than the requests and used again."""
+    rng = np.random.default_rng(8)
+    m = {"heads": H, "kv_heads": G, "dim": n, "vdim": P, "conv": K}
+    w, width = delta_weights(rng, m)
+    lengths = [1, 2, 37, 90, 203]
+    xs = [rounded(rng.standard_normal((t, width)), F32) for t in lengths]
+    want = [plain.delta(w, "d.", m, x, 1e-5) for x in xs]
+    mixer = Delta(w, m, 7, dtype, 1e-5)
+    mixer.state.fill_(3.0)  # what a slot's last user left
+    for cuts, slots_of, count in (((1, 2, 3, 17, 190), [5, 0, 3, 6, 1], 5), ((1,), [2, 4, 5, 0], 4)):
+        for s in slots_of:
+            mixer.state[s].zero_()  # as the engine does when a request is admitted
+        for r, got in enumerate(walk(lengths[:count], cuts, slots_of, xs, mixer)):
+            assert_close(got, want[r], KERNEL_TOL[dtype] * (2 if dtype == F32 else 1), f"cuts {cuts}: request of {lengths[r]} tokens")
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_a_far_token_is_read_back_from_the_state(dtype):
+    """Token 2 of 400 writes a large value under a key that nothing else points to and the decays are near one: the last
+    query points that way and reads it back, which a state lost at a step's border or a slot mixed up would not give."""
+    rng = np.random.default_rng(9)
+    m = {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 8, "conv": 2}
+    w, width = delta_weights(rng, m, slow=True)
+    for s in ("q", "k", "v"):
+        w[f"d.{s}.conv"] = np.tile([0.0, 1.0], (w[f"d.{s}.conv"].shape[0], 1))
+    x = rounded(rng.standard_normal((400, width)) * 0.3, F32)
+    x[:, 16:24], x[:, 24:32] = -20.0, rounded(rng.standard_normal((400, 8)) + 2.0, F32)  # keys live in the second half (silu(-20) is nothing) ...
+    x[2, 16:24], x[2, 24:32] = 4.0, -20.0  # ... but token 2's in the first
+    x[2, 32:48] = 60.0
+    x[399, :8], x[399, 8:16] = 4.0, -20.0  # and so does the last query
+    want = plain.delta(w, "d.", m, x, 1e-5)
+    quiet = x.copy()
+    quiet[2, 32:48] = 0.0
+    assert np.abs(want[399] - plain.delta(w, "d.", m, quiet, 1e-5)[399]).max() > 0.1, "the test's far token leaves no trace"
+    mixer = Delta(w, m, 3, dtype, 1e-5)
+    got = walk([400], (3, 1, 150, 1, 1, 2, 90), [1], [x], mixer)
+    assert_close(got[0], want, KERNEL_TOL[dtype] * (2 if dtype == F32 else 1), "every token")
+
+
+# ---------------------------------------------------------------------------------------------------
+# gates, router, norm
+# ---------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("tokens", [1, 5, 17, 40, 130, 300])
+@pytest.mark.parametrize("hidden,ff,limit", [(128, 96, 0.8), (72, 100, 1.7), (256, 264, None), (50, 36, 1.0)])
+def test_clamped_gate_in_the_products_that_have_one(dtype, tokens, hidden, ff, limit):
+    """The dense feed-forward as the part runs it (decode and prompt products, with and without a depth split)."""
+    from alofa_b200.csrc import ops
+    from alofa_b200.parts.linear import GATED, Linear
+
+    rng = np.random.default_rng(16)
+    gate = (1.702, float("inf") if limit is None else limit)
+    x = rounded(rng.standard_normal((tokens, hidden)), dtype)
+    wt = rounded(2.5 * rng.standard_normal((2 * ff, hidden)) / np.sqrt(hidden), dtype)
+    g, u = x @ wt[:ff].T, x @ wt[ff:].T
+    lim = gate[1]
+    want = np.minimum(g, lim) * plain.sigmoid(1.702 * np.minimum(g, lim)) * (np.clip(u, -lim, lim) + 1.0)
+    assert limit is None or (np.abs(g - np.minimum(g, lim)).max() > 0.3 and np.abs(u - np.clip(u, -lim, lim)).max() > 0.3), "nothing is clamped"
+    out = torch.empty((tokens, ff), dtype=dtype, device="cuda")
+    Linear(dev(wt, dtype), None, GATED, gate=gate)(out, dev(x, dtype))
+    assert_close(out.float().cpu(), want, 3e-6 if dtype == F32 else 6e-3, "gated product")
+    both = dev(np.concatenate([g, u], axis=1), F32)
+    mid = torch.empty((tokens, ff), dtype=dtype, device="cuda")
+    ops.gate_up(mid, both, gate)
+    assert_close(mid.float().cpu(), want, 3e-6 if dtype == F32 else 6e-3, "gate_up")
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("E,top,hidden,ff,groups", [(8, 3, 64, 48, (4, 2)), (6, 2, 100, 28, (3, 2)), (5, 1, 128, 64, None), (9, 3, 64, 16, (3, 1))])
+def test_routed_experts_with_the_clamped_gate(dtype, E, top, hidden, ff, groups):
+    from alofa_b200.config.spec import PartSpec
+    from alofa_b200.parts.base import Runtime
+    from alofa_b200.parts.routed import RoutedExperts
+
+    class Ctx:
+        buf = staticmethod(lambda shape, dt: torch.empty(shape, dtype=dt, device="cuda"))
+
+    rng = np.random.default_rng(17)
+    w = {"m.router": rounded(3 * rng.standard_normal((E, hidden)) / np.sqrt(hidden), BF16)}
+    for e in range(E):
+        w.update({f"m.e{e}.gate": rounded(2 * rng.standard_normal((ff, hidden)) / np.sqrt(hidden), BF16), f"m.e{e}.up": rounded(2 * rng.standard_normal((ff, hidden)) / np.sqrt(hidden), BF16),
+                  f"m.e{e}.down": rounded(rng.standard_normal((hidden, ff)) / np.sqrt(ff), BF16)})
+    mlp = {"expert": {"ff": ff, "limit": 0.9}, "router": {"experts": E, "top": top}}
+    if groups:
+        mlp["router"]["groups"] = {"count": groups[0], "keep": groups[1]}
+    part = RoutedExperts(PartSpec("routed_experts", {"hidden_size": hidden, "experts": E, "top": top, "expert_ff": ff, "gated": True, "activation": "clamped_silu", "gate_alpha": 1.702,
+                                                     "gate_limit": 0.9, "score": "softmax", "renormalize": True, "renorm_eps": 1e-20, "groups": groups[0] if groups else 1,
+                                                     "keep": groups[1] if groups else 1, "group_score": "best"}, prefix="m."), Runtime(torch.device("cuda"), dtype))
+    part.load({k: dev(v, dtype) for k, v in w.items()})
+    for tokens in (1, 7, 150):
+        x = rounded(rng.standard_normal((tokens, hidden)), BF16)
+        sure = plain.route(w, "m.", mlp["router"], x)[2] > 1e-3
+        h = dev(np.zeros((tokens, hidden)), F32)
+        part.forward(Ctx, dev(x, dtype), h)
+        assert_close(h.cpu().numpy()[sure], plain.routed(w, "m.", mlp, x)[sure], 1e-5 if dtype == F32 else 1e-2, f"{tokens} tokens")
+
+
+@pytest.mark.parametrize("experts,top,groups,keep", [(6, 2, 3, 1), (12, 4, 4, 2), (4, 1, 4, 2), (9, 3, 3, 1), (64, 6, 8, 4), (40, 5, 40, 7), (8, 2, 1, 1)])
+def test_router_takes_the_groups_of_the_largest_scores(experts, top, groups, keep):
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(11)
+    n, hidden = 97, 48
+    x = rounded(rng.standard_normal((n, hidden)), F32)
+    w = {"m.router": rounded(2 * rng.standard_normal((experts, hidden)) / np.sqrt(hidden), F32)}
+    r = {"experts": experts, "top": top}
+    if groups > 1:
+        r["groups"] = {"count": groups, "keep": keep}
+    chosen, weight, margin = plain.route(w, "m.", r, x)
+    if 1 < groups and keep < top:  # the best of each kept group come first: with as many groups as choices nothing changes
+        assert (np.sort(chosen, 1) != np.sort(plain.route(w, "m.", {"experts": experts, "top": top}, x)[0], 1)).any(), "the test's groups change no choice"
+    choice, wgt = torch.empty((n, top), dtype=torch.int32, device="cuda"), torch.empty((n, top), dtype=F32, device="cuda")
+    ops.moe_router(choice, wgt, None, dev(x, F32), dev(w["m.router"], F32), experts, top, True, True, None, 1e-20, groups, keep, 1.0, True)
+    sure = margin > 1e-5
+    assert sure.mean() > 0.9
+    assert (choice.cpu().numpy()[sure] == chosen[sure]).all()
+    assert_close(wgt.cpu().numpy()[sure], weight[sure], 1e-5, "weights")
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("rows,width", [(1, 96), (9, 100), (7, 30), (300, 64), (300, 1030), (300, 2560), (260, 1024), (33, 4096)])
+def test_layer_norm_with_and_without_owed_sums(dtype, rows, width):
+    """Rows far from zero mean (a variance taken as the mean of squares less the squared mean would lose them), picked
+    rows, and a product's split sums added on the way."""
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(12)
+    h = rounded(rng.standard_normal((rows, width)) + 200.0, F32)
+    g, b = rounded(1 + 0.3 * rng.standard_normal(width), F32), rounded(rng.standard_normal(width), F32)
+    tol = 1e-4 if dtype == F32 else 1e-2
+    want = plain.layer_norm(h, g, b, 1e-5)
+    out = torch.empty((rows, width), dtype=dtype, device="cuda")
+    ops.rmsnorm(out, dev(h, F32), dev(g, F32), 1e-5, None, dev(b, F32))
+    assert_close(out.float().cpu(), want, tol, "every size")
+    pick = rng.permutation(rows)[: max(1, rows // 2)].astype(np.int32)
+    few = torch.empty((len(pick), width), dtype=dtype, device="cuda")
+    ops.rmsnorm(few, dev(h, F32), dev(g, F32), 1e-5, dev(pick), dev(b, F32))
+    assert_close(few.float().cpu(), want[pick], tol, "picked rows")
+    out.zero_()
+    if not ops.norm_fused(out, dev(h, F32), dev(g, F32), 1e-5, shift=dev(b, F32)):
+        assert width % 4
+        return
+    assert_close(out.float().cpu(), want, tol, "vectorised")
+    planes, bias = rounded(rng.standard_normal((3, rows, width)), F32), rounded(rng.standard_normal(width), F32)
+    hd = dev(h, F32)
+    assert ops.norm_fused(out, hd, dev(g, F32), 1e-5, None, dev(planes, F32), 3, dev(bias, F32), shift=dev(b, F32))
+    full = h + planes.sum(axis=0) + bias
+    assert_close(hd.cpu(), full, 1e-6, "stream")
+    assert_close(out.float().cpu(), plain.layer_norm(full, g, b, 1e-5), tol, "with owed sums")
+
+
+# ---------------------------------------------------------------------------------------------------
+# whole models
+# ---------------------------------------------------------------------------------------------------
+LENGTHS = {"A": [1, 2, 23, 64, 65, 129, 200], "B": [3, 16, 17, 33, 80, 131], "C": [5, 64, 190, 257], "D": [2, 63, 150, 300], "E": [4, 65, 189, 400]}
+DECODED = 12
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    base = tmp_path_factory.mktemp("pekerax_gpu")
+    return {name: tiny.write(base / name, name, seed=10 + i) for i, name in enumerate(tiny.CONFIGS)}
+
+
+def make_requests(name):
+    reqs, prompts = {}, {}
+    for i, n in enumerate(LENGTHS[name]):
+        reqs[f"r{i}"] = tiny.tokens(name, n + DECODED, seed=i)
+        prompts[f"r{i}"] = n
+    return reqs, prompts
+
+
+@pytest.fixture(scope="module")
+def plain_logits(folders):
+    out = {}
+    for name, folder in folders.items():
+        w, cfg = plain.load(folder)
+        logits, sure = {}, {}
+        for rid, toks in make_requests(name)[0].items():
+            logits[rid], margins = plain.forward(w, cfg, toks, margins=True)
+            sure[rid] = plain.sure_prefix(margins, 0.05)
+        out[name] = (logits, sure)
+    return out
+
+
+def runner_for(folder, dtype, block, pages, max_requests=4, graphs=True):
+    from alofa_b200.engine.loading import load_model
+    from alofa_b200.engine.step import StepRunner
+
+    model, *_ = load_model(folder, dtype)
+    return StepRunner(model, block_size=block, num_pages=pages, max_requests=max_requests, max_tokens=pages * block, max_step_tokens=512, cuda_graphs=graphs)
+
+
+def assert_most_close(errors, tol, what):
+    errors = np.asarray(errors)
+    assert (errors > tol).mean() <= 0.25 and np.median(errors) <= tol / 3, \
+        f"{what}: {(errors > tol).sum()} of {len(errors)} positions beyond {tol:.1e}, median {np.median(errors):.3e}, worst {errors.max():.3e}"
+
+
+def compare(steps, outputs, want, vocab, tol, what, sure=None):
+    """Every position within ``tol`` in 32-bit.  In bfloat16 strictly up to a request's first close call of a router
+    (``sure``: two scores within rounding of one another, where bfloat16 may rightly take the other expert); over all
+    positions three quarters keep the bound and the median a third of it: a lost state, a wrong key or page moves
+    every position by order one."""
+    got = replay.collect(steps, outputs, vocab)
+    errors = []
+    for rid, rows in got.items():
+        ref = want[rid][: len(rows)]
+        assert rows.shape == ref.shape, f"{what} {rid}: {rows.shape} vs {ref.shape}"
+        err = np.abs(rows - ref).max(axis=-1) / max(1.0, float(np.abs(ref).max()))
+        n = len(rows) if sure is None else min(len(rows), sure[rid])
+        if n:
+            assert err[:n].max() <= tol, f"{what} {rid}: position {int(err[:n].argmax())} differs by {err[:n].max():.3e} > {tol:.1e}"
+        errors.append(err)
+    assert_most_close(np.concatenate(errors), tol, what)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", list(tiny.CONFIGS))
+def test_whole_decoded_portions_and_mixed_batches(folders, plain_logits, name, dtype):
+    """The same requests whole, with the last tokens decoded one by one, in portions down to two tokens, and mixed
+    (portions beside single tokens, four live at most, four state slots) in a pool that holds two of the longest: pages
+    and slots are given back and used again.  Every position against plain."""
+    reqs, prompts = make_requests(name)
+    vocab = tiny.CONFIGS[name]["vocab"]
+    block = 16 if name in ("B", "D") else 64
+    per_request = -(-max(len(t) for t in reqs.values()) // block)
+    schedules = {
+        "whole": (replay.whole(reqs), per_request),
+        "decoded": (replay.tail_decoded(reqs, tail=DECODED + 20), per_request),
+        "portions": (replay.portions(reqs), per_request),
+        "mixed": (replay.mixed(reqs, prompts, 2 * per_request * block + block, block, seed=3), 2 * per_request + 1),
+    }
+    for what, (steps, pages) in schedules.items():
+        runner = runner_for(folders[name], dtype, block, pages, max_requests=4)
+        out = replay.run_inprocess(runner, steps)
+        compare(steps, out, plain_logits[name][0], vocab, TOL[dtype], f"{name}/{dtype}/{what}", sure=plain_logits[name][1] if dtype == "bfloat16" else None)
+        assert set(runner.manager.free_pages()) == {pages} and runner.manager.live_requests() == 0
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "C", "D", "E"])
+def test_long_decoding_from_the_first_token(folders, name, dtype):
+    """One prompt token, then 170 tokens one by one (past page borders, past every window's edge and the kept tokens), two
+    requests side by side that started 40 steps apart; decode steps are replayed as graphs."""
+    from alofa_b200.engine.step import StepEntry
+
+    w, cfg = plain.load(folders[name])
+    a, b = tiny.tokens(name, 171, seed=50), tiny.tokens(name, 131, seed=51)
+    (want_a, ma), (want_b, mb) = plain.forward(w, cfg, a, margins=True), plain.forward(w, cfg, b, margins=True)
+    sure_a, sure_b = (plain.sure_prefix(ma, 0.05), plain.sure_prefix(mb, 0.05)) if dtype == "bfloat16" else (171, 131)
+    runner = runner_for(folders[name], dtype, 16, 22, max_requests=2)
+    sa, sb, errors = runner.admit(0), None, []
+    for i in range(171):
+        entries = [StepEntry(sa, [a[i]], [0])]
+        if i >= 40:
+            if sb is None:
+                sb = runner.admit(1)
+            entries.append(StepEntry(sb, [b[i - 40]], [0]))
+        rows = runner.forward(entries).float().cpu().numpy()
+        for row, want, k, sure, who in ((rows[0], want_a, i, sure_a, "first"),) + (((rows[1], want_b, i - 40, sure_b, "second"),) if i >= 40 else ()):
+            if k < sure:
+                assert_close(row, want[k], TOL[dtype], f"{who} request, token {k}")
+            errors.append(np.abs(row - want[k]).max() / max(1.0, float(np.abs(want).max())))
+    assert_most_close(errors, TOL[dtype], "long decoding")
+    runner.check_status()
+    assert runner.manager.defects() == 0
+
+
+def test_batches_and_cuts_do_not_change_a_request(folders):
+    """float32: a request's logits in portions and in a mixed batch equal, to rounding of the sums' order, those it gets alone and whole."""
+    name = "D"
+    reqs, prompts = make_requests(name)
+    vocab = tiny.CONFIGS[name]["vocab"]
+    alone = replay.collect(replay.whole(reqs), replay.run_inprocess(runner_for(folders[name], "float32", 16, 20), replay.whole(reqs)), vocab)
+    for what, steps, pages in (("portions", replay.portions(reqs), 20), ("mixed", replay.mixed(reqs, prompts, 700, 16, seed=9), 44)):
+        other = replay.collect(steps, replay.run_inprocess(runner_for(folders[name], "float32", 16, pages, max_requests=4), steps), vocab)
+        for rid in reqs:
+            assert np.abs(alone[rid] - other[rid]).max() <= 1e-5 * max(1.0, np.abs(alone[rid]).max()), f"{what} {rid}"
+
+
+def test_a_single_kept_page_is_held_and_the_rest_given_back(folders):
+    """After a long prompt a request of configuration D holds, in its windowed groups, the kept pages and the window's."""
+    from alofa_b200.engine.step import StepEntry
+
+    runner = runner_for(folders["D"], "bfloat16", 16, 25)
+    slot = runner.admit(0)
+    runner.forward([StepEntry(slot, tiny.tokens("D", 390, seed=3), [389])])
+    runner.check_status()
+    assert [(g.window, g.keep_first) for g in runner.group_specs] == [(37, 3), (100, 50)]
+    for gi, (window, keep) in enumerate(((37, 3), (100, 50))):
+        table = runner.manager.block_table(slot, gi)
+        kept, passed = -(-keep // 16), (390 - window + 1) // 16
+        assert (table[:kept] >= 0).all() and (table[kept:passed] < 0).all() and (table[passed:] >= 0).all()
+
+
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_the_stream_after_every_layer(folders, name):
+    """float32: the residual stream after each layer."""
+    import alofa_b200.parts.block as block
+    from alofa_b200.engine.step import StepEntry
+
+    w, cfg = plain.load(folders[name])
+    ids = tiny.tokens(name, 30, seed=77)
+    _, want = plain.forward(w, cfg, ids, streams=True)
+    seen, original = [], block.PrenormResidual.forward
+
+    def recording(self, ctx, h, cache, writes=True):
+        original(self, ctx, h, cache, writes)
+        ctx.flush_pending()
+        seen.append(h.double().cpu().numpy())
+
+    block.PrenormResidual.forward = recording
+    try:
+        runner = runner_for(folders[name], "float32", 64, 1, graphs=False)
+        runner.forward([StepEntry(runner.admit(0), ids, [0])])
+    finally:
+        block.PrenormResidual.forward = original
+    assert len(seen) == len(want) == len(cfg["layers"])
+    for k, (got, ref) in enumerate(zip(seen, want)):
+        assert_close(got, ref, TOL["float32"], f"after layer {k}")
+
+
+@pytest.mark.parametrize("name", list(tiny.CONFIGS))
+def test_greedy_generation_through_the_engine(folders, name):
+    """Engine.generate (scheduler, chunked prefill, decode graphs): float32 tokens equal plain greedy; bfloat16 tokens
+    are each within rounding of the plain maximum, up to the first close call of a router."""
+    from alofa_b200.engine.engine import Engine
+
+    w, cfg = plain.load(folders[name])
+    prompts = [tiny.tokens(name, n, seed=200 + i) for i, n in enumerate([1, 7, 40, 90, 18])]
+    want = [plain.greedy(w, cfg, p, 6) for p in prompts]
+    eng = Engine(str(folders[name]), dtype="float32", block_size=16, max_batch=3, token_budget=48, max_chunk=32, max_tokens=128)
+    assert eng.generate(prompts, max_new_tokens=6) == want
+    assert eng.stats()["defects"] == 0
+    eng16 = Engine(str(folders[name]), dtype="bfloat16", block_size=16, max_batch=3, token_budget=48, max_chunk=32, max_tokens=128)
+    for p, out in zip(prompts, eng16.generate(prompts, max_new_tokens=6)):
+        seq = list(p)
+        for tok in out:
+            logits, margins = plain.forward(w, cfg, seq, margins=True)
+            if plain.sure_prefix(margins, 0.05) < len(seq):
+                break
+            row = logits[-1]
+            assert row.max() - row[tok] <= 8e-2 * max(1.0, float(np.abs(row).max())), "a bfloat16 token is not near the plain maximum"
+            seq.append(tok)
+    eng16.runner.check_status()
+
+
+def test_the_programs_take_the_architecture(folders, tmp_path):
+    """bin/trace_run replays a schedule and bin/generate generates, both choosing the model by config.json."""
+    name = "C"
+    reqs, _ = make_requests(name)
+    reqs = {k: reqs[k] for k in ("r0", "r2")}
+    w, cfg = plain.load(folders[name])
+    want = {rid: plain.forward(w, cfg, t) for rid, t in reqs.items()}
+    steps = replay.portions(reqs, sizes=(40, 2, 3, 64, 1))
+    out = replay.run_trace_program(folders[name], "float32", steps, tmp_path / "out", 512)
+    compare(steps, out, want, cfg["vocab"], TOL["float32"], "trace_run")
+    prompt = tiny.tokens(name, 12, seed=5)
+    done = subprocess.run([sys.executable, str(replay.ROOT / "bin" / "generate"), "--model", str(folders[name]), "--dtype", "float32", "--prompt-ids",
+                           ",".join(map(str, prompt)), "--max-new-tokens", "5", "--max-tokens", "64", "--json"], capture_output=True, text=True, timeout=600)
+    assert done.returncode == 0, done.stderr[-2000:]
+    assert json.loads(done.stdout.strip().splitlines()[-1])["out_ids"] == [plain.greedy(w, cfg, prompt, 5)]
