@@ -1296,6 +1296,9 @@ def _delta():
         sigs = {
             "alofa_min_gru": [_P, _P, _I, _I, _I, _I, _P, _L, _P, _P, _I, _I, _I, _I, _P],
             "alofa_delta_prepare": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
+            "alofa_delta_pairs": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+            "alofa_delta_pair_words": [],
+            "alofa_delta_group_scan": [_P, _P, _I, _I, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
             "alofa_delta_scan": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         }
         for name, args in sigs.items():
@@ -1363,6 +1366,41 @@ def delta_scan(y, v, v_off: int, kn, qn, kq, g, beta, state, q_start, state_slot
     _done(_delta().alofa_delta_scan(_dev(y, "y", f32), _dev(v, "v", f32), v.shape[1], v_off, _dev(kn, "kn", f32), _dev(qn, "qn", f32), _dev(kq, "kq", f32), _dev(g, "g", f32),
                                     _dev(beta, "beta", f32), state.data_ptr(), state.stride(0), _dev(q_start, "q_start", i32), _dev(state_slots, "state_slots", i32),
                                     rows, n_seqs, heads, groups, n, p, 1 if one else 0, spread, _stream()), "delta_scan", f"heads={heads} groups={groups} n={n} p={p}")
+
+
+def delta_pair_words() -> int:
+    """Numbers per token and head of :func:`delta_pairs`."""
+    return _delta().alofa_delta_pair_words()
+
+
+def delta_pairs(pairs, kn, qn, kq, g, beta, heads: int, groups: int, n: int) -> None:
+    """What :func:`delta_group_scan` reads of a token beside its key, query and
+    values, per head: beta, its decay, and the decayed products of its key and
+    query with the keys of the three tokens before it; ``pairs`` fp32 [T, heads *
+    delta_pair_words()], the other operands as :func:`delta_prepare` leaves
+    them (one decay per head)."""
+    f32 = torch.float32
+    rows = kn.shape[0]
+    if (tuple(pairs.shape) != (rows, heads * delta_pair_words()) or tuple(kn.shape) != (rows, groups * n) or tuple(qn.shape) != (rows, groups * n) or tuple(kq.shape) != (rows, groups)
+            or tuple(g.shape) != (rows, heads) or tuple(beta.shape) != (rows, heads)):
+        raise AlofaError("invalid_argument", "delta_pairs sizes disagree", f"pairs={tuple(pairs.shape)} kn={tuple(kn.shape)} heads={heads} groups={groups} n={n}")
+    _done(_delta().alofa_delta_pairs(_dev(pairs, "pairs", f32), _dev(kn, "kn", f32), _dev(qn, "qn", f32), _dev(kq, "kq", f32), _dev(g, "g", f32), _dev(beta, "beta", f32),
+                                     rows, heads, groups, n, _stream()), "delta_pairs", f"heads={heads} groups={groups} n={n}")
+
+
+def delta_group_scan(y, v, v_off: int, kn, qn, pairs, state, q_start, state_slots, n_seqs: int, heads: int, groups: int, n: int, p: int, spread: int = 0) -> None:
+    """:func:`delta_scan` with one decay per head, four tokens at a time (their
+    dot products with the state side by side, the state decayed and written
+    once): the same sums in another order.  ``pairs`` from :func:`delta_pairs`."""
+    f32, i32 = torch.float32, torch.int32
+    rows = y.shape[0]
+    if (tuple(y.shape) != (rows, heads * p) or v.shape[0] != rows or v_off + heads * p > v.shape[1] or tuple(kn.shape) != (rows, groups * n) or tuple(qn.shape) != (rows, groups * n)
+            or tuple(pairs.shape) != (rows, heads * delta_pair_words())):
+        raise AlofaError("invalid_argument", "delta_group_scan sizes disagree", f"y={tuple(y.shape)} v={tuple(v.shape)} heads={heads} groups={groups} n={n} p={p}")
+    _slot_state(state, heads * p * n, "delta_group_scan")
+    _done(_delta().alofa_delta_group_scan(_dev(y, "y", f32), _dev(v, "v", f32), v.shape[1], v_off, _dev(kn, "kn", f32), _dev(qn, "qn", f32), _dev(pairs, "pairs", f32), state.data_ptr(),
+                                          state.stride(0), _dev(q_start, "q_start", i32), _dev(state_slots, "state_slots", i32), rows, n_seqs, heads, groups, n, p, spread,
+                                          _stream()), "delta_group_scan", f"heads={heads} groups={groups} n={n} p={p}")
 
 
 # -- the real-gated linear recurrent unit ------------------------------------------------------------

@@ -60,6 +60,8 @@ from .linear import RESIDUAL, STORE, Linear, add_into_stream
 
 # blocks a scan launch should have before its value channels stop being dealt to more of them (about one per SM)
 SCAN_SPREAD = 128
+# tokens a request of the step, on average, from which the delta rule with one decay per head goes four tokens at a time
+GROUPED_FROM = 2
 
 
 def _project_out(ctx, linear_add: Linear, linear_store: Linear, h, x, store: bool) -> None:
@@ -278,7 +280,7 @@ class GatedDelta(Part):
         return SlotState((self.scan_words + self.conv_words,), torch.float32)
 
     def scratch_row_bytes(self) -> int:
-        return 4 * (self.in_rows + self.channels + 2 * (self.decays + self.v) + 2 * self.qk + 2 * self.heads + self.kv_heads + 2 * self.v) + 8 * self.hidden + 512
+        return 4 * (self.in_rows + self.channels + 2 * (self.decays + self.v) + 2 * self.qk + 2 * self.heads + self.kv_heads + 2 * self.v + 12 * self.heads) + 8 * self.hidden + 512
 
     def tensors(self):
         pre = self.prefix
@@ -341,7 +343,12 @@ class GatedDelta(Part):
         kq, g, beta = ctx.buf((n, G), f32), ctx.buf((n, self.decays), f32), ctx.buf((n, H), f32)
         ops.delta_prepare(qn, kn, kq, g, beta, xc, z, u, self.channels, self.dt_bias, self.a_log, H, G, N, self.UNIT_EPS, N ** -0.5, at)
         y = ctx.buf((n, self.v), f32)
-        ops.delta_scan(y, xc, 2 * self.qk, kn, qn, kq, g, beta, st, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, G, N, P, spread=SCAN_SPREAD)
+        if self.decays == H and n >= GROUPED_FROM * ctx.n_seqs:  # portions of prompts: four tokens at a time
+            pairs = ctx.buf((n, H * ops.delta_pair_words()), f32)
+            ops.delta_pairs(pairs, kn, qn, kq, g, beta, H, G, N)
+            ops.delta_group_scan(y, xc, 2 * self.qk, kn, qn, pairs, st, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, G, N, P, spread=SCAN_SPREAD)
+        else:
+            ops.delta_scan(y, xc, 2 * self.qk, kn, qn, kq, g, beta, st, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, G, N, P, spread=SCAN_SPREAD)
         normed = ctx.buf((n, self.v), self.rt.dtype)
         ops.gated_group_norm(normed, y, z, at + self.decays, self.norm_w, H, self.eps, gate_first=False, sigmoid=self.gate_sigmoid)
         _project_out(ctx, self.out_add, self.out_store, h, normed, store)

@@ -656,7 +656,7 @@ class KernelClock:
 
     PRODUCTS = ("gemm_tc", "gemm_generic", "gemm_batched", "gemm_tc_rope")
     ATTENTION = ("attention_bf16", "latent_attention_bf16", "latent_attention", "paged_attention_generic")
-    STATE = ("linear_scan", "causal_conv", "delta_scan", "min_gru", "lru_scan")  # read and leave a state per request
+    STATE = ("linear_scan", "causal_conv", "delta_scan", "delta_group_scan", "min_gru", "lru_scan")  # read and leave a state per request
 
     def __init__(self, peaks: dict):
         self.peaks = peaks
@@ -710,6 +710,15 @@ class KernelClock:
             fp32_rate = _t.cuda.get_device_properties(0).multi_processor_count * 128 * 2 * 1.965e9
             ideal = max(7.0 * rows * heads * n * p / fp32_rate, byts / (self.peaks["hbm_gbs"] * 1e9)) * 1e6
             return ideal, 7.0 * rows * heads * n * p, byts
+        elif name == "delta_group_scan":
+            # y, v, ., kn, qn, pairs, state, q_start, slots, n_seqs, heads, groups, n, p; the flops of the recurrence itself, as above
+            y, n_seqs, heads, groups, n, p = args[0], args[9], args[10], args[11], args[12], args[13]
+            rows = y.shape[0]
+            byts = 4 * rows * (2 * heads * p + 2 * groups * n + args[5].shape[1]) + 8 * n_seqs * heads * n * p
+            import torch as _t
+
+            fp32_rate = _t.cuda.get_device_properties(0).multi_processor_count * 128 * 2 * 1.965e9
+            return max(7.0 * rows * heads * n * p / fp32_rate, byts / (self.peaks["hbm_gbs"] * 1e9)) * 1e6, 7.0 * rows * heads * n * p, byts
         elif name == "qkv_prepare_rows":
             # q_out, k_cache, v_cache, qkv: a step's rows of the projection (or its split sums) read, q, keys and values written, the shared values once
             q, k, v, qkv = args[:4]
@@ -759,7 +768,7 @@ class KernelClock:
         self.pairs = pairs
         names = [n for n in dir(ops) if not n.startswith("_") and callable(getattr(ops, n)) and getattr(getattr(ops, n), "__module__", "") == ops.__name__
                  and n not in ("launch_count", "count_launches", "bound_stream", "attention_decode_wide_warps", "attention_decode_slots", "attention_bf16_supported",
-                               "gemm_tc_rope_splits", "gemm_tc_splits", "latent_attention_bf16_supported", "load_library", "gemm_by_tile")]  # gemm_by_tile only chooses: its product is timed
+                               "gemm_tc_rope_splits", "gemm_tc_splits", "delta_pair_words", "latent_attention_bf16_supported", "load_library", "gemm_by_tile")]  # gemm_by_tile only chooses: its product is timed
         originals = {n: getattr(ops, n) for n in names}
         records = []
 

@@ -334,10 +334,10 @@ def delta_weights(rng, m, slow=False, prefix="d."):
 
 
 class Delta:
-    """The kernels of the mixer with a state per slot, as the part runs them."""
+    """The kernels of the mixer with a state per slot, as the part runs them (``grouped`` False: token by token in every step)."""
 
-    def __init__(self, w, m, slots, dtype, eps, prefix="d."):
-        self.m, self.dtype, self.eps = m, dtype, eps
+    def __init__(self, w, m, slots, dtype, eps, grouped=True, prefix="d."):
+        self.m, self.dtype, self.eps, self.grouped = m, dtype, eps, grouped
         H, G, n, P = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         self.channels, self.words = 2 * G * n + H * P, H * n * P
         self.state = torch.zeros((slots, self.words + (m["conv"] - 1) * self.channels), dtype=F32, device="cuda")
@@ -357,7 +357,12 @@ class Delta:
         ops.causal_conv(xc, u, 0, self.conv, None, self.state[:, self.words :], q_start, slots, seq, len(counts))
         qn, kn, kq, g, beta, y = new(T, G * n), new(T, G * n), new(T, G), new(T, H), new(T, H), new(T, H * P)
         ops.delta_prepare(qn, kn, kq, g, beta, xc, u, u, self.channels, self.dt_bias, self.a_log, H, G, n, 1e-6, n ** -0.5, self.channels + H)
-        ops.delta_scan(y, xc, 2 * G * n, kn, qn, kq, g, beta, self.state, q_start, slots, len(counts), H, G, n, P, spread=128)
+        if self.grouped and T >= 2 * len(counts):
+            pairs = new(T, H * ops.delta_pair_words())
+            ops.delta_pairs(pairs, kn, qn, kq, g, beta, H, G, n)
+            ops.delta_group_scan(y, xc, 2 * G * n, kn, qn, pairs, self.state, q_start, slots, len(counts), H, G, n, P, spread=128)
+        else:
+            ops.delta_scan(y, xc, 2 * G * n, kn, qn, kq, g, beta, self.state, q_start, slots, len(counts), H, G, n, P, spread=128)
         out = torch.empty((T, H * P), dtype=self.dtype, device="cuda")
         ops.gated_group_norm(out, y, u, self.channels + 2 * H, self.norm, H, self.eps, gate_first=False)
         return out.float().cpu().numpy()
@@ -382,7 +387,7 @@ def walk(lengths, cuts, slots_of, xs, mixer):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("H,G,n,P,K", [(6, 3, 12, 20, 4), (2, 2, 16, 8, 1), (5, 1, 7, 9, 3), (4, 2, 64, 32, 2), (1, 1, 128, 256, 4), (2, 1, 130, 6, 2), (3, 3, 1, 4, 2), (2, 1, 300, 12, 3)])
+@pytest.mark.parametrize("H,G,n,P,K", [(6, 3, 12, 20, 4), (2, 2, 16, 8, 1), (5, 1, 7, 9, 3), (4, 2, 64, 32, 2), (1, 1, 128, 256, 4), (2, 1, 130, 6, 2), (3, 3, 1, 4, 2), (2, 1, 300, 12, 3), (2, 2, 40, 16, 2), (1, 1, 600, 8, 2)])
 def test_delta_rule_with_one_decay_a_head_over_portions_in_slots_used_out_of_order(dtype, H, G, n, P, K):
     """Convolutions and recurrence carried from step to step: portions of 1, 2 and many tokens, requests that sit steps
     out, slots in another order than the requests and used again."""
@@ -392,13 +397,14 @@ def test_delta_rule_with_one_decay_a_head_over_portions_in_slots_used_out_of_ord
     lengths = [1, 2, 37, 90, 203]
     xs = [rounded(rng.standard_normal((t, width)), F32) for t in lengths]
     want = [plain.delta(w, "d.", m, x, 1e-5) for x in xs]
-    mixer = Delta(w, m, 7, dtype, 1e-5)
-    mixer.state.fill_(3.0)  # what a slot's last user left
-    for cuts, slots_of, count in (((1, 2, 3, 17, 190), [5, 0, 3, 6, 1], 5), ((1,), [2, 4, 5, 0], 4)):
-        for s in slots_of:
-            mixer.state[s].zero_()  # as the engine does when a request is admitted
-        for r, got in enumerate(walk(lengths[:count], cuts, slots_of, xs, mixer)):
-            assert_close(got, want[r], KERNEL_TOL[dtype] * (2 if dtype == F32 else 1), f"cuts {cuts}: request of {lengths[r]} tokens")
+    for grouped in (True, False):
+        mixer = Delta(w, m, 7, dtype, 1e-5, grouped)
+        mixer.state.fill_(3.0)  # what a slot's last user left
+        for cuts, slots_of, count in (((1, 2, 3, 17, 190), [5, 0, 3, 6, 1], 5), ((4, 5, 6, 7, 64), [4, 2, 1, 0, 6], 5), ((1,), [2, 4, 5, 0], 4)):
+            for s in slots_of:
+                mixer.state[s].zero_()  # as the engine does when a request is admitted
+            for r, got in enumerate(walk(lengths[:count], cuts, slots_of, xs, mixer)):
+                assert_close(got, want[r], KERNEL_TOL[dtype] * (2 if dtype == F32 else 1), f"cuts {cuts}: request of {lengths[r]} tokens")
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
