@@ -122,7 +122,7 @@ def test_decode_with_more_work_than_the_device_holds_at_once(folders, name, monk
         # kernel; eight, twice, whose splits the output product merges; nineteen with one split each on the wide kernel's eight or six warps
         for step, (live, room, wide) in enumerate(((range(20), 40, 0), (range(4, 12), 16, 0), (range(4, 12), 16, 0), (range(19), 40, 40))):  # nineteen: a graph of its own
             monkeypatch.setattr(ops, "attention_decode_slots",
-                                lambda hd, page, warps=4, room=room, wide=wide: room if warps == 4 else min(wide, real_slots(hd, page, warps)))
+                                lambda hd, page, warps=4, *library, room=room, wide=wide: room if warps == 4 else min(wide, real_slots(hd, page, warps, *library)))
             logits = runner.forward([StepEntry(slots[i], [seqs[i][lens[i] + len(got[i])]], [0]) for i in live]).float().cpu().numpy()
             for row, i in zip(logits, live):
                 got[i].append(row)
