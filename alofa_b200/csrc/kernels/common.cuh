@@ -74,6 +74,8 @@ __device__ __forceinline__ float fast_gate_times(float g, float u, float alpha, 
 // Activations that an epilogue may apply to its fp32 sums (after the bias): the precise library
 // functions, the same in every kernel that takes an activation code.
 enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_RELU = 4, ACT_RELU_SQUARED = 5 };
+__device__ __forceinline__ float logistic(float z) { return 1.0f / (1.0f + expf(-z)); }
+
 __device__ __forceinline__ float activate(float z, int act) {
   switch (act) {
     case ACT_GELU_ERF: return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));  // the exact gelu: z Phi(z)

@@ -5,7 +5,7 @@
 // batch the tile names (experts of a routed feed-forward, rows sorted by
 // expert and padded to whole tiles).  64 x 64 output tile per CTA, 32-deep
 // slices by cp.async into two shared-memory buffers, four warps of 32 x 32
-// (mma.sync m16n8k16, fp32 sums), bias and activation on the fp32 sums.  The
+// (mma.sync m16n8k16, fp32 sums), bias, activation and gate on the fp32 sums.  The
 // depth, the row strides and the batch strides are multiples of 8 elements and
 // the operands start on 16-byte boundaries (the caller checks).
 #include "common.cuh"
@@ -29,7 +29,8 @@ template <typename TO>
 __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__ out, const bf16* __restrict__ x, const bf16* __restrict__ w,
                                                                 const float* __restrict__ bias, const int* __restrict__ tile_batch, int M, int N,
                                                                 int K, long long ldx, long long x_batch, long long ldw, long long w_batch,
-                                                                long long ldo, long long out_batch, long long bias_batch, int act, int tile_rows) {
+                                                                long long ldo, long long out_batch, long long bias_batch, int act, int tile_rows,
+                                                                const float* __restrict__ gate, long long ldg, long long gate_batch) {
   __shared__ __align__(16) bf16 As[2][TM * LD];
   __shared__ __align__(16) bf16 Bs[2][TN * LD];
   pdl_begin();
@@ -43,6 +44,7 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
   }
   w += (size_t)b * w_batch;
   if (bias) bias += (size_t)b * bias_batch;
+  if (gate) gate += (size_t)b * gate_batch;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int wm = warp & 1, wn = warp >> 1, g = lane >> 2, t = lane & 3;
   const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
@@ -101,7 +103,11 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
       for (int k = 0; k < 4; ++k) {
         const int gm = m0 + wm * 32 + i * 16 + g + (k >> 1) * 8;
         const int gn = n0 + wn * 32 + j * 8 + 2 * t + (k & 1);
-        if (gm < M && gn < N) out[(size_t)gm * ldo + gn] = from_f<TO>(activate(acc[i][j][k] + (bias ? bias[gn] : 0.f), act));
+        if (gm < M && gn < N) {
+          float v = activate(acc[i][j][k] + (bias ? bias[gn] : 0.f), act);
+          if (gate) v *= logistic(gate[(size_t)gm * ldg + gn]);
+          out[(size_t)gm * ldo + gn] = from_f<TO>(v);
+        }
       }
 }
 
@@ -109,17 +115,18 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
 
 ALOFA_API int alofa_gemm_batched_bf16(void* out, const void* x, const void* w, const float* bias, const int* tile_batch, int batches, int M, int N, int K,
                                       long long ldx, long long x_batch, long long ldw, long long w_batch, long long ldo, long long out_batch,
-                                      long long bias_batch, int act, int tile_rows, int out_bf16, cudaStream_t stream) {
+                                      long long bias_batch, int act, int tile_rows, const float* gate, long long ldg, long long gate_batch, int out_bf16,
+                                      cudaStream_t stream) {
   if (M <= 0 || N <= 0 || batches <= 0) return ALOFA_OK;
-  if (tile_batch && (tile_rows <= 0 || tile_rows % TM)) return ALOFA_ERR_ARGUMENT;
+  if (tile_batch && (tile_rows <= 0 || tile_rows % TM || gate)) return ALOFA_ERR_ARGUMENT;
   if (K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || (x_batch & 7) || (w_batch & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return ALOFA_ERR_ARGUMENT;
   if ((M + TM - 1) / TM > 65535 || batches > 65535) return ALOFA_ERR_ARGUMENT;
   dim3 grid((N + TN - 1) / TN, (M + TM - 1) / TM, tile_batch ? 1 : batches);
   if (out_bf16)
     launch_dep(gemm_batched_bf16_kernel<bf16>, grid, dim3(128), 0, stream, (bf16*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx, x_batch,
-               ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows);
+               ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch);
   else
     launch_dep(gemm_batched_bf16_kernel<float>, grid, dim3(128), 0, stream, (float*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx,
-               x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows);
+               x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch);
   return launch_status();
 }

@@ -88,7 +88,7 @@ ALOFA_API int alofa_latent_prepare(void* cq, void* cache, const float* lat, cons
                                    const int* positions, const int* slot_map, int n_tokens, int q_rank, int kv_rank, int rot, int rot_dims,
                                    float eps, int ld, int halves, float mag, int is_bf16, cudaStream_t stream) {
   if (n_tokens <= 0) return ALOFA_OK;
-  if (q_rank < 0 || kv_rank <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || ld < q_rank + kv_rank + rot) return ALOFA_ERR_ARGUMENT;
+  if (q_rank < 0 || kv_rank <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || ld < q_rank + (cache ? kv_rank + rot : 0)) return ALOFA_ERR_ARGUMENT;
   if (is_bf16)
     launch_dep(latent_prepare_kernel<bf16>, n_tokens, 256, 0, stream, (bf16*)cq, (bf16*)cache, lat, wq, wkv, freq, positions, slot_map, q_rank, kv_rank,
                rot, rot_dims, eps, ld, halves, mag);
@@ -172,7 +172,8 @@ ALOFA_API int alofa_rotary_interleaved(void* x, const float* freq, const int* po
 // ---------------------------------------------------------------------------
 // Batched product with strides: for batch b, out_b[m, n] = act(sum_k x_b[m, k] * w_b[n, k] + bias_b[n]),
 //   x_b = x + b * x_batch (row stride ldx), w_b = w + b * w_batch (row stride ldw),
-//   out_b = out + b * out_batch (row stride ldo), bias_b = bias + b * bias_batch.
+//   out_b = out + b * out_batch (row stride ldo), bias_b = bias + b * bias_batch; with a gate (fp32 logits, not with
+//   tile_batch) times 1 / (1 + exp(-gate_b[m, n])), gate_b = gate + b * gate_batch (row stride ldg).
 // With tile_batch (one entry per tile of tile_rows rows of M, a multiple of 64) there is one x and one out,
 // and tile i multiplies by the weight of batch tile_batch[i] (negative: the
 // tile is empty): rows sorted by expert, each expert's rows padded to whole tiles.
@@ -182,7 +183,8 @@ template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256) gemm_batched_kernel(TO* __restrict__ out, const TA* __restrict__ x, const TW* __restrict__ w,
                                                            const float* __restrict__ bias, const int* __restrict__ tile_batch, int M, int N, int K,
                                                            long long ldx, long long x_batch, long long ldw, long long w_batch, long long ldo,
-                                                           long long out_batch, long long bias_batch, int act, int tile_rows) {
+                                                           long long out_batch, long long bias_batch, int act, int tile_rows, const float* __restrict__ gate,
+                                                           long long ldg, long long gate_batch) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float xs[BK][BM + 1];
   __shared__ float ws[BK][BN + 1];
@@ -198,6 +200,7 @@ __global__ void __launch_bounds__(256) gemm_batched_kernel(TO* __restrict__ out,
     w += (size_t)b * w_batch;
     out += (size_t)b * out_batch;
     if (bias) bias += (size_t)b * bias_batch;
+    if (gate) gate += (size_t)b * gate_batch;
   }
   const int tid = threadIdx.x;
   const int tx = tid & 15, ty = tid >> 4;
@@ -241,7 +244,9 @@ __global__ void __launch_bounds__(256) gemm_batched_kernel(TO* __restrict__ out,
       if (gn >= N) continue;
       float v = acc[i][j];
       if (bias) v += bias[gn];
-      out[(size_t)gm * ldo + gn] = from_f<TO>(activate(v, act));
+      v = activate(v, act);
+      if (gate) v *= logistic(gate[(size_t)gm * ldg + gn]);
+      out[(size_t)gm * ldo + gn] = from_f<TO>(v);
     }
   }
 }
@@ -249,22 +254,23 @@ __global__ void __launch_bounds__(256) gemm_batched_kernel(TO* __restrict__ out,
 template <typename TA, typename TW, typename TO>
 static int gemm_batched_launch(void* out, const void* x, const void* w, const float* bias, const int* tile_batch, int batches, int M, int N, int K,
                                long long ldx, long long x_batch, long long ldw, long long w_batch, long long ldo, long long out_batch,
-                               long long bias_batch, int act, int tile_rows, cudaStream_t stream) {
+                               long long bias_batch, int act, int tile_rows, const float* gate, long long ldg, long long gate_batch, cudaStream_t stream) {
   dim3 grid((N + 63) / 64, (M + 63) / 64, tile_batch ? 1 : batches);
   launch_dep(gemm_batched_kernel<TA, TW, TO>, grid, dim3(256), 0, stream, (TO*)out, (const TA*)x, (const TW*)w, bias, tile_batch, M, N, K, ldx,
-             x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows);
+             x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch);
   return launch_status();
 }
 
 // dtype flags: 0 = fp32, 1 = bf16.  x and w share a dtype flag pair as in alofa_gemm_generic.
 ALOFA_API int alofa_gemm_batched(void* out, const void* x, const void* w, const float* bias, const int* tile_batch, int batches, int M, int N, int K,
                                  long long ldx, long long x_batch, long long ldw, long long w_batch, long long ldo, long long out_batch,
-                                 long long bias_batch, int act, int tile_rows, int x_bf16, int w_bf16, int out_bf16, cudaStream_t stream) {
+                                 long long bias_batch, int act, int tile_rows, const float* gate, long long ldg, long long gate_batch, int x_bf16, int w_bf16,
+                                 int out_bf16, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || batches <= 0) return ALOFA_OK;
-  if (K <= 0 || (M + 63) / 64 > 65535 || batches > 65535 || (tile_batch && (tile_rows <= 0 || tile_rows % 64))) return ALOFA_ERR_ARGUMENT;
+  if (K <= 0 || (M + 63) / 64 > 65535 || batches > 65535 || (tile_batch && (tile_rows <= 0 || tile_rows % 64 || gate))) return ALOFA_ERR_ARGUMENT;
   const int key = (x_bf16 ? 4 : 0) | (w_bf16 ? 2 : 0) | (out_bf16 ? 1 : 0);
 #define ALOFA_BATCHED(TA, TW, TO) \
-  return gemm_batched_launch<TA, TW, TO>(out, x, w, bias, tile_batch, batches, M, N, K, ldx, x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, stream)
+  return gemm_batched_launch<TA, TW, TO>(out, x, w, bias, tile_batch, batches, M, N, K, ldx, x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch, stream)
   switch (key) {
     case 0: ALOFA_BATCHED(float, float, float);
     case 1: ALOFA_BATCHED(float, float, bf16);

@@ -590,7 +590,10 @@ ALOFA_API int alofa_qkv_prepare(void* q_out, void* k_cache, void* v_cache, const
 // k: G * d | v: G * dv | more].  q / sqrt(mean(q^2) + eps) * q_w (q_w [H * d]) to its buffer, k likewise (k_w [G * d]) and v to
 // the token's cache slot.  v_first (optional, fp32 [T, G * dv]): the values of the first of several layers that mix
 // theirs.  mix null: this is that layer, its values are left there; else v <- (1 - mix) v + mix v_first before it is
-// stored.  One block per token: the row's q and k wait in shared memory for their sums.
+// stored.  With rot.dims > 0 the first rot.dims numbers of every q and k head (d numbers each) are then turned by the token's
+// position: neighbouring pairs or (rot.halves) number i with number i + dims / 2, by the angle p * freq[i] (an fp32 product,
+// precise sine and cosine, once per token), cosine and sine times mag.  One block per token: the row's q and k wait in shared
+// memory for their sums.
 // ---------------------------------------------------------------------------
 template <typename T, int V>
 struct PackedStore;
@@ -631,16 +634,30 @@ __device__ __forceinline__ void row_columns(float (&x)[V], const float* row, int
   }
 }
 
+struct RowRotation {
+  const int* positions;
+  const float* freq;
+  int d, dims, halves;
+  float mag;
+};
+
 template <typename T, int V>
 __global__ void __launch_bounds__(1024) qkv_prepare_rows_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const float* __restrict__ qkv, int ld,
                                                                 const int* __restrict__ slot_map, int nq, int nk, int nv, const float* __restrict__ q_w,
                                                                 const float* __restrict__ k_w, float eps, float* __restrict__ v_first, const float* __restrict__ mix,
                                                                 int splits, long long plane, const float* __restrict__ bias, float* __restrict__ extra_out, int extra_at,
-                                                                int extra_n) {
-  extern __shared__ __align__(16) float row_smem[];  // nq + nk numbers
+                                                                int extra_n, RowRotation rot) {
+  extern __shared__ __align__(16) float row_smem[];  // nq + nk numbers, then rot.dims: cosine and sine of every pair
   __shared__ float scratch[32];
   pdl_begin();
   const int t = blockIdx.x;
+  float* turns = row_smem + nq + nk;
+  for (int i = threadIdx.x; i < rot.dims / 2; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)rot.positions[t] * rot.freq[i], &sn, &cs);
+    turns[2 * i] = cs * rot.mag;
+    turns[2 * i + 1] = sn * rot.mag;
+  }
   const float* row = qkv + (size_t)t * ld;
   const int slot = slot_map[t];
   float sq = 0.f, sk = 0.f;
@@ -688,6 +705,21 @@ __global__ void __launch_bounds__(1024) qkv_prepare_rows_kernel(T* __restrict__ 
     float x[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) x[i] = row_smem[c + i] * r * w[i];
+    if (rot.dims > 0) {
+      const int e0 = (is_q ? c : c - nq) % rot.d;
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        int e = e0 + i;
+        if (e >= rot.d) e %= rot.d;  // a quad may run over a head's end
+        if (e >= rot.dims) continue;
+        const int half = rot.dims / 2;
+        const bool second = rot.halves ? e >= half : (e & 1);
+        const int pair = rot.halves ? (second ? e - half : e) : e >> 1;
+        const int away = rot.halves ? (second ? -half : half) : (second ? -1 : 1);
+        const float other = row_smem[c + i + away] * r * w[i + away];
+        x[i] = second ? x[i] * turns[2 * pair] + other * turns[2 * pair + 1] : x[i] * turns[2 * pair] - other * turns[2 * pair + 1];
+      }
+    }
     PackedStore<T, V>::put(is_q ? q_out + (size_t)t * nq + c : k_cache + (size_t)slot * nk + (c - nq), x);
   }
 }
@@ -695,8 +727,8 @@ __global__ void __launch_bounds__(1024) qkv_prepare_rows_kernel(T* __restrict__ 
 template <typename T, int V>
 static int qkv_prepare_rows_launch(void* q_out, void* k_cache, void* v_cache, const float* qkv, int ld, const int* slot_map, int n_tokens, int nq, int nk, int nv,
                                    const float* q_w, const float* k_w, float eps, float* v_first, const float* mix, int splits, long long plane, const float* bias,
-                                   float* extra_out, int extra_at, int extra_n, cudaStream_t stream) {
-  const size_t smem = (size_t)(nq + nk) * sizeof(float);
+                                   float* extra_out, int extra_at, int extra_n, const RowRotation& rot, cudaStream_t stream) {
+  const size_t smem = (size_t)(nq + nk + rot.dims) * sizeof(float);
   if (smem > 200 * 1024) return ALOFA_ERR_ARGUMENT;
   static size_t set = 48 * 1024;
   if (smem > set) {
@@ -707,15 +739,19 @@ static int qkv_prepare_rows_launch(void* q_out, void* k_cache, void* v_cache, co
   int threads = groups >= 1024 ? 1024 : (groups + 31) / 32 * 32;
   if (n_tokens > 148 && threads > 256) threads = 256;
   launch_dep(qkv_prepare_rows_kernel<T, V>, n_tokens, threads, smem, stream, (T*)q_out, (T*)k_cache, (T*)v_cache, qkv, ld, slot_map, nq, nk, nv, q_w, k_w, eps, v_first,
-             mix, splits, plane, bias, extra_out, extra_at, extra_n);
+             mix, splits, plane, bias, extra_out, extra_at, extra_n, rot);
   return launch_status();
 }
 
-// nq, nk, nv: columns of q (all heads), k and v.  splits, plane, bias and the extra columns as in alofa_qkv_prepare.
+// nq, nk, nv: columns of q (all heads), k and v.  splits, plane, bias and the extra columns as in alofa_qkv_prepare.  d (the
+// head size), positions and freq are read only when rot_dims > 0.
 ALOFA_API int alofa_qkv_prepare_rows(void* q_out, void* k_cache, void* v_cache, const float* qkv, int ld, const int* slot_map, int n_tokens, int nq, int nk, int nv,
                                      const float* q_w, const float* k_w, float eps, float* v_first, const float* mix, int is_bf16, int splits, long long plane,
-                                     const float* bias, float* extra_out, int extra_at, int extra_n, cudaStream_t stream) {
+                                     const float* bias, float* extra_out, int extra_at, int extra_n, const int* positions, const float* freq, int d, int rot_dims,
+                                     int halves, float mag, cudaStream_t stream) {
   if (n_tokens <= 0) return ALOFA_OK;
+  if (rot_dims < 0 || (rot_dims & 1) || (rot_dims > 0 && (!positions || !freq || d < rot_dims || nq % d || nk % d))) return ALOFA_ERR_ARGUMENT;
+  const RowRotation rot{positions, freq, d, rot_dims, halves, mag};
   if (nq <= 0 || nk <= 0 || nv <= 0 || !q_w || !k_w || (mix && !v_first) || ld < nq + nk + nv || splits < 0 || (splits > 0 && plane < (long long)n_tokens * ld) ||
       (extra_out && (extra_n <= 0 || extra_at < 0 || extra_at + extra_n > ld)))
     return ALOFA_ERR_ARGUMENT;
@@ -724,7 +760,7 @@ ALOFA_API int alofa_qkv_prepare_rows(void* q_out, void* k_cache, void* v_cache, 
                     (uintptr_t)k_cache % 16 == 0 && (uintptr_t)v_cache % 16 == 0;
 #define ROWS_CASE(TT, VV) \
   return qkv_prepare_rows_launch<TT, VV>(q_out, k_cache, v_cache, qkv, ld, slot_map, n_tokens, nq, nk, nv, q_w, k_w, eps, v_first, mix, splits, plane, bias, extra_out, \
-                                         extra_at, extra_n, stream)
+                                         extra_at, extra_n, rot, stream)
   if (is_bf16) {
     if (four) ROWS_CASE(bf16, 4);
     ROWS_CASE(bf16, 1);

@@ -613,8 +613,8 @@ def _latent():
             "alofa_latent_prepare": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P],
             "alofa_latent_query_turn": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
             "alofa_rotary_interleaved": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-            "alofa_gemm_batched": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _L, _L, _L, _I, _I, _I, _I, _I, _P],
-            "alofa_gemm_batched_bf16": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _L, _L, _L, _I, _I, _I, _P],
+            "alofa_gemm_batched": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _L, _L, _L, _I, _I, _P, _L, _L, _I, _I, _I, _P],
+            "alofa_gemm_batched_bf16": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _L, _L, _L, _I, _I, _P, _L, _L, _I, _P],
             "alofa_activate": [_P, _P, _P, _L, _I, _I, _I, _P],
             "alofa_latent_attention": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
             "alofa_sandwich_norm": [_P, _P, _P, _F, _P, _P, _F, _I, _I, _I, _I, _L, _P, _P],
@@ -643,10 +643,11 @@ def latent_prepare(cq, cache_rows, lat, wq, wkv, freq, positions, slot_map, q_ra
     each token = [RMSNorm of the second part | the third part, its first
     ``rot_dims`` numbers turned by the token's position: neighbouring pairs, or
     with ``halves`` number i with number i + rot_dims / 2; cosine and sine
-    times ``mag``].  ``cache_rows`` None: no write."""
+    times ``mag``].  ``cache_rows`` None: no write, and the second and third parts (and
+    ``wkv``) need not be there."""
     f32 = torch.float32
     n = lat.shape[0]
-    if lat.shape[1] < q_rank + kv_rank + rot or (q_rank and tuple(cq.shape) != (n, q_rank)) or (cache_rows is not None and cache_rows.shape[1] != kv_rank + rot):
+    if lat.shape[1] < q_rank + (kv_rank + rot if cache_rows is not None else 0) or (q_rank and tuple(cq.shape) != (n, q_rank)) or (cache_rows is not None and cache_rows.shape[1] != kv_rank + rot):
         raise AlofaError("invalid_argument", "latent_prepare sizes disagree", f"lat={tuple(lat.shape)} q_rank={q_rank} kv_rank={kv_rank} rot={rot}")
     if q_rank == 0 and cache_rows is None:
         return
@@ -655,7 +656,7 @@ def latent_prepare(cq, cache_rows, lat, wq, wkv, freq, positions, slot_map, q_ra
         _latent().alofa_latent_prepare(
             _dev(cq, "cq") if q_rank else None, _dev(cache_rows, "cache", dt) if cache_rows is not None else None, _dev(lat, "lat", f32),
             _dev(wq, "wq", f32) if q_rank else None,
-            _dev(wkv, "wkv", f32), _dev(freq, "freq", f32) if rot_dims else None, _dev(positions, "positions", torch.int32),
+            _dev(wkv, "wkv", f32) if cache_rows is not None else None, _dev(freq, "freq", f32) if rot_dims else None, _dev(positions, "positions", torch.int32),
             _dev(slot_map, "slot_map", torch.int32) if cache_rows is not None else None, n, q_rank, kv_rank, rot, rot_dims, float(eps), lat.shape[1],
             1 if halves else 0, float(mag), 1 if dt == torch.bfloat16 else 0, _stream(),
         ),
@@ -695,17 +696,24 @@ def rotary_interleaved(x, freq, positions, heads: int, hd: int, rot_dims: int) -
 
 
 def gemm_batched(out, x, w, batches: int, m: int, n: int, k: int, ldx: int, x_batch: int, ldw: int, w_batch: int, ldo: int, out_batch: int,
-                 bias=None, bias_batch: int = 0, act: str = "none", tile_batch=None, tile_rows: int = 64) -> None:
+                 bias=None, bias_batch: int = 0, act: str = "none", tile_batch=None, tile_rows: int = 64, gate=None, gate_at: int = 0, gate_batch: int = 0) -> None:
     """``out_b[m, n] = act(x_b[m, :] . w_b[n, :] + bias_b[n])`` for every batch
     b, operands addressed by row and batch strides (in elements) from the
     tensors' first elements.  With ``tile_batch`` (int32, one entry per tile of
     ``tile_rows`` rows, a multiple of 64) there is one x and one out and tile i
-    uses the weight of batch ``tile_batch[i]``; negative entries are skipped.  bfloat16 operands whose
+    uses the weight of batch ``tile_batch[i]``; negative entries are skipped.  ``gate`` (fp32 [m, columns],
+    sums of a projection): out_b is multiplied by ``sigmoid(gate[m, gate_at + b * gate_batch + n])``.  bfloat16 operands whose
     depth and strides are multiples of 8 go to the tensor-core kernel, all
     others to the one that takes every size."""
     for t, name in ((out, "out"), (x, "x"), (w, "w")):
         if not t.is_cuda:
             raise AlofaError("unsupported", "kernels run on CUDA tensors only", f"{name} is on {t.device}")
+    gate_ptr, ldg = None, 0
+    if gate is not None:
+        ldg = gate.shape[1]
+        if gate.shape[0] < m or gate_at < 0 or gate_at + (batches - 1) * gate_batch + n > ldg:
+            raise AlofaError("invalid_argument", "gemm_batched: the gate lies outside its rows", f"gate={tuple(gate.shape)} at={gate_at} batches={batches} M={m} N={n}")
+        gate_ptr = _dev(gate, "gate", torch.float32) + 4 * gate_at
     bf = torch.bfloat16
     if (x.dtype == bf and w.dtype == bf and not (k % 8 or ldx % 8 or ldw % 8 or x_batch % 8 or w_batch % 8 or x.data_ptr() % 16 or w.data_ptr() % 16)
             and os.environ.get("ALOFA_BATCHED_TC", "1") != "0"):
@@ -713,7 +721,7 @@ def gemm_batched(out, x, w, batches: int, m: int, n: int, k: int, ldx: int, x_ba
             _latent().alofa_gemm_batched_bf16(
                 out.data_ptr(), x.data_ptr(), w.data_ptr(), _dev(bias, "bias", torch.float32) if bias is not None else None,
                 _dev(tile_batch, "tile_batch", torch.int32) if tile_batch is not None else None, batches, m, n, k, ldx, x_batch, ldw, w_batch, ldo, out_batch,
-                bias_batch, ACTIVATIONS[act], tile_rows, _is_bf16(out, "out"), _stream(),
+                bias_batch, ACTIVATIONS[act], tile_rows, gate_ptr, ldg, gate_batch, _is_bf16(out, "out"), _stream(),
             ),
             "gemm_batched_bf16", f"batches={batches} M={m} N={n} K={k}",
         )
@@ -722,7 +730,7 @@ def gemm_batched(out, x, w, batches: int, m: int, n: int, k: int, ldx: int, x_ba
         _latent().alofa_gemm_batched(
             out.data_ptr(), x.data_ptr(), w.data_ptr(), _dev(bias, "bias", torch.float32) if bias is not None else None,
             _dev(tile_batch, "tile_batch", torch.int32) if tile_batch is not None else None, batches, m, n, k, ldx, x_batch, ldw, w_batch, ldo, out_batch,
-            bias_batch, ACTIVATIONS[act], tile_rows, _is_bf16(x, "x"), _is_bf16(w, "w"), _is_bf16(out, "out"), _stream(),
+            bias_batch, ACTIVATIONS[act], tile_rows, gate_ptr, ldg, gate_batch, _is_bf16(x, "x"), _is_bf16(w, "w"), _is_bf16(out, "out"), _stream(),
         ),
         "gemm_batched", f"batches={batches} M={m} N={n} K={k}",
     )
@@ -968,7 +976,7 @@ def _recurrent():
             "alofa_gated_group_norm": [_P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _F, _I, _I, _P],
             "alofa_branch_norm_add": [_P, _P, _P, _P, _P, _I, _I, _F, _F, _P],
             "alofa_qkv_prepare": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _F, _I, _P, _I, _F, _I, _I, _I, _I, _L, _P, _P, _I, _I, _P],
-            "alofa_qkv_prepare_rows": [_P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _I, _L, _P, _P, _I, _I, _P],
+            "alofa_qkv_prepare_rows": [_P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _I, _L, _P, _P, _I, _I, _P, _P, _I, _I, _I, _F, _P],
             "alofa_heads_finish": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _I, _I, _P],
         }
         for name, args in sigs.items():
@@ -1163,13 +1171,16 @@ def _owed_or_finished(qkv, what: str):
     return sums[0], int(qkv.splits), sums.shape[1] * sums.shape[2], qkv.bias
 
 
-def qkv_prepare_rows(q_out, k_cache, v_cache, qkv, slot_map, q_weight, k_weight, eps: float, v_first=None, mix=None, extra_out=None, extra_at: int = 0) -> None:
+def qkv_prepare_rows(q_out, k_cache, v_cache, qkv, slot_map, q_weight, k_weight, eps: float, v_first=None, mix=None, extra_out=None, extra_at: int = 0,
+                     positions=None, freq=None, rot_dims: int = 0, halves: bool = False, magnitude: float = 1.0) -> None:
     """:func:`qkv_prepare` where q and k are each normed over all their heads at
     once: from rows of fp32 sums [q | k | v | more], ``q / sqrt(mean(q^2) + eps)
     * q_weight`` (fp32, one number per column) to ``q_out`` [T, nq], k likewise
     and v to the tokens' cache slots.  ``v_first`` (fp32 [T, nv]): without
     ``mix`` the values are also left there; with ``mix`` (one fp32 number on the
     device) they become ``(1 - mix) v + mix v_first`` before they are stored.
+    ``rot_dims`` > 0: the first so many numbers of every q and k head are then
+    turned by the token's position as :func:`latent_prepare` turns them.
     ``qkv`` may be the partial sums a product left owed, ``extra_out`` /
     ``extra_at`` are as in :func:`qkv_prepare`."""
     f32 = torch.float32
@@ -1177,6 +1188,8 @@ def qkv_prepare_rows(q_out, k_cache, v_cache, qkv, slot_map, q_weight, k_weight,
     n, nq = q_out.shape
     dt = q_out.dtype
     nk, nv = k_cache.shape[1] * k_cache.shape[2], v_cache.shape[1] * v_cache.shape[2]
+    if rot_dims and (rot_dims > k_cache.shape[2] or freq.shape[0] < rot_dims // 2 or positions.shape[0] != n):
+        raise AlofaError("invalid_argument", "qkv_prepare_rows: the rotation disagrees with the heads", f"rot_dims={rot_dims} d={k_cache.shape[2]} freq={tuple(freq.shape)}")
     if (qkv.shape[0] != n or qkv.shape[1] < nq + nk + nv or q_weight.shape[0] != nq or k_weight.shape[0] != nk or (v_first is not None and tuple(v_first.shape) != (n, nv))
             or (mix is not None and (v_first is None or mix.numel() != 1)) or (extra_out is not None and (extra_out.shape[0] != n or extra_at + extra_out.shape[1] > qkv.shape[1]))):
         raise AlofaError("invalid_argument", "qkv_prepare_rows sizes disagree", f"qkv={tuple(qkv.shape)} q={tuple(q_out.shape)} k={tuple(k_cache.shape)} v={tuple(v_cache.shape)}")
@@ -1185,7 +1198,9 @@ def qkv_prepare_rows(q_out, k_cache, v_cache, qkv, slot_map, q_weight, k_weight,
         _recurrent().alofa_qkv_prepare_rows(_dev(q_out, "q_out"), _dev(k_cache, "k_cache", dt), _dev(v_cache, "v_cache", dt), _dev(qkv, "qkv", f32), qkv.shape[1],
                                             _dev(slot_map, "slot_map", torch.int32), n, nq, nk, nv, _dev(q_weight, "q_weight", f32), _dev(k_weight, "k_weight", f32), float(eps),
                                             opt(v_first, "v_first"), opt(mix, "mix"), _is_bf16(q_out, "q_out"), splits, plane, opt(bias, "bias"),
-                                            opt(extra_out, "extra_out"), int(extra_at), extra_out.shape[1] if extra_out is not None else 0, _stream()),
+                                            opt(extra_out, "extra_out"), int(extra_at), extra_out.shape[1] if extra_out is not None else 0,
+                                            _dev(positions, "positions", torch.int32) if rot_dims else None, _dev(freq, "freq", f32) if rot_dims else None, k_cache.shape[2],
+                                            int(rot_dims), 1 if halves else 0, float(magnitude), _stream()),
         "qkv_prepare_rows", f"nq={nq} nk={nk} nv={nv}",
     )
 

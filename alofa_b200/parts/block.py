@@ -30,6 +30,8 @@ from ..errors import AlofaError
 from .base import Part, TensorSpec, as_float32_vector, build_part, register_part
 from .linear import STORE, Linear
 
+DEFER_ABOVE = 64  # tokens in a step above which a sublayer's last product leaves its split sums for the norm's kernel to add: with few the kernel that settles them first measured faster
+
 
 class PrenormResidual(Part):
     family = "block"
@@ -90,8 +92,8 @@ class SandwichResidual(Part):
     """Norms on both sides of each sublayer.  The sublayer's output goes to an
     fp32 buffer of its own (parts that say ``stores_output`` write it, any
     other part adds into a zeroed one); one kernel then normalises it, adds it
-    to the stream and, for the mixer, also yields the normed input of the
-    feed-forward."""
+    to the stream and also yields the normed rows of what comes next: the
+    feed-forward, or the next such block's mixer."""
 
     family = "block"
 
@@ -126,29 +128,55 @@ class SandwichResidual(Part):
         return self.mixer.cache_spec()
 
     def scratch_row_bytes(self) -> int:
-        return 12 * self.mixer_norm.size + sum(getattr(part, "scratch_row_bytes", lambda: 0)() for part in self.parts())
+        return 16 * self.mixer_norm.size + sum(getattr(part, "scratch_row_bytes", lambda: 0)() for part in self.parts())
+
+    @property
+    def first_norm(self):
+        """The norm this block starts with: the block before may make its rows (``ctx.next_norm``, ``ctx.stream_rows``)."""
+        return self.mixer_norm
 
     def _sublayer(self, ctx, part, x, h, *args):
-        """The part's output for the rows ``x``, fp32, in a buffer of its own."""
+        """The part's output for the rows ``x``: an fp32 buffer of its own, or the split sums its last product left for the norm's kernel to add."""
         y = ctx.buf(tuple(h.shape), h.dtype)
-        if getattr(part, "stores_output", False):
-            part.forward(ctx, x, y, *args, store=True)
-        else:
+        if not getattr(part, "stores_output", False):
             y.zero_()
             part.forward(ctx, x, y, *args)
             ctx.flush_pending()
+        elif getattr(part, "defers_output", False) and x.shape[0] > DEFER_ABOVE:
+            owed = part.forward(ctx, x, y, *args, store=True, defer=True)
+            return y if owed is None else owed
+        else:
+            part.forward(ctx, x, y, *args, store=True)
         return y
 
+    def _rows(self, ctx, h):
+        """The normed rows of ``h`` that the mixer reads: those the block before left, else made now."""
+        left, ctx.stream_rows = ctx.stream_rows, None
+        if left is not None and left[0] is h and left[2] is self.mixer_norm:
+            return left[1]
+        return self.mixer_norm.forward(ctx, h)
+
+    def _close(self, ctx, h, y, post):
+        """The layer's last norm, which adds to the stream and also leaves the rows the next block starts from (a scratch buffer of a
+        layer lives until the layer after next begins)."""
+        nxt = ctx.next_norm
+        if nxt is None:
+            ops.sandwich_norm(h, y, post.weight, post.eps)
+            return
+        x = ctx.buf(tuple(h.shape), self.rt.dtype)
+        ops.sandwich_norm(h, y, post.weight, post.eps, x, nxt.weight, nxt.eps)
+        ctx.stream_rows = (h, x, nxt)
+
     def forward(self, ctx, h, cache, writes=True):
-        x = self.mixer_norm.forward(ctx, h)
+        x = self._rows(ctx, h)
         y = self._sublayer(ctx, self.mixer, x, h, cache, writes)
         if self.feed_forward is None:
-            ops.sandwich_norm(h, y, self.mixer_post.weight, self.mixer_post.eps)
+            self._close(ctx, h, y, self.mixer_post)
             return
         x = ctx.buf(tuple(h.shape), self.rt.dtype)
         ops.sandwich_norm(h, y, self.mixer_post.weight, self.mixer_post.eps, x, self.feed_forward_norm.weight, self.feed_forward_norm.eps)
         y = self._sublayer(ctx, self.feed_forward, x, h)
-        ops.sandwich_norm(h, y, self.feed_forward_post.weight, self.feed_forward_post.eps)
+        self._close(ctx, h, y, self.feed_forward_post)
 
 
 class PostnormResidual(Part):
@@ -198,7 +226,7 @@ class PostnormResidual(Part):
     def _output(ctx, part, h, x, *args):
         """The sublayer's output for the rows ``x``: an fp32 buffer, or the split sums its last product left for the norm's kernel to add."""
         y = ctx.buf(tuple(h.shape), torch.float32)
-        if getattr(part, "defers_output", False) and x.shape[0] > 64:  # in steps of a few tokens the kernel that settles the sums first measured faster
+        if getattr(part, "defers_output", False) and x.shape[0] > DEFER_ABOVE:
             owed = part.forward(ctx, x, y, *args, store=True, defer=True)
             return y if owed is None else owed
         part.forward(ctx, x, y, *args, store=True)

@@ -19,8 +19,13 @@ The stacked ``[Wdq; Wdkv]`` makes both down-projections one product.
 Options: ``q_rank`` 0 or absent: no query latent, ``q = x Wq^T`` (tensor
 ``q``) and the down-projection is ``Wdkv`` alone; ``gate``: head h's output is
 multiplied by ``sigmoid(x Wg^T)_h`` (tensor ``g`` [heads, hidden], stacked
-under the down-projection); the position part may pair halves and carry a
-magnitude (:class:`~alofa_b200.parts.position.RotaryInterleaved`)."""
+under the down-projection), or ("channel") every channel of it by a gate of its
+own (``g`` [heads * vdim, hidden]; taken in the epilogue of the per-head value
+product); ``position`` absent: no rotated part; it may pair halves and carry a
+magnitude (:class:`~alofa_b200.parts.position.RotaryInterleaved`);
+``own_latent`` False: the layer has no ``Wdkv`` and attends, with its own
+``Wuk`` and ``Wuv``, to the rows that another layer keeps (its run names that
+layer's cache)."""
 from __future__ import annotations
 
 import torch
@@ -36,9 +41,11 @@ class LatentAttention(Part):
     family = "mixer"
     stores_output = True  # forward(..., store=True) writes its output instead of adding it
 
+    defers_output = True  # forward(..., store=True, defer=True) may hand back the output product's split sums instead of the finished output
+
     @property
     def graph_safe(self):
-        return self.position.graph_safe
+        return self.position is None or self.position.graph_safe
 
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
@@ -50,77 +57,93 @@ class LatentAttention(Part):
         self.vdim = int(p("vdim"))
         self.kv_rank = int(p("kv_rank"))
         self.q_rank = int(self.params.get("q_rank") or 0)  # 0: queries come straight from x
-        self.gate = bool(self.params.get("gate", False))
+        gate = self.params.get("gate", False)
+        if gate not in (False, True, None, "channel"):
+            raise AlofaError("unsupported", "a latent attention's gate is one per head or one per channel", f"gate={gate}")
+        self.gate_channels = gate == "channel"
+        self.gate_cols = self.heads * self.vdim if self.gate_channels else self.heads if gate else 0  # columns of the gate's projection
+        self.own_latent = bool(self.params.get("own_latent", True))
         self.scale = float(p("scale"))
         self.eps = float(p("eps"))
         self.has_sink = bool(p("sink", False))
         self.window = self.params.get("window")
         if self.dim + self.rot <= 0 or self.kv_rank > 1024:
             raise AlofaError("unsupported", "latent attention wants a head of at least one dimension and a latent of at most 1024", f"dim={self.dim} rot={self.rot} kv_rank={self.kv_rank}")
-        self.position = build_part("position", p("position"), rt)
+        position = self.params.get("position")
+        self.position = build_part("position", position, rt) if position is not None else None
         self.rot_dims = int(getattr(self.position, "dims", 0))
         self.halves = bool(getattr(self.position, "halves", False))
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
+        if self.position is None and self.rot:
+            raise AlofaError("invalid_argument", "a rotated part needs a position encoding", f"rot_dim={self.rot}")
         if self.rot_dims > self.rot:
             raise AlofaError("invalid_argument", "more rotated dimensions than the rotated part has", f"dims={self.rot_dims} rot_dim={self.rot}")
         self.width = self.kv_rank + self.rot  # a cache row
-        self.down = self.up_q = self.out = self.uk_t = self.uv = self.sink = None
+        # columns of the stacked down-projection: [query latent | latent and rotated part | gate]
+        self.gate_at = self.q_rank + (self.width if self.own_latent else 0)
+        self.down = self.up_q = self.out = self.uk_t = self.uv = self.sink = self.kv_norm = None
 
     def cache_spec(self):
         return PagedRows(self.width, self.window)
 
     def scratch_row_bytes(self) -> int:
         h = self.heads
-        return 4 * (self.q_rank + self.width + h) + 4 * self.q_rank + 4 * h * (self.dim + self.rot) + 4 * h * self.width + 4 * h * self.kv_rank + 4 * h * self.vdim + 4 * self.hidden
+        return 4 * (self.q_rank + self.width + self.gate_cols) + 4 * self.q_rank + 4 * h * (self.dim + self.rot) + 4 * h * self.width + 4 * h * self.kv_rank + 4 * h * self.vdim + 4 * self.hidden
 
     def tensors(self):
         pre, h = self.prefix, self.heads
         t = {
-            pre + "dkv": TensorSpec((self.width, self.hidden)),
-            pre + "dkv.norm": TensorSpec((self.kv_rank,), "ones"),
             pre + "uk": TensorSpec((h * self.dim, self.kv_rank)),
             pre + "uv": TensorSpec((h * self.vdim, self.kv_rank)),
             pre + "o": TensorSpec((self.hidden, h * self.vdim)),
         }
+        if self.own_latent:
+            t.update({pre + "dkv": TensorSpec((self.width, self.hidden)), pre + "dkv.norm": TensorSpec((self.kv_rank,), "ones")})
         if self.q_rank:
             t.update({pre + "dq": TensorSpec((self.q_rank, self.hidden)), pre + "dq.norm": TensorSpec((self.q_rank,), "ones"),
                       pre + "uq": TensorSpec((h * (self.dim + self.rot), self.q_rank))})
         else:
             t[pre + "q"] = TensorSpec((h * (self.dim + self.rot), self.hidden))
-        if self.gate:
-            t[pre + "g"] = TensorSpec((h, self.hidden))
+        if self.gate_cols:
+            t[pre + "g"] = TensorSpec((self.gate_cols, self.hidden))
         if self.has_sink:
             t[pre + "sink"] = TensorSpec((h,))
-        t.update(self.position.tensors())
+        if self.position is not None:
+            t.update(self.position.tensors())
         return t
 
     def load(self, state):
         pre, h = self.prefix, self.heads
         # one product for everything that leaves fp32 sums: [Wdq; Wdkv; Wg]
-        stacked = ([state[pre + "dq"]] if self.q_rank else []) + [state[pre + "dkv"]] + ([state[pre + "g"]] if self.gate else [])
-        self.down = Linear(torch.cat(stacked, dim=0), None, STORE)
+        stacked = [state[pre + n] for n, there in (("dq", self.q_rank), ("dkv", self.own_latent), ("g", self.gate_cols)) if there]
+        self.down = Linear(torch.cat(stacked, dim=0), None, STORE) if stacked else None
         self.q_norm = as_float32_vector(state[pre + "dq.norm"]) if self.q_rank else None
-        self.kv_norm = as_float32_vector(state[pre + "dkv.norm"])
+        self.kv_norm = as_float32_vector(state[pre + "dkv.norm"]) if self.own_latent else None
         self.up_q = Linear(state[pre + "uq"] if self.q_rank else state[pre + "q"], None, STORE)
         # [heads, kv_rank, dim]: row c of head h holds column c of Wuk_h, so the per-head product q_h -> Wuk_h^T q_h reads rows
         self.uk_t = state[pre + "uk"].view(h, self.dim, self.kv_rank).transpose(1, 2).contiguous() if self.dim else None
         self.uv = state[pre + "uv"].contiguous()
         self.out = Linear(state[pre + "o"], None, STORE)
         self.sink = as_float32_vector(state[pre + "sink"]) if self.has_sink else None
-        self.position.load(state)
+        if self.position is not None:
+            self.position.load(state)
 
-    def forward(self, ctx, x, h, cache, writes=True, store=False):
+    def forward(self, ctx, x, h, cache, writes=True, store=False, defer=False):
         """``h`` += (or, with ``store``, =) the mixer's output for the rows ``x``;
         ``h`` is fp32 [tokens, hidden]."""
+        if writes and not self.own_latent:
+            raise AlofaError("state", "a latent attention without a latent of its own runs on another layer's cache", f"prefix={self.prefix}")
         n, dt, heads = x.shape[0], self.rt.dtype, self.heads
         group = ctx.groups[cache.group]
-        freq = self.position.frequencies()
-        gate_at = self.q_rank + self.width
-        lat = ctx.buf((n, gate_at + (heads if self.gate else 0)), torch.float32)
-        self.down(lat, x, buf=ctx.buf)
+        freq = self.position.frequencies() if self.rot_dims else None
+        lat = None
+        if self.down is not None:
+            lat = ctx.buf((n, self.gate_at + self.gate_cols), torch.float32)
+            self.down(lat, x, buf=ctx.buf)
         cq = ctx.buf((n, self.q_rank), dt) if self.q_rank else None
-        ops.latent_prepare(cq, cache.k if writes else None, lat, self.q_norm, self.kv_norm, freq, ctx.positions, group.slot_map,
-                           self.q_rank, self.kv_rank, self.rot, self.rot_dims, self.eps, self.halves, self.magnitude)
+        if lat is not None:
+            ops.latent_prepare(cq, cache.k if writes else None, lat, self.q_norm, self.kv_norm, freq, ctx.positions, group.slot_map,
+                               self.q_rank, self.kv_rank, self.rot, self.rot_dims, self.eps, self.halves, self.magnitude)
         q = ctx.buf((n, heads * (self.dim + self.rot)), dt)
         self.up_q(q, cq if self.q_rank else x, buf=ctx.buf)
         qa = ctx.buf((n, heads * self.width), dt)
@@ -134,13 +157,13 @@ class LatentAttention(Part):
         o_lat = ctx.buf((n, heads * self.kv_rank), dt)
         self.attend(ctx, o_lat, qa, cache, group)
         o = ctx.buf((n, heads * self.vdim), dt)
-        # per head: o[:, h] = o_lat[:, h] Wuv_h^T
+        # per head: o[:, h] = o_lat[:, h] Wuv_h^T (times the channels' gates)
         ops.gemm_batched(o, o_lat, self.uv, heads, n, self.vdim, self.kv_rank, heads * self.kv_rank, self.kv_rank, self.kv_rank, self.vdim * self.kv_rank,
-                         heads * self.vdim, self.vdim)
-        if self.gate:
-            ops.head_gate(o, lat, gate_at, heads, self.vdim)
+                         heads * self.vdim, self.vdim, gate=lat if self.gate_channels else None, gate_at=self.gate_at, gate_batch=self.vdim)
+        if self.gate_cols and not self.gate_channels:
+            ops.head_gate(o, lat, self.gate_at, heads, self.vdim)
         if store:
-            self.out(h, o, buf=ctx.buf)
+            return self.out(h, o, defer=defer, buf=ctx.buf)  # None, or the split sums a caller that asked for them adds up itself
         else:
             y = ctx.buf(tuple(h.shape), torch.float32)
             self.out(y, o, buf=ctx.buf)

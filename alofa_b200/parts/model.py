@@ -25,6 +25,9 @@ class Model:
         self.final_norm = build_part("norm", spec.final_norm, rt)
         self.head = build_part("head", spec.head, rt)
         self.run = [(e.layer, i if e.cache is None else e.cache) for i, e in enumerate(spec.run)]
+        # per run entry: the norm that what follows starts with, where a block before it may make those rows (the final norm only when every row is wanted)
+        norms = [getattr(self.layers[layer], "first_norm", None) for layer, _ in self.run[1:]] + [self.final_norm]
+        self.next_norms = [n if n is not None and n.spec.kind == "rmsnorm" else None for n in norms]
         # a block may read the embedding output of the step's tokens later on (ctx.embedding_output)
         self.keeps_embedding = any(getattr(block, "needs_embedding_output", False) for block in self.layers)
         # blocks that keep several copies of the residual stream say how many (ctx.streams); every block of a model says the same
@@ -81,11 +84,15 @@ class Model:
             ctx.first_values = ctx.buf((ctx.n_tokens, self.shared_value_width), torch.float32)
         if self.stream_copies:
             ctx.open_streams(h, self.stream_copies)
+        # every row wanted, in order (a decode step): no picking, and the last block or a norm that reads the stream as base + accumulator may make them
+        all_rows = ctx.n_out == ctx.n_tokens and bool((ctx.host_field("logit_rows") == np.arange(ctx.n_tokens, dtype=np.int32)).all())
+        last = len(self.run) - 1
         for i, (layer, cache) in enumerate(self.run):
             block = self.layers[layer]
             if not getattr(block, "absorbs_pending", False):
                 ctx.flush_pending()
             ctx.begin_layer()
+            ctx.next_norm = self.next_norms[i] if i < last or all_rows else None
             block.forward(ctx, h, caches.get(cache), writes=(cache == i))
         ctx.end_layers()
         if self.stream_copies:
@@ -95,11 +102,11 @@ class Model:
             return None
         if not getattr(self.final_norm, "absorbs_pending", False):
             ctx.flush_pending()
-        # every row wanted, in order (a decode step): no picking, and a norm that reads the stream as base + accumulator may
-        rows = ctx.logit_rows
-        if ctx.n_out == ctx.n_tokens and bool((ctx.host_field("logit_rows") == np.arange(ctx.n_tokens, dtype=np.int32)).all()):
-            rows = None
-        x = self.final_norm.forward(ctx, h, rows)
+        left, ctx.stream_rows = ctx.stream_rows, None
+        if all_rows and left is not None and left[0] is h and left[2] is self.final_norm:
+            x = left[1]
+        else:
+            x = self.final_norm.forward(ctx, h, None if all_rows else ctx.logit_rows)
         ctx.close_stream()
         return self.head.forward(ctx, x)
 

@@ -1,6 +1,7 @@
 """RMSNorm: ``y = x / sqrt(mean(x^2) + eps) * w`` per row, fp32 sums; no bias,
 no mean subtraction, the weight is used as stored
-(src/alofa/kernels/cpu/scalar.mojo:93-129).  Layer norm: ``y = (x - mean) /
+(src/alofa/kernels/cpu/scalar.mojo:93-129), or (``weight_offset``) that number
+more than stored, added in fp32.  Layer norm: ``y = (x - mean) /
 sqrt(variance + eps) * w + b``, the variance being the mean of the squared
 deviations, ``b`` the tensor of the weight's name with ``.b`` added."""
 from __future__ import annotations
@@ -21,14 +22,17 @@ class RMSNorm(Part):
         self.size = int(self.param("size"))
         self.eps = float(self.param("eps"))
         self.name = self.prefix + str(self.params.get("weight_name", "weight"))  # the tensor's name: prefix + "weight" unless the spec says otherwise
+        self.offset = float(self.params.get("weight_offset") or 0.0)
         self.weight = None
         self.shift = None  # a layer norm's bias
 
     def tensors(self):
-        return {self.name: TensorSpec((self.size,), "ones")}
+        return {self.name: TensorSpec((self.size,), "normal" if self.offset else "ones")}
 
     def load(self, state):
         self.weight = as_float32_vector(state[self.name])
+        if self.offset:
+            self.weight = self.weight + self.offset
 
     absorbs_pending = True  # adds split-K partial sums owed to h while reading it
     gives_normed_rows = True  # forward(lazy=True) may hand its reader rows still to be made

@@ -1,5 +1,5 @@
-"""Softmax attention without rotation over a paged key/value cache, with the
-options of designs that take positions in by other means:
+"""Softmax attention over a paged key/value cache with the options of designs
+that norm their queries and keys or take positions in by other means:
 
 * ``qk_norm``: q and k are divided by their root mean square over the head's
   channels (eps inside the root); with ``norm_weight`` then multiplied by a
@@ -12,8 +12,9 @@ options of designs that take positions in by other means:
 * ``scale``: scores are ``(q . k) * scale``;
 * ``softcap``: then ``softcap * tanh(score / softcap)``;
 * ``bias``: q, k and v have biases (``<tensor>.b``), added in the projection;
-* ``position``: a position part whose rotation (neighbouring pairs, angles in
-  fp32 in the kernel) turns the first dimensions of every q and k head;
+* ``position``: a position part whose rotation (neighbouring pairs, or with
+  ``norm_over`` "projection" also pairs of halves; angles in fp32 in the
+  kernel) turns the first dimensions of every q and k head, after the norm;
 * ``sink``: the softmax's denominator holds one more term ``exp(sink)`` that
   belongs to no key and has no value (0.0: "one added to the denominator";
   "learned": a number per head, tensor ``sink``);
@@ -97,7 +98,7 @@ class NormedAttention(PagedAttend, Part):
         self.position = build_part("position", self.params["position"], rt) if self.params.get("position") is not None else None
         self.rot_dims = int(getattr(self.position, "dims", 0)) if self.position is not None else 0
         if self.position is not None and (not hasattr(self.position, "frequencies") or self.rot_dims > self.dim):
-            raise AlofaError("unsupported", "this attention rotates neighbouring pairs only, at most the head's dimensions", f"position={self.params['position']}")
+            raise AlofaError("unsupported", "this attention rotates pairs by frequencies, at most the head's dimensions", f"position={self.params['position']}")
         if min(self.heads, self.kv_heads, self.dim, self.vdim) <= 0 or self.heads % self.kv_heads:
             raise AlofaError("invalid_argument", "kv heads must divide heads, sizes must be positive", f"params={self.params}")
         if self.vdim > 256:
@@ -108,8 +109,10 @@ class NormedAttention(PagedAttend, Part):
             raise AlofaError("invalid_argument", "keys that are also the values have the values' size", f"dim={self.dim} vdim={self.vdim}")
         if self.chunk < 0 or (self.chunk and self.window):
             raise AlofaError("invalid_argument", "a chunked mask takes a positive size and no window beside it", f"chunk={self.chunk} window={self.window}")
-        if self.norm_rows and (not self.norm_weight or self.maps > 1 or self.values_from_keys or self.position is not None or self.coef):
-            raise AlofaError("unsupported", "norms over the whole projection have weights, one map a head, values of their own and no rotation or temperature", f"params={self.params}")
+        if self.norm_rows and (not self.norm_weight or self.maps > 1 or self.values_from_keys or self.coef):
+            raise AlofaError("unsupported", "norms over the whole projection have weights, one map a head, values of their own and no temperature", f"params={self.params}")
+        if self.position is not None and getattr(self.position, "halves", False) and not self.norm_rows:
+            raise AlofaError("unsupported", "pairs of halves are turned by the kernel that norms whole projections", f"position={self.params['position']}")
         if self.value_mix not in (None, "first", "later") or (self.value_mix and not self.norm_rows):
             raise AlofaError("unsupported", "values are mixed by the kernel that norms whole projections", f"params={self.params}")
         if self.keep_first < 0 or (self.distance_bias and self.maps > 1):
@@ -201,17 +204,20 @@ class NormedAttention(PagedAttend, Part):
         owed = self.qkv(sums, x, defer=n > DEFER_ABOVE, buf=ctx.buf)
         q = ctx.buf((n, self.q_dim), dt)
         rotated = self.rot_dims > 0
+        magnitude = float(getattr(self.position, "magnitude", 1.0)) if rotated else 1.0
         g_off = self.q_dim + self.k_dim + self.v_dim  # the gates' column in the stacked projection's sums
         gates, gates_at = (sums, g_off) if self.gate else (None, 0)
         if owed is not None and self.gate:
             gates, gates_at = ctx.buf((n, self.heads), torch.float32), 0  # the gates' logits, finished, for the kernel after the attention
         if self.norm_rows:
             ops.qkv_prepare_rows(q, cache.k, cache.v, sums if owed is None else owed, group.slot_map, self.q_weight, self.k_weight, self.eps,
-                                 ctx.first_values if self.value_mix else None, self.mix, gates if owed is not None and self.gate else None, g_off)
+                                 ctx.first_values if self.value_mix else None, self.mix, gates if owed is not None and self.gate else None, g_off,
+                                 ctx.positions if rotated else None, self.position.frequencies() if rotated else None, self.rot_dims,
+                                 bool(getattr(self.position, "halves", False)), magnitude)
         else:
             ops.qkv_prepare(q, cache.k, cache.v, sums if owed is None else owed, ctx.positions, group.slot_map, self.heads, self.kv_heads, self.dim, self.vdim, self.qk_norm,
                             self.eps, self.coef, self.every, self.position.frequencies() if rotated else None, self.rot_dims, self.maps, self.q_weight, self.k_weight,
-                            float(getattr(self.position, "magnitude", 1.0)) if rotated else 1.0, self.values_from_keys, self.v_copies,
+                            magnitude, self.values_from_keys, self.v_copies,
                             gates if owed is not None and self.gate else None, g_off)
         if self.tensor_cores:
             # the tensor-core kernels, which multiply a head's gate in where they complete its rows

@@ -66,8 +66,12 @@ class RotaryInterleaved(Part):
 
     ``layout`` "halves" pairs dimension i with i + dims / 2 instead (kernels
     that take a ``halves`` flag; :meth:`apply` does neighbouring pairs only).
-    ``scaling`` = ``{factor, original, fast, slow}`` stretches the slow
-    frequencies (YaRN): with ``turns(t) = dims * ln(original / (2 pi t)) / (2 ln
+    ``scaling`` stretches the slow frequencies.  ``{kind: "wavelength", factor,
+    original, low, high}`` (as in Llama 3.1) goes by the wavelength ``l_i = 2 pi
+    / f_i``: ``f_i`` where ``l_i < original / high``, ``f_i / factor`` where
+    ``l_i > original / low``, and between the two ``(1 - s) f_i / factor + s
+    f_i`` with ``s = (original / l_i - low) / (high - low)``.  ``{factor,
+    original, fast, slow}`` (YaRN): with ``turns(t) = dims * ln(original / (2 pi t)) / (2 ln
     base)``, ``lo = max(floor(turns(fast)), 0)``, ``hi = min(ceil(turns(slow)),
     dims - 1)`` and ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` the
     frequency is ``f_i / factor * ramp_i + f_i * (1 - ramp_i)``, and cosine and
@@ -86,11 +90,15 @@ class RotaryInterleaved(Part):
             raise AlofaError("unsupported", "rotary dims must be even, the base positive, the layout 'pairs' or 'halves'", f"dims={self.dims} base={self.base} layout={self.layout}")
         self.magnitude = 1.0
         if self.scaling:
-            sc = {k: float(self.scaling[k]) for k in ("factor", "original", "fast", "slow")}
+            self.by_wavelength = str(self.scaling.get("kind", "turns")) == "wavelength"
+            sc = {k: float(self.scaling[k]) for k in (("factor", "original", "low", "high") if self.by_wavelength else ("factor", "original", "fast", "slow"))}
             if min(sc.values()) <= 0 or self.base == 1.0:
                 raise AlofaError("invalid_argument", "rotary scaling wants positive numbers and a base other than 1", f"scaling={self.scaling}")
             self.scaling = sc
-            self.magnitude = 0.1 * math.log(sc["factor"]) + 1.0
+            if self.by_wavelength and sc["high"] < sc["low"]:
+                raise AlofaError("invalid_argument", "rotary scaling by wavelength wants high not below low", f"scaling={self.scaling}")
+            if not self.by_wavelength:
+                self.magnitude = 0.1 * math.log(sc["factor"]) + 1.0
         self._freq = None
 
     @property
@@ -104,7 +112,14 @@ class RotaryInterleaved(Part):
         """f_i, i < dims / 2, in float64 (rounded to fp32 once, by the caller)."""
         i = np.arange(max(self.dims // 2, 1), dtype=np.float64)
         freq = np.power(np.float64(self.base), -2.0 * i / max(self.dims, 1))
-        if self.scaling:
+        if self.scaling and self.by_wavelength:
+            sc = self.scaling
+            wave = 2.0 * math.pi / freq
+            span = sc["high"] - sc["low"]
+            s = (sc["original"] / wave - sc["low"]) / span if span > 0 else np.zeros_like(wave)
+            between = (1.0 - s) * freq / sc["factor"] + s * freq
+            freq = np.where(wave < sc["original"] / sc["high"], freq, np.where(wave > sc["original"] / sc["low"], freq / sc["factor"], between))
+        elif self.scaling:
             sc = self.scaling
 
             def turns(t):
