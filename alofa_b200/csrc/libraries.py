@@ -19,6 +19,8 @@ def all_libraries() -> list:
         # latent attention on tensor cores is built per latent size at first use; the size of the tests' model is built ahead
         {"name": "alofa_latent_attention_kv64_r32", "sources": ["kernels/latent_attention_bf16.cu"], "defines": {"KV_RANK": 64, "ROT": 32}},
         {"name": "alofa_latent_attention_kv96_r16", "sources": ["kernels/latent_attention_bf16.cu"], "defines": {"KV_RANK": 96, "ROT": 16}},
+        *[{"name": f"alofa_latent_attention_kv{kv}_r0", "sources": ["kernels/latent_attention_bf16.cu"], "defines": {"KV_RANK": kv, "ROT": 0}} for kv in (32, 64, 128, 512)],
+        *[{"name": f"alofa_attention_hd{hd}_v{vd}", "sources": ["kernels/attention_bf16.cu"], "defines": {"HEAD_DIM": hd, "V_DIM": vd}} for hd, vd in ((64, 128), (128, 64), (32, 48), (32, 64))],
         *[{"name": f"alofa_attention_hd{hd}", "sources": ["kernels/attention_bf16.cu"], "defines": {"HEAD_DIM": hd}} for hd in (16, 32, 48, 64, 80, 96, 128)],
         # the build that takes a distance bias off its scores, per sizes of key and value heads at first use; the tests' sizes ahead
         *[{"name": f"alofa_attention_hd{hd}" + (f"_v{vd}" if vd != hd else "") + "_dist", "sources": ["kernels/attention_bf16.cu"],

@@ -127,7 +127,7 @@ class NormedAttention(PagedAttend, Part):
         # the bfloat16 tensor-core kernels take keys and values of one size and as many value heads as key heads: with several maps a
         # head the values are then kept once per map (the every-size kernel reads one value head for all of a key head's maps)
         self.tensor_cores = (rt.dtype == torch.bfloat16 and (self.dim == self.vdim or self.maps == 1) and ops.attention_bf16_supported(self.dim, self.vdim)
-                             and (self.scale > 0 or not self.distance_bias))  # there the bias is taken off in units of the scale
+                             and self.scale > 0)  # there a row's maximum is scaled once, and a bias is taken off in units of the scale
         self.v_copies = self.maps if self.tensor_cores else 1
         self.nh, self.nkv, self.hd, self.vd = self.heads * self.maps, self.kv_heads * self.maps, self.dim, self.vdim  # what the shared choice of kernels goes by
         self.shared_value_width = self.v_dim if self.value_mix else 0

@@ -6,6 +6,7 @@
     python bench.py --design darolix [--size 1k|2k]     (another line: that design beside Kotutar at equal layer sizes)
     python bench.py --design dibulix [--size 1k|2k]     (another line: that design beside Darolix at equal layer sizes)
     python bench.py --design kikerax [--size 1k|2k]     (another line: that design beside Darolix at equal layer sizes)
+    python bench.py --design nugopel [--size 1k|2k]     (another line: that design beside Kotutar and Pekerax at equal layer sizes)
 
 The default run has the layer sizes of the Qwen2.5-0.5B shape with random
 weights, a batch of 8 requests with 2,048-token prompts inside a 4,096-token
@@ -649,6 +650,47 @@ def pekerax_numbers(z: dict, b: dict) -> dict:
             "head_flops": 2.0 * w * z["vocab"], "state_bytes_per_request": 2 * state_bytes + window_bytes}
 
 
+# --design nugopel: latent attention without positions and windowed attention with one added to the softmax's denominator in turn, a
+# mixture of experts with a shared one in every layer, beside the Kotutar design (latent attention, norms on both sides, routed experts
+# with a shared one) and, for norms over whole projections and windowed attention, the Pekerax design, at the same width, layers, heads,
+# experts and vocabulary.  The latent's sizes are Kotutar's without the rotated part, the other attention's Pekerax's; the second
+# latent attention reads the first one's latent.
+NUGOPEL_SIZES = {
+    "1k": dict(kv_heads=2, att_dim=128, att_vdim=128, window=1024, rot_dims=64),
+    "2k": dict(kv_heads=4, att_dim=128, att_vdim=128, window=1024, rot_dims=64),
+}
+
+
+def nugopel_config(z: dict, b: dict):
+    """Latent attention with a latent of its own, attention, latent attention on the first one's latent, attention, in turn."""
+    from alofa_b200.models.nugopel import AttentionConfig, ExpertsConfig, LatentConfig, NugopelConfig, NugopelLayer
+
+    attention = AttentionConfig(z["heads"], b["kv_heads"], b["att_dim"], b["att_vdim"], b["att_dim"] ** -0.5, 5e5, b["rot_dims"], {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192.0},
+                                b["window"])
+    experts = ExpertsConfig(z["experts"], z["top"], z["expert_ff"], z["shared_ff"])
+    latent = lambda source: LatentConfig(z["heads"], z["dim"], z["vdim"], z["kv_rank"], z["dim"] ** -0.5, source)
+    kinds = lambda i: (("latent_attention", latent(None)), ("attention", attention), ("latent_attention", latent(i - 2)), ("attention", attention))[i % 4]
+    return NugopelConfig(z["vocab"], z["width"], 1e-6, [NugopelLayer(*kinds(i), experts) for i in range(z["layers"])])
+
+
+def nugopel_numbers(z: dict, b: dict) -> dict:
+    """Bytes a decode step reads and flops a token costs for the Nugopel sizes (bf16).  The bench's prompts are longer than the
+    window, so a decode step reads the window's rows per request whatever the context (counted as state), and every latent
+    attention reads the whole latent."""
+    w, h, g, r = z["width"], z["heads"], b["kv_heads"], z["kv_rank"]
+    latent = w * h * (z["dim"] + z["vdim"]) + h * (z["dim"] + z["vdim"]) * r + h * z["vdim"] * w
+    att = w * ((h + g) * b["att_dim"] + g * b["att_vdim"]) + h * b["att_vdim"] * w
+    n_lat, n_own, n_att = (sum(i % 4 in kinds for i in range(z["layers"])) for kinds in ((0, 2), (0,), (1, 3)))
+    mixers = n_lat * latent + n_own * w * r + n_att * att
+    expert, around = 2 * w * z["expert_ff"], 2 * w * z["shared_ff"] + z["experts"] * w
+    whole, inside = PROMPT_LEN * (PROMPT_LEN + 1) / 2, min(b["window"], PROMPT_LEN)
+    seen = (inside * (inside + 1) / 2 + (PROMPT_LEN - inside) * inside) / whole  # the part of a prompt's (query, key) pairs that the window leaves
+    return {"weight_bytes": 2 * (mixers + z["layers"] * (z["experts"] * expert + around) + z["vocab"] * w), "kv_bytes_per_token": n_lat * r * 2,
+            "flops_per_token": 2.0 * (mixers + z["layers"] * (z["top"] * expert + around)),
+            "attn_flops_per_pair": n_lat * 4.0 * h * r + seen * n_att * 2.0 * h * (b["att_dim"] + b["att_vdim"]),
+            "head_flops": 2.0 * w * z["vocab"], "state_bytes_per_request": 2 * b["window"] * n_att * g * (b["att_dim"] + b["att_vdim"])}
+
+
 class KernelClock:
     """Times every kernel call of the package's ops module with its own pair of CUDA events during one
     step (run outright, no graph), and sets each beside the time its own operands allow: the larger of
@@ -755,17 +797,23 @@ class KernelClock:
             caches = [a for a in args[2:4] if isinstance(a, torch.Tensor) and a.dim() >= 2 and a.dtype == q.dtype]
             row_bytes = sum(c[0].numel() * c.element_size() for c in caches)
             byts = out.numel() * out.element_size() + q.numel() * q.element_size() + kv_rows * row_bytes
-            flops = 2.0 * self.pairs * (q.shape[1] + out.shape[1])  # per (query token, key) pair: heads * (score width + value width) multiply-adds
+            pairs = self.pairs
+            if self.windowed is not None:  # mixers of one design that see different numbers of keys: by the call's own window
+                window = args[{"attention_bf16": 14, "latent_attention_bf16": 13}[name]]
+                rows_seen, pairs = self.windowed(window)
+                byts += (rows_seen - kv_rows) * row_bytes
+            flops = 2.0 * pairs * (q.shape[1] + out.shape[1])  # per (query token, key) pair: heads * (score width + value width) multiply-adds
         ideal = max(flops / (self.peaks["bf16_tflops"] * 1e12), byts / (self.peaks["hbm_gbs"] * 1e9)) * 1e6
         return ideal, flops, byts
 
-    def run(self, step, kv_rows: int, pairs: float) -> list:
-        """``step()`` runs one step; ``kv_rows``: cache rows the step's requests hold; ``pairs``: (query token, visible key) pairs."""
+    def run(self, step, kv_rows: int, pairs: float, windowed=None) -> list:
+        """``step()`` runs one step; ``kv_rows``: cache rows the step's requests hold; ``pairs``: (query token, visible key) pairs;
+        ``windowed`` (optional): window (None: all keys) -> (cache rows, pairs) of an attention with it."""
         import torch
 
         from alofa_b200.csrc import ops
 
-        self.pairs = pairs
+        self.pairs, self.windowed = pairs, windowed
         names = [n for n in dir(ops) if not n.startswith("_") and callable(getattr(ops, n)) and getattr(getattr(ops, n), "__module__", "") == ops.__name__
                  and n not in ("launch_count", "count_launches", "bound_stream", "attention_decode_wide_warps", "attention_decode_slots", "attention_bf16_supported",
                                "gemm_tc_rope_splits", "gemm_tc_splits", "delta_pair_words", "latent_attention_bf16_supported", "load_library", "gemm_by_tile")]  # gemm_by_tile only chooses: its product is timed
@@ -808,7 +856,7 @@ class DesignBench(Bench):
     """One engine of one design at one size, measured like the headline bench's."""
 
     def __init__(self, architecture: str, cfg, label: str, vocab: int, weight_bytes: int, kv_bytes_per_token: int, flops_per_token: float, attn_flops_per_pair: float, max_batch: int,
-                 state_bytes_per_request: int = 0, window: int = 0):
+                 state_bytes_per_request: int = 0, window: int = 0, by_call: bool = False):
         import numpy as np
 
         from alofa_b200.engine.engine import Engine
@@ -821,17 +869,19 @@ class DesignBench(Bench):
         self.numbers = {"weight_bytes": weight_bytes, "kv_bytes_per_token": kv_bytes_per_token, "state_bytes_per_request": state_bytes_per_request}
         self.flops_per_token, self.attn_flops_per_pair = flops_per_token, attn_flops_per_pair
         self.window = window  # every attention of the design sees this many keys at most (0: all)
+        self.by_call = by_call  # the design's attentions have windows of their own
         self.peaks, self.peaks_kind = peaks()
         self.rng = np.random.default_rng(0)
 
     def prompt(self, n: int) -> list:
         return [int(t) for t in self.rng.integers(0, self.vocab, size=n)]
 
-    def pairs(self, tokens: int) -> float:
+    def pairs(self, tokens: int, window: int = 0) -> float:
         """(query, visible key) pairs of one prompt of ``tokens`` tokens."""
-        if not self.window or self.window >= tokens:
+        window = window or self.window
+        if not window or window >= tokens:
             return tokens * (tokens + 1) / 2
-        return self.window * (self.window + 1) / 2 + (tokens - self.window) * self.window
+        return window * (window + 1) / 2 + (tokens - window) * window
 
     def prefill(self, warmup: int, reps: int = 10) -> dict:
         from alofa_b200.engine.step import StepEntry
@@ -863,7 +913,8 @@ class DesignBench(Bench):
             runner.forward_logits([StepEntry(slot, tokens, (PROMPT_LEN - 1,))])  # loads every kernel
             runner.release(slot)
             slot = runner.admit(30_001)
-            prefill = clock.run(lambda: runner.forward_logits([StepEntry(slot, tokens, (PROMPT_LEN - 1,))]), PROMPT_LEN, self.pairs(PROMPT_LEN))
+            prefill = clock.run(lambda: runner.forward_logits([StepEntry(slot, tokens, (PROMPT_LEN - 1,))]), PROMPT_LEN, self.pairs(PROMPT_LEN),
+                                (lambda w: (PROMPT_LEN, self.pairs(PROMPT_LEN, w or 0))) if self.by_call else None)
             runner.release(slot)
             slots = [runner.admit(31_000 + i) for i in range(batch)]
             for s_ in slots:
@@ -871,7 +922,7 @@ class DesignBench(Bench):
             one = lambda: runner.forward_logits([StepEntry(s_, (1,), (0,)) for s_ in slots])
             one()
             seen = min(PROMPT_LEN + 2, self.window or PROMPT_LEN + 2)
-            decode = clock.run(one, batch * seen, batch * seen)
+            decode = clock.run(one, batch * seen, batch * seen, (lambda w: (batch * min(seen, w or seen),) * 2) if self.by_call else None)
             for s_ in slots:
                 runner.release(s_)
         finally:
@@ -922,16 +973,20 @@ def darolix_numbers(z: dict, d: dict) -> dict:
 def run_designs(args) -> dict:
     """Prefill and decode of a design beside its closest existing design at equal layer sizes (Kotutar
     beside Qwen2, Darolix beside Kotutar, Dibulix and Kikerax beside Darolix, Pekerax beside Dibulix and
-    Kikerax), and the kernels of one step of each against their own rooflines."""
-    from alofa_b200.models import darolix, dibulix, kikerax, kotutar, pekerax, qwen2
+    Kikerax, Nugopel beside Kotutar and Pekerax), and the kernels of one step of each against their own rooflines."""
+    from alofa_b200.models import darolix, dibulix, kikerax, kotutar, nugopel, pekerax, qwen2
 
-    pair = {"pekerax": "Pekerax design beside Dibulix and Kikerax", "kikerax": "Kikerax design beside Darolix", "dibulix": "Dibulix design beside Darolix", "darolix": "Darolix design beside Kotutar", "kotutar": "Kotutar design beside Qwen2"}[args.design]
+    pair = {"nugopel": "Nugopel design beside Kotutar and Pekerax", "pekerax": "Pekerax design beside Dibulix and Kikerax", "kikerax": "Kikerax design beside Darolix", "dibulix": "Dibulix design beside Darolix", "darolix": "Darolix design beside Kotutar", "kotutar": "Kotutar design beside Qwen2"}[args.design]
     out = {"metric": f"prefill and decode of the {pair} at equal layer sizes", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
            "prompt_tokens": PROMPT_LEN, "context": CONTEXT, "steps": args.steps, "warmup": args.warmup, "sizes": {}}
     for size in ([args.size] if args.size else sorted(DESIGN_SIZES)):
         z = DESIGN_SIZES[size]
         row = {"sizes": z}
-        if args.design == "pekerax":
+        if args.design == "nugopel":
+            row["nugopel_sizes"], row["pekerax_sizes"] = NUGOPEL_SIZES[size], PEKERAX_SIZES[size]
+            arms = (("nugopel", nugopel.NAME, nugopel_config(z, NUGOPEL_SIZES[size])), ("kotutar", kotutar.NAME, kotutar_config(z)),
+                    ("pekerax", pekerax.NAME, pekerax_config(z, PEKERAX_SIZES[size])))
+        elif args.design == "pekerax":
             row["pekerax_sizes"], row["dibulix_sizes"], row["kikerax_sizes"] = PEKERAX_SIZES[size], DIBULIX_SIZES[size], KIKERAX_SIZES[size]
             arms = (("pekerax", pekerax.NAME, pekerax_config(z, PEKERAX_SIZES[size])), ("dibulix", dibulix.NAME, dibulix_config(z, DIBULIX_SIZES[size])),
                     ("kikerax", kikerax.NAME, kikerax_config(z, KIKERAX_SIZES[size])))
@@ -947,7 +1002,9 @@ def run_designs(args) -> dict:
         else:
             arms = (("kotutar", kotutar.NAME, kotutar_config(z)), ("qwen2", qwen2.NAME, qwen2_config_like(z)))
         for design, name, cfg in arms:
-            if design == "pekerax":
+            if design == "nugopel":
+                n = nugopel_numbers(z, NUGOPEL_SIZES[size])
+            elif design == "pekerax":
                 n = pekerax_numbers(z, PEKERAX_SIZES[size])
             elif design == "kikerax":
                 n = kikerax_numbers(z, KIKERAX_SIZES[size])
@@ -959,7 +1016,7 @@ def run_designs(args) -> dict:
                 n = design_numbers(design, z, routed_only=args.design == "darolix")
             window = {"dibulix": DIBULIX_SIZES[size]["window"], "pekerax": PEKERAX_SIZES[size]["window"] + PEKERAX_SIZES[size]["keep_first"]}.get(design, 0)
             bench = DesignBench(name, cfg, f"{design} {size}", z["vocab"], n["weight_bytes"], n["kv_bytes_per_token"], n["flops_per_token"], n["attn_flops_per_pair"], 64,
-                                n.get("state_bytes_per_request", 0), window=window)
+                                n.get("state_bytes_per_request", 0), window=window, by_call=design == "nugopel")
             res = {"prefill_2048": bench.prefill(args.warmup)}
             for batch in (8, 64):
                 point = bench.decode(batch, min(args.steps, 64), args.warmup)
@@ -989,7 +1046,7 @@ def main() -> int:
     ap.add_argument("--phase", choices=["all", "decode", "prefill"], default="all", help="profiling aid: run only one part; the JSON line then lacks the others")
     ap.add_argument("--shape", choices=sorted(SHAPES), default="0.5b", help="whose layer sizes the headline run has")
     ap.add_argument("--no-extra", dest="extra", action="store_false", help="leave out the measurements beside the headline (long contexts, the 1.5B and 7B shapes)")
-    ap.add_argument("--design", choices=["kotutar", "darolix", "dibulix", "kikerax", "pekerax"], help="instead of the headline run: this design beside its closest existing one (Qwen2 for kotutar, Kotutar for darolix, Darolix for dibulix and kikerax, Dibulix and Kikerax for pekerax) at equal layer sizes (prefill, decode, kernels against their rooflines)")
+    ap.add_argument("--design", choices=["kotutar", "darolix", "dibulix", "kikerax", "pekerax", "nugopel"], help="instead of the headline run: this design beside its closest existing one (Qwen2 for kotutar, Kotutar for darolix, Darolix for dibulix and kikerax, Dibulix and Kikerax for pekerax, Kotutar and Pekerax for nugopel) at equal layer sizes (prefill, decode, kernels against their rooflines)")
     ap.add_argument("--size", choices=sorted(DESIGN_SIZES), help="with --design: one of the sizes only")
     args = ap.parse_args()
     if args.impl == "reference":
