@@ -3,8 +3,8 @@
 // every batch b (per-head products of latent attention), or, with tile_batch,
 // one x and one out whose 64-row tiles each multiply by the weight of the
 // batch the tile names (experts of a routed feed-forward, rows sorted by
-// expert and padded to whole tiles).  64 x 64 output tile per CTA, 32-deep
-// slices by cp.async into two shared-memory buffers, four warps of 32 x 32
+// expert and padded to whole tiles).  64 x 64 output tile per CTA, 64-deep
+// slices by cp.async into a ring of three shared-memory buffers, four warps of 32 x 32
 // (mma.sync m16n8k16, fp32 sums), bias, activation and gate on the fp32 sums.  The
 // depth, the row strides and the batch strides are multiples of 8 elements and
 // the operands start on 16-byte boundaries (the caller checks).
@@ -12,7 +12,8 @@
 
 namespace {
 
-constexpr int TM = 64, TN = 64, TK = 32, LD = TK + 8;
+constexpr int TM = 64, TN = 64, TK = 64, LD = TK + 8, STAGES = 3;
+constexpr size_t SMEM_BYTES = (size_t)STAGES * (TM + TN) * LD * 2;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
@@ -31,8 +32,9 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
                                                                 int K, long long ldx, long long x_batch, long long ldw, long long w_batch,
                                                                 long long ldo, long long out_batch, long long bias_batch, int act, int tile_rows,
                                                                 const float* __restrict__ gate, long long ldg, long long gate_batch) {
-  __shared__ __align__(16) bf16 As[2][TM * LD];
-  __shared__ __align__(16) bf16 Bs[2][TN * LD];
+  extern __shared__ __align__(16) uint8_t tiles_smem[];
+  bf16(*As)[TM * LD] = reinterpret_cast<bf16(*)[TM * LD]>(tiles_smem);
+  bf16(*Bs)[TN * LD] = reinterpret_cast<bf16(*)[TN * LD]>(tiles_smem + (size_t)STAGES * TM * LD * 2);
   pdl_begin();
   int b = blockIdx.z;
   if (tile_batch) {
@@ -50,9 +52,9 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
   const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
   auto fetch = [&](int kt, int buf) {
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < TM * TK / 8 / 128; ++i) {
       const int e = tid + 128 * i;
-      const int r = e >> 2, c = (e & 3) * 8;
+      const int r = e / (TK / 8), c = (e % (TK / 8)) * 8;
       const int gk = kt * TK + c;
       bf16* da = &As[buf][r * LD + c];
       if (m0 + r < M && gk < K) cp16(smem_addr(da), x + (size_t)(m0 + r) * ldx + gk);
@@ -70,14 +72,17 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
 #pragma unroll
       for (int k = 0; k < 4; ++k) acc[i][j][k] = 0.f;
   const int slices = (K + TK - 1) / TK;
-  fetch(0, 0);
-  asm volatile("cp.async.commit_group;");
-  for (int kt = 0; kt < slices; ++kt) {
-    const int buf = kt & 1;
-    if (kt + 1 < slices) fetch(kt + 1, buf ^ 1);
+#pragma unroll
+  for (int st = 0; st < STAGES - 1; ++st) {
+    if (st < slices) fetch(st, st);
     asm volatile("cp.async.commit_group;");
-    asm volatile("cp.async.wait_group 1;");
-    __syncthreads();
+  }
+  for (int kt = 0; kt < slices; ++kt) {
+    const int buf = kt % STAGES;
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2));
+    __syncthreads();  // the slice is there for every warp, and the buffer of the slice before it is read out
+    if (kt + STAGES - 1 < slices) fetch(kt + STAGES - 1, (kt + STAGES - 1) % STAGES);
+    asm volatile("cp.async.commit_group;");
 #pragma unroll
     for (int ks = 0; ks < TK; ks += 16) {
       uint32_t a[2][4], bb[2][4];
@@ -93,7 +98,6 @@ __global__ void __launch_bounds__(128) gemm_batched_bf16_kernel(TO* __restrict__
           mma16816(acc[i][2 * j + 1], a[i], bb[j][2], bb[j][3]);
         }
     }
-    __syncthreads();
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -122,11 +126,18 @@ ALOFA_API int alofa_gemm_batched_bf16(void* out, const void* x, const void* w, c
   if (K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || (x_batch & 7) || (w_batch & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return ALOFA_ERR_ARGUMENT;
   if ((M + TM - 1) / TM > 65535 || batches > 65535) return ALOFA_ERR_ARGUMENT;
   dim3 grid((N + TN - 1) / TN, (M + TM - 1) / TM, tile_batch ? 1 : batches);
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(gemm_batched_bf16_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES) != cudaSuccess ||
+        cudaFuncSetAttribute(gemm_batched_bf16_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES) != cudaSuccess)
+      return ALOFA_ERR_LAUNCH;
+    set = true;
+  }
   if (out_bf16)
-    launch_dep(gemm_batched_bf16_kernel<bf16>, grid, dim3(128), 0, stream, (bf16*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx, x_batch,
+    launch_dep(gemm_batched_bf16_kernel<bf16>, grid, dim3(128), SMEM_BYTES, stream, (bf16*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx, x_batch,
                ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch);
   else
-    launch_dep(gemm_batched_bf16_kernel<float>, grid, dim3(128), 0, stream, (float*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx,
+    launch_dep(gemm_batched_bf16_kernel<float>, grid, dim3(128), SMEM_BYTES, stream, (float*)out, (const bf16*)x, (const bf16*)w, bias, tile_batch, M, N, K, ldx,
                x_batch, ldw, w_batch, ldo, out_batch, bias_batch, act, tile_rows, gate, ldg, gate_batch);
   return launch_status();
 }

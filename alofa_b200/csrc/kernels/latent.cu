@@ -668,25 +668,46 @@ __global__ void moe_route_kernel(int* __restrict__ choice, float* __restrict__ w
   if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-zr[E]));
 }
 
-// The router's product and the choice in one kernel: z = x Wr^T in fp32 (x in the compute dtype, Wr fp32
-// [E (+1), hidden]).  A block takes up to eight tokens, whose rows it keeps in shared memory; a warp takes
-// the experts warp, warp + 8, ... and, for each, sums all the block's tokens at once: every lane reads its
-// share of the expert's weights once and multiplies it into each token's row, then the warp adds the
-// lanes' shares in butterfly order.  The order of additions of a (token, expert) sum depends on the depth
-// alone.  The logits stay in shared memory; then a warp per token takes scores and choice as above.
-template <typename T, int TT>
+// The router's product and the choice in one kernel: z = x Wr^T, fp32 sums (x in the compute dtype, Wr [E (+1), hidden]
+// fp32 or bfloat16).  A cluster of blocks takes up to TT tokens and deals the experts among its blocks, so that a
+// handful of tokens pulls the weights through several SMs; every block keeps the tokens' rows in shared memory, a warp
+// takes one of the block's experts at a time and sums all tokens at once: every lane reads its share of the expert's
+// weights once and multiplies it into each token's row, then the warp adds the lanes' shares in butterfly order.  The
+// order of additions of a (token, expert) sum depends on the depth alone.  A token's logits go to the shared memory of
+// the block that then takes its scores and choice, a warp per token, as above.
+template <typename T>
+__device__ __forceinline__ void eight_floats(float (&v)[8], const T* p);  // p on a 16-byte boundary
+template <>
+__device__ __forceinline__ void eight_floats<float>(float (&v)[8], const float* p) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+template <>
+__device__ __forceinline__ void eight_floats<bf16>(float (&v)[8], const bf16* p) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const uint32_t u[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(u[i] << 16);
+    v[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+  }
+}
+
+template <typename T, typename WT, int TT>
 __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate,
-                                                         const T* __restrict__ x, const float* __restrict__ wr, int T_, int E, int top, int hidden,
+                                                         const T* __restrict__ x, const WT* __restrict__ wr, int T_, int E, int top, int hidden,
                                                          int gated, int softmax, int renormalize, const float* __restrict__ correction,
-                                                         float renorm_eps, int groups, int keep, float route_scale, int group_best) {
+                                                         float renorm_eps, int groups, int keep, float route_scale, int group_best, int blocks) {
   extern __shared__ __align__(16) uint8_t router_smem[];
   const int cols = E + (gated ? 1 : 0);
   float* z = reinterpret_cast<float*>(router_smem);      // [TT][cols]
   float* gsc = z + TT * cols;                            // [TT][groups]: the groups' scores
   T* xs = reinterpret_cast<T*>(z + ((TT * (cols + groups) + 3) & ~3));  // [TT][hidden], on a 16-byte boundary
+  if (blocks > 1) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");  // every block of the cluster runs before its memory is written to
   pdl_begin();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t0 = blockIdx.x * TT;
+  const int rank = blockIdx.x % blocks;  // of the `blocks` blocks of this cluster
+  const int t0 = blockIdx.x / blocks * TT;
   const int live = min(TT, T_ - t0);
   if ((hidden * sizeof(T)) % 16 == 0) {  // rows start on 16-byte boundaries: 16 bytes a thread
     constexpr int PER = 16 / sizeof(T);
@@ -700,26 +721,29 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
       for (int c = threadIdx.x; c < hidden; c += 256) xs[r * hidden + c] = r < live ? x[(size_t)(t0 + r) * hidden + c] : from_f<T>(0.f);
   }
   __syncthreads();
-  for (int e = warp; e < cols; e += 8) {
-    const float* w = wr + (size_t)e * hidden;
+  if (blocks > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+  const int per = (cols + blocks - 1) / blocks;
+  for (int e = rank * per + warp; e < min(cols, (rank + 1) * per); e += 8) {
+    const WT* w = wr + (size_t)e * hidden;
     float dot[TT];
 #pragma unroll
     for (int r = 0; r < TT; ++r) dot[r] = 0.f;
-    if ((hidden & 3) == 0) {
-      // four depth entries a lane and several loads in flight: with one scalar load at a time a warp spent
-      // its time waiting for the weights (190 us a call at 64 experts, whatever the number of tokens)
+    if ((hidden & 7) == 0) {
 #pragma unroll 4
-      for (int c = lane * 4; c < hidden; c += 128) {
-        const float4 wv = *reinterpret_cast<const float4*>(w + c);
+      for (int c = lane * 8; c < hidden; c += 256) {
+        float wv[8];
+        eight_floats<WT>(wv, w + c);
 #pragma unroll
         for (int r = 0; r < TT; ++r) {
-          const T* xr = xs + r * hidden + c;
-          dot[r] = fmaf(to_f(xr[3]), wv.w, fmaf(to_f(xr[2]), wv.z, fmaf(to_f(xr[1]), wv.y, fmaf(to_f(xr[0]), wv.x, dot[r]))));
+          float xv[8];
+          eight_floats<T>(xv, xs + r * hidden + c);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) dot[r] = fmaf(xv[i], wv[i], dot[r]);
         }
       }
     } else {
       for (int c = lane; c < hidden; c += 32) {
-        const float wv = w[c];
+        const float wv = to_f(w[c]);
 #pragma unroll
         for (int r = 0; r < TT; ++r) dot[r] = fmaf(to_f(xs[r * hidden + c]), wv, dot[r]);
       }
@@ -727,11 +751,22 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
 #pragma unroll
     for (int r = 0; r < TT; ++r) {
       const float v = warp_sum(dot[r]);
-      if (lane == 0) z[r * cols + e] = v;
+      if (lane != 0) continue;
+      if (blocks > 1) {  // to the block that takes token r
+        uint32_t at;
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"((uint32_t)__cvta_generic_to_shared(z + r * cols + e)), "r"(r % blocks));
+        asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(at), "f"(v) : "memory");
+      } else {
+        z[r * cols + e] = v;
+      }
     }
   }
+  if (blocks > 1) {
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+  }
   __syncthreads();
-  for (int r = warp; r < live; r += 8) {
+  for (int r = rank + blocks * warp; r < live; r += 8 * blocks) {
     const int t = t0 + r;
     float* s = z + r * cols;
     const float zg = gated ? s[E] : 0.f;
@@ -806,40 +841,41 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
   }
 }
 
-template <typename T, int TT>
-static int moe_router_launch(int* choice, float* weight, float* gate, const void* x, const float* wr, int T_, int E, int top, int hidden, int softmax,
+template <typename T, typename WT, int TT>
+static int moe_router_launch(int* choice, float* weight, float* gate, const void* x, const void* wr, int T_, int E, int top, int hidden, int softmax,
                              int renormalize, const float* correction, float renorm_eps, int groups, int keep, float route_scale, int group_best, cudaStream_t stream) {
   const int cols = E + (gate ? 1 : 0);
   const size_t smem = ((size_t)TT * (cols + groups) + 4) * sizeof(float) + (size_t)TT * hidden * sizeof(T);
   static size_t set = 0;
   if (smem > set) {
-    if (cudaFuncSetAttribute(moe_router_kernel<T, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
+    if (cudaFuncSetAttribute(moe_router_kernel<T, WT, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
     set = smem;
   }
-  launch_dep(moe_router_kernel<T, TT>, (T_ + TT - 1) / TT, 256, smem, stream, choice, weight, gate, (const T*)x, wr, T_, E, top, hidden, gate ? 1 : 0, softmax,
-             renormalize, correction, renorm_eps, groups, keep, route_scale, group_best);
+  const int blocks = T_ <= 1024 && cols >= 16 ? 8 : 1;  // with more tokens there are enough clusters of one block
+  launch_dep_cluster(moe_router_kernel<T, WT, TT>, (T_ + TT - 1) / TT * blocks, 256, smem, stream, blocks, choice, weight, gate, (const T*)x, (const WT*)wr, T_, E, top, hidden,
+                     gate ? 1 : 0, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, blocks);
   return launch_status();
 }
 
-// correction (optional, fp32 [E]): added to the scores for the choice only.  renorm_eps: added to the sum the weights are divided by.
-// groups > 1: the experts form that many equal groups of neighbours, of which only the `keep` best (by the sum of their two largest
-// choice scores) can be chosen.  route_scale: a factor on the weights.
-ALOFA_API int alofa_moe_router(int* choice, float* weight, float* gate, const void* x, const float* wr, int T, int E, int top, int hidden, int softmax,
-                               int renormalize, int x_bf16, const float* correction, float renorm_eps, int groups, int keep, float route_scale,
+// wr in fp32 or (x in bfloat16 too) bfloat16.  correction (optional, fp32 [E]): added to the scores for the choice only.  renorm_eps: added
+// to the sum the weights are divided by.  groups > 1: the experts form that many equal groups of neighbours, of which only the `keep` best
+// (by the sum of their two largest choice scores) can be chosen.  route_scale: a factor on the weights.
+ALOFA_API int alofa_moe_router(int* choice, float* weight, float* gate, const void* x, const void* wr, int T, int E, int top, int hidden, int softmax,
+                               int renormalize, int x_bf16, int w_bf16, const float* correction, float renorm_eps, int groups, int keep, float route_scale,
                                int group_best, cudaStream_t stream) {
   if (T <= 0) return ALOFA_OK;
-  if (E <= 0 || top <= 0 || top > E || top > 32) return ALOFA_ERR_ARGUMENT;
+  if (E <= 0 || top <= 0 || top > E || top > 32 || (w_bf16 && !x_bf16)) return ALOFA_ERR_ARGUMENT;
   if (groups < 1) groups = 1;
   if (groups > 1 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top)) return ALOFA_ERR_ARGUMENT;
   const size_t row = (size_t)hidden * (x_bf16 ? 2 : 4) + (size_t)(E + groups + 1) * 4;
   const size_t room = 200 * 1024;
-  // few tokens: two to a block, so that a decode step's tokens are spread over more than a handful of SMs
-  if (8 * row <= room && T > 512)
-    return x_bf16 ? moe_router_launch<bf16, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
-                  : moe_router_launch<float, 8>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream);
-  if (2 * row <= room)
-    return x_bf16 ? moe_router_launch<bf16, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
-                  : moe_router_launch<float, 2>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream);
+#define ROUTER_CASE(TT) \
+  return !x_bf16  ? moe_router_launch<float, float, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream) \
+         : w_bf16 ? moe_router_launch<bf16, bf16, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream) \
+                  : moe_router_launch<bf16, float, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
+  if (8 * row + 16 <= room) ROUTER_CASE(8);
+  if (2 * row + 16 <= room) ROUTER_CASE(2);
+#undef ROUTER_CASE
   return ALOFA_ERR_ARGUMENT;
 }
 
@@ -890,28 +926,29 @@ __global__ void moe_sort_kernel(int* __restrict__ dest, int* __restrict__ tile_e
 // The same result faster, for as many experts as shared memory holds a count per thread for: thread i
 // takes the pairs [i * share, (i + 1) * share), counts them per expert, the counts of each expert are
 // summed over the threads in thread order (so the order within an expert stays the order of the pairs),
-// and every thread numbers its pairs from there.
-constexpr int SORT_THREADS = 256;
-__global__ void __launch_bounds__(SORT_THREADS) moe_sort_counted_kernel(int* __restrict__ dest, int* __restrict__ tile_expert, const int* __restrict__ choice,
-                                                                        int pairs, int E, int tile, int max_tiles) {
-  extern __shared__ int counted[];  // [E][SORT_THREADS] counts, then offsets; then [E] first rows
+// and every thread numbers its pairs from there.  C: the type of a count and of a place among an expert's pairs.
+template <int THREADS, typename C>
+__global__ void __launch_bounds__(THREADS) moe_sort_counted_kernel(int* __restrict__ dest, int* __restrict__ tile_expert, const int* __restrict__ choice,
+                                                                   int pairs, int E, int tile, int max_tiles) {
+  extern __shared__ __align__(16) uint8_t sort_smem[];
+  int* first = reinterpret_cast<int*>(sort_smem);                    // [E] counts, then first rows
+  C* counted = reinterpret_cast<C*>(first + E);                     // [E][THREADS] counts, then offsets
   pdl_begin();
-  int* first = counted + E * SORT_THREADS;
-  const int tid = threadIdx.x;
-  const int share = (pairs + SORT_THREADS - 1) / SORT_THREADS;
+  constexpr int SHARE = THREADS / 32;  // threads a lane sums
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int share = (pairs + THREADS - 1) / THREADS;
   const int lo = min(pairs, tid * share), hi = min(pairs, lo + share);
-  for (int e = 0; e < E; ++e) counted[e * SORT_THREADS + tid] = 0;
+  for (int e = 0; e < E; ++e) counted[e * THREADS + tid] = 0;
   for (int i = lo; i < hi; ++i)
-    if (choice[i] < E) counted[choice[i] * SORT_THREADS + tid] += 1;
+    if (choice[i] < E) counted[choice[i] * THREADS + tid] += 1;
   __syncthreads();
-  // an exclusive sum over the threads, per expert: a warp takes experts in turn, a lane eight threads' counts
-  const int warp = tid >> 5, lane = tid & 31;
-  for (int e = warp; e < E; e += SORT_THREADS / 32) {
-    int* row = counted + e * SORT_THREADS;
-    int v[8], sum = 0;
+  // an exclusive sum over the threads, per expert: a warp takes experts in turn, a lane SHARE threads' counts
+  for (int e = warp; e < E; e += THREADS / 32) {
+    C* row = counted + e * THREADS + lane * SHARE;
+    int v[SHARE], sum = 0;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      v[j] = row[lane * 8 + j];
+    for (int j = 0; j < SHARE; ++j) {
+      v[j] = row[j];
       sum += v[j];
     }
     int incl = sum;
@@ -922,57 +959,79 @@ __global__ void __launch_bounds__(SORT_THREADS) moe_sort_counted_kernel(int* __r
     }
     int at = incl - sum;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      row[lane * 8 + j] = at;
+    for (int j = 0; j < SHARE; ++j) {
+      row[j] = (C)at;
       at += v[j];
     }
     if (lane == 31) first[e] = incl;  // the expert's count, for now
   }
   __syncthreads();
-  if (tid == 0) {
-    int at = 0;
-    for (int e = 0; e < E; ++e) {
-      const int n = first[e], tiles = (n + tile - 1) / tile;
-      first[e] = at;
-      for (int i = 0; i < tiles; ++i) tile_expert[at / tile + i] = e;
-      at += tiles * tile;
+  if (warp == 0) {
+    int at = 0;  // tiles handed out
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, tiles = e < E ? (first[e] + tile - 1) / tile : 0;
+      int incl = tiles;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += up;
+      }
+      const int mine = at + incl - tiles;
+      if (e < E) first[e] = mine * tile;
+      for (int i = 0; i < tiles; ++i) tile_expert[mine + i] = e;
+      at += __shfl_sync(0xffffffffu, incl, 31);
     }
-    for (int i = at / tile; i < max_tiles; ++i) tile_expert[i] = -1;
+    for (int i = at + lane; i < max_tiles; i += 32) tile_expert[i] = -1;
   }
   __syncthreads();
   for (int i = lo; i < hi; ++i) {
     const int e = choice[i];
-    dest[i] = e < E ? first[e] + counted[e * SORT_THREADS + tid]++ : -1;  // no row for a choice that is no expert with weights
+    dest[i] = e < E ? first[e] + counted[e * THREADS + tid]++ : -1;  // no row for a choice that is no expert with weights
   }
+}
+
+template <int THREADS, typename C>
+static int moe_sort_counted_launch(int* dest, int* tile_expert, const int* choice, int pairs, int E, int tile, int max_tiles, cudaStream_t stream) {
+  const size_t smem = (size_t)E * (THREADS * sizeof(C) + sizeof(int));
+  static size_t set = 0;
+  if (smem > set) {
+    if (cudaFuncSetAttribute(moe_sort_counted_kernel<THREADS, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
+    set = smem;
+  }
+  launch_dep(moe_sort_counted_kernel<THREADS, C>, 1, THREADS, smem, stream, dest, tile_expert, choice, pairs, E, tile, max_tiles);
+  return launch_status();
 }
 
 ALOFA_API int alofa_moe_sort(int* dest, int* tile_expert, const int* choice, int pairs, int E, int tile, int max_tiles, cudaStream_t stream) {
   if (pairs <= 0) return ALOFA_OK;
   if (E <= 0 || tile <= 0 || (size_t)2 * E * 4 > 48 * 1024 || max_tiles < (pairs + tile - 1) / tile) return ALOFA_ERR_ARGUMENT;
-  const size_t counted = ((size_t)E * SORT_THREADS + E) * sizeof(int);
-  if (counted <= 200 * 1024) {
-    static size_t set = 0;
-    if (counted > set) {
-      if (cudaFuncSetAttribute(moe_sort_counted_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)counted) != cudaSuccess) return ALOFA_ERR_LAUNCH;
-      set = counted;
-    }
-    launch_dep(moe_sort_counted_kernel, 1, SORT_THREADS, counted, stream, dest, tile_expert, choice, pairs, E, tile, max_tiles);
-    return launch_status();
-  }
+  const size_t room = 200 * 1024;
+  if (pairs <= 65535 && pairs > 1024 && (size_t)E * (1024 * 2 + 4) <= room) return moe_sort_counted_launch<1024, uint16_t>(dest, tile_expert, choice, pairs, E, tile, max_tiles, stream);
+  if (pairs <= 65535 && (size_t)E * (256 * 2 + 4) <= room) return moe_sort_counted_launch<256, uint16_t>(dest, tile_expert, choice, pairs, E, tile, max_tiles, stream);
+  if ((size_t)E * (256 * 4 + 4) <= room) return moe_sort_counted_launch<256, int>(dest, tile_expert, choice, pairs, E, tile, max_tiles, stream);
   launch_dep(moe_sort_kernel, 1, 256, (size_t)2 * E * sizeof(int), stream, dest, tile_expert, choice, pairs, E, tile, max_tiles);
   return launch_status();
 }
 
 // scatter: xs[dest[pair]] = x[token] * (weight[pair] if the weight multiplies the input) in the compute dtype.
 template <typename T>
+__device__ __forceinline__ void place_row(T* __restrict__ to, const T* __restrict__ from, const float* weight, int hidden) {
+  if (!weight && (hidden * sizeof(T)) % 16 == 0) {  // rows of whole 16-byte pieces, as they are
+    const int chunks = hidden * (int)sizeof(T) / 16;
+    for (int c = threadIdx.x; c < chunks; c += blockDim.x) reinterpret_cast<uint4*>(to)[c] = reinterpret_cast<const uint4*>(from)[c];
+    return;
+  }
+  const float w = weight ? *weight : 1.0f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) to[c] = weight ? from_f<T>(to_f(from[c]) * w) : from[c];
+}
+
+template <typename T>
 __global__ void moe_scatter_kernel(T* __restrict__ xs, const T* __restrict__ x, const float* __restrict__ weight, const int* __restrict__ dest, int top,
                                    int hidden) {
   pdl_begin();
-  const int pair = blockIdx.x, t = pair / top;
-  const float w = weight ? weight[pair] : 1.0f;
+  const int pair = blockIdx.x;
   if (dest[pair] < 0) return;
-  const size_t to = (size_t)dest[pair] * hidden, from = (size_t)t * hidden;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) xs[to + c] = weight ? from_f<T>(to_f(x[from + c]) * w) : x[from + c];
+  place_row(xs + (size_t)dest[pair] * hidden, x + (size_t)(pair / top) * hidden, weight ? weight + pair : nullptr, hidden);
 }
 
 ALOFA_API int alofa_moe_scatter(void* xs, const void* x, const float* weight, const int* dest, int pairs, int top, int hidden, int is_bf16,
@@ -983,31 +1042,134 @@ ALOFA_API int alofa_moe_scatter(void* xs, const void* x, const float* weight, co
   return launch_status();
 }
 
+// Both in one launch for a decode step's few pairs: every block finds the place of its own pair (the experts' counts, their
+// first rows, and how many pairs of the same expert come before) and copies the row; the first block also names the tiles' experts.
+constexpr int PLACE_PAIRS = 1024, PLACE_EXPERTS = 1024;
+template <typename T>
+__global__ void __launch_bounds__(256) moe_place_kernel(T* __restrict__ xs, int* __restrict__ dest, int* __restrict__ tile_expert, const int* __restrict__ choice,
+                                                        const T* __restrict__ x, const float* __restrict__ weight, int pairs, int E, int tile, int max_tiles, int top,
+                                                        int hidden) {
+  __shared__ int count[PLACE_EXPERTS];  // counts, then first rows
+  __shared__ int ahead;
+  pdl_begin();
+  const int pair = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
+  for (int e = tid; e < E; e += 256) count[e] = 0;
+  if (tid == 0) ahead = 0;
+  __syncthreads();
+  const int mine = choice[pair];
+  int before = 0;
+  for (int i = tid; i < pairs; i += 256) {
+    const int e = choice[i];
+    if (e < E) atomicAdd(&count[e], 1);
+    before += i < pair && e == mine;
+  }
+  before = __reduce_add_sync(0xffffffffu, before);
+  if (lane == 0 && before) atomicAdd(&ahead, before);
+  __syncthreads();
+  if (tid < 32) {
+    int at = 0;  // tiles handed out
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, tiles = e < E ? (count[e] + tile - 1) / tile : 0;
+      int incl = tiles;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += up;
+      }
+      const int begin = at + incl - tiles;
+      if (e < E) count[e] = begin * tile;
+      if (pair == 0)
+        for (int i = 0; i < tiles; ++i) tile_expert[begin + i] = e;
+      at += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (pair == 0)
+      for (int i = at + lane; i < max_tiles; i += 32) tile_expert[i] = -1;
+  }
+  __syncthreads();
+  const int to = mine < E ? count[mine] + ahead : -1;  // no row for a choice that is no expert with weights
+  if (tid == 0) dest[pair] = to;
+  if (to >= 0) place_row(xs + (size_t)to * hidden, x + (size_t)(pair / top) * hidden, weight ? weight + pair : nullptr, hidden);
+}
+
+// 1 (nothing launched): more pairs or experts than this kernel takes.
+ALOFA_API int alofa_moe_place(void* xs, int* dest, int* tile_expert, const int* choice, const void* x, const float* weight, int pairs, int E, int tile, int max_tiles,
+                              int top, int hidden, int is_bf16, cudaStream_t stream) {
+  if (pairs <= 0) return ALOFA_OK;
+  if (E <= 0 || tile <= 0 || top <= 0 || max_tiles < (pairs + tile - 1) / tile) return ALOFA_ERR_ARGUMENT;
+  if (pairs > PLACE_PAIRS || E > PLACE_EXPERTS) return 1;
+  if (is_bf16) launch_dep(moe_place_kernel<bf16>, pairs, 256, 0, stream, (bf16*)xs, dest, tile_expert, choice, (const bf16*)x, weight, pairs, E, tile, max_tiles, top, hidden);
+  else launch_dep(moe_place_kernel<float>, pairs, 256, 0, stream, (float*)xs, dest, tile_expert, choice, (const float*)x, weight, pairs, E, tile, max_tiles, top, hidden);
+  return launch_status();
+}
+
 // combine: y[t] = sum_k (weight[t, k] if the weight multiplies the output) * ys[dest[t, k]] + gate[t] * shared[t]  (fp32; k ascending).
 // A pair without a row (dest < 0: an identity expert) contributes the token's own input x[t]; with `add` the sum is added to y.
-template <typename T>
-__global__ void moe_combine_kernel(float* __restrict__ y, const float* __restrict__ ys, const int* __restrict__ dest, const float* __restrict__ weight,
-                                   const float* __restrict__ shared, const float* __restrict__ gate, int top, int hidden, const T* __restrict__ x, int add) {
+// V columns a thread; a block takes COMBINE_COLUMNS of a token, so that a handful of tokens is spread over more SMs.
+constexpr int COMBINE_THREADS = 128;
+template <typename T, int V>
+__global__ void __launch_bounds__(COMBINE_THREADS) moe_combine_kernel(float* __restrict__ y, const float* __restrict__ ys, const int* __restrict__ dest,
+                                                                      const float* __restrict__ weight, const float* __restrict__ shared,
+                                                                      const float* __restrict__ gate, int top, int hidden, const T* __restrict__ x, int add) {
+  __shared__ int row_of[32];
+  __shared__ float weight_of[32];
   pdl_begin();
   const int t = blockIdx.x;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-    float v = 0.f;
-    for (int k = 0; k < top; ++k) {
-      const int row = dest[(size_t)t * top + k];
-      const float e = row >= 0 ? ys[(size_t)row * hidden + c] : (x ? to_f(x[(size_t)t * hidden + c]) : 0.f);
-      v += weight ? weight[(size_t)t * top + k] * e : e;
+  if (threadIdx.x < top) {
+    row_of[threadIdx.x] = dest[(size_t)t * top + threadIdx.x];
+    weight_of[threadIdx.x] = weight ? weight[(size_t)t * top + threadIdx.x] : 1.0f;
+  }
+  __syncthreads();
+  const int c = (blockIdx.y * COMBINE_THREADS + threadIdx.x) * V;
+  if (c >= hidden) return;
+  float v[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) v[i] = 0.f;
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const int row = row_of[k];
+    const float g = weight_of[k];
+    float e[V];
+    if (row >= 0) {
+      if constexpr (V == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(ys + (size_t)row * hidden + c);
+        e[0] = a.x, e[1] = a.y, e[2] = a.z, e[3] = a.w;
+      } else {
+        e[0] = ys[(size_t)row * hidden + c];
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) e[i] = x ? to_f(x[(size_t)t * hidden + c + i]) : 0.f;
     }
-    if (shared) v += (gate ? gate[t] : 1.0f) * shared[(size_t)t * hidden + c];
-    if (add) y[(size_t)t * hidden + c] += v;
-    else y[(size_t)t * hidden + c] = v;
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] += g * e[i];
+  }
+  const float gs = gate ? gate[t] : 1.0f;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const size_t at = (size_t)t * hidden + c + i;
+    if (shared) v[i] += gs * shared[at];
+    if (add) v[i] += y[at];
+  }
+  if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(y + (size_t)t * hidden + c) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    y[(size_t)t * hidden + c] = v[0];
   }
 }
 
 ALOFA_API int alofa_moe_combine(float* y, const float* ys, const int* dest, const float* weight, const float* shared, const float* gate, int T, int top,
                                 int hidden, const void* x, int x_bf16, int add, cudaStream_t stream) {
   if (T <= 0) return ALOFA_OK;
-  if (x_bf16) launch_dep(moe_combine_kernel<bf16>, T, 256, 0, stream, y, ys, dest, weight, shared, gate, top, hidden, (const bf16*)x, add);
-  else launch_dep(moe_combine_kernel<float>, T, 256, 0, stream, y, ys, dest, weight, shared, gate, top, hidden, (const float*)x, add);
+  if (top <= 0 || top > 32) return ALOFA_ERR_ARGUMENT;
+  const bool four = (hidden & 3) == 0 && !(((uintptr_t)y | (uintptr_t)ys) & 15);
+  const int columns = COMBINE_THREADS * (four ? 4 : 1);
+  const dim3 grid(T, (hidden + columns - 1) / columns);
+#define COMBINE_CASE(TX, V) launch_dep(moe_combine_kernel<TX, V>, grid, COMBINE_THREADS, 0, stream, y, ys, dest, weight, shared, gate, top, hidden, (const TX*)x, add)
+  if (x_bf16 && four) COMBINE_CASE(bf16, 4);
+  else if (x_bf16) COMBINE_CASE(bf16, 1);
+  else if (four) COMBINE_CASE(float, 4);
+  else COMBINE_CASE(float, 1);
+#undef COMBINE_CASE
   return launch_status();
 }
 

@@ -620,9 +620,10 @@ def _latent():
             "alofa_sandwich_norm": [_P, _P, _P, _F, _P, _P, _F, _I, _I, _I, _I, _L, _P, _P],
             "alofa_concat_rows": [_P, _P, _P, _I, _I, _I, _P],
             "alofa_moe_route": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-            "alofa_moe_router": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _I, _P],
+            "alofa_moe_router": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _I, _P],
             "alofa_cast_rows": [_P, _P, _L, _I, _P],
             "alofa_moe_sort": [_P, _P, _P, _I, _I, _I, _I, _P],
+            "alofa_moe_place": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
             "alofa_moe_scatter": [_P, _P, _P, _P, _I, _I, _I, _I, _P],
             "alofa_moe_combine": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _I, _P],
             "alofa_gate_up": [_P, _P, _L, _I, _I, _F, _F, _P],
@@ -805,6 +806,7 @@ def concat_rows(out, a, b) -> None:
 
 
 MOE_TILE = 64  # rows per tile of the sorted matrix: every expert's rows are padded to whole tiles
+GEMM_BY_TILE_FILL = 296  # tiles of a product by tile from which on wide ones are taken
 MOE_TILE_TC = 128  # the same where the tcgen05 product takes the tiles (its token tile)
 
 
@@ -818,7 +820,8 @@ def gemm_by_tile(out, x, w, tile_batch, tile_rows: int, act: str = "none") -> No
     rows = x.shape[0]
     if (tile_rows == MOE_TILE_TC and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and k % 8 == 0 and rows % 128 == 0
             and os.environ.get("ALOFA_BY_TILE_TC", "1") != "0"):
-        wide = -256 if n > 128 else -128
+        # tiles of 256 weight rows, unless they are so few (a decode step's) that half as wide ones keep more SMs pulling weights
+        wide = -256 if n > 128 and tile_batch.numel() * -(-n // 256) >= GEMM_BY_TILE_FILL else -128
         if gemm_tc(out, x, w.view(batches * n, k), None, EPI_STORE, wide, act=ACTIVATIONS[act], tile_batch=tile_batch, batches=batches):
             return
     gemm_batched(out, x, w, 1, rows, n, k, k, 0, k, n * k, n, 0, act=act, tile_batch=tile_batch, tile_rows=tile_rows)
@@ -854,8 +857,8 @@ def moe_route(choice, weight, gate, z, experts: int, top: int, softmax: bool = F
 def moe_router(choice, weight, gate, x, wr, experts: int, top: int, softmax: bool = False, renormalize: bool = False, correction=None,
                renorm_eps: float = 0.0, groups: int = 1, keep: int = 1, route_scale: float = 1.0, group_best: bool = False) -> None:
     """:func:`moe_route` with the router's product in the same kernel: ``x``
-    [T, hidden] in the compute dtype, ``wr`` fp32 [experts (+1 with ``gate``),
-    hidden]; logits and scores are fp32.  ``correction`` (fp32 [experts]) is
+    [T, hidden] in the compute dtype, ``wr`` [experts (+1 with ``gate``),
+    hidden] in fp32 or, with ``x``, in bfloat16; sums, logits and scores are fp32.  ``correction`` (fp32 [experts]) is
     added to the scores for the choice only, the weights stay the scores;
     ``renorm_eps`` is added to the sum that ``renormalize`` divides by.
     ``groups`` > 1: the experts form that many equal groups of neighbours; a
@@ -867,7 +870,7 @@ def moe_router(choice, weight, gate, x, wr, experts: int, top: int, softmax: boo
         raise AlofaError("invalid_argument", "router sizes disagree", f"wr={tuple(wr.shape)} x={tuple(x.shape)} experts={experts}")
     _done(
         _latent().alofa_moe_router(_dev(choice, "choice", i32), _dev(weight, "weight", f32), _dev(gate, "gate", f32) if gate is not None else None, _dev(x, "x"),
-                                   _dev(wr, "wr", f32), x.shape[0], experts, top, x.shape[1], 1 if softmax else 0, 1 if renormalize else 0, _is_bf16(x, "x"),
+                                   _dev(wr, "wr"), x.shape[0], experts, top, x.shape[1], 1 if softmax else 0, 1 if renormalize else 0, _is_bf16(x, "x"), _is_bf16(wr, "wr"),
                                    _dev(correction, "correction", f32) if correction is not None else None, float(renorm_eps), int(groups), int(keep), float(route_scale),
                                    1 if group_best else 0, _stream()),
         "moe_router", f"experts={experts} top={top} groups={groups} keep={keep}",
@@ -886,6 +889,19 @@ def moe_scatter(xs, x, weight, dest, top: int) -> None:
     """xs[dest[t, k]] = x[t] (times weight[t, k] when given)."""
     _done(_latent().alofa_moe_scatter(_dev(xs, "xs", x.dtype), _dev(x, "x"), _dev(weight, "weight", torch.float32) if weight is not None else None,
                                       _dev(dest, "dest", torch.int32), dest.numel(), top, x.shape[1], _is_bf16(x, "x"), _stream()), "moe_scatter")
+
+
+def moe_place(xs, dest, tile_expert, choice, x, weight, experts: int, tile: int, top: int) -> bool:
+    """:func:`moe_sort` and :func:`moe_scatter` in one kernel for the few pairs of
+    a decode step; False, having launched nothing, for more."""
+    i32 = torch.int32
+    rc = _latent().alofa_moe_place(_dev(xs, "xs", x.dtype), _dev(dest, "dest", i32), _dev(tile_expert, "tile_expert", i32), _dev(choice, "choice", i32), _dev(x, "x"),
+                                   _dev(weight, "weight", torch.float32) if weight is not None else None, choice.numel(), experts, tile, tile_expert.numel(), top, x.shape[1],
+                                   _is_bf16(x, "x"), _stream())
+    if rc == 1:
+        return False
+    _done(rc, "moe_place")
+    return True
 
 
 def moe_combine(y, ys, dest, weight, shared, gate, top: int, x=None, add: bool = False) -> None:

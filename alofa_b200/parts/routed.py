@@ -102,7 +102,7 @@ class RoutedExperts(Part):
     def load(self, state):
         pre = self.prefix
         rows = [state[pre + "router"]] + ([state[pre + "shared.sg"]] if self.shared_gate else [])
-        self.router = torch.cat(rows, dim=0).to(torch.float32).contiguous()  # the router is fp32 whatever the compute dtype
+        self.router = torch.cat(rows, dim=0).contiguous()  # the router's products and sums are fp32 whatever the compute dtype: bfloat16 weights widen exactly
         if self.gated:  # gate rows first, then up rows: one product yields both
             self.up = torch.stack([torch.cat([state[pre + f"e{e}.gate"], state[pre + f"e{e}.up"]], dim=0) for e in range(self.experts)]).contiguous()
         else:
@@ -127,10 +127,11 @@ class RoutedExperts(Part):
         pairs = n * top
         tiles = -(-pairs // tile) + self.experts  # every expert may end on a tile that is not full
         dest, tile_expert = ctx.buf((n, top), i32), ctx.buf((tiles,), i32)
-        ops.moe_sort(dest, tile_expert, choice, self.experts, tile)
         rows = tiles * tile
         xs = ctx.buf((rows, self.hidden), dt)
-        ops.moe_scatter(xs, x, weight if self.weight_on_input else None, dest, top)
+        if not ops.moe_place(xs, dest, tile_expert, choice, x, weight if self.weight_on_input else None, self.experts, tile, top):
+            ops.moe_sort(dest, tile_expert, choice, self.experts, tile)
+            ops.moe_scatter(xs, x, weight if self.weight_on_input else None, dest, top)
         mid = ctx.buf((rows, self.ff), dt)
         if self.gated:
             # gate and up in one product whose epilogue multiplies them (the tcgen05 kernel), else the sums of both and a kernel that gates

@@ -445,6 +445,79 @@ def test_router_weights_are_the_softmax_over_the_chosen_logits(experts, top):
             assert len(kept) == top and all(abs(kept.get(e, 0.0) - v) <= 2e-5 for e, v in want.items() if v > 1e-30), f"token {t}: {kept} {want}"
 
 
+@pytest.mark.parametrize("tokens,experts,top,hidden", [(1, 64, 6, 2048), (9, 17, 3, 264), (70, 200, 8, 72), (1100, 33, 2, 136), (5, 4, 2, 100), (3, 20, 2, 8192)])
+@pytest.mark.parametrize("x_type,w_type", [(F32, F32), (BF16, F32), (BF16, BF16)])
+def test_router_for_few_and_many_tokens_and_experts(tokens, experts, top, hidden, x_type, w_type):
+    """Experts dealt over a cluster of blocks and on one block, depths that are and are not multiples of 8, weights in either
+    type: 32-bit sums, and a token's logits do not depend on which others come with it."""
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(18)
+    x, wr = rounded(rng.standard_normal((tokens, hidden)), x_type), rounded(2 * rng.standard_normal((experts, hidden)) / np.sqrt(hidden), w_type)
+    chosen, weight, margin = plain.route({"m.router": wr}, "m.", {"experts": experts, "top": top}, x)
+
+    def run(rows):
+        choice, wgt = torch.empty((len(rows), top), dtype=torch.int32, device="cuda"), torch.empty((len(rows), top), dtype=F32, device="cuda")
+        ops.moe_router(choice, wgt, None, dev(rows, x_type), dev(wr, w_type), experts, top, True, True)
+        return choice.cpu().numpy(), wgt.cpu().numpy()
+
+    choice, wgt = run(x)
+    sure = margin > 1e-4
+    assert sure.mean() > 0.8 or tokens < 10
+    assert (choice[sure] == chosen[sure]).all()
+    assert_close(wgt[sure], weight[sure], 1e-5, "weights")
+    alone = run(x[tokens // 2 : tokens // 2 + 1])
+    assert (alone[0][0] == choice[tokens // 2]).all() and (alone[1][0] == wgt[tokens // 2]).all()
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("tokens,top,experts,tile,hidden,identity", [(1, 1, 4, 64, 24, 0), (8, 6, 64, 128, 256, 0), (37, 3, 5, 64, 30, 2), (128, 8, 40, 128, 8, 0), (129, 8, 70, 128, 20, 3), (3000, 4, 90, 128, 16, 0)])
+def test_pairs_are_placed_by_expert_in_one_kernel_or_two(dtype, tokens, top, experts, tile, hidden, identity):
+    """Few pairs in one launch, more in two: the same places, tiles and rows (experts past the last are the identity: no row)."""
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(19)
+    choice = np.stack([rng.permutation(experts + identity)[:top] if top <= experts else rng.integers(0, experts, top) for _ in range(tokens)]).astype(np.int32)
+    tiles = -(-tokens * top // tile) + experts
+    x, weight = rounded(rng.standard_normal((tokens, hidden)), dtype), rounded(rng.standard_normal((tokens, top)), F32)
+    for scaled in (False, True):
+        results = []
+        for one in (True, False):
+            dest, te = torch.full((tokens, top), -7, dtype=torch.int32, device="cuda"), torch.full((tiles,), -7, dtype=torch.int32, device="cuda")
+            xs = torch.zeros((tiles * tile, hidden), dtype=dtype, device="cuda")
+            w = dev(weight, F32) if scaled else None
+            if one:
+                assert ops.moe_place(xs, dest, te, dev(choice), dev(x, dtype), w, experts, tile, top) == (tokens * top <= 1024)
+            if not one or tokens * top > 1024:
+                ops.moe_sort(dest, te, dev(choice), experts, tile)
+                ops.moe_scatter(xs, dev(x, dtype), w, dest, top)
+            results.append((dest.cpu().numpy().ravel(), te.cpu().numpy(), xs.float().cpu().numpy()))
+        d, te, xs = results[0]
+        assert all((a == b).all() for a, b in zip(results[0], results[1]))
+        flat, rows = choice.ravel(), np.repeat(x, top, axis=0) * (weight.reshape(-1, 1) if scaled else 1.0)
+        real = flat < experts
+        assert (d[~real] == -1).all() and len(set(d[real].tolist())) == real.sum() and (te[d[real] // tile] == flat[real]).all()
+        for e in range(experts):
+            assert (np.diff(d[flat == e]) == 1).all()
+        used = te[te >= 0]
+        assert (np.diff(used) >= 0).all() and (te[len(used):] == -1).all()
+        assert_close(xs[d[real]], rows[real], 1e-6 if dtype == F32 else 8e-3, "rows")
+
+
+@pytest.mark.parametrize("tokens,top,hidden", [(1, 1, 30), (5, 6, 2048), (70, 32, 100), (9, 2, 516)])
+def test_combine_adds_choices_in_order_and_the_shared_output(tokens, top, hidden):
+    from alofa_b200.csrc import ops
+
+    rng = np.random.default_rng(20)
+    ys, shared, y0 = (rounded(rng.standard_normal(s), F32) for s in ((tokens * top + 3, hidden), (tokens, hidden), (tokens, hidden)))
+    dest, weight = rng.permutation(tokens * top + 3)[: tokens * top].reshape(tokens, top).astype(np.int32), rounded(rng.standard_normal((tokens, top)), F32)
+    for w, sh, add in ((weight, shared, False), (None, None, True), (weight, None, True)):
+        y = dev(y0, F32)
+        ops.moe_combine(y, dev(ys, F32), dev(dest), dev(w, F32) if w is not None else None, dev(sh, F32) if sh is not None else None, None, top, add=add)
+        want = (ys[dest] * (w[:, :, None] if w is not None else 1.0)).sum(axis=1) + (sh if sh is not None else 0.0) + (y0 if add else 0.0)
+        assert_close(y.cpu(), want, 3e-6, "combined")
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("rows,width", [(1, 96), (9, 100), (7, 30), (300, 1024)])
 def test_norm_with_its_weight_stored_less_one(dtype, rows, width):
