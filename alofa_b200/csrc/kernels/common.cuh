@@ -184,6 +184,17 @@ static inline void launch_dep(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
 
+// An ordinary launch: no block is placed before the kernel before it has left.
+template <typename... KArgs, typename... Args>
+static inline void launch_whole(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+}
+
 // The same with the grid's blocks in clusters of `cluster` neighbours along x (which must divide the grid; 1: none).
 template <typename... KArgs, typename... Args>
 static inline void launch_dep_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, int cluster, Args&&... args) {

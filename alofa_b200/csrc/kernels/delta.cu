@@ -642,7 +642,8 @@ static int delta_group_scan_launch(const DeltaGroupArgs& a, int n_seqs, int thre
     if (cudaFuncSetAttribute(delta_group_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;
     set = smem;
   }
-  launch_dep(delta_group_scan_kernel<R>, dim3(a.H, n_seqs, (a.P + a.PC - 1) / a.PC), threads, smem, stream, a);
+  // an ordinary launch: its few long-lived CTAs would otherwise settle beside what is left of the kernel before, several to an SM (375 us a call, or 647)
+  launch_whole(delta_group_scan_kernel<R>, dim3(a.H, n_seqs, (a.P + a.PC - 1) / a.PC), threads, smem, stream, a);
   return launch_status();
 }
 

@@ -1077,6 +1077,10 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = tmem_base_smem;
+  // by tile (the experts of a routed feed-forward): a token tile's batch, whose first weight row in the stacked weight is row_of;
+  // a tile that names none is passed over by every role alike
+  auto skipped = [&](int tile) { return args.tile_batch && args.tile_batch[tile / n_ftiles] < 0; };
+  auto row_of = [&](int tile) { return args.tile_batch ? args.tile_batch[tile / n_ftiles] * (GATED ? 2 : 1) * args.N : 0; };
   auto load_weights = [&](int it, int i, int f0) {  // the weight tile of slice i of a tile into the stage of ring position it
     const int s = it % PERSISTENT_STAGES;
     uint8_t* stage = tiles + (size_t)s * STAGE_BYTES;
@@ -1092,7 +1096,7 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
   int early_slices = 0;
   if (threadIdx.x == 0) {
     asm volatile("griddepcontrol.launch_dependents;");
-    if ((int)blockIdx.x < n_tiles) {
+    if ((int)blockIdx.x < n_tiles && !args.tile_batch) {
       early_slices = min(PERSISTENT_STAGES, n_slices);
       for (int i = 0; i < early_slices; ++i) load_weights(i, i, ((int)blockIdx.x % n_ftiles) * FEATS);
     }
@@ -1105,7 +1109,8 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
     if (lane == 0) {
       int it = 0;  // slices asked for so far, over all tiles
       for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
-        const int f0 = (tile % n_ftiles) * FEATS, t0 = (tile / n_ftiles) * 128;
+        if (skipped(tile)) continue;
+        const int f0 = (tile % n_ftiles) * FEATS + row_of(tile), t0 = (tile / n_ftiles) * 128;
         for (int i = 0; i < n_slices; ++i, ++it) {
           const int s = it % PERSISTENT_STAGES;
           if (it >= PERSISTENT_STAGES && !mbar_wait(&empty_bar[s], ((it / PERSISTENT_STAGES) - 1) & 1, &abort_flag)) break;
@@ -1119,7 +1124,8 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
     if (lane == 0) {
       int it = 0, j = 0;  // slices consumed; tiles of this CTA so far
       bool ok = true;
-      for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x, ++j) {
+      for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
+        if (skipped(tile)) continue;
         const int buf = j & 1;
         if (j >= 2) ok = mbar_wait(&acc_free[buf], ((j >> 1) - 1) & 1, &abort_flag);
         if (!ok) break;
@@ -1137,12 +1143,14 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
           umma_commit(&empty_bar[s]);
         }
         if (ok) umma_commit(&acc_full[buf]);
+        ++j;
       }
     }
   } else {
     const int q = warp & 3, half = (warp - 2) >> 2;
     int j = 0;
-    for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++j) {
+    for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
+      if (skipped(tile)) continue;
       const int buf = j & 1;
       const int f0 = (tile % n_ftiles) * FEATS, t0 = (tile / n_ftiles) * 128;
       bool ok = mbar_wait(&acc_full[buf], (j >> 1) & 1, &abort_flag);
@@ -1156,6 +1164,7 @@ gemm_tc_tokens_persistent_kernel(const __grid_constant__ CUtensorMap map_w, cons
         __syncwarp();
         if (lane == 0) mbar_arrive(&acc_free[buf]);
       }
+      ++j;
     }
   }
   tc_fence_before();
@@ -1504,6 +1513,8 @@ static int few_tokens_product(int bnf, int splits, int T, int N, int K, int epi)
   return T <= 32 ? 32 : 64;
 }
 
+constexpr int BY_TILE_PERSISTENT_ROWS = 4096;  // sorted rows (padding counted) from which on a product by tile runs on the persistent kernel: prompt portions
+
 template <int BNF, int EPI>
 static int launch_tokens(const CUtensorMap& mw, const CUtensorMap& mx, const GemmArgs& args, int splits, cudaStream_t stream) {
   constexpr size_t STAGE = (size_t)128 * BK * 2 + (size_t)BNF * BK * 2;
@@ -1534,7 +1545,7 @@ static int launch_tokens(const CUtensorMap& mw, const CUtensorMap& mx, const Gem
     prefer_max_shared(gemm_tc_tokens_kernel<BNF, EPI>);
     configured = true;
   }
-  if (BNF == 256 && splits == 1 && (args.N & 3) == 0 && (args.K <= 2048 || args.pair) && !args.tile_batch) {
+  if (BNF == 256 && splits == 1 && (args.N & 3) == 0 && (args.K <= 2048 || args.pair) && (!args.tile_batch || args.T >= BY_TILE_PERSISTENT_ROWS)) {
     // More tiles than SMs and a shallow depth, where a tile's epilogue is a large share of its
     // time: one resident CTA per SM works through the tiles, epilogues beside MMAs.  (Deep
     // products measured faster as two CTAs per SM, which keep four stages in flight per SM.)

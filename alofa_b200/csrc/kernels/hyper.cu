@@ -181,9 +181,31 @@ __global__ void head_gate_kernel(T* __restrict__ o, const float* __restrict__ g,
   o[i] = from_f<T>(to_f(o[i]) / (1.0f + expf(-z)));
 }
 
+// A gate per channel: four a thread.
+template <typename T>
+__global__ void channel_gate_kernel(T* __restrict__ o, const float* __restrict__ g, int ldg, int quads, long long count) {
+  pdl_begin();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= count) return;
+  const long long t = i / quads;
+  const float4 z = *reinterpret_cast<const float4*>(g + t * ldg + 4 * (i - t * quads));
+  T* p = o + 4 * i;
+  const float a = to_f(p[0]) * logistic(z.x), b = to_f(p[1]) * logistic(z.y), c = to_f(p[2]) * logistic(z.z), d = to_f(p[3]) * logistic(z.w);
+  p[0] = from_f<T>(a);
+  p[1] = from_f<T>(b);
+  p[2] = from_f<T>(c);
+  p[3] = from_f<T>(d);
+}
+
 ALOFA_API int alofa_head_gate(void* o, const float* g, int ldg, int g_off, int n_tokens, int heads, int vdim, int is_bf16, cudaStream_t stream) {
   const long long count = (long long)n_tokens * heads * vdim;
   if (count <= 0) return ALOFA_OK;
+  if (vdim == 1 && heads % 4 == 0 && ldg % 4 == 0 && g_off % 4 == 0 && !((uintptr_t)g & 15)) {
+    const long long quads = count / 4;
+    if (is_bf16) launch_dep(channel_gate_kernel<bf16>, (unsigned)((quads + 255) / 256), 256, 0, stream, (bf16*)o, g + g_off, ldg, heads / 4, quads);
+    else launch_dep(channel_gate_kernel<float>, (unsigned)((quads + 255) / 256), 256, 0, stream, (float*)o, g + g_off, ldg, heads / 4, quads);
+    return launch_status();
+  }
   if (is_bf16) launch_dep(head_gate_kernel<bf16>, (unsigned)((count + 255) / 256), 256, 0, stream, (bf16*)o, g, ldg, g_off, heads, vdim, count);
   else launch_dep(head_gate_kernel<float>, (unsigned)((count + 255) / 256), 256, 0, stream, (float*)o, g, ldg, g_off, heads, vdim, count);
   return launch_status();

@@ -99,6 +99,47 @@ ALOFA_API int alofa_latent_prepare(void* cq, void* cache, const float* lat, cons
 }
 
 // ---------------------------------------------------------------------------
+// The cached rows of a step whose requests all start in it, brought together: request after request, each on a page border
+// (page rows to a page, as many as the request needs), what its last page has left over zero; and the block table that finds
+// them there.  What is made of such rows row by row is then a paged cache of its own.  One block per token.
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) latent_gather_kernel(T* __restrict__ out, int* __restrict__ table, const T* __restrict__ cache, const int* __restrict__ q_start,
+                                                            const int* __restrict__ seq_of_token, const int* __restrict__ slot_map, int width, int page, int max_blocks,
+                                                            int rows) {
+  __shared__ int first_page;
+  pdl_begin();
+  const int t = blockIdx.x, s = seq_of_token[t];
+  if (threadIdx.x < 32) {
+    int pages = 0;
+    for (int i = threadIdx.x; i < s; i += 32) pages += (q_start[i + 1] - q_start[i] + page - 1) / page;
+    pages = __reduce_add_sync(0xffffffffu, pages);
+    if (threadIdx.x == 0) first_page = pages;
+  }
+  __syncthreads();
+  const int n = q_start[s + 1] - q_start[s], p = t - q_start[s], row = first_page * page + p;
+  if (row >= rows) return;
+  if (threadIdx.x == 0 && p % page == 0 && p / page < max_blocks) table[(size_t)s * max_blocks + p / page] = first_page + p / page;
+  const int slot = slot_map[t];
+  for (int c = threadIdx.x; c < width; c += blockDim.x) out[(size_t)row * width + c] = slot >= 0 ? cache[(size_t)slot * width + c] : from_f<T>(0.f);
+  if (p != n - 1) return;
+  const int end = min(rows, (first_page + (n + page - 1) / page) * page);
+  for (int r = row + 1; r < end; ++r)
+    for (int c = threadIdx.x; c < width; c += blockDim.x) out[(size_t)r * width + c] = from_f<T>(0.f);
+}
+
+ALOFA_API int alofa_latent_gather(void* out, int* table, const void* cache, const int* q_start, const int* seq_of_token, const int* slot_map, int n_tokens, int width,
+                                  int page, int max_blocks, int rows, int is_bf16, cudaStream_t stream) {
+  if (n_tokens <= 0) return ALOFA_OK;
+  if (width <= 0 || page <= 0 || max_blocks <= 0 || rows <= 0) return ALOFA_ERR_ARGUMENT;
+  if (is_bf16)
+    launch_dep(latent_gather_kernel<bf16>, n_tokens, 128, 0, stream, (bf16*)out, table, (const bf16*)cache, q_start, seq_of_token, slot_map, width, page, max_blocks, rows);
+  else
+    launch_dep(latent_gather_kernel<float>, n_tokens, 128, 0, stream, (float*)out, table, (const float*)cache, q_start, seq_of_token, slot_map, width, page, max_blocks, rows);
+  return launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // The rotated part of the queries: q [T, H, dim + rot] -> qa [T, H, kv_rank + rot]
 // at columns kv_rank.. (the first kv_rank columns are the absorbed unrotated
 // part, written by the batched product).  One block per token.
@@ -619,43 +660,65 @@ ALOFA_API int alofa_concat_rows(void* out, const float* a, const float* b, int r
 // `top` largest are chosen (ties: the lower index), their scores are the
 // weights, optionally divided by their sum.  One warp per token.
 // ---------------------------------------------------------------------------
-__global__ void moe_route_kernel(int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate, const float* __restrict__ z, int T,
-                                 int E, int top, int cols, int softmax, int renormalize) {
-  extern __shared__ float sc[];  // [warps][E]
-  pdl_begin();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
-  if (t >= T) return;
-  float* s = sc + warp * E;
-  const float* zr = z + (size_t)t * cols;
+__device__ __forceinline__ void choose_experts(int* __restrict__ choice, float* __restrict__ weight, float* s, float* gs, int lane, int t, int E, int top, int softmax,
+                                               int renormalize, const float* __restrict__ correction, float renorm_eps, int groups, int keep, float route_scale,
+                                               int group_best) {
   if (softmax) {
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s[e]);
     mx = warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) {
-      s[e] = expf(zr[e] - mx);
+      s[e] = expf(s[e] - mx);
       sum += s[e];
     }
     sum = warp_sum(sum);
     for (int e = lane; e < E; e += 32) s[e] /= sum;
   } else {
-    for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
+    for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
   }
   __syncwarp();
+  if (groups > 1) {
+    // experts form `groups` equal groups of neighbours; a group's score is the sum of its two largest choice
+    // scores (score + correction), or (group_best) the largest alone; only experts of the `keep` best groups can be chosen (ties: the lower group)
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;  // the largest and the second
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = correction ? s[e] + correction[e] : s[e];
+        if (v > a) b = a, a = v;
+        else if (v > b) b = v;
+      }
+      gs[g] = per > 1 && !group_best ? a + b : a;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      const float mine = gs[g];
+      int ahead = 0;
+      for (int o = 0; o < groups; ++o) ahead += (gs[o] > mine || (gs[o] == mine && o < g)) ? 1 : 0;
+      if (ahead >= keep)
+        for (int e = g * per; e < (g + 1) * per; ++e) s[e] = -INFINITY;  // never the largest: score + correction stays -inf
+    }
+    __syncwarp();
+  }
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
+    // the choice goes by score + correction (when given), the weight is the score itself
     float best = -INFINITY;
     int arg = 0x7fffffff;
-    for (int e = lane; e < E; e += 32)
-      if (s[e] > best) best = s[e], arg = e;  // ascending e: the first of equals
+    for (int e = lane; e < E; e += 32) {
+      const float v = correction ? s[e] + correction[e] : s[e];
+      if (v > best) best = v, arg = e;
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
       const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
       if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa;
     }
-    if (arg >= E) arg = k, best = 0.f;  // scores that are no numbers: some expert, weight zero
+    if (arg >= E) arg = k, best = 0.f;
+    else if (correction) best = s[arg];
+    __syncwarp();
     if (lane == 0) {
       choice[(size_t)t * top + k] = arg;
       weight[(size_t)t * top + k] = best;
@@ -664,7 +727,24 @@ __global__ void moe_route_kernel(int* __restrict__ choice, float* __restrict__ w
     total += best;
     __syncwarp();
   }
-  if (renormalize && lane < top) weight[(size_t)t * top + lane] /= total;
+  if (renormalize && lane < top) weight[(size_t)t * top + lane] = weight[(size_t)t * top + lane] / (total + renorm_eps) * route_scale;
+  else if (route_scale != 1.0f && lane < top) weight[(size_t)t * top + lane] *= route_scale;
+}
+
+// The choice from logits in memory (cols of them a row, fp32), a warp per token.
+__global__ void __launch_bounds__(256) moe_route_kernel(int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate, const float* __restrict__ z, int T,
+                                                        int E, int top, int cols, int softmax, int renormalize, const float* __restrict__ correction, float renorm_eps,
+                                                        int groups, int keep, float route_scale, int group_best) {
+  extern __shared__ float sc[];  // [8][E + groups]
+  pdl_begin();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 8 + warp;
+  if (t >= T) return;
+  float* s = sc + warp * (E + groups);
+  const float* zr = z + (size_t)t * cols;
+  for (int e = lane; e < E; e += 32) s[e] = zr[e];
+  __syncwarp();
+  choose_experts(choice, weight, s, s + E, lane, t, E, top, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best);
   if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-zr[E]));
 }
 
@@ -770,73 +850,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(int* __restrict__ choic
     const int t = t0 + r;
     float* s = z + r * cols;
     const float zg = gated ? s[E] : 0.f;
-    if (softmax) {
-      float mx = -INFINITY;
-      for (int e = lane; e < E; e += 32) mx = fmaxf(mx, s[e]);
-      mx = warp_max(mx);
-      float sum = 0.f;
-      for (int e = lane; e < E; e += 32) {
-        s[e] = expf(s[e] - mx);
-        sum += s[e];
-      }
-      sum = warp_sum(sum);
-      for (int e = lane; e < E; e += 32) s[e] /= sum;
-    } else {
-      for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
-    }
-    __syncwarp();
-    if (groups > 1) {
-      // experts form `groups` equal groups of neighbours; a group's score is the sum of its two largest choice
-      // scores (score + correction), or (group_best) the largest alone; only experts of the `keep` best groups can be chosen (ties: the lower group)
-      const int per = E / groups;
-      float* gs = gsc + r * groups;
-      for (int g = lane; g < groups; g += 32) {
-        float a = -INFINITY, b = -INFINITY;  // the largest and the second
-        for (int e = g * per; e < (g + 1) * per; ++e) {
-          const float v = correction ? s[e] + correction[e] : s[e];
-          if (v > a) b = a, a = v;
-          else if (v > b) b = v;
-        }
-        gs[g] = per > 1 && !group_best ? a + b : a;
-      }
-      __syncwarp();
-      for (int g = lane; g < groups; g += 32) {
-        const float mine = gs[g];
-        int ahead = 0;
-        for (int o = 0; o < groups; ++o) ahead += (gs[o] > mine || (gs[o] == mine && o < g)) ? 1 : 0;
-        if (ahead >= keep)
-          for (int e = g * per; e < (g + 1) * per; ++e) s[e] = -INFINITY;  // never the largest: score + correction stays -inf
-      }
-      __syncwarp();
-    }
-    float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-      // the choice goes by score + correction (when given), the weight is the score itself
-      float best = -INFINITY;
-      int arg = 0x7fffffff;
-      for (int e = lane; e < E; e += 32) {
-        const float v = correction ? s[e] + correction[e] : s[e];
-        if (v > best) best = v, arg = e;
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-        if (ob > best || (ob == best && oa < arg)) best = ob, arg = oa;
-      }
-      if (arg >= E) arg = k, best = 0.f;
-      else if (correction) best = s[arg];
-      __syncwarp();
-      if (lane == 0) {
-        choice[(size_t)t * top + k] = arg;
-        weight[(size_t)t * top + k] = best;
-        s[arg] = -INFINITY;
-      }
-      total += best;
-      __syncwarp();
-    }
-    if (renormalize && lane < top) weight[(size_t)t * top + lane] = weight[(size_t)t * top + lane] / (total + renorm_eps) * route_scale;
-    else if (route_scale != 1.0f && lane < top) weight[(size_t)t * top + lane] *= route_scale;
+    choose_experts(choice, weight, s, gsc + r * groups, lane, t, E, top, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best);
     if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-zg));
   }
 }
@@ -873,17 +887,21 @@ ALOFA_API int alofa_moe_router(int* choice, float* weight, float* gate, const vo
   return !x_bf16  ? moe_router_launch<float, float, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream) \
          : w_bf16 ? moe_router_launch<bf16, bf16, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream) \
                   : moe_router_launch<bf16, float, TT>(choice, weight, gate, x, wr, T, E, top, hidden, softmax, renormalize, correction, renorm_eps, groups, keep, route_scale, group_best, stream)
-  if (8 * row + 16 <= room) ROUTER_CASE(8);
+  if (8 * row + 16 <= room && T > 64) ROUTER_CASE(8);  // few tokens: two to a cluster, so that more of them work side by side
   if (2 * row + 16 <= room) ROUTER_CASE(2);
 #undef ROUTER_CASE
   return ALOFA_ERR_ARGUMENT;
 }
 
+// z: [T, cols] logits, cols at least E (and one more with a gate).  The rest as in alofa_moe_router.
 ALOFA_API int alofa_moe_route(int* choice, float* weight, float* gate, const float* z, int T, int E, int top, int cols, int softmax, int renormalize,
-                              cudaStream_t stream) {
+                              const float* correction, float renorm_eps, int groups, int keep, float route_scale, int group_best, cudaStream_t stream) {
   if (T <= 0) return ALOFA_OK;
-  if (E <= 0 || top <= 0 || top > E || top > 32 || cols < E + (gate ? 1 : 0) || (size_t)8 * E * 4 > 48 * 1024) return ALOFA_ERR_ARGUMENT;
-  launch_dep(moe_route_kernel, (T + 7) / 8, 256, (size_t)8 * E * sizeof(float), stream, choice, weight, gate, z, T, E, top, cols, softmax, renormalize);
+  if (groups < 1) groups = 1;
+  if (E <= 0 || top <= 0 || top > E || top > 32 || cols < E + (gate ? 1 : 0) || (size_t)8 * (E + groups) * 4 > 48 * 1024) return ALOFA_ERR_ARGUMENT;
+  if (groups > 1 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top)) return ALOFA_ERR_ARGUMENT;
+  launch_dep(moe_route_kernel, (T + 7) / 8, 256, (size_t)8 * (E + groups) * sizeof(float), stream, choice, weight, gate, z, T, E, top, cols, softmax, renormalize, correction,
+             renorm_eps, groups, keep, route_scale, group_best);
   return launch_status();
 }
 
@@ -932,25 +950,36 @@ __global__ void __launch_bounds__(THREADS) moe_sort_counted_kernel(int* __restri
                                                                    int pairs, int E, int tile, int max_tiles) {
   extern __shared__ __align__(16) uint8_t sort_smem[];
   int* first = reinterpret_cast<int*>(sort_smem);                    // [E] counts, then first rows
-  C* counted = reinterpret_cast<C*>(first + E);                     // [E][THREADS] counts, then offsets
+  C* counted = reinterpret_cast<C*>(first + ((E + 3) & ~3));        // [E][THREADS] counts, then offsets; rows on 16-byte boundaries
   pdl_begin();
   constexpr int SHARE = THREADS / 32;  // threads a lane sums
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int share = (pairs + THREADS - 1) / THREADS;
   const int lo = min(pairs, tid * share), hi = min(pairs, lo + share);
+  constexpr int HELD = 16;  // choices a thread keeps in registers: their loads are all in flight at once
+  int held[HELD];
+#pragma unroll
+  for (int j = 0; j < HELD; ++j) held[j] = lo + j < hi ? choice[lo + j] : E;
   for (int e = 0; e < E; ++e) counted[e * THREADS + tid] = 0;
-  for (int i = lo; i < hi; ++i)
+#pragma unroll
+  for (int j = 0; j < HELD; ++j)
+    if (held[j] < E) counted[held[j] * THREADS + tid] += 1;
+  for (int i = lo + HELD; i < hi; ++i)
     if (choice[i] < E) counted[choice[i] * THREADS + tid] += 1;
   __syncthreads();
   // an exclusive sum over the threads, per expert: a warp takes experts in turn, a lane SHARE threads' counts
   for (int e = warp; e < E; e += THREADS / 32) {
-    C* row = counted + e * THREADS + lane * SHARE;
-    int v[SHARE], sum = 0;
+    constexpr int PIECES = SHARE * (int)sizeof(C) / 16;  // 16 bytes at a time: element by element the lanes meet in two banks
+    uint4* row = reinterpret_cast<uint4*>(counted + e * THREADS + lane * SHARE);
+    union {
+      uint4 piece[PIECES];
+      C v[SHARE];
+    } held;
+    int sum = 0;
 #pragma unroll
-    for (int j = 0; j < SHARE; ++j) {
-      v[j] = row[j];
-      sum += v[j];
-    }
+    for (int j = 0; j < PIECES; ++j) held.piece[j] = row[j];
+#pragma unroll
+    for (int j = 0; j < SHARE; ++j) sum += held.v[j];
     int incl = sum;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -960,9 +989,12 @@ __global__ void __launch_bounds__(THREADS) moe_sort_counted_kernel(int* __restri
     int at = incl - sum;
 #pragma unroll
     for (int j = 0; j < SHARE; ++j) {
-      row[j] = (C)at;
-      at += v[j];
+      const int n = held.v[j];
+      held.v[j] = (C)at;
+      at += n;
     }
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j) row[j] = held.piece[j];
     if (lane == 31) first[e] = incl;  // the expert's count, for now
   }
   __syncthreads();
@@ -984,15 +1016,18 @@ __global__ void __launch_bounds__(THREADS) moe_sort_counted_kernel(int* __restri
     for (int i = at + lane; i < max_tiles; i += 32) tile_expert[i] = -1;
   }
   __syncthreads();
-  for (int i = lo; i < hi; ++i) {
-    const int e = choice[i];
+  auto place = [&](int i, int e) {
     dest[i] = e < E ? first[e] + counted[e * THREADS + tid]++ : -1;  // no row for a choice that is no expert with weights
-  }
+  };
+#pragma unroll
+  for (int j = 0; j < HELD; ++j)
+    if (lo + j < hi) place(lo + j, held[j]);
+  for (int i = lo + HELD; i < hi; ++i) place(i, choice[i]);
 }
 
 template <int THREADS, typename C>
 static int moe_sort_counted_launch(int* dest, int* tile_expert, const int* choice, int pairs, int E, int tile, int max_tiles, cudaStream_t stream) {
-  const size_t smem = (size_t)E * (THREADS * sizeof(C) + sizeof(int));
+  const size_t smem = (size_t)E * (THREADS * sizeof(C) + sizeof(int)) + 16;
   static size_t set = 0;
   if (smem > set) {
     if (cudaFuncSetAttribute(moe_sort_counted_kernel<THREADS, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return ALOFA_ERR_LAUNCH;

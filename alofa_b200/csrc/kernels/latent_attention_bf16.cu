@@ -16,7 +16,9 @@
 // (exp2 of scores scaled by scale * log2 e), round the weights to bfloat16 -
 // one warp's 16 keys are exactly one A fragment of the second product -,
 // exchange fragments and sums, and each adds P V for its half of the columns
-// into fp32 accumulators in registers (KV_RANK / 4 per thread).  The sink enters as the initial state of a row:
+// into fp32 accumulators in registers (KV_RANK / 4 per thread).  Where a row group
+// is alone in its CTA (few heads, decode) four warps share it in the same way, each
+// with eight keys and a quarter of the columns.  The sink enters as the initial state of a row:
 // maximum = sink, sum = 1, nothing added to the output.
 //
 // Causal bound and window go by the row's own position; keys past the request's
@@ -41,12 +43,11 @@ constexpr int D = KV_RANK + ROT;
 constexpr int PITCH = D + 8;          // elements per row in shared memory: 16 bytes of padding keep ldmatrix off bank conflicts
 constexpr int BN = 32;                // keys per block
 // Two shapes of the CTA.  Wide: four row groups (64 rows), eight warps, three key blocks in flight: prompt
-// portions, and decode tokens of more than 16 heads.  Narrow: one row group (16 rows), two warps, two key
+// portions, and decode tokens of more than 16 heads.  Narrow: one row group (16 rows), two warps or four, two key
 // blocks in flight, two CTAs to an SM: decode tokens of up to 16 heads, whose rows would fill a quarter of
-// the wide tile while its other warps only fetched.
+// the wide tile while its other warps only fetched.  W warps share a row group: two, or four in the narrow shape.
 constexpr int MIN_CTAS_WIDE = KV_RANK <= 256 ? 2 : 1;  // the output accumulators are KV_RANK / 4 registers a thread
-constexpr int HALF = KV_RANK / 2;     // value columns per warp
-constexpr int NT = HALF / 8;          // n-tiles of the output per warp
+constexpr int NARROW_WARPS = KV_RANK % 64 == 0 ? 4 : 2;
 static_assert(KV_RANK % 32 == 0 && D % 16 == 0, "latent sizes this kernel takes");
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -64,29 +65,34 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src)); }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
-constexpr int XCHG_BYTES = 2 * 16 * 4 + 2 * 16 * 4 + 2 * 32 * 16;  // per row group
-// the two warps of row group `rg` meet (named barriers 1..4; barrier 0 is the block's)
-__device__ __forceinline__ void pair_sync(int rg) { asm volatile("bar.sync %0, 64;" ::"r"(rg + 1) : "memory"); }
+constexpr int xchg_bytes(int w) { return 2 * w * 16 * 4 + 1024; }  // per row group
+// the W warps of row group `rg` meet (named barriers 1..4; barrier 0 is the block's)
+template <int W>
+__device__ __forceinline__ void group_sync(int rg) { asm volatile("bar.sync %0, %1;" ::"r"(rg + 1), "n"(32 * W) : "memory"); }
 __device__ __forceinline__ uint32_t pack2(float a, float b) {
   __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
-template <int GROUPS, int STAGES>
-__global__ void __launch_bounds__(GROUPS * 64, GROUPS == 1 ? 2 : MIN_CTAS_WIDE)
+template <int GROUPS, int STAGES, int W>
+__global__ void __launch_bounds__(GROUPS * W * 32, GROUPS == 1 ? 2 : MIN_CTAS_WIDE)
 latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa, const bf16* __restrict__ cache, const float* __restrict__ sink,
                              const int* __restrict__ q_start, const int* __restrict__ kv_len, const int* __restrict__ block_table, int max_blocks,
                              int page_size, int heads, int window, float scale_log2, float* __restrict__ part_o, float* __restrict__ part_ml,
                              int blocks_per_split, int total_rows) {
-  constexpr int BM = 16 * GROUPS, THREADS = 64 * GROUPS;
+  constexpr int BM = 16 * GROUPS, THREADS = 32 * W * GROUPS;
+  constexpr int COLS = KV_RANK / W;      // value columns per warp
+  constexpr int NT = COLS / 8;           // n-tiles of the output per warp
+  constexpr int KN = BN / W / 8;         // n-tiles of the scores per warp (8 keys each)
+  static_assert(KV_RANK % (16 * W) == 0, "whole pairs of n-tiles");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* Qs = reinterpret_cast<bf16*>(smem_raw);      // [BM][PITCH]
   bf16* Ks = Qs + BM * PITCH;                        // [STAGES][BN][PITCH]
-  // what the two warps of a row group hand one another per key block: maxima and sums of their 16 keys per row, their weight fragments
-  uint8_t* xchg = reinterpret_cast<uint8_t*>(Ks + (size_t)STAGES * BN * PITCH) + (size_t)((threadIdx.x >> 5) % GROUPS) * XCHG_BYTES;
-  float* x_max = reinterpret_cast<float*>(xchg);           // [2][16]
-  float* x_sum = x_max + 32;                                // [2][16]
-  uint4* x_frag = reinterpret_cast<uint4*>(x_sum + 32);     // [2][32]
+  // what the warps of a row group hand one another per key block: maxima and sums of their keys per row, their weight fragments
+  uint8_t* xchg = reinterpret_cast<uint8_t*>(Ks + (size_t)STAGES * BN * PITCH) + (size_t)((threadIdx.x >> 5) % GROUPS) * xchg_bytes(W);
+  float* x_max = reinterpret_cast<float*>(xchg);           // [W][16]
+  float* x_sum = x_max + 16 * W;                            // [W][16]
+  uint32_t* x_frag = reinterpret_cast<uint32_t*>(x_sum + 16 * W);  // [W][32][2 * KN]
   pdl_begin();
   const int seq = blockIdx.y, tile = blockIdx.x;
   const int t0 = q_start[seq], q_len = q_start[seq + 1] - t0;
@@ -174,29 +180,48 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
       __syncthreads();
       continue;
     }
-    // S = Q K^T for 16 rows x this warp's 16 keys of the block (the group's other warp takes the other 16)
-    float s[2][4];
+    // S = Q K^T for 16 rows x this warp's keys of the block (the group's other warps take the others)
+    float s[KN][4];
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
+    for (int j = 0; j < KN; ++j)
 #pragma unroll
       for (int k = 0; k < 4; ++k) s[j][k] = 0.f;
-    const uint32_t k_base = smem_addr(Kb + (ch * 16 + (lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 8);
+    if constexpr (KN == 2) {
+      const uint32_t k_base = smem_addr(Kb + (ch * 16 + (lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 8);
 #pragma unroll 4
-    for (int k0 = 0; k0 < D; k0 += 16) {
-      uint32_t a[4], kb[4];
-      ldsm4(a, q_base + k0 * 2);
-      ldsm4(kb, k_base + k0 * 2);
-      mma16816(s[0], a, kb[0], kb[1]);
-      mma16816(s[1], a, kb[2], kb[3]);
+      for (int k0 = 0; k0 < D; k0 += 16) {
+        uint32_t a[4], kb[4];
+        ldsm4(a, q_base + k0 * 2);
+        ldsm4(kb, k_base + k0 * 2);
+        mma16816(s[0], a, kb[0], kb[1]);
+        mma16816(s[KN - 1], a, kb[2], kb[3]);
+      }
+    } else {  // eight keys, 32 of the depth at a time
+      const uint32_t k_base = smem_addr(Kb + (ch * 8 + (lane & 7)) * PITCH + (lane >> 3) * 8);
+#pragma unroll 4
+      for (int k0 = 0; k0 + 32 <= D; k0 += 32) {
+        uint32_t a[4], c[4], kb[4];
+        ldsm4(kb, k_base + k0 * 2);
+        ldsm4(a, q_base + k0 * 2);
+        ldsm4(c, q_base + (k0 + 16) * 2);
+        mma16816(s[0], a, kb[0], kb[1]);
+        mma16816(s[0], c, kb[2], kb[3]);
+      }
+      if constexpr (D % 32 != 0) {  // a last 16; the other half of what is read lies in the row's padding and beyond, and is not used
+        uint32_t a[4], kb[4];
+        ldsm4(kb, k_base + (D - 16) * 2);
+        ldsm4(a, q_base + (D - 16) * 2);
+        mma16816(s[0], a, kb[0], kb[1]);
+      }
     }
     // mask; the rows' maxima over the warp's keys, then over the group's (in units of log2)
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
+    for (int j = 0; j < KN; ++j)
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const int i = k >> 1;
-        const int key = b * BN + ch * 16 + j * 8 + 2 * t + (k & 1);
+        const int key = b * BN + ch * (BN / W) + j * 8 + 2 * t + (k & 1);
         const float v = (key <= pos[i] && key >= first[i]) ? s[j][k] * scale_log2 : -INFINITY;
         s[j][k] = v;
         mx[i] = fmaxf(mx[i], v);
@@ -207,17 +232,19 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
       if (t == 0) x_max[ch * 16 + g + 8 * i] = mx[i];
     }
-    pair_sync(rg);
+    group_sync<W>(rg);
     float corr[2], sum[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-      const float m_new = fmaxf(m[i], fmaxf(mx[i], x_max[(ch ^ 1) * 16 + g + 8 * i]));
+      float m_new = m[i];
+#pragma unroll
+      for (int o = 0; o < W; ++o) m_new = fmaxf(m_new, x_max[o * 16 + g + 8 * i]);
       const float m_use = m_new == -INFINITY ? 0.f : m_new;
       corr[i] = exp2f(m[i] - m_use);  // m = -inf: 0
       m[i] = m_new;
       sum[i] = 0.f;
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
+      for (int j = 0; j < KN; ++j) {
         s[j][2 * i] = exp2f(s[j][2 * i] - m_use);
         s[j][2 * i + 1] = exp2f(s[j][2 * i + 1] - m_use);
         sum[i] += s[j][2 * i] + s[j][2 * i + 1];
@@ -226,17 +253,20 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
       sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
       if (t == 0) x_sum[ch * 16 + g + 8 * i] = sum[i];
     }
-    // the weights of the warp's 16 keys, rounded, are one A fragment of the second product: both warps need both
-    uint4 mine;
-    mine.x = pack2(s[0][0], s[0][1]);
-    mine.y = pack2(s[0][2], s[0][3]);
-    mine.z = pack2(s[1][0], s[1][1]);
-    mine.w = pack2(s[1][2], s[1][3]);
-    x_frag[ch * 32 + lane] = mine;
-    pair_sync(rg);
-    const uint4 other = x_frag[(ch ^ 1) * 32 + lane];
+    // the weights of 16 keys, rounded, are one A fragment of the second product (of 8 keys, half of one): every warp needs all
 #pragma unroll
-    for (int i = 0; i < 2; ++i) l[i] = l[i] * corr[i] + (x_sum[g + 8 * i] + x_sum[16 + g + 8 * i]);  // keys 0-15 first, in both warps
+    for (int j = 0; j < KN; ++j) {
+      x_frag[((ch * KN + j) * 2) * 32 + lane] = pack2(s[j][0], s[j][1]);
+      x_frag[((ch * KN + j) * 2 + 1) * 32 + lane] = pack2(s[j][2], s[j][3]);
+    }
+    group_sync<W>(rg);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {  // the first keys' sum first, in every warp
+      float all = x_sum[g + 8 * i];
+#pragma unroll
+      for (int o = 1; o < W; ++o) all += x_sum[o * 16 + g + 8 * i];
+      l[i] = l[i] * corr[i] + all;
+    }
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       o[j][0] *= corr[0];
@@ -244,12 +274,13 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
       o[j][2] *= corr[1];
       o[j][3] *= corr[1];
     }
-    // O += P V over this warp's half of the value columns, all 32 keys
-    const uint32_t v_base = smem_addr(Kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + ch * HALF + (lane >> 4) * 8);
+    // O += P V over this warp's value columns, all 32 keys
+    const uint32_t v_base = smem_addr(Kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + ch * COLS + (lane >> 4) * 8);
 #pragma unroll
     for (int kk = 0; kk < 2; ++kk) {
-      const uint4 f = kk == ch ? mine : other;
-      const uint32_t p[4] = {f.x, f.y, f.z, f.w};
+      uint32_t p[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) p[i] = x_frag[(kk * 4 + i) * 32 + lane];
 #pragma unroll
       for (int j = 0; j < NT; j += 2) {
         uint32_t v[4];
@@ -268,13 +299,13 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
     const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
     if (split) {
       const size_t row = (size_t)blockIdx.z * total_rows + (size_t)t0 * heads + r;
-      float* dst = part_o + row * KV_RANK + ch * HALF + 2 * t;
+      float* dst = part_o + row * KV_RANK + ch * COLS + 2 * t;
 #pragma unroll
       for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[j][2 * i] * inv, o[j][2 * i + 1] * inv);
       if (ch == 0 && t == 0) *reinterpret_cast<float2*>(part_ml + row * 2) = make_float2(m[i], l[i]);
       continue;
     }
-    bf16* dst = out + ((size_t)t0 * heads + r) * KV_RANK + ch * HALF + 2 * t;
+    bf16* dst = out + ((size_t)t0 * heads + r) * KV_RANK + ch * COLS + 2 * t;
 #pragma unroll
     for (int j = 0; j < NT; ++j)
       *reinterpret_cast<uint32_t*>(dst + j * 8) = pack2(o[j][2 * i] * inv, o[j][2 * i + 1] * inv);
@@ -282,21 +313,31 @@ latent_attention_bf16_kernel(bf16* __restrict__ out, const bf16* __restrict__ qa
 }
 
 // out[row] = sum_z w_z o_z / sum_z w_z with w_z = l_z 2^(m_z - max m), splits in ascending order.
-__global__ void latent_attention_merge_kernel(bf16* __restrict__ out, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
-                                              int total_rows) {
+constexpr int MAX_SPLITS = 512;
+__global__ void __launch_bounds__(128) latent_attention_merge_kernel(bf16* __restrict__ out, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
+                                                                     int total_rows) {
+  __shared__ float2 ml[MAX_SPLITS];
+  __shared__ float weight[MAX_SPLITS];
   pdl_begin();
   const size_t row = blockIdx.x;
+  for (int z = threadIdx.x; z < splits; z += blockDim.x) ml[z] = *reinterpret_cast<const float2*>(part_ml + ((size_t)z * total_rows + row) * 2);
+  __syncthreads();
   float top = -INFINITY;
-  for (int z = 0; z < splits; ++z) top = fmaxf(top, part_ml[((size_t)z * total_rows + row) * 2]);
-  for (int c = threadIdx.x; c < KV_RANK; c += blockDim.x) {
-    float num = 0.f, den = 0.f;
+  for (int z = 0; z < splits; ++z) top = fmaxf(top, ml[z].x);
+  for (int z = threadIdx.x; z < splits; z += blockDim.x) weight[z] = ml[z].y > 0.f ? ml[z].y * exp2f(ml[z].x - top) : 0.f;
+  __syncthreads();
+  float den = 0.f;
+  for (int z = 0; z < splits; ++z) den += weight[z];
+  for (int c = threadIdx.x * 4; c < KV_RANK; c += blockDim.x * 4) {
+    float4 num = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
     for (int z = 0; z < splits; ++z) {
-      const float2 ml = *reinterpret_cast<const float2*>(part_ml + ((size_t)z * total_rows + row) * 2);
-      const float w = ml.y > 0.f ? ml.y * exp2f(ml.x - top) : 0.f;
-      num = fmaf(w, part_o[((size_t)z * total_rows + row) * KV_RANK + c], num);
-      den += w;
+      const float w = weight[z];
+      const float4 o = *reinterpret_cast<const float4*>(part_o + ((size_t)z * total_rows + row) * KV_RANK + c);
+      num.x = fmaf(w, o.x, num.x), num.y = fmaf(w, o.y, num.y), num.z = fmaf(w, o.z, num.z), num.w = fmaf(w, o.w, num.w);
     }
-    out[row * KV_RANK + c] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+    const bool any = den > 0.f;
+    *reinterpret_cast<uint2*>(out + row * KV_RANK + c) = make_uint2(pack2(any ? num.x / den : 0.f, any ? num.y / den : 0.f), pack2(any ? num.z / den : 0.f, any ? num.w / den : 0.f));
   }
 }
 
@@ -311,25 +352,25 @@ ALOFA_API int alofa_latent_attention_bf16(void* out, const void* qa, const void*
   if (n_seqs <= 0 || max_q_len <= 0) return ALOFA_OK;
   if (heads <= 0 || page_size <= 0) return ALOFA_ERR_ARGUMENT;
   if (splits < 1) splits = 1;
-  if (splits > 1 && (!part_o || !part_ml || blocks_per_split <= 0 || total_rows <= 0 || splits > 65535)) return ALOFA_ERR_ARGUMENT;
+  if (splits > 1 && (!part_o || !part_ml || blocks_per_split <= 0 || total_rows <= 0 || splits > MAX_SPLITS)) return ALOFA_ERR_ARGUMENT;
   const bool narrow = (long long)max_q_len * heads <= 16;
   const int bm = narrow ? 16 : 64, stages = narrow ? 2 : 3;
-  const size_t smem = (size_t)(bm + stages * BN) * PITCH * sizeof(bf16) + (size_t)(narrow ? 1 : 4) * XCHG_BYTES;
+  const size_t smem = (size_t)(bm + stages * BN) * PITCH * sizeof(bf16) + (size_t)(narrow ? xchg_bytes(NARROW_WARPS) : 4 * xchg_bytes(2));
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(latent_attention_bf16_kernel<4, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)((64 + 3 * BN) * PITCH * sizeof(bf16) + 4 * XCHG_BYTES)) != cudaSuccess ||
-        cudaFuncSetAttribute(latent_attention_bf16_kernel<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)((16 + 2 * BN) * PITCH * sizeof(bf16) + XCHG_BYTES)) != cudaSuccess)
+    if (cudaFuncSetAttribute(latent_attention_bf16_kernel<4, 3, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)((64 + 3 * BN) * PITCH * sizeof(bf16) + 4 * xchg_bytes(2))) != cudaSuccess ||
+        cudaFuncSetAttribute(latent_attention_bf16_kernel<1, 2, NARROW_WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)((16 + 2 * BN) * PITCH * sizeof(bf16) + xchg_bytes(NARROW_WARPS))) != cudaSuccess)
       return ALOFA_ERR_LAUNCH;
     set = true;
   }
   const long long tiles = ((long long)max_q_len * heads + bm - 1) / bm;
   if (tiles > 2147483647LL || n_seqs > 65535) return ALOFA_ERR_ARGUMENT;
   if (narrow)
-    launch_dep(latent_attention_bf16_kernel<1, 2>, dim3((unsigned)tiles, n_seqs, splits), dim3(64), smem, stream, (bf16*)out, (const bf16*)qa, (const bf16*)cache,
+    launch_dep(latent_attention_bf16_kernel<1, 2, NARROW_WARPS>, dim3((unsigned)tiles, n_seqs, splits), dim3(32 * NARROW_WARPS), smem, stream, (bf16*)out, (const bf16*)qa, (const bf16*)cache,
                sink, q_start, kv_len, block_table, max_blocks, page_size, heads, window, scale * 1.4426950408889634f, part_o, part_ml, blocks_per_split,
                total_rows);
   else
-    launch_dep(latent_attention_bf16_kernel<4, 3>, dim3((unsigned)tiles, n_seqs, splits), dim3(256), smem, stream, (bf16*)out, (const bf16*)qa, (const bf16*)cache,
+    launch_dep(latent_attention_bf16_kernel<4, 3, 2>, dim3((unsigned)tiles, n_seqs, splits), dim3(256), smem, stream, (bf16*)out, (const bf16*)qa, (const bf16*)cache,
                sink, q_start, kv_len, block_table, max_blocks, page_size, heads, window, scale * 1.4426950408889634f, part_o, part_ml, blocks_per_split,
                total_rows);
   if (splits > 1) launch_dep(latent_attention_merge_kernel, dim3(total_rows), dim3(128), 0, stream, (bf16*)out, part_o, part_ml, splits, total_rows);
@@ -339,5 +380,5 @@ ALOFA_API int alofa_latent_attention_bf16(void* out, const void* qa, const void*
 ALOFA_API int alofa_latent_attention_bf16_sizes(int* kv_rank, int* rot) {
   *kv_rank = KV_RANK;
   *rot = ROT;
-  return (int)((64 + 3 * BN) * PITCH * sizeof(bf16) + 4 * XCHG_BYTES);
+  return (int)((64 + 3 * BN) * PITCH * sizeof(bf16) + 4 * xchg_bytes(2));
 }

@@ -611,6 +611,7 @@ def _latent():
         lib = load_library("alofa_latent", ["kernels/latent.cu", "kernels/gemm_batched_bf16.cu"])
         sigs = {
             "alofa_latent_prepare": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P],
+            "alofa_latent_gather": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
             "alofa_latent_query_turn": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
             "alofa_rotary_interleaved": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
             "alofa_gemm_batched": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _L, _L, _L, _I, _I, _P, _L, _L, _I, _I, _I, _P],
@@ -619,7 +620,7 @@ def _latent():
             "alofa_latent_attention": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
             "alofa_sandwich_norm": [_P, _P, _P, _F, _P, _P, _F, _I, _I, _I, _I, _L, _P, _P],
             "alofa_concat_rows": [_P, _P, _P, _I, _I, _I, _P],
-            "alofa_moe_route": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+            "alofa_moe_route": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _I, _P],
             "alofa_moe_router": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _F, _I, _I, _F, _I, _P],
             "alofa_cast_rows": [_P, _P, _L, _I, _P],
             "alofa_moe_sort": [_P, _P, _P, _I, _I, _I, _I, _P],
@@ -662,6 +663,23 @@ def latent_prepare(cq, cache_rows, lat, wq, wkv, freq, positions, slot_map, q_ra
             1 if halves else 0, float(mag), 1 if dt == torch.bfloat16 else 0, _stream(),
         ),
         "latent_prepare",
+    )
+
+
+def latent_gather(out, table, cache_rows, q_start, seq_of_token, slot_map, page: int) -> None:
+    """The cached rows of a step whose requests all start in it, request after
+    request from ``out``'s first row on, each on a border of ``page`` rows (the
+    rest of its last page zero), and in ``table`` [requests, blocks] (int32)
+    the pages they take.  Rows of ``out`` that no page covers stay as they are."""
+    i32 = torch.int32
+    n = slot_map.shape[0]
+    if out.shape[1] != cache_rows.shape[1] or table.shape[0] != q_start.shape[0] - 1 or table.shape[1] * page < n - table.shape[0] + 1 or out.shape[0] < n:
+        raise AlofaError("invalid_argument", "latent_gather sizes disagree", f"out={tuple(out.shape)} cache={tuple(cache_rows.shape)} table={tuple(table.shape)} tokens={n}")
+    _done(
+        _latent().alofa_latent_gather(_dev(out, "out", cache_rows.dtype), _dev(table, "table", i32), _dev(cache_rows, "cache"), _dev(q_start, "q_start", i32),
+                                      _dev(seq_of_token, "seq_of_token", i32), _dev(slot_map, "slot_map", i32), n, out.shape[1], int(page), table.shape[1], out.shape[0],
+                                      _is_bf16(out, "out"), _stream()),
+        "latent_gather", f"tokens={n} requests={table.shape[0]}",
     )
 
 
@@ -842,14 +860,18 @@ def gemm_by_tile_gated(out, x, w, tile_batch, tile_rows: int, gate=SILU_GATE) ->
     return gemm_tc(out, x, w.view(batches * n2, k), None, EPI_GATED, -256, tile_batch=tile_batch, batches=batches, gate=gate)
 
 
-def moe_route(choice, weight, gate, z, experts: int, top: int, softmax: bool = False, renormalize: bool = False) -> None:
+def moe_route(choice, weight, gate, z, experts: int, top: int, softmax: bool = False, renormalize: bool = False, correction=None, renorm_eps: float = 0.0, groups: int = 1,
+              keep: int = 1, route_scale: float = 1.0, group_best: bool = False) -> None:
     """From router logits z [T, experts (+1)] fp32: the ``top`` experts of each
     token by score (sigmoid, or softmax over the experts), their scores as
-    weights, and ``gate`` = sigmoid of the last column when given."""
+    weights, and ``gate`` = sigmoid of the last column when given.  The rest as
+    in :func:`moe_router`."""
     i32, f32 = torch.int32, torch.float32
     _done(
         _latent().alofa_moe_route(_dev(choice, "choice", i32), _dev(weight, "weight", f32), _dev(gate, "gate", f32) if gate is not None else None, _dev(z, "z", f32),
-                                  z.shape[0], experts, top, z.shape[1], 1 if softmax else 0, 1 if renormalize else 0, _stream()),
+                                  z.shape[0], experts, top, z.shape[1], 1 if softmax else 0, 1 if renormalize else 0,
+                                  _dev(correction, "correction", f32) if correction is not None else None, float(renorm_eps), int(groups), int(keep), float(route_scale),
+                                  1 if group_best else 0, _stream()),
         "moe_route", f"experts={experts} top={top}",
     )
 

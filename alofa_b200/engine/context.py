@@ -129,6 +129,7 @@ class StepContext:
         self.streams_owed = None
         # (h, rows, layer): the stream's rows in the compute dtype as the kernel that last added to the stream left them, and the
         # number of the layer that did; a block whose first sublayer reads the stream itself takes them if it is the very next layer
+        self.fresh = False  # every request of the step starts in it (set by the step runner)
         self.next_norm = None  # the norm the block after this one starts with, for a block whose last kernel can make its rows
         self.stream_rows = None
         self.layer_no = 0

@@ -105,7 +105,7 @@ class StepRunner:
             self._stream_acc = torch.zeros((2, self.STREAM_TOKENS, model.spec.hidden_size), dtype=torch.int64, device=self.rt.device)
         self._layouts = {}
         self.cuda_graphs = cuda_graphs and on_gpu and model.graph_safe()
-        self._graphs = {}  # decode steps by batch size; steps with prompt portions by (tokens, requests, wanted rows)
+        self._graphs = {}  # decode steps by batch size; steps with prompt portions by (tokens, requests, wanted rows), and apart for those whose requests all start in them where a mixer tells them apart
         self.prompt_graphs = self.cuda_graphs and os.environ.get("ALOFA_PROMPT_GRAPHS", "1") != "0"
         self.max_prompt_graphs = 4
         self._seen_shapes = {}
@@ -158,8 +158,10 @@ class StepRunner:
             tokens = np.concatenate([np.asarray(e.tokens, dtype=np.int64) for e in entries])
         if tokens.min() < 0 or tokens.max() >= self.model.spec.vocab_size:
             raise AlofaError("out_of_range", "token id outside the vocabulary", f"vocab={self.model.spec.vocab_size}")
+        lengths_fresh = True
         for e, n in zip(entries, counts):
             have = self.manager.computed_len(e.slot)
+            lengths_fresh = lengths_fresh and have == 0
             if have + n > self.max_tokens:
                 raise AlofaError("out_of_range", "history would outgrow the context window", f"slot={e.slot} have={have} add={n} max_tokens={self.max_tokens}")
         if n_out == n_seqs and n_tokens == n_seqs:
@@ -205,6 +207,7 @@ class StepRunner:
         ctx.stream_acc = self._stream_acc
         ctx.max_q_len, ctx.max_kv_len = max_q, max_kv
         ctx.decode_only = max_q == 1
+        ctx.fresh = self.model.tells_fresh and not ctx.decode_only and lengths_fresh
         ctx.max_context = self.max_tokens
         ctx.slots, ctx.counts = slots, counts
         ctx.any_hot = any(e.temperature > 0.0 for e in entries)
@@ -239,7 +242,7 @@ class StepRunner:
             # A step with prompt portions is some two hundred launches, about as long to issue from
             # Python as to run: a shape (tokens, requests, wanted rows) met a third time is recorded
             # and replayed from then on.  A few shapes are kept, the least recently used one goes.
-            key = (ctx.n_tokens, ctx.n_seqs, ctx.n_out)
+            key = (ctx.n_tokens, ctx.n_seqs, ctx.n_out) + (("fresh",) if ctx.fresh else ())
             g = self._graphs.pop(key, None)
             if g is None:
                 seen = self._seen_shapes.get(key, 0)
@@ -247,7 +250,7 @@ class StepRunner:
                     self._seen_shapes.clear()
                 self._seen_shapes[key] = seen + 1
                 if seen >= 2:
-                    kept = [k for k in self._graphs if len(k) == 3 and k[2] != "decode"]
+                    kept = [k for k in self._graphs if k[2] != "decode"]
                     if len(kept) >= self.max_prompt_graphs:
                         del self._graphs[kept[0]]
                     logits, tokens = self._capture(ctx, key, sample)

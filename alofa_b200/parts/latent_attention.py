@@ -16,6 +16,12 @@ first kv_rank numbers also serve as the value; ``Wuv_h`` is applied to the
 attention output of the head.  Both per-head products are one batched launch.
 The stacked ``[Wdq; Wdkv]`` makes both down-projections one product.
 
+A step of prompts alone (every request starts in it; no rotated part, bfloat16,
+head sizes the tensor-core attention takes) goes the other way round: the
+step's cached rows are brought together, keys and values of all heads made from
+them by two products, and ordinary causal attention runs over those; per (query,
+key) pair that is ``dim + vdim`` numbers a head instead of ``2 kv_rank``.
+
 Options: ``q_rank`` 0 or absent: no query latent, ``q = x Wq^T`` (tensor
 ``q``) and the down-projection is ``Wdkv`` alone; ``gate``: head h's output is
 multiplied by ``sigmoid(x Wg^T)_h`` (tensor ``g`` [heads, hidden], stacked
@@ -33,8 +39,24 @@ import torch
 from ..csrc import ops
 from ..errors import AlofaError
 from . import fast_linear
+from .attention import PagedAttend
 from .base import PagedRows, Part, TensorSpec, as_float32_vector, build_part, register_part
 from .linear import STORE, Linear
+
+
+UNFOLD_TOKENS = 128  # tokens a request from which on (on average) keys and values made from a step's latents pay
+UNFOLD_PAGE = 64  # rows to a page of those keys and values: whole key blocks of the attention kernels
+
+
+class UnfoldedHeads(PagedAttend):
+    """Ordinary attention over keys and values made from a step's own latents: they are a paged cache of their own."""
+
+    page_size = UNFOLD_PAGE
+
+    def __init__(self, mixer, k, v, block_table):
+        self.nh = self.nkv = mixer.heads
+        self.hd, self.vd, self.scale, self.window, self.sink = mixer.dim, mixer.vdim, mixer.scale, mixer.window, mixer.sink
+        self.k, self.v, self.block_table = k, v, block_table
 
 
 class LatentAttention(Part):
@@ -79,6 +101,8 @@ class LatentAttention(Part):
         if self.rot_dims > self.rot:
             raise AlofaError("invalid_argument", "more rotated dimensions than the rotated part has", f"dims={self.rot_dims} rot_dim={self.rot}")
         self.width = self.kv_rank + self.rot  # a cache row
+        # steps of prompts alone take another way through the layer (ctx.fresh)
+        self.tells_fresh = (rt.dtype == torch.bfloat16 and not self.rot and self.dim > 0 and self.scale > 0 and ops.attention_bf16_supported(self.dim, self.vdim))
         # columns of the stacked down-projection: [query latent | latent and rotated part | gate]
         self.gate_at = self.q_rank + (self.width if self.own_latent else 0)
         self.down = self.up_q = self.out = self.uk_t = self.uv = self.sink = self.kv_norm = None
@@ -88,7 +112,8 @@ class LatentAttention(Part):
 
     def scratch_row_bytes(self) -> int:
         h = self.heads
-        return 4 * (self.q_rank + self.width + self.gate_cols) + 4 * self.q_rank + 4 * h * (self.dim + self.rot) + 4 * h * self.width + 4 * h * self.kv_rank + 4 * h * self.vdim + 4 * self.hidden
+        unfolded = 2 * (self.kv_rank + h * (self.dim + self.vdim)) if self.tells_fresh else 0
+        return unfolded + 4 * (self.q_rank + self.width + self.gate_cols) + 4 * self.q_rank + 4 * h * (self.dim + self.rot) + 4 * h * self.width + 4 * h * self.kv_rank + 4 * h * self.vdim + 4 * self.hidden
 
     def tensors(self):
         pre, h = self.prefix, self.heads
@@ -123,6 +148,8 @@ class LatentAttention(Part):
         # [heads, kv_rank, dim]: row c of head h holds column c of Wuk_h, so the per-head product q_h -> Wuk_h^T q_h reads rows
         self.uk_t = state[pre + "uk"].view(h, self.dim, self.kv_rank).transpose(1, 2).contiguous() if self.dim else None
         self.uv = state[pre + "uv"].contiguous()
+        self.keys_up = Linear(state[pre + "uk"], None, STORE) if self.tells_fresh else None
+        self.values_up = Linear(self.uv, None, STORE) if self.tells_fresh else None
         self.out = Linear(state[pre + "o"], None, STORE)
         self.sink = as_float32_vector(state[pre + "sink"]) if self.has_sink else None
         if self.position is not None:
@@ -146,6 +173,35 @@ class LatentAttention(Part):
                                self.q_rank, self.kv_rank, self.rot, self.rot_dims, self.eps, self.halves, self.magnitude)
         q = ctx.buf((n, heads * (self.dim + self.rot)), dt)
         self.up_q(q, cq if self.q_rank else x, buf=ctx.buf)
+        if self.tells_fresh and ctx.fresh and n >= UNFOLD_TOKENS * ctx.n_seqs:
+            o = self.attend_unfolded(ctx, q, cache, group)
+            if self.gate_cols:
+                ops.head_gate(o, lat, self.gate_at, self.gate_cols, heads * self.vdim // self.gate_cols)
+        else:
+            o = self.attend_latent(ctx, q, cache, group, freq, lat)
+        if store:
+            return self.out(h, o, defer=defer, buf=ctx.buf)  # None, or the split sums a caller that asked for them adds up itself
+        y = ctx.buf(tuple(h.shape), torch.float32)
+        self.out(y, o, buf=ctx.buf)
+        h.add_(y)
+
+    def attend_unfolded(self, ctx, q, cache, group):
+        """Attention of a step whose requests all start in it, over keys and values made from its latents."""
+        n, dt, heads = q.shape[0], self.rt.dtype, self.heads
+        # by the step's shape alone: each request's rows end with a whole page
+        rows = UNFOLD_PAGE * ((n + ctx.n_seqs * (UNFOLD_PAGE - 1)) // UNFOLD_PAGE)
+        c = ctx.buf((rows, self.kv_rank), dt)
+        table = ctx.buf((ctx.n_seqs, -(-n // UNFOLD_PAGE)), torch.int32)
+        ops.latent_gather(c, table, cache.k, ctx.q_start, ctx.seq_of_token, group.slot_map, UNFOLD_PAGE)
+        k, v = ctx.buf((rows, heads, self.dim), dt), ctx.buf((rows, heads, self.vdim), dt)
+        self.keys_up(k.view(rows, -1), c, buf=ctx.buf)
+        self.values_up(v.view(rows, -1), c, buf=ctx.buf)
+        unfolded = UnfoldedHeads(self, k, v, table)
+        return unfolded.attend(ctx, q, unfolded, unfolded)
+
+    def attend_latent(self, ctx, q, cache, group, freq, lat):
+        """Attention over the cached rows themselves, the queries carried into the latent space."""
+        n, dt, heads = q.shape[0], self.rt.dtype, self.heads
         qa = ctx.buf((n, heads * self.width), dt)
         ops.latent_query_turn(qa, q, freq, ctx.positions, heads, self.dim, self.rot, self.rot_dims, self.kv_rank, self.halves, self.magnitude)
         if self.dim:
@@ -162,12 +218,7 @@ class LatentAttention(Part):
                          heads * self.vdim, self.vdim, gate=lat if self.gate_channels else None, gate_at=self.gate_at, gate_batch=self.vdim)
         if self.gate_cols and not self.gate_channels:
             ops.head_gate(o, lat, self.gate_at, heads, self.vdim)
-        if store:
-            return self.out(h, o, defer=defer, buf=ctx.buf)  # None, or the split sums a caller that asked for them adds up itself
-        else:
-            y = ctx.buf(tuple(h.shape), torch.float32)
-            self.out(y, o, buf=ctx.buf)
-            h.add_(y)
+        return o
 
     def attend(self, ctx, o_lat, qa, cache, group):
         """Attention of the step's rows over the cached latent rows: on tensor

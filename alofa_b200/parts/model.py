@@ -30,6 +30,8 @@ class Model:
         self.next_norms = [n if n is not None and n.spec.kind == "rmsnorm" else None for n in norms]
         # a block may read the embedding output of the step's tokens later on (ctx.embedding_output)
         self.keeps_embedding = any(getattr(block, "needs_embedding_output", False) for block in self.layers)
+        # whether a mixer goes another way in steps whose requests all start in them
+        self.tells_fresh = any(getattr(getattr(block, "mixer", None), "tells_fresh", False) for block in self.layers)
         # blocks that keep several copies of the residual stream say how many (ctx.streams); every block of a model says the same
         # mixers that mix their values with those of the first of them: the values of a step's tokens are kept for it (ctx.first_values)
         widths = {int(getattr(block, "shared_value_width", 0)) for block in self.layers} - {0}

@@ -38,6 +38,9 @@ from .feed_forward import DenseMLP, gate_form
 from .linear import STORE, Linear
 
 
+ROUTER_PRODUCT_TOKENS = 256  # tokens in a step from which on the router's logits are a tensor-core product and the choice a kernel of its own
+
+
 class RoutedExperts(Part):
     family = "feed_forward"
     graph_safe = True
@@ -103,6 +106,8 @@ class RoutedExperts(Part):
         pre = self.prefix
         rows = [state[pre + "router"]] + ([state[pre + "shared.sg"]] if self.shared_gate else [])
         self.router = torch.cat(rows, dim=0).contiguous()  # the router's products and sums are fp32 whatever the compute dtype: bfloat16 weights widen exactly
+        # over prompt portions the logits are a product of their own: bfloat16 operands as they are, fp32 sums
+        self.logits = Linear(self.router, None, STORE) if self.router.dtype == torch.bfloat16 else None
         if self.gated:  # gate rows first, then up rows: one product yields both
             self.up = torch.stack([torch.cat([state[pre + f"e{e}.gate"], state[pre + f"e{e}.up"]], dim=0) for e in range(self.experts)]).contiguous()
         else:
@@ -113,7 +118,7 @@ class RoutedExperts(Part):
             self.shared.load(state)
 
     def scratch_row_bytes(self) -> int:
-        return 2 * self.top * (4 * self.hidden + (12 if self.gated else 4) * self.ff + 4 * self.hidden) + 8 * self.hidden + 4 * self.shared_ff + 4 * (self.experts + 1)
+        return 2 * self.top * (4 * self.hidden + (12 if self.gated else 4) * self.ff + 4 * self.hidden) + 8 * self.hidden + 4 * self.shared_ff + 12 * (self.experts + 1)
 
     def forward(self, ctx, x, h, store=False):
         n, dt, top = x.shape[0], self.rt.dtype, self.top
@@ -122,8 +127,13 @@ class RoutedExperts(Part):
         i32, f32 = torch.int32, torch.float32
         choice, weight = ctx.buf((n, top), i32), ctx.buf((n, top), f32)
         gate = ctx.buf((n,), f32) if self.shared_gate else None
-        ops.moe_router(choice, weight, gate, x, self.router, self.routed, top, self.score == "softmax", self.renormalize, self.correction, self.renorm_eps,
-                       self.groups, self.keep, self.route_scale, self.group_best)
+        how = (self.routed, top, self.score == "softmax", self.renormalize, self.correction, self.renorm_eps, self.groups, self.keep, self.route_scale, self.group_best)
+        if self.logits is not None and x.dtype == torch.bfloat16 and n >= ROUTER_PRODUCT_TOKENS:
+            z = ctx.buf((n, self.router.shape[0]), f32)
+            self.logits(z, x, buf=ctx.buf)
+            ops.moe_route(choice, weight, gate, z, *how)
+        else:
+            ops.moe_router(choice, weight, gate, x, self.router, *how)
         pairs = n * top
         tiles = -(-pairs // tile) + self.experts  # every expert may end on a tile that is not full
         dest, tile_expert = ctx.buf((n, top), i32), ctx.buf((tiles,), i32)

@@ -676,7 +676,7 @@ def nugopel_config(z: dict, b: dict):
 def nugopel_numbers(z: dict, b: dict) -> dict:
     """Bytes a decode step reads and flops a token costs for the Nugopel sizes (bf16).  The bench's prompts are longer than the
     window, so a decode step reads the window's rows per request whatever the context (counted as state), and every latent
-    attention reads the whole latent."""
+    attention reads the whole latent; a prompt alone attends to keys and values made from it."""
     w, h, g, r = z["width"], z["heads"], b["kv_heads"], z["kv_rank"]
     latent = w * h * (z["dim"] + z["vdim"]) + h * (z["dim"] + z["vdim"]) * r + h * z["vdim"] * w
     att = w * ((h + g) * b["att_dim"] + g * b["att_vdim"]) + h * b["att_vdim"] * w
@@ -687,7 +687,7 @@ def nugopel_numbers(z: dict, b: dict) -> dict:
     seen = (inside * (inside + 1) / 2 + (PROMPT_LEN - inside) * inside) / whole  # the part of a prompt's (query, key) pairs that the window leaves
     return {"weight_bytes": 2 * (mixers + z["layers"] * (z["experts"] * expert + around) + z["vocab"] * w), "kv_bytes_per_token": n_lat * r * 2,
             "flops_per_token": 2.0 * (mixers + z["layers"] * (z["top"] * expert + around)),
-            "attn_flops_per_pair": n_lat * 4.0 * h * r + seen * n_att * 2.0 * h * (b["att_dim"] + b["att_vdim"]),
+            "attn_flops_per_pair": n_lat * 2.0 * h * (z["dim"] + z["vdim"]) + seen * n_att * 2.0 * h * (b["att_dim"] + b["att_vdim"]),
             "head_flops": 2.0 * w * z["vocab"], "state_bytes_per_request": 2 * b["window"] * n_att * g * (b["att_dim"] + b["att_vdim"])}
 
 

@@ -93,6 +93,7 @@ class Step:
         counts = [hi - lo for _, lo, hi in spans]
         self.n_tokens, self.n_seqs, self.max_q_len = sum(counts), len(spans), max(counts)
         self.decode_only = self.max_q_len == 1
+        self.fresh = not self.decode_only and all(lo == 0 for _, lo, _ in spans)
         self.max_kv_len = self.max_context = max(hi for _, _, hi in spans)
         self.positions = dev(np.concatenate([np.arange(lo, hi, dtype=np.int32) for _, lo, hi in spans]))
         self.seq_of_token = dev(np.concatenate([np.full(c, s, dtype=np.int32) for s, c in enumerate(counts)]))
@@ -205,6 +206,34 @@ def test_latent_attention_on_its_own_latent_and_on_another_layers(dtype, H, d, d
             for what, got in zip(("whole", f"portions of {cuts}"), in_steps(first, case, rows, dtype, cuts, reader)):
                 for i, n in enumerate(lengths):
                     assert_close(got[i], want[i], KERNEL_TOL[dtype], f"{what}: request of {n} tokens, own {reader is None}")
+
+
+@pytest.mark.parametrize("H,d,dv,r,page", [(4, 32, 48, 64, 64), (3, 64, 64, 128, 16), (2, 128, 64, 40, 48), (16, 16, 16, 96, 64)])
+@pytest.mark.parametrize("lengths", [[128], [130, 257, 192], [500, 1, 64, 63], [65, 300]])
+def test_prompts_alone_attend_to_keys_and_values_made_from_their_latents(H, d, dv, r, page, lengths):
+    """bfloat16 steps of prompts that all start in them, of whole pages and not, then a portion and single tokens over the same
+    cache, which go the other way; a second layer on the same rows."""
+    rng = np.random.default_rng(21)
+    m, m2 = latent_mixer(H, d, dv, r), latent_mixer(H + 1, 32, 16, r)
+    w, width = latent_weights(rng, m, BF16)
+    n2 = (H + 1) * 48
+    w2, _ = latent_weights(rng, m2, BF16, "b.", False, (width, 0, width + (H + 1) * 32, width + n2))
+    w = {n: np.pad(v, ((0, 0), (0, n2))) if v.ndim == 2 and v.shape[1] == width else v for n, v in w.items()}
+    rows = [rounded(rng.standard_normal((n + 6, width + n2)), BF16) for n in lengths]
+    first, second = latent_part(w, m, width + n2, BF16, True), latent_part(w2, m2, width + n2, BF16, False, prefix="b.")
+    assert first.tells_fresh and second.tells_fresh and not latent_part(w, m, width + n2, F32, True).tells_fresh
+    case = Paged(rng, [n + 6 for n in lengths], page, (r,), dtype=BF16)
+    latents = [plain.latent(w, "a.", x, 1e-5) for x in rows]
+    want = [[plain.latent_attention(w, "a.", m, x, c) for x, c in zip(rows, latents)], [plain.latent_attention(w2, "b.", m2, x, c) for x, c in zip(rows, latents)]]
+    calls = []
+    for part in (first, second):
+        part.attend_unfolded = lambda *a, f=part.attend_unfolded: calls.append(1) or f(*a)
+    for lo, hi in ((0, 0), (0, 4), (4, 5), (5, 6)):  # the prompts; four tokens more of each; two single ones
+        spans = [(i, n + lo if hi else 0, n + hi) for i, n in enumerate(lengths)]
+        for part, ref, writes in ((first, want[0], True), (second, want[1], False)):
+            got = run_part(part, case, rows, spans, BF16, writes)
+            assert_close(got, np.concatenate([ref[i][a:b] for i, a, b in spans]), KERNEL_TOL[BF16], f"tokens {lo} to {hi}")
+    assert len(calls) == 2, "the prompts alone should have gone over keys and values of their own"
 
 
 @pytest.mark.parametrize("dtype,H,d,dv,r", [(F32, 2, 16, 8, 24), (BF16, 2, 16, 8, 24), (BF16, 4, 32, 16, 64), (BF16, 17, 16, 16, 64)])

@@ -67,9 +67,9 @@ CONFIGS = {
     # no router anywhere, so that bfloat16 is held to its bound at every position, on the tensor-core kernels; windows that end inside pages
     "D": {"architecture": "Nugopel", "vocab": 222, "width": 160, "norm": {"eps": 5e-6},
           "layers": [layer(attention(4, 4, 48, 48, 0.15, 300.0, 24, (5.0, 1.0, 4.0, 150.0), 37), None),
-                     layer(latent(4, 40, 40, 64, 0.16), None),
+                     layer(latent(4, 48, 32, 64, 0.16), None),
                      layer(attention(8, 2, 32, 64, 0.18, 700.0, 20, (2.0, 1.0, 3.0, 256.0), 100), None),
-                     layer(latent(3, 24, 56, 64, 0.2, 1), None)]},
+                     layer(latent(3, 32, 64, 64, 0.2, 1), None)]},
     # every expert for every token, so that no choice is close: the mixture too at every position
     "E": {"architecture": "Nugopel", "vocab": 180, "width": 64, "norm": {"eps": 1e-5},
           "layers": [layer(latent(2, 16, 24, 32, 0.3), moe(4, 4, 32, 24)),
