@@ -824,7 +824,7 @@ def concat_rows(out, a, b) -> None:
 
 
 MOE_TILE = 64  # rows per tile of the sorted matrix: every expert's rows are padded to whole tiles
-GEMM_BY_TILE_FILL = 296  # tiles of a product by tile from which on wide ones are taken
+GEMM_BY_TILE_FILL, GEMM_BY_TILE_FEW = 296, 100  # tiles of a product by tile from which on wide ones, and half as wide ones, are taken
 MOE_TILE_TC = 128  # the same where the tcgen05 product takes the tiles (its token tile)
 
 
@@ -838,8 +838,9 @@ def gemm_by_tile(out, x, w, tile_batch, tile_rows: int, act: str = "none") -> No
     rows = x.shape[0]
     if (tile_rows == MOE_TILE_TC and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and k % 8 == 0 and rows % 128 == 0
             and os.environ.get("ALOFA_BY_TILE_TC", "1") != "0"):
-        # tiles of 256 weight rows, unless they are so few (a decode step's) that half as wide ones keep more SMs pulling weights
-        wide = -256 if n > 128 and tile_batch.numel() * -(-n // 256) >= GEMM_BY_TILE_FILL else -128
+        # tiles of 256 weight rows, unless they are so few (a decode step's) that narrower ones keep more SMs pulling weights
+        tiles = tile_batch.numel()
+        wide = -256 if n > 128 and tiles * -(-n // 256) >= GEMM_BY_TILE_FILL else -128 if tiles * -(-n // 128) >= GEMM_BY_TILE_FEW else -64
         if gemm_tc(out, x, w.view(batches * n, k), None, EPI_STORE, wide, act=ACTIVATIONS[act], tile_batch=tile_batch, batches=batches):
             return
     gemm_batched(out, x, w, 1, rows, n, k, k, 0, k, n * k, n, 0, act=act, tile_batch=tile_batch, tile_rows=tile_rows)

@@ -826,7 +826,8 @@ class KernelClock:
                 a.record()
                 result = fn(*args, **kwargs)
                 b.record()
-                records.append((name, a, b, self.ideal_us(name, args, kwargs, kv_rows)))
+                if result is not False:  # False: the kernel does not take these sizes, nothing was launched
+                    records.append((name, a, b, self.ideal_us(name, args, kwargs, kv_rows)))
                 return result
             return timed
 
