@@ -307,7 +307,7 @@ def attention_weights(rng, m, dtype, ones=False, prefix="a."):
 
 ATTENTIONS = [(F32, 4, 2, 16, 24, 9, 16, 16), (F32, 3, 3, 12, 8, 21, 6, 16), (F32, 2, 1, 10, 30, None, 2, 16), (F32, 1, 1, 8, 130, 2, 8, 16), (F32, 6, 2, 40, 72, 32, 24, 64),
               (BF16, 3, 1, 12, 20, 17, 12, 16), (BF16, 4, 2, 64, 64, 64, 64, 64), (BF16, 4, 1, 64, 64, 1, 32, 64), (BF16, 2, 2, 64, 64, 130, 20, 16), (BF16, 6, 2, 64, 128, 100, 64, 64),
-              (BF16, 2, 1, 128, 64, 90, 96, 32), (BF16, 4, 4, 128, 128, 200, 64, 64), (BF16, 20, 1, 32, 48, 40, 32, 16), (BF16, 3, 3, 96, 96, 72, 48, 64), (BF16, 34, 2, 48, 48, None, 24, 48),
+              (BF16, 2, 1, 128, 64, 90, 96, 32), (BF16, 4, 4, 128, 128, 200, 64, 64), (BF16, 20, 1, 32, 48, 40, 32, 16), (BF16, 3, 3, 96, 96, 81, 32, 64), (BF16, 34, 2, 48, 48, None, 24, 48),
               (BF16, 5, 5, 80, 80, 33, 40, 64)]
 
 
